@@ -99,7 +99,7 @@ __device__ __forceinline__ float tanh_approx(float x) {
 }
 
 // SOFTCAP is a template flag so that the (rare) tanh path never sits in the hot loop's instruction stream: with it
-// inline the unrolled softmax body was ~150 KB of SASS and the four softmax warps ran out of the instruction cache.
+// inline the unrolled softmax body measured several times slower (instruction-fetch bound).
 template <int D, bool SOFTCAP>
 __global__ void __launch_bounds__(THREADS, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
@@ -329,7 +329,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
         const int kv0 = (j0 + it) * BK;
         // The softmax threads are instruction-issue bound (a polynomial ex2 on the FMA pipe made the kernel 20% SLOWER),
         // so the row is touched as little as possible: the max is taken over the RAW scores (scale > 0 commutes with
-        // max), the scale and the max subtraction are one packed FFMA2 per column pair, the row sum one packed FADD2.
+        // max), the scale and the max subtraction are one packed fma per column pair, the row sum one packed add.
         float m_raw = -INFINITY;
         // blocks wholly inside every row's [row_lo, row_hi) of this warp need no mask (the common case away from
         // the causal diagonal and the window edge)

@@ -21,8 +21,7 @@
 //   * A super-tile is 256 weight rows = two UMMA M=128 tiles that share every x tile (B operand):
 //     x is re-read from L2 by every CTA, so sharing halves the L2->SM traffic per weight byte.
 //   * 16 dequant warps (one thread per row and k-half) expand int4/int8 -> fp16 with the magic-number
-//     trick (int4: 1 SHF + 4 LOP3 + 4 HADD2 + 4 HFMA2 per 8 weights, no PRMT; int8: 2 PRMT + 2 HADD2
-//     + 2 HFMA2 per 4) and store the A tile straight into TENSOR MEMORY (tcgen05.st); the MMA is the
+//     trick (masks, packed adds and packed fmas, no conversions) and store the A tile straight into TENSOR MEMORY (tcgen05.st); the MMA is the
 //     TS form, fp16 A x bf16/fp16 B -> fp32 in TMEM.  fp16 keeps 11 significant bits of s*q+b (bf16: 8),
 //     which is what holds the 2e-2/1e-2 parity bound at K = 25600 / 28672.
 //   * Accumulators are double-buffered in TMEM; 4 epilogue warps drain tile i (bias, SwiGLU, bf16,

@@ -11,7 +11,7 @@
 // of x (UMMA N = NB in {16..256}); the fp32 accumulator [128 x NB] lives in TMEM.
 //
 //   warps 0..DQW-1     dequant: DQW/4 threads per weight row, each unpacks its share of the 64-wide
-//                      k block (int4/int8 -> s*q+b, bf16x2 HFMA2, single rounding) -> A ring in the
+//                      k block (int4/int8 -> s*q+b, packed fma, single rounding) -> A ring in the
 //                      canonical K-major SWIZZLE_128B layout
 //   warp DQW   (1 thr)  TMA: packed uint32 weight tiles [128 rows x 128 B] -> smem ring (PS deep)
 //   warp DQW+1 (1 thr)  TMA: x tiles [NB x 64] bf16, 128B-swizzled K-major  -> B ring (NS deep)
@@ -113,7 +113,7 @@ __device__ __forceinline__ uint4 dequant_word4(uint32_t w, typename Cvt<T>::T2 s
 }
 // 4 bytes of one packed word -> 4 fp16 values s*q+b: a byte under the exponent byte 0x64 reads 1024 + q exactly
 // (q < 1024), the subtraction is exact and the FMA rounds once -- the same single rounding as an fp32 fma followed
-// by a conversion, in 2 PRMT + 2 HADD2 + 2 HFMA2 instead of 4 I2F + 4 FFMA + 2 F2F per word (the int8 GEMM at
+// by a conversion, in six packed operations instead of ten scalar ones per word (the int8 GEMM at
 // M >= 256 was dequant-bound on the conversions: 0.28-0.47 of the bf16 peak, profiles/r02_gemm_bigm.txt).
 template <typename T>
 __device__ __forceinline__ uint2 dequant_word8(uint32_t w, float s, float b) {
@@ -327,8 +327,8 @@ qgemm_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_constant
     }
   } else if (warp == W_MMA) {
     // ===== MMA issuer: whole-warp loop with warp-uniform operands, issue under elect_one().  Under `if (lane == 0)`
-    // ptxas wrapped every tcgen05.mma in an ELECT + R2UR waterfall (~80 cycles per MMA): at NB = 64 (32 cycles of
-    // tensor pipe per MMA) that WAS the "0.3 us per k block whatever the math" of round 1's ablation. =====
+    // an issue measured ~80 cycles per MMA: at NB = 64 (32 cycles of tensor pipe per MMA) that was 0.3 us per k
+    // block whatever the math. =====
     constexpr uint32_t idesc = make_idesc(C::kFmt, ROWS, NB);
     const uint32_t tb = __shfl_sync(0xffffffffu, tmem_base, 0);
     for (int kb = 0; kb < my_kb; ++kb) {
