@@ -1,0 +1,177 @@
+/*
+ * b200_hybrid_ops.h -- C-ABI of the mixers of hybrid decoders: latent attention over a paged latent cache, gated
+ * linear recurrences (Mamba-2, mLSTM) over per-request state slots, and the norms / gates either side of them.
+ * Same conventions as b200_paged_ops.h: device pointers, element strides, `stream` is a cudaStream_t, 0 on success.
+ *
+ * A batch is a list of segments (one per request) of consecutive rows: rows [cu_seqlens[s], cu_seqlens[s+1]) are the
+ * new tokens of segment s, seq_lens[s] its length INCLUDING them, so its first row is at position
+ * seq_lens[s] - (cu_seqlens[s+1] - cu_seqlens[s]).  A segment that starts at position 0 finds a zero state whatever
+ * its slot holds.
+ */
+#ifndef B200_HYBRID_OPS_H_
+#define B200_HYBRID_OPS_H_
+
+#include <stddef.h>
+#include <stdint.h>
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+/* out[r, :] = table[ids[r], :] widened to fp32 (a 32-bit residual stream). */
+int b200_embed_rows(const int32_t* ids, const void* table, float* out, int rows, int vocab, int dim,
+                    int64_t out_stride, int dtype, void* stream);
+
+/* out[r, :] = x[row_ids ? row_ids[r] : r, :] / sqrt(mean(x^2) + eps) * (weight + weight_offset); x and weight fp32,
+ * out in out_dtype.  weight_offset = 1: weights stored around zero. */
+int b200_stream_norm(const float* x, const int64_t* row_ids, const float* weight, void* out, int rows, int dim,
+                     int64_t x_stride, int64_t out_stride, float eps, float weight_offset, int out_dtype,
+                     void* stream);
+
+/* The element-wise end of a layer's two parallel halves, one launch:
+ *   out[r, 0:inner)              = post(gate) * weight * group_norm(y * pre(z))
+ *     pre(z) = silu(z) if pre_gate, post(g) = sigmoid(g) if post_gate; group_norm divides each of inner / group_size
+ *     parts by its own root mean square (group_size = 0: no norm); weight fp32 or NULL.
+ *   out[r, act_offset + i]       = gelu(act_in[r, i]) (erf form), i in [0, act_dim)
+ *   out[r, i] = 0 for the remaining columns below out_cols (alignment padding of the next product's operand).
+ * Any of the two halves may be absent (act_dim = 0; y = NULL: the columns below inner are somebody else's). */
+typedef struct b200_mixer_finish_args {
+  const void* y;
+  const void* pre_gate;
+  const void* post_gate;
+  const float* weight;
+  const void* act_in;
+  void* out;
+  int64_t y_stride, pre_stride, post_stride, act_stride, out_stride;
+  int32_t rows, inner, group_size, act_dim, act_offset, out_cols;
+  int32_t y_head_dim, y_head_stride; /* y column c is at (c / y_head_dim) * y_head_stride + c % y_head_dim (0: c) */
+  float eps;
+  int32_t dtype;
+} b200_mixer_finish_args;
+int b200_mixer_finish(const b200_mixer_finish_args* a, void* stream);
+
+/* Causal depthwise convolution over segments, then silu if `activation` = 1:
+ *   out[t, c] = act(bias[c] + sum_k weight[k, c] * in[t - (taps - 1) + k, c])
+ * inputs before the segment come from state[slot, taps-1, channels] (oldest first), which is replaced by the last
+ * taps - 1 inputs.  weight fp32 [taps, channels], bias fp32 [channels]. */
+int b200_causal_conv(const void* in, const float* weight, const float* bias, void* state, const int32_t* cu_seqlens,
+                     const int32_t* seq_lens, const int32_t* slots, void* out, int num_seqs, int max_q_len,
+                     int channels, int taps, int64_t in_stride, int64_t out_stride, int activation, int dtype,
+                     void* stream);
+
+/* Gated linear recurrence per (segment, head), state S [key_dim, value_dim] in fp32:
+ *   kind 0 (Mamba-2): dt = softplus(gate_a + bias_a[h]);
+ *       S <- exp(-rate[h] dt) S + dt k v^T;  out = S^T q + skip[h] v;  q / k shared by num_heads / num_groups heads.
+ *   kind 1 (mLSTM): i = cap tanh((gate_a + bias_a[h]) / cap), f = logsigmoid(cap tanh((gate_b + bias_b[h]) / cap)),
+ *       m' = max(f + m, i); S <- exp(f + m - m') S + exp(i - m') k v^T; n likewise with k alone;
+ *       out = S^T q' / (max(|n . q'|, exp(-m')) + 1e-6), q' = q_scale q.
+ * state [slots, heads, key_dim, value_dim]; mLSTM also norm_state [slots, heads, vtiles, key_dim] and max_state
+ * [slots, heads, vtiles] with vtiles = ceil(value_dim / 64): one copy per 64-wide value tile, so that the tiles of a
+ * head never wait for one another.
+ * Segments of at most seq_limit rows run token by token; longer ones (16-bit types only) in chunks of
+ * B200_RECURRENCE_CHUNK rows listed by chunk_seq / chunk_row (segment and first row of every chunk of every longer
+ * segment, in order; seq_chunk0[s] = index of segment s's first chunk).  workspace: see
+ * b200_recurrence_workspace_bytes. */
+#define B200_RECURRENCE_CHUNK 64
+typedef struct b200_recurrence_args {
+  const void* q;
+  const void* k;
+  const void* v;
+  const void* gate_a;
+  const void* gate_b;
+  const float* bias_a;
+  const float* bias_b;
+  const float* rate;
+  const float* skip;
+  float* state;
+  float* norm_state;
+  float* max_state;
+  const int32_t* cu_seqlens;
+  const int32_t* seq_lens;
+  const int32_t* slots;
+  const int32_t* chunk_seq;
+  const int32_t* chunk_row;
+  const int32_t* seq_chunk0;
+  void* out;
+  void* workspace;
+  size_t workspace_bytes;
+  int64_t q_stride, k_stride, v_stride, gate_stride, out_stride;
+  int32_t kind, dtype, num_tokens, num_seqs, num_heads, num_groups, key_dim, value_dim;
+  int32_t num_chunks, seq_limit;
+  float q_scale, gate_cap;
+} b200_recurrence_args;
+size_t b200_recurrence_workspace_bytes(const b200_recurrence_args* a);
+/* 1 if the chunked form covers this call's type and sizes (it needs 16-bit operands and 16-multiples). */
+int b200_recurrence_can_chunk(const b200_recurrence_args* a);
+int b200_recurrence(const b200_recurrence_args* a, void* stream);
+int b200_recurrence_num_launches(const b200_recurrence_args* a);
+
+/* Before latent attention, per row: the latent is normed (weight fp32, plain), the shared key part is rotated
+ * (interleaved pairs), both go to the latent cache row slot_mapping[t]:
+ * [latent kv_rank | key part rot_dim]; the rotated part of every query head goes to
+ * q_out[t, h, rot_offset + ...], and with copy_nope the unrotated part to q_out[t, h, 0 : dim), columns from
+ * rot_offset + rot_dim to q_cols zeroed. */
+typedef struct b200_latent_prep_args {
+  const void* q;
+  const void* down;
+  const float* norm_weight;
+  const int32_t* positions;
+  const int64_t* slot_mapping;
+  const float* inv_freq; /* [rot_dims / 2], base^(-2i/rot_dims) */
+  void* cache;
+  void* q_out;
+  int64_t q_stride, down_stride, q_out_stride;
+  int64_t num_slots;
+  int32_t num_tokens, heads, dim, rot_dim, rot_dims, kv_rank;
+  int32_t q_cols, rot_offset, copy_nope;
+  float eps;
+  int32_t dtype;
+} b200_latent_prep_args;
+int b200_latent_prep(const b200_latent_prep_args* a, void* stream);
+
+/* y[t, h, n] = sum_k w[h, n, k] x[t, h, k], times sigmoid(gate[t, h * n_dim + n]) if gate: the per-head products of
+ * latent attention (queries into the latent space, latent outputs into value space). */
+typedef struct b200_head_linear_args {
+  const void* x;
+  const void* w;
+  const void* gate;
+  void* y;
+  int64_t x_stride, x_head_stride, y_stride, y_head_stride, gate_stride;
+  int32_t rows, heads, n, k, dtype;
+} b200_head_linear_args;
+int b200_head_linear(const b200_head_linear_args* a, void* stream);
+
+/* Latent attention in the latent space: every query head attends over the same cached rows
+ * [latent kv_rank | key part rot_dim]; values are the latents.  q [T, heads, kv_rank + rot_dim], out
+ * [T, heads, kv_rank].  Only segments of at most max_q_len rows are computed.  window <= 0: none. */
+typedef struct b200_latent_attn_args {
+  const void* q;
+  const void* cache;
+  const int32_t* block_tables;
+  const int32_t* seq_lens;
+  const int32_t* cu_seqlens;
+  void* out;
+  void* workspace;
+  size_t workspace_bytes;
+  int64_t q_stride, out_stride;
+  int64_t num_slots;
+  int32_t num_tokens, num_seqs, heads, kv_rank, rot_dim, block_size, max_blocks_per_seq, max_seq_len, window;
+  int32_t max_q_len;
+  int32_t dtype, kernel, force_splits;
+  float scale;
+} b200_latent_attn_args;
+size_t b200_latent_attention_workspace_bytes(const b200_latent_attn_args* a);
+int b200_latent_attention_num_launches(const b200_latent_attn_args* a);
+int b200_latent_attention(const b200_latent_attn_args* a, void* stream);
+
+/* Rows [first[i], first[i] + count[i]) of request i's cached latents, gathered from the pages into consecutive rows
+ * of out [rows, kv_rank + rot_dim] starting at out_row[i] (the operand of the products that expand keys and values);
+ * rows between out_row[i] + count[i] and the next multiple of `pad` are zeroed. */
+int b200_latent_gather(const void* cache, const int32_t* block_tables, const int32_t* first, const int32_t* count,
+                       const int32_t* out_row, void* out, int num_seqs, int max_count, int width, int block_size,
+                       int max_blocks_per_seq, int64_t num_slots, int pad, int dtype, void* stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif /* B200_HYBRID_OPS_H_ */

@@ -25,7 +25,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 3
+#define B200_ABI_VERSION 4
 
 /* Element types of activations / caches (reference: dtype_to_metal,
  * paged_ops.cpp:185-196 -- float, half, bfloat16 are the supported set). */
@@ -167,6 +167,8 @@ typedef struct b200_paged_attn_args {
                               floor(16 / (H_q/H_kv)) query rows of one sequence per CTA share every KV read
                               (pagedattention.metal:1396-1914) -- and never the tile kernel (paged_ops.cpp:468-476).
                               Results are bitwise those of the expanded one-row-per-segment dispatch. */
+  int32_t wide_weights; /* 1: the prefill tile kernel feeds the softmax weights to the value product as a two-term
+                         * bf16 split (16 significant bits instead of 8); other kernels ignore it */
 } b200_paged_attn_args;
 
 size_t b200_paged_attention_workspace_bytes(const b200_paged_attn_args* args);

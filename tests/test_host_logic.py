@@ -153,7 +153,7 @@ def test_quantized_linear_module_protocol():
 
 def _declared_symbols() -> set[str]:
     names = set()
-    for h in ("b200_paged_ops.h", "b200_decoder_ops.h", "b200_tp_ops.h"):
+    for h in ("b200_paged_ops.h", "b200_decoder_ops.h", "b200_tp_ops.h", "b200_hybrid_ops.h"):
         path = os.path.join(ROOT, "include", h)
         if not os.path.exists(path):
             continue
@@ -169,7 +169,7 @@ def test_library_exports_every_declared_symbol():
     assert declared == set(EXPORTED_SYMBOLS)
     for name in sorted(declared):
         assert hasattr(lib, name), f"{name} declared in include/*.h but not exported"
-    assert lib.b200_abi_version() == 3  # round 2: x_dtype / out_dtype arguments, args.out_dtype, args.window_seqlen_q
+    assert lib.b200_abi_version() == 4  # args.out_dtype, args.window_seqlen_q, args.wide_weights
     assert lib.b200_partition_size() == 512
 
 

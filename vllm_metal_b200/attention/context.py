@@ -48,6 +48,8 @@ class PagedAttentionContext:
     num_decode_requests: int = 0
     verify_window_q: int = 1
     kv_groups: tuple[PagedKVGroupContext, ...] | None = None
+    # state slot of every segment (recurrent layers); set by the runner, None for models without such layers
+    state_slots: list[int] | None = None
     # (group index, cache block size) -> device tensors, filled by impls.sdpa
     kernel_metadata_cache: dict[tuple[int | None, int], Any] = field(default_factory=dict)
     # per-token RoPE positions (device int32), memoised by impls.sdpa

@@ -1,0 +1,121 @@
+"""Device metadata of one packed step for recurrent and latent-attention layers: what ``_KernelMetadata`` holds for the
+paged caches, plus the state slot of every segment, the chunk list of the recurrences and the split of the batch into
+rows that attend in the latent space and rows whose keys and values are expanded first.  Built once per step, shared
+by all layers."""
+
+from __future__ import annotations
+
+from dataclasses import dataclass, field
+
+import numpy as np
+import torch
+
+from ...metal.hybrid_ops import RECURRENCE_CHUNK
+from .sdpa import _KernelMetadata, _positions, _to_device
+
+# Segments of at most this many rows go through the recurrences token by token (their state is streamed once per row);
+# longer ones in chunks.
+CHUNK_LIMIT = 4
+EXPAND_PAGE = 32  # page size of the expanded key / value buffer
+
+
+@dataclass(frozen=True, eq=False)
+class ExpandPlan:
+    """Segments ``first_seq ..`` of the batch, whose visible keys and values are expanded from the latents."""
+
+    first_row: int
+    rows_total: int           # rows of the expanded buffer (whole pages)
+    max_count: int
+    first: torch.Tensor       # int32 [S'] first visible position
+    count: torch.Tensor       # int32 [S'] visible rows
+    out_row: torch.Tensor     # int32 [S'] where they start in the buffer
+    source_tables: torch.Tensor
+    cu_seqlens_q: torch.Tensor
+    block_tables: torch.Tensor  # of the expanded buffer
+
+
+@dataclass(frozen=True, eq=False)
+class SegmentMetadata(_KernelMetadata):
+    state_slots: torch.Tensor = None  # int32 [S]
+    max_q_len: int = 1
+    num_chunks: int = 0
+    has_short: bool = True
+    chunk_limit: int = CHUNK_LIMIT
+    chunk_seq: torch.Tensor | None = None
+    chunk_row: torch.Tensor | None = None
+    seq_chunk0: torch.Tensor | None = None
+    # host copies the expansion plans are made from (None on the all-decode path, which never expands)
+    q_lens: np.ndarray | None = None
+    context_lens: np.ndarray | None = None
+    _plans: dict = field(default_factory=dict)
+
+    def split(self, threshold: int) -> tuple[int, int, int]:
+        """``(segments, rows, longest)`` of the leading part that attends in the latent space: everything before the
+        trailing run of segments of at least ``threshold`` rows."""
+        if self.q_lens is None:
+            return self.seq_lens.shape[0], self.positions.shape[0], self.max_q_len
+        n = len(self.q_lens)
+        while n > 0 and self.q_lens[n - 1] >= threshold:
+            n -= 1
+        return n, int(self.q_lens[:n].sum()), int(self.q_lens[:n].max(initial=0))
+
+    def expand_plan(self, threshold: int, window: int) -> ExpandPlan | None:
+        key = (threshold, window)
+        if key not in self._plans:
+            self._plans[key] = self._make_plan(threshold, window)
+        return self._plans[key]
+
+    def _make_plan(self, threshold: int, window: int) -> ExpandPlan | None:
+        n, row0, _ = self.split(threshold)
+        if self.q_lens is None or n == len(self.q_lens):
+            return None
+        q, ctx = self.q_lens[n:].astype(np.int64), self.context_lens[n:].astype(np.int64)
+        first = np.maximum(0, ctx - q - window + 1) if window > 0 else np.zeros_like(ctx)
+        count = ctx - first
+        pages = -(-count // EXPAND_PAGE)
+        page0 = np.concatenate([[0], np.cumsum(pages)])
+        table = np.zeros((len(q), int(pages.max())), dtype=np.int32)
+        for i, p in enumerate(pages):
+            table[i, :p] = page0[i] + np.arange(p)
+        dev = self.seq_lens.device
+        i32 = [np.asarray(x, dtype=np.int32) for x in (first, count, page0[:-1] * EXPAND_PAGE,
+                                                       np.concatenate([[0], np.cumsum(q)]))]
+        f, c, o, cu = (_to_device(x, torch.int32, dev) for x in i32)
+        return ExpandPlan(row0, int(page0[-1]) * EXPAND_PAGE, int(count.max()), f, c, o, self.block_tables[n:], cu,
+                          _to_device(table, torch.int32, dev))
+
+
+def segment_metadata(ctx, block_size: int, device) -> SegmentMetadata:
+    """From a step context whose ``state_slots`` are set (``prepare_unified`` + the runner)."""
+    key = ("segments", block_size)
+    meta = ctx.kernel_metadata_cache.get(key)
+    if meta is not None:
+        return meta
+    cu = np.asarray(ctx.cu_seqlens, dtype=np.int64)
+    q = np.diff(cu)
+    n = len(q)
+    # the any-size page arithmetic of these kernels takes the cache's own block size: no kernel-page translation
+    width = max(1, max(len(r) for r in ctx.block_tables))
+    table = np.zeros((n, width), dtype=np.int32)
+    for i, row in enumerate(ctx.block_tables):
+        table[i, :len(row)] = row
+    slots = ctx.state_slots if ctx.state_slots is not None else [0] * n
+    long = np.nonzero(q > CHUNK_LIMIT)[0]
+    chunk_seq, chunk_row = [], []
+    seq_chunk0 = np.zeros(n, dtype=np.int32)
+    for s in long:
+        seq_chunk0[s] = len(chunk_seq)
+        rows = range(int(cu[s]), int(cu[s + 1]), RECURRENCE_CHUNK)
+        chunk_seq += [int(s)] * len(rows)
+        chunk_row += list(rows)
+    dev = lambda x, t=torch.int32: _to_device(np.asarray(x), t, device)  # noqa: E731
+    meta = SegmentMetadata(
+        slot_mapping=dev(np.asarray(ctx.slot_mapping, dtype=np.int64), torch.int64),
+        seq_lens=dev(np.asarray(ctx.context_lens, dtype=np.int32)), cu_seqlens_q=dev(cu.astype(np.int32)),
+        block_tables=dev(table), block_size=block_size, max_seq_len=max(ctx.context_lens), positions=dev(_positions(ctx)),
+        state_slots=dev(np.asarray(slots, dtype=np.int32)), max_q_len=int(q.max()), num_chunks=len(chunk_seq),
+        has_short=len(long) < n, chunk_seq=dev(np.asarray(chunk_seq, dtype=np.int32)) if chunk_seq else None,
+        chunk_row=dev(np.asarray(chunk_row, dtype=np.int32)) if chunk_seq else None,
+        seq_chunk0=dev(seq_chunk0) if chunk_seq else None, q_lens=q, context_lens=np.asarray(ctx.context_lens))
+    ctx.kernel_metadata_cache[key] = meta
+    return meta

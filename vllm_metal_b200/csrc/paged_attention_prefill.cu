@@ -100,7 +100,9 @@ __device__ __forceinline__ float tanh_approx(float x) {
 
 // SOFTCAP is a template flag so that the (rare) tanh path never sits in the hot loop's instruction stream: with it
 // inline the unrolled softmax body measured several times slower (instruction-fetch bound).
-template <int D, bool SOFTCAP>
+// WIDE keeps two bf16 terms of every softmax weight: the high terms take the first half of S's columns as usual, the low
+// terms the second half, and the value product runs over both.
+template <int D, bool SOFTCAP, bool WIDE>
 __global__ void __launch_bounds__(THREADS, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                   const __grid_constant__ CUtensorMap v_map, const Params p) {
@@ -281,6 +283,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           for (int k = 0; k < BK / 16; ++k) {
             const uint64_t dv = make_smem_desc_mn(sm_v + st * SM::KV_BYTES + k * 16 * 128, SM::HALF_BYTES, 1024);
             tc_mma_f16_ts(tb + TM_O + i * D, tb + TM_SP + i * BK + 8 * k, dv, idesc_o, (it | k) != 0 ? 1u : 0u);
+            if (WIDE) tc_mma_f16_ts(tb + TM_O + i * D, tb + TM_SP + i * BK + BK / 2 + 8 * k, dv, idesc_o, 1u);
           }
           if (i == ntile - 1) tc_commit(bar_v_empty + 8 * st);
           tc_commit(bar_o_full + 8 * i);
@@ -354,13 +357,32 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
         const float m_eff = (m_new == -INFINITY) ? 0.f : m_new;
         const float2 sc2 = make_float2(sc, sc), nm2 = make_float2(-m_eff, -m_eff);
         float2 sum2 = make_float2(0.f, 0.f);
-        uint32_t pk[BK / 2];
+        uint32_t pk[WIDE ? 1 : BK / 2];
+        if (WIDE) {
+          // S_i(it) is complete, so PV_i(it - 1), issued before it, is: the whole of SP_i may be overwritten here
 #pragma unroll
-        for (int c = 0; c < BK; c += 2) {
-          const float2 x2 = __ffma2_rn(make_float2(s[c], s[c + 1]), sc2, nm2);  // s * scale*log2e - m
-          const float2 p2 = make_float2(ex2(x2.x), ex2(x2.y));
-          sum2 = __fadd2_rn(sum2, p2);
-          pk[c >> 1] = pack2(p2.x, p2.y, p.is_fp16);
+          for (int g = 0; g < 2; ++g) {
+            uint32_t hi[32], lo[32];
+#pragma unroll
+            for (int c = 0; c < 64; c += 2) {
+              const float2 x2 = __ffma2_rn(make_float2(s[g * 64 + c], s[g * 64 + c + 1]), sc2, nm2);
+              const float2 p2 = make_float2(ex2(x2.x), ex2(x2.y));
+              sum2 = __fadd2_rn(sum2, p2);
+              hi[c >> 1] = pack2(p2.x, p2.y, 0);
+              const float2 h2 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi[c >> 1]));
+              lo[c >> 1] = pack2(p2.x - h2.x, p2.y - h2.y, 0);
+            }
+            tmem_st32(t_sp + g * 32, hi);
+            tmem_st32(t_sp + BK / 2 + g * 32, lo);
+          }
+        } else {
+#pragma unroll
+          for (int c = 0; c < BK; c += 2) {
+            const float2 x2 = __ffma2_rn(make_float2(s[c], s[c + 1]), sc2, nm2);  // s * scale*log2e - m
+            const float2 p2 = make_float2(ex2(x2.x), ex2(x2.y));
+            sum2 = __fadd2_rn(sum2, p2);
+            pk[c >> 1] = pack2(p2.x, p2.y, p.is_fp16);
+          }
         }
         const float sum = sum2.x + sum2.y;
         l = l * alpha + sum;
@@ -380,8 +402,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           }
         }
         m_used = m_new;
-        tmem_st32(t_sp, pk);        // P_i over the first half of S_i's columns (every thread has read its S row)
-        tmem_st32(t_sp + 32, pk + 32);
+        if (!WIDE) {
+          tmem_st32(t_sp, pk);        // P_i over the first half of S_i's columns (every thread has read its S row)
+          tmem_st32(t_sp + 32, pk + 32);
+        }
         tmem_st_wait();
         tc_fence_before();
         __syncwarp();
@@ -438,10 +462,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   }
 }
 
-template <int D, bool SOFTCAP>
+template <int D, bool SOFTCAP, bool WIDE>
 static int launch(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) {
   using SM = Smem<D>;
-  auto kern = prefill_tc_kernel<D, SOFTCAP>;
+  auto kern = prefill_tc_kernel<D, SOFTCAP, WIDE>;
   static int configured_dev[16] = {0};
   int dev = 0;
   B200_CUDA_OK(cudaGetDevice(&dev));
@@ -503,9 +527,9 @@ bool prefill_tc_supported(const b200_paged_attn_args& a) {
   if (a.dtype != B200_BF16 && a.dtype != B200_F16) return false;
   if (a.head_dim != 64 && a.head_dim != 128) return false;
   if (a.block_size < 8 || a.block_size > 128 || (128 % a.block_size) != 0) return false;
-  // the TMA maps view each cache as one [num_blocks * block_size tokens, H_kv * D] matrix
+  // the TMA maps view each cache as one [num_blocks * block_size tokens, H_kv * D] matrix (rows may be wider)
   if (a.kv_head_stride != a.head_dim) return false;
-  if (a.kv_token_stride != (int64_t)a.num_kv_heads * a.head_dim) return false;
+  if (a.kv_token_stride < (int64_t)a.num_kv_heads * a.head_dim || a.kv_token_stride % 8) return false;
   if (a.kv_block_stride != (int64_t)a.block_size * a.kv_token_stride) return false;
   if (((uintptr_t)a.query % 16) || ((uintptr_t)a.key_cache % 16) || ((uintptr_t)a.value_cache % 16)) return false;
   if ((a.q_stride * 2) % 16) return false;
@@ -514,8 +538,11 @@ bool prefill_tc_supported(const b200_paged_attn_args& a) {
 }
 
 int launch_prefill_tc(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) {
-  if (a.softcap > 0.f) return a.head_dim == 128 ? pf::launch<128, true>(a, min_qlen, st) : pf::launch<64, true>(a, min_qlen, st);
-  return a.head_dim == 128 ? pf::launch<128, false>(a, min_qlen, st) : pf::launch<64, false>(a, min_qlen, st);
+  if (a.softcap > 0.f)
+    return a.head_dim == 128 ? pf::launch<128, true, false>(a, min_qlen, st) : pf::launch<64, true, false>(a, min_qlen, st);
+  if (a.wide_weights && a.dtype == B200_BF16)
+    return a.head_dim == 128 ? pf::launch<128, false, true>(a, min_qlen, st) : pf::launch<64, false, true>(a, min_qlen, st);
+  return a.head_dim == 128 ? pf::launch<128, false, false>(a, min_qlen, st) : pf::launch<64, false, false>(a, min_qlen, st);
 }
 
 }  // namespace b200

@@ -1,0 +1,81 @@
+"""Dense (unquantized) linears of the hybrid decoders.  Layers that feed several projections from one input run them as
+ONE product (rows of all weights stacked), and the two halves of a parallel layer leave through one product as well:
+their outputs are columns of one operand, their weights lie side by side along K, and the product accumulates straight
+into the fp32 residual stream.  The products themselves are plain library GEMMs (fp32 accumulation)."""
+
+from __future__ import annotations
+
+import torch
+
+_ALIGN = 8  # columns: 16 bytes of a 16-bit type, what vector loads and the tensor-core GEMMs want
+
+
+def pin_matmul_precision() -> None:
+    """fp32 stays fp32 and 16-bit products accumulate in fp32 whatever the process had set before."""
+    torch.backends.cuda.matmul.allow_tf32 = False
+    torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
+
+
+def _up(n: int) -> int:
+    return -(-n // _ALIGN) * _ALIGN
+
+
+class StackedLinear:
+    """``y = x W^T`` for several weights ``[out_i, in]`` that share ``x``; ``split(y)`` gives the parts as views."""
+
+    def __init__(self, parts: dict[str, torch.Tensor], dtype: torch.dtype, device) -> None:
+        self.slices: dict[str, tuple[int, int]] = {}
+        at = 0
+        for name, w in parts.items():
+            self.slices[name] = (at, at + w.shape[0])
+            at = _up(at + w.shape[0])
+        width = next(iter(parts.values())).shape[1]
+        self.weight = torch.zeros((at, width), dtype=dtype, device=device)
+        for name, w in parts.items():
+            if w.shape[1] != width:
+                raise ValueError(f"'{name}' takes {w.shape[1]} inputs, the others {width}")
+            lo, hi = self.slices[name]
+            self.weight[lo:hi].copy_(w)
+
+    def __call__(self, x: torch.Tensor) -> torch.Tensor:
+        return torch.mm(x, self.weight.t())
+
+    def split(self, y: torch.Tensor) -> dict[str, torch.Tensor]:
+        return {name: y[:, lo:hi] for name, (lo, hi) in self.slices.items()}
+
+
+class SideBySideLinear:
+    """``x += [a | b] [W_a | W_b]^T`` with an fp32 ``x``."""
+
+    def __init__(self, parts: dict[str, torch.Tensor], dtype: torch.dtype, device) -> None:
+        self.offsets: dict[str, int] = {}
+        at = 0
+        for name, w in parts.items():
+            self.offsets[name] = at
+            at = _up(at + w.shape[1])
+        self.columns = at
+        rows = next(iter(parts.values())).shape[0]
+        self.weight = torch.zeros((rows, at), dtype=dtype, device=device)
+        for name, w in parts.items():
+            self.weight[:, self.offsets[name]:self.offsets[name] + w.shape[1]].copy_(w)
+
+    def operand(self, rows: int) -> torch.Tensor:
+        return torch.empty((rows, self.columns), dtype=self.weight.dtype, device=self.weight.device)
+
+    def add_into(self, x: torch.Tensor, y: torch.Tensor) -> None:
+        if y.dtype == torch.float32:
+            torch.addmm(x, y, self.weight.t(), out=x)
+        else:
+            torch.addmm(x, y, self.weight.t(), out_dtype=torch.float32, out=x)
+
+
+class DenseHead:
+    """Logits in fp32."""
+
+    def __init__(self, weight: torch.Tensor, dtype: torch.dtype, device) -> None:
+        self.weight = weight.to(device=device, dtype=dtype).contiguous()
+
+    def __call__(self, x: torch.Tensor) -> torch.Tensor:
+        if x.dtype == torch.float32:
+            return torch.mm(x, self.weight.t())
+        return torch.mm(x, self.weight.t(), out_dtype=torch.float32)

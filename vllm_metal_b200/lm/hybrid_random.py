@@ -1,0 +1,67 @@
+"""Random weights for a hybrid configuration (benchmarks, tests, dummy loading): variances that keep the residual
+stream, the gates and the decays in a range where every mechanism matters."""
+
+from __future__ import annotations
+
+import torch
+
+from .hybrid_config import HybridArgs, LatentAttentionArgs, Mamba2Args, MLSTMArgs
+
+
+def tensor_shapes(args: HybridArgs) -> dict[str, tuple[int, ...]]:
+    """Checkpoint tensor names and shapes of a configuration."""
+    w = args.width
+    shapes: dict[str, tuple[int, ...]] = {"embed": (args.vocab, w)}
+    for i, layer in enumerate(args.layers):
+        if layer.weights != i:
+            continue
+        m, p = layer.mixer, f"l{i}.mix."
+        shapes[f"l{i}.norm1"] = (w,)
+        if isinstance(m, Mamba2Args):
+            shapes |= {p + "in": (2 * m.inner + 2 * m.groups * m.state + m.heads, w), p + "conv": (m.conv_channels, m.conv),
+                       p + "conv.b": (m.conv_channels,), p + "dt_bias": (m.heads,), p + "A_log": (m.heads,),
+                       p + "D": (m.heads,), p + "norm": (m.inner,), p + "o": (w, m.inner)}
+        elif isinstance(m, MLSTMArgs):
+            qk, v = m.heads * m.dim, m.heads * m.vdim
+            shapes |= {p + "q": (qk, w), p + "k": (qk, w), p + "v": (v, w), p + "g": (v, w), p + "o": (w, v),
+                       p + "norm": (v,), p + "i": (m.heads, w), p + "i.b": (m.heads,), p + "f": (m.heads, w),
+                       p + "f.b": (m.heads,)}
+        elif isinstance(m, LatentAttentionArgs):
+            shapes |= {p + "q": (m.heads * (m.dim + m.rot_dim), w), p + "dkv": (m.kv_rank + m.rot_dim, w),
+                       p + "dkv.norm": (m.kv_rank,), p + "uk": (m.heads * m.dim, m.kv_rank),
+                       p + "uv": (m.heads * m.vdim, m.kv_rank), p + "g": (m.heads * m.vdim, w),
+                       p + "o": (w, m.heads * m.vdim)}
+        if layer.ff:
+            shapes |= {f"l{i}.mlp.up": (layer.ff, w), f"l{i}.mlp.down": (w, layer.ff)}
+    return shapes | {"final.norm": (w,), "head": (args.vocab, w)}
+
+
+def random_tensors(args: HybridArgs, device="cpu", seed: int = 0):
+    """A ``get(name, shape)`` for ``HybridModel`` whose tensors are drawn when asked for."""
+    shapes = tensor_shapes(args)
+
+    def get(name: str, shape: tuple[int, ...]) -> torch.Tensor:
+        if shapes[name] != tuple(shape):
+            raise ValueError(f"tensor '{name}': asked for {shape}, the configuration says {shapes[name]}")
+        gen = torch.Generator(device=device).manual_seed(seed * 1000003 + list(shapes).index(name))
+        t = torch.empty(shape, dtype=torch.float32, device=device).normal_(0.0, 1.0, generator=gen)
+        leaf = name.split(".", 1)[-1]
+        if leaf in ("mix.dkv.norm", "mix.norm"):
+            t = 1.0 + 0.1 * t
+        elif leaf in ("norm1", "norm"):        # stored around zero
+            t = 0.1 * t
+        elif leaf == "mix.A_log":
+            t = t.abs() * 0.7
+        elif leaf == "mix.dt_bias":
+            t = t - 2.0
+        elif leaf == "mix.f.b":
+            t = t + 2.0
+        elif leaf == "mix.conv":
+            t = t * shape[1] ** -0.5
+        elif leaf in ("mix.D", "mix.i.b", "mix.conv.b", "embed"):
+            t = 0.5 * t
+        elif len(shape) == 2:
+            t = t * shape[1] ** -0.5
+        return t.to(torch.bfloat16)
+
+    return get

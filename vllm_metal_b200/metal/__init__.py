@@ -28,6 +28,7 @@ from typing import Any
 import torch
 
 from . import constants
+from .hybrid_ops import HYBRID_SYMBOLS, HybridOps, bind_hybrid
 from .constants import DTYPE_BF16, DTYPE_F16, DTYPE_F32, PA_WINDOW_MAX_HEAD_SIZE as PA_WINDOW_MAX_HEAD, PARTITION_SIZE
 
 logger = logging.getLogger(__name__)
@@ -77,6 +78,7 @@ class PagedAttnArgs(ctypes.Structure):
         ("softcap", ctypes.c_float),
         ("out_dtype", ctypes.c_int32),
         ("window_seqlen_q", ctypes.c_int32),
+        ("wide_weights", ctypes.c_int32),
     ]
 
 
@@ -127,6 +129,7 @@ EXPORTED_SYMBOLS = (
     "b200_allreduce_add_rmsnorm",
     "b200_allreduce_add_rmsnorm_push",
     "b200_argmax_vocab_parallel",
+    *HYBRID_SYMBOLS,
 )
 
 
@@ -134,6 +137,36 @@ def library_path() -> str:
     from .build import output_path
 
     return str(output_path())
+
+
+class _Missing:
+    """A symbol that a component library does not hold: binding it is fine, calling it is not."""
+
+    def __init__(self, name: str, path: str) -> None:
+        self._name, self._path = name, path
+
+    def __call__(self, *args):
+        raise RuntimeError(f"{self._path} holds no {self._name}: build the full library with "
+                           f"`python -m vllm_metal_b200.metal.build`")
+
+
+class _Library(ctypes.CDLL):
+    def __getattr__(self, name: str):
+        try:
+            return super().__getattr__(name)
+        except AttributeError:
+            if not name.startswith("b200_"):
+                raise
+            missing = _Missing(name, self._name)
+            setattr(self, name, missing)
+            return missing
+
+
+def _component_library():
+    """A fresh component library, if one was built (``metal.build.ensure``)."""
+    from .build import COMPONENTS, output_path, stale_artifacts
+
+    return next((output_path(c) for c in COMPONENTS if not stale_artifacts(c)), None)
 
 
 def load_library() -> ctypes.CDLL:
@@ -149,20 +182,23 @@ def load_library() -> ctypes.CDLL:
         from pathlib import Path
 
         so = Path(override)
+    component = None if override or not stale_artifacts() else _component_library()
+    if component is not None:
+        so = component
     if not so.exists():
         raise RuntimeError(
             f"Prebuilt native extension not found at {so}. Run "
             f"`python -m vllm_metal_b200.metal.build` (needs nvcc) or set "
             f"VLLM_METAL_BUILD_FROM_SOURCE=1; there is no CPU fallback."
         )
-    stale = [] if override else stale_artifacts()
+    stale = [] if override or component is not None else stale_artifacts()
     if stale:
         raise RuntimeError(
             f"Prebuilt CUDA artifacts are stale vs the current sources "
             f"({', '.join(p.name for p in stale)}): a kernel source was edited without "
             f"rebuilding. Run `python -m vllm_metal_b200.metal.build`."
         )
-    lib = ctypes.CDLL(str(so))
+    lib = _Library(str(so))
     lib.b200_last_error.restype = ctypes.c_char_p
     lib.b200_paged_attention_workspace_bytes.restype = ctypes.c_size_t
     lib.b200_paged_attention_workspace_bytes.argtypes = [ctypes.POINTER(PagedAttnArgs)]
@@ -195,6 +231,7 @@ def load_library() -> ctypes.CDLL:
     lib.b200_argmax.argtypes = [vp, vp, i32, i32, i64, i32, vp]
     lib.b200_add_inplace.argtypes = [vp, vp, i32, i32, i64, i64, i32, vp]
     lib.b200_advance_decode.argtypes = [vp, vp, vp, vp, vp, vp, i32, i32, i32, vp]
+    bind_hybrid(lib)
     if lib.b200_partition_size() != PARTITION_SIZE:
         raise RuntimeError("PARTITION_SIZE mismatch between constants.py and the library")
     return lib
@@ -224,7 +261,7 @@ def _dtype_code(name: str, t: torch.Tensor) -> int:
         raise RuntimeError(f"{name}: unsupported dtype {t.dtype}; expected float32/float16/bfloat16") from None
 
 
-class _Ops:
+class _Ops(HybridOps):
     """The operator object ``get_ops()`` returns (reference: module ``_paged_ops``)."""
 
     PARTITION_SIZE = PARTITION_SIZE
@@ -342,13 +379,15 @@ class _Ops:
         window_seqlen_q: int = 1,
         sinks: torch.Tensor | None = None,
         *,
+        wide_weights: bool = False,
         _force_partitions: int = 0,
         _kernel: int = 0,
     ) -> None:
         """Unified paged varlen attention; fills ``out`` in place.
 
         Same positional/keyword surface as the reference binding.  TurboQuant KV
-        compression is out of scope for this build and raises.
+        compression is out of scope for this build and raises.  ``wide_weights``: the prefill
+        tile kernel keeps 16 instead of 8 significant bits of the softmax weights in the value product.
         """
         if use_turboquant or key_scale_cache is not None or value_scale_cache is not None:
             if sinks is not None:
@@ -461,6 +500,7 @@ class _Ops:
         a.scale, a.softcap = float(scale), float(softcap)
         a.out_dtype = _dtype_code("out", out)
         a.window_seqlen_q = int(window_seqlen_q)
+        a.wide_weights = int(bool(wide_weights))
         need = self._lib.b200_paged_attention_workspace_bytes(ctypes.byref(a))
         ws = self._workspace(query.device, need)
         a.workspace = _ptr(ws)

@@ -22,6 +22,13 @@ CSRC_DIR = _PKG_DIR / "csrc"
 INCLUDE_DIR = _PKG_DIR.parent / "include"
 LIB_NAME = "lib_b200_paged_ops.so"
 
+# Parts of the library that stand on their own: a model family that needs no more than such a part can be built and
+# served without compiling the rest (a first call in a fresh checkout).
+COMPONENTS: dict[str, tuple[str, ...]] = {
+    "hybrid": ("c_abi", "decoder_ops", "hybrid_ops", "latent_attention", "latent_ops", "paged_attention_decode",
+               "paged_attention_generic", "paged_attention_prefill", "recurrence"),
+}
+
 NVCC_FLAGS = [
     "-gencode",
     "arch=compute_100a,code=sm_100a",
@@ -37,21 +44,24 @@ NVCC_FLAGS = [
 ]
 
 
-def output_path() -> Path:
-    return _PKG_DIR / LIB_NAME
+def output_path(component: str | None = None) -> Path:
+    return _PKG_DIR / (LIB_NAME if component is None else f"lib_b200_{component}_ops.so")
 
 
-def stamp_path() -> Path:
-    return _PKG_DIR / (LIB_NAME + ".stamp")
+def stamp_path(component: str | None = None) -> Path:
+    out = output_path(component)
+    return out.with_name(out.name + ".stamp")
 
 
-def sources() -> list[Path]:
+def sources(component: str | None = None) -> list[Path]:
+    if component is not None:
+        return [CSRC_DIR / f"{name}.cu" for name in COMPONENTS[component]]
     return sorted(CSRC_DIR.glob("*.cu"))
 
 
-def source_hash() -> str:
+def source_hash(component: str | None = None) -> str:
     h = hashlib.sha256()
-    files = sorted(list(CSRC_DIR.glob("*.cu")) + list(CSRC_DIR.glob("*.cuh")) + list(INCLUDE_DIR.glob("*.h")))
+    files = sorted(sources(component) + list(CSRC_DIR.glob("*.cuh")) + list(INCLUDE_DIR.glob("*.h")))
     for f in files:
         h.update(f.name.encode())
         h.update(f.read_bytes())
@@ -59,14 +69,15 @@ def source_hash() -> str:
     return h.hexdigest()
 
 
-def stale_artifacts() -> list[Path]:
+def stale_artifacts(component: str | None = None) -> list[Path]:
     """Artifacts whose stamp no longer matches the sources (empty if no sources
     are present, e.g. on a box that only received the built library)."""
-    if not output_path().exists():
-        return [output_path()]
-    if not stamp_path().exists() or not CSRC_DIR.exists():
+    out, stamp = output_path(component), stamp_path(component)
+    if not out.exists():
+        return [out]
+    if not stamp.exists() or not CSRC_DIR.exists():
         return []
-    return [] if stamp_path().read_text().strip() == source_hash() else [output_path()]
+    return [] if stamp.read_text().strip() == source_hash(component) else [out]
 
 
 def find_nvcc() -> str:
@@ -85,13 +96,20 @@ def _file_hash(src: Path, extra: list[str]) -> str:
     return h.hexdigest()
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every ``csrc/*.cu`` to an object (in parallel, cached by content hash under
-    ``build/``) and link them into the one shared library."""
+def ensure(component: str) -> Path:
+    """The full library if it is there and fresh, else the component's, compiled now if need be."""
+    if not stale_artifacts():
+        return output_path()
+    return build(component=component)
+
+
+def build(force: bool = False, verbose: bool = False, component: str | None = None) -> Path:
+    """Compile every ``csrc/*.cu`` (or a component's) to an object (in parallel, cached by content hash under
+    ``build/``) and link them into one shared library."""
     from concurrent.futures import ThreadPoolExecutor
 
-    out = output_path()
-    if not force and out.exists() and not stale_artifacts():
+    out = output_path(component)
+    if not force and out.exists() and not stale_artifacts(component):
         return out
     extra = os.environ.get("B200_NVCC_EXTRA", "").split()  # tuning experiments (-DQGEMM_...), not for shipping
     nvcc = find_nvcc()
@@ -115,7 +133,7 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         return obj
 
     with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 1)) as ex:
-        objs = list(ex.map(compile_one, sources()))
+        objs = list(ex.map(compile_one, sources(component)))
     cmd = [nvcc, "--shared", "-o", str(out), *[str(o) for o in objs]]
     proc = subprocess.run(cmd, capture_output=True, text=True)
     logs.append(" ".join(cmd) + "\n" + proc.stdout + proc.stderr)
@@ -124,7 +142,7 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         raise RuntimeError(f"link failed ({proc.returncode}):\n{(proc.stdout + proc.stderr)[-4000:]}")
     if verbose:
         print("\n".join(logs))
-    stamp_path().write_text(source_hash() + "\n")
+    stamp_path(component).write_text(source_hash(component) + "\n")
     return out
 
 

@@ -1,0 +1,312 @@
+"""Operator surface of ``include/b200_hybrid_ops.h``: the mixers of hybrid decoders (latent attention, gated linear
+recurrences) and the norms / gates either side of them.  ``HybridOps`` is mixed into the object ``get_ops()`` returns;
+like there, a CPU tensor or an unsupported size raises and nothing falls back."""
+
+from __future__ import annotations
+
+import ctypes
+
+import torch
+
+from .constants import DTYPE_BF16, DTYPE_F16, DTYPE_F32
+
+_DTYPE = {torch.float32: DTYPE_F32, torch.float16: DTYPE_F16, torch.bfloat16: DTYPE_BF16}
+_P, _I, _L, _F, _Z = ctypes.c_void_p, ctypes.c_int32, ctypes.c_int64, ctypes.c_float, ctypes.c_size_t
+
+HYBRID_SYMBOLS = (
+    "b200_embed_rows",
+    "b200_stream_norm",
+    "b200_mixer_finish",
+    "b200_causal_conv",
+    "b200_recurrence",
+    "b200_recurrence_workspace_bytes",
+    "b200_recurrence_can_chunk",
+    "b200_recurrence_num_launches",
+    "b200_latent_prep",
+    "b200_head_linear",
+    "b200_latent_attention",
+    "b200_latent_attention_workspace_bytes",
+    "b200_latent_attention_num_launches",
+    "b200_latent_gather",
+)
+
+RECURRENCE_CHUNK = 64
+RECURRENCE_TILE_V = 64
+
+
+def _struct(name: str, doc: str, **fields):
+    flat = []
+    for ctype, names in fields.items():
+        flat += [(n, {"P": _P, "I": _I, "L": _L, "F": _F, "Z": _Z}[ctype[0]]) for n in names.split()]
+    return type(name, (ctypes.Structure,), {"_fields_": flat, "__doc__": doc})
+
+
+MixerFinishArgs = _struct(
+    "MixerFinishArgs", "b200_mixer_finish_args",
+    P="y pre_gate post_gate weight act_in out",
+    L="y_stride pre_stride post_stride act_stride out_stride",
+    I="rows inner group_size act_dim act_offset out_cols y_head_dim y_head_stride",
+    F="eps", I2="dtype")
+RecurrenceArgs = _struct(
+    "RecurrenceArgs", "b200_recurrence_args",
+    P="q k v gate_a gate_b bias_a bias_b rate skip state norm_state max_state cu_seqlens seq_lens slots chunk_seq "
+      "chunk_row seq_chunk0 out workspace",
+    Z="workspace_bytes",
+    L="q_stride k_stride v_stride gate_stride out_stride",
+    I="kind dtype num_tokens num_seqs num_heads num_groups key_dim value_dim num_chunks seq_limit",
+    F="q_scale gate_cap")
+LatentPrepArgs = _struct(
+    "LatentPrepArgs", "b200_latent_prep_args",
+    P="q down norm_weight positions slot_mapping inv_freq cache q_out",
+    L="q_stride down_stride q_out_stride num_slots",
+    I="num_tokens heads dim rot_dim rot_dims kv_rank q_cols rot_offset copy_nope",
+    F="eps", I2="dtype")
+HeadLinearArgs = _struct(
+    "HeadLinearArgs", "b200_head_linear_args",
+    P="x w gate y", L="x_stride x_head_stride y_stride y_head_stride gate_stride", I="rows heads n k dtype")
+LatentAttnArgs = _struct(
+    "LatentAttnArgs", "b200_latent_attn_args",
+    P="q cache block_tables seq_lens cu_seqlens out workspace", Z="workspace_bytes",
+    L="q_stride out_stride num_slots",
+    I="num_tokens num_seqs heads kv_rank rot_dim block_size max_blocks_per_seq max_seq_len window max_q_len dtype "
+      "kernel force_splits",
+    F="scale")
+
+
+def bind_hybrid(lib: ctypes.CDLL) -> None:
+    vp, i32, i64, f32 = ctypes.c_void_p, ctypes.c_int, ctypes.c_int64, ctypes.c_float
+    lib.b200_embed_rows.argtypes = [vp, vp, vp, i32, i32, i32, i64, i32, vp]
+    lib.b200_stream_norm.argtypes = [vp, vp, vp, vp, i32, i32, i64, i64, f32, f32, i32, vp]
+    lib.b200_causal_conv.argtypes = [vp] * 8 + [i32, i32, i32, i32, i64, i64, i32, i32, vp]
+    lib.b200_latent_gather.argtypes = [vp] * 6 + [i32, i32, i32, i32, i32, i64, i32, i32, vp]
+    for name, struct in (("mixer_finish", MixerFinishArgs), ("recurrence", RecurrenceArgs),
+                         ("latent_prep", LatentPrepArgs), ("head_linear", HeadLinearArgs),
+                         ("latent_attention", LatentAttnArgs)):
+        getattr(lib, "b200_" + name).argtypes = [ctypes.POINTER(struct), vp]
+    for name, struct in (("recurrence", RecurrenceArgs), ("latent_attention", LatentAttnArgs)):
+        getattr(lib, f"b200_{name}_workspace_bytes").argtypes = [ctypes.POINTER(struct)]
+        getattr(lib, f"b200_{name}_workspace_bytes").restype = ctypes.c_size_t
+        getattr(lib, f"b200_{name}_num_launches").argtypes = [ctypes.POINTER(struct)]
+    lib.b200_recurrence_can_chunk.argtypes = [ctypes.POINTER(RecurrenceArgs)]
+
+
+def _rows(name: str, t: torch.Tensor, dtype: torch.dtype | None = None) -> torch.Tensor:
+    if not t.is_cuda:
+        raise RuntimeError(f"{name} must live on a CUDA device; this path has no CPU implementation")
+    if t.dim() != 2 or t.stride(1) != 1:
+        raise ValueError(f"{name} must be [rows, columns] with unit column stride, got {tuple(t.shape)}")
+    if dtype is not None and t.dtype != dtype:
+        raise ValueError(f"{name} must be {dtype}, got {t.dtype}")
+    return t
+
+
+def _f32(name: str, t: torch.Tensor | None, n: int) -> int | None:
+    if t is None:
+        return None
+    if not t.is_cuda or t.dtype != torch.float32 or not t.is_contiguous() or t.numel() != n:
+        raise ValueError(f"{name} must be {n} contiguous float32 values on the device, got {tuple(t.shape)} {t.dtype}")
+    return t.data_ptr()
+
+
+def _stream() -> int:
+    return torch.cuda.current_stream().cuda_stream
+
+
+class HybridOps:
+    """Methods over ``self._lib`` / ``self._check`` / ``self._workspace`` / ``self.launches`` of the operator object."""
+
+    def embed_rows(self, ids: torch.Tensor, table: torch.Tensor) -> torch.Tensor:
+        """Rows of ``table`` as an fp32 residual stream ``[T, dim]``."""
+        _rows("table", table)
+        if ids.dtype != torch.int32 or not table.is_contiguous():
+            raise ValueError("embed_rows takes int32 ids and a contiguous table")
+        out = torch.empty((ids.shape[0], table.shape[1]), dtype=torch.float32, device=table.device)
+        self._check(self._lib.b200_embed_rows(ids.data_ptr(), table.data_ptr(), out.data_ptr(), ids.shape[0],
+                                              table.shape[0], table.shape[1], out.stride(0), _DTYPE[table.dtype],
+                                              _stream()))
+        self.launches += 1
+        return out
+
+    def stream_norm(self, x, weight, eps: float, weight_offset: float, out_dtype, rows=None) -> torch.Tensor:
+        """RMS norm of the fp32 stream (or of the rows listed in int64 ``rows``)."""
+        _rows("x", x, torch.float32)
+        if rows is not None and (rows.dtype != torch.int64 or not rows.is_cuda):
+            raise ValueError("rows must be int64 on the device")
+        n = x.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n, x.shape[1]), dtype=out_dtype, device=x.device)
+        self._check(self._lib.b200_stream_norm(
+            x.data_ptr(), None if rows is None else rows.data_ptr(), _f32("weight", weight, x.shape[1]), out.data_ptr(),
+            n, x.shape[1], x.stride(0), out.stride(0), float(eps), float(weight_offset), _DTYPE[out_dtype], _stream()))
+        self.launches += 1
+        return out
+
+    def mixer_finish(self, out, inner: int, act_in=None, act_offset: int = 0, y=None, pre_gate=None, post_gate=None,
+                     weight=None, group_size: int = 0, eps: float = 0.0, y_head_dim: int = 0,
+                     y_head_stride: int = 0) -> None:
+        """Gate -> group norm -> gate into ``out[:, :inner]`` and gelu into ``out[:, act_offset:]``, one launch; ``y``
+        may be given per head with padding (``y_head_dim`` used of every ``y_head_stride`` columns)."""
+        _rows("out", out)
+        a = MixerFinishArgs()
+        for name, t in (("y", y), ("pre_gate", pre_gate), ("post_gate", post_gate), ("act_in", act_in)):
+            if t is not None:
+                _rows(name, t, out.dtype)
+                if t.shape[0] != out.shape[0]:
+                    raise ValueError(f"{name} has {t.shape[0]} rows, out {out.shape[0]}")
+                setattr(a, name, t.data_ptr())
+        a.y_stride = 0 if y is None else y.stride(0)
+        a.pre_stride = 0 if pre_gate is None else pre_gate.stride(0)
+        a.post_stride = 0 if post_gate is None else post_gate.stride(0)
+        a.act_stride = 0 if act_in is None else act_in.stride(0)
+        a.weight = _f32("weight", weight, inner)
+        a.out, a.out_stride, a.out_cols, a.rows = out.data_ptr(), out.stride(0), out.shape[1], out.shape[0]
+        a.inner, a.group_size, a.eps, a.dtype = inner, group_size, float(eps), _DTYPE[out.dtype]
+        a.act_dim, a.act_offset = (0 if act_in is None else act_in.shape[1]), act_offset
+        a.y_head_dim, a.y_head_stride = y_head_dim, y_head_stride
+        self._check(self._lib.b200_mixer_finish(ctypes.byref(a), _stream()))
+        self.launches += 1
+
+    def causal_conv(self, x, weight, bias, state, seg, silu: bool = True) -> torch.Tensor:
+        """Depthwise causal convolution of ``x [T, C]`` over the segments of ``seg`` (carried inputs in
+        ``state [slots, taps-1, C]``); ``weight`` fp32 ``[taps, C]``, ``bias`` fp32 ``[C]``."""
+        _rows("x", x)
+        taps, ch = weight.shape
+        if x.shape[1] != ch or state.dtype != x.dtype or tuple(state.shape[1:]) != (taps - 1, ch):
+            raise ValueError("causal_conv: x, weight and state disagree")
+        out = torch.empty((x.shape[0], ch), dtype=x.dtype, device=x.device)
+        self._check(self._lib.b200_causal_conv(
+            x.data_ptr(), _f32("weight", weight, taps * ch), _f32("bias", bias, ch),
+            state.data_ptr() if state.numel() else None, seg.cu_seqlens_q.data_ptr(), seg.seq_lens.data_ptr(),
+            seg.state_slots.data_ptr(), out.data_ptr(), seg.cu_seqlens_q.shape[0] - 1, seg.max_q_len, ch, taps,
+            x.stride(0), out.stride(0), int(silu), _DTYPE[x.dtype], _stream()))
+        self.launches += 1
+        return out
+
+    def recurrence(self, kind: str, q, k, v, gate_a, gate_b, seg, state, *, heads: int, groups: int, key_dim: int,
+                   value_dim: int, bias_a, bias_b=None, rate=None, skip=None, norm_state=None, max_state=None,
+                   q_scale: float = 1.0, gate_cap: float = 0.0, force_sequential: bool = False) -> torch.Tensor:
+        """Gated linear recurrence (``kind`` "ssd" / "mlstm") over the segments of ``seg``: outputs ``[T, heads *
+        value_dim]``, the slots' fp32 states updated in place.  Segments longer than ``seg.chunk_limit`` rows run in
+        chunks on tensor cores where type and sizes allow."""
+        a = RecurrenceArgs()
+        for name, t in (("q", q), ("k", k), ("v", v), ("gate_a", gate_a), ("gate_b", gate_b)):
+            if t is not None:
+                _rows(name, t, v.dtype)
+                setattr(a, name, t.data_ptr())
+        if gate_b is not None and gate_b.stride(0) != gate_a.stride(0):
+            raise ValueError("both gates must share one row stride")
+        if q.shape[1] != groups * key_dim or v.shape[1] != heads * value_dim:
+            raise ValueError("recurrence: q / k / v columns do not match the heads")
+        slots = state.shape[0]
+        if tuple(state.shape) != (slots, heads, key_dim, value_dim):
+            raise ValueError(f"state must be [slots, {heads}, {key_dim}, {value_dim}], got {tuple(state.shape)}")
+        tiles = -(-value_dim // RECURRENCE_TILE_V)
+        a.bias_a, a.bias_b = _f32("bias_a", bias_a, heads), _f32("bias_b", bias_b, heads)
+        a.rate, a.skip = _f32("rate", rate, heads), _f32("skip", skip, heads)
+        a.state = _f32("state", state, state.numel())
+        a.norm_state = _f32("norm_state", norm_state, slots * heads * tiles * key_dim)
+        a.max_state = _f32("max_state", max_state, slots * heads * tiles)
+        a.cu_seqlens, a.seq_lens = seg.cu_seqlens_q.data_ptr(), seg.seq_lens.data_ptr()
+        a.slots = seg.state_slots.data_ptr()
+        out = torch.empty((v.shape[0], heads * value_dim), dtype=v.dtype, device=v.device)
+        a.out, a.out_stride = out.data_ptr(), out.stride(0)
+        a.q_stride, a.k_stride, a.v_stride, a.gate_stride = q.stride(0), k.stride(0), v.stride(0), gate_a.stride(0)
+        a.kind, a.dtype = {"ssd": 0, "mlstm": 1}[kind], _DTYPE[v.dtype]
+        a.num_tokens, a.num_seqs = v.shape[0], seg.cu_seqlens_q.shape[0] - 1
+        a.num_heads, a.num_groups, a.key_dim, a.value_dim = heads, groups, key_dim, value_dim
+        a.q_scale, a.gate_cap = float(q_scale), float(gate_cap)
+        a.seq_limit = 0x7FFFFFFF
+        if seg.num_chunks > 0 and not force_sequential and self._lib.b200_recurrence_can_chunk(ctypes.byref(a)):
+            a.num_chunks = seg.num_chunks
+            # the sequential launch only exists for the segments that need it
+            a.seq_limit = seg.chunk_limit if seg.has_short else 0
+            a.chunk_seq, a.chunk_row = seg.chunk_seq.data_ptr(), seg.chunk_row.data_ptr()
+            a.seq_chunk0 = seg.seq_chunk0.data_ptr()
+            need = self._lib.b200_recurrence_workspace_bytes(ctypes.byref(a))
+            ws = self._workspace(v.device, need)
+            a.workspace, a.workspace_bytes = ws.data_ptr(), ws.numel()
+        self._check(self._lib.b200_recurrence(ctypes.byref(a), _stream()))
+        self.launches += self._lib.b200_recurrence_num_launches(ctypes.byref(a))
+        return out
+
+    def latent_prep(self, q, down, norm_weight, positions, slot_mapping, inv_freq, cache, q_out, *, heads: int, dim: int,
+                    rot_dim: int, kv_rank: int, eps: float, rot_offset: int, copy_nope: bool) -> None:
+        """Latent norm + rotation + cache write (``cache [slots, kv_rank + rot_dim]``), and the queries' rotated (with
+        ``copy_nope`` also the unrotated) parts into ``q_out [T, heads, columns]``."""
+        t = q.shape[0]
+        for name, x in (("q", q), ("down", down), ("cache", cache)):
+            _rows(name, x, q_out.dtype)
+        if not cache.is_contiguous() or cache.shape[1] != kv_rank + rot_dim or down.shape != (t, kv_rank + rot_dim):
+            raise ValueError(f"cache and down must have {kv_rank + rot_dim} columns")
+        if not q_out.is_contiguous() or q_out.shape[:2] != (t, heads) or q.shape[1] != heads * (dim + rot_dim):
+            raise ValueError("q must be [T, heads * (dim + rot_dim)] and q_out contiguous [T, heads, columns]")
+        if positions.dtype != torch.int32 or slot_mapping.dtype != torch.int64 or \
+                positions.shape != (t,) or slot_mapping.shape != (t,):
+            raise ValueError("positions must be int32 [T] and slot_mapping int64 [T]")
+        a = LatentPrepArgs()
+        a.q, a.down, a.cache, a.q_out = q.data_ptr(), down.data_ptr(), cache.data_ptr(), q_out.data_ptr()
+        a.norm_weight = _f32("norm_weight", norm_weight, kv_rank)
+        a.positions, a.slot_mapping = positions.data_ptr(), slot_mapping.data_ptr()
+        a.inv_freq = _f32("inv_freq", inv_freq, inv_freq.numel()) if inv_freq.numel() else None
+        a.rot_dims = 2 * inv_freq.numel()
+        a.q_stride, a.down_stride, a.num_slots = q.stride(0), down.stride(0), cache.shape[0]
+        a.q_out_stride, a.q_cols = q_out.stride(0), q_out.shape[2]
+        a.num_tokens, a.heads, a.dim, a.rot_dim, a.kv_rank = t, heads, dim, rot_dim, kv_rank
+        a.rot_offset, a.copy_nope = rot_offset, int(copy_nope)
+        a.eps, a.dtype = float(eps), _DTYPE[q.dtype]
+        self._check(self._lib.b200_latent_prep(ctypes.byref(a), _stream()))
+        self.launches += 1
+
+    def head_linear(self, x, w, y, gate=None) -> None:
+        """``y[t, h] = w[h] x[t, h]`` (``w [H, n, k]``), times ``sigmoid(gate[t, h * n + i])``; ``x`` / ``y`` are
+        ``[T, H, k]`` / ``[T, H, n]`` views with unit inner stride."""
+        h, n, k = w.shape
+        if x.shape[1:] != (h, k) or y.shape != (x.shape[0], h, n) or x.stride(2) != 1 or y.stride(2) != 1:
+            raise ValueError("head_linear: x [T, H, k], w [H, n, k] and y [T, H, n] disagree")
+        if not (x.dtype == w.dtype == y.dtype) or not w.is_contiguous() or not w.is_cuda:
+            raise ValueError("head_linear: one dtype and a contiguous w on the device")
+        a = HeadLinearArgs()
+        a.x, a.w, a.y = x.data_ptr(), w.data_ptr(), y.data_ptr()
+        if gate is not None:
+            _rows("gate", gate, x.dtype)
+            a.gate, a.gate_stride = gate.data_ptr(), gate.stride(0)
+        a.x_stride, a.x_head_stride, a.y_stride, a.y_head_stride = x.stride(0), x.stride(1), y.stride(0), y.stride(1)
+        a.rows, a.heads, a.n, a.k, a.dtype = x.shape[0], h, n, k, _DTYPE[x.dtype]
+        self._check(self._lib.b200_head_linear(ctypes.byref(a), _stream()))
+        self.launches += 1
+
+    def latent_attention(self, q, cache, meta, scale: float, window: int, kv_rank: int, max_q_len: int,
+                         num_seqs: int | None = None, *, kernel: int = 0, force_splits: int = 0) -> torch.Tensor:
+        """Attention of ``q [T, H, kv_rank + rot]`` over the paged latent rows; returns ``[T, H, kv_rank]``.  The
+        first ``num_seqs`` segments of ``meta`` cover q's rows; ``window <= 0``: causal only.  ``kernel``: 0 auto,
+        1 any-size, 2 tensor cores (raises where it does not apply)."""
+        t, heads, width = q.shape
+        if not q.is_contiguous() or not q.is_cuda or cache.dtype != q.dtype or cache.shape[1] != width:
+            raise ValueError("latent_attention: q must be contiguous and match the cache rows")
+        out = torch.empty((t, heads, kv_rank), dtype=q.dtype, device=q.device)
+        a = LatentAttnArgs()
+        a.q, a.cache, a.out = q.data_ptr(), cache.data_ptr(), out.data_ptr()
+        a.block_tables, a.seq_lens = meta.block_tables.data_ptr(), meta.seq_lens.data_ptr()
+        a.cu_seqlens = meta.cu_seqlens_q.data_ptr()
+        a.q_stride, a.out_stride, a.num_slots = q.stride(0), out.stride(0), cache.shape[0]
+        a.num_tokens, a.num_seqs = t, meta.seq_lens.shape[0] if num_seqs is None else num_seqs
+        a.heads, a.kv_rank, a.rot_dim = heads, kv_rank, width - kv_rank
+        a.block_size, a.max_blocks_per_seq = meta.block_size, max(1, meta.block_tables.stride(0))
+        a.max_seq_len, a.window, a.max_q_len = meta.max_seq_len, window, max_q_len
+        a.dtype, a.kernel, a.force_splits, a.scale = _DTYPE[q.dtype], kernel, force_splits, float(scale)
+        need = self._lib.b200_latent_attention_workspace_bytes(ctypes.byref(a))
+        ws = self._workspace(q.device, need)
+        a.workspace, a.workspace_bytes = (None, 0) if ws is None else (ws.data_ptr(), ws.numel())
+        self._check(self._lib.b200_latent_attention(ctypes.byref(a), _stream()))
+        self.launches += self._lib.b200_latent_attention_num_launches(ctypes.byref(a))
+        return out
+
+    def latent_gather(self, cache, block_tables, first, count, out_row, out, max_count: int, block_size: int,
+                      pad: int) -> None:
+        """Cached rows ``first .. first + count`` of every request into consecutive rows of ``out``; the rows up
+        to the next multiple of ``pad`` are zeroed."""
+        _rows("cache", cache)
+        self._check(self._lib.b200_latent_gather(
+            cache.data_ptr(), block_tables.data_ptr(), first.data_ptr(), count.data_ptr(), out_row.data_ptr(),
+            out.data_ptr(), first.shape[0], max_count, cache.shape[1], block_size, max(1, block_tables.stride(0)),
+            cache.shape[0], pad, _DTYPE[cache.dtype], _stream()))
+        self.launches += 1

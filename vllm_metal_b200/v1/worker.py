@@ -22,36 +22,11 @@ from vllm.v1.kv_cache_interface import FullAttentionSpec, KVCacheConfig, KVCache
 from vllm.v1.worker.worker_base import WorkerBase
 
 from ..attention.caches.kv_cache import B200PagedKVCache
-from ..lm.decoder import PRESETS, Model, ModelArgs
+from ..lm.decoder import Model
+from ..lm.registry import FAMILIES, HybridFamily, model_args_from_hf_config
 from .model_runner import PagedModelRunner
 
 logger = logging.getLogger(__name__)
-
-
-def model_args_from_hf_config(hf_config: Any, quant: dict | None = None) -> ModelArgs:
-    """Map a HF/mlx-lm ``config.json`` onto the decoder's ``ModelArgs`` (weights themselves are
-    loaded or random-initialised by ``Model``).  ``quant`` is the ``quantization`` dict."""
-    import dataclasses
-
-    q = quant or getattr(hf_config, "quantization", None) or {}
-    n_heads = int(hf_config.num_attention_heads)
-    hidden = int(hf_config.hidden_size)
-    fields = dict(
-        num_layers=int(hf_config.num_hidden_layers), hidden=hidden, n_heads=n_heads,
-        n_kv_heads=int(getattr(hf_config, "num_key_value_heads", n_heads)),
-        head_dim=int(getattr(hf_config, "head_dim", None) or hidden // n_heads),
-        intermediate=int(hf_config.intermediate_size), vocab=int(hf_config.vocab_size),
-        rms_eps=float(getattr(hf_config, "rms_norm_eps", 1e-6)),
-        rope_base=float(getattr(hf_config, "rope_theta", 10000.0)),
-        tie_embeddings=bool(getattr(hf_config, "tie_word_embeddings", False)),
-        qk_norm=str(getattr(hf_config, "model_type", "")).startswith("qwen3"),
-        sliding_window=int(getattr(hf_config, "sliding_window", None) or -1),
-        layer_types=list(getattr(hf_config, "layer_types", None) or []),
-        name=str(getattr(hf_config, "model_type", "hf")),
-        bits=int(q.get("bits", 4)), group_size=int(q.get("group_size", 64)),
-    )
-    known = {f.name for f in dataclasses.fields(ModelArgs)}
-    return dataclasses.replace(PRESETS["tiny"], **{k: v for k, v in fields.items() if k in known})
 
 
 class _RequestState:
