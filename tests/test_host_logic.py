@@ -174,8 +174,8 @@ def test_library_exports_every_declared_symbol():
 
 
 def test_args_struct_matches_header_layout():
-    # 10 pointers/size_t + 12 int32 + 6 int64 + 2 float + 2 int32 (out_dtype, window_seqlen_q)
-    assert ctypes.sizeof(PagedAttnArgs) == 10 * 8 + 12 * 4 + 6 * 8 + 2 * 4 + 4 + 4
+    # 10 pointers/size_t + 12 int32 + 6 int64 + 2 float + 3 int32 (out_dtype, window_seqlen_q, wide_weights), padded to 8
+    assert ctypes.sizeof(PagedAttnArgs) == 10 * 8 + 12 * 4 + 6 * 8 + 2 * 4 + 4 * 4
     assert PagedAttnArgs.out_dtype.offset == 10 * 8 + 12 * 4 + 6 * 8 + 2 * 4
     assert PagedAttnArgs.window_seqlen_q.offset == PagedAttnArgs.out_dtype.offset + 4
     assert PagedAttnArgs.q_stride.offset == 10 * 8 + 12 * 4

@@ -84,6 +84,8 @@ class HybridModel:
             layer.add_to(x, self.args, meta, cache, i)
             if self.residual_hook is not None:
                 self.residual_hook(i, x)
+        if logits_rows is not None and logits_rows.shape[0] == 0:
+            return torch.empty((0, self.args.vocab), dtype=torch.float32, device=self.device)
         x = get_ops().stream_norm(x, self.final_norm, self.args.eps, 1.0, self.dtype, rows=logits_rows)
         return self.head(x)
 
