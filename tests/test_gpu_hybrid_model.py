@@ -1,0 +1,395 @@
+"""Hybrid decoders on the device, whole: norms, gates and activations, then the model through the engine's step against
+the whole-sequence oracle -- portions, batches, reused pages and slots, windows, long decoding, generation."""
+
+from __future__ import annotations
+
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+from oracle import hybrid as oracle
+
+from .hybrid_helpers import (LATENT, MAMBA2, MLSTM, default_config, layer, make_config, make_engine, random_checkpoint,
+                             shared, to_oracle, write_folder)
+
+pytestmark = pytest.mark.gpu
+
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+BOTH = pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+
+
+# -- element-wise mechanisms ---------------------------------------------------------------------------------
+
+@BOTH
+@pytest.mark.parametrize("dim", [1, 30, 88, 4096, 5000])
+def test_stream_norm_with_weights_around_zero(ops, dtype, dim):
+    g = torch.Generator().manual_seed(dim)
+    x, w = torch.randn((9, dim), generator=g), torch.randn(dim, generator=g) * 0.3
+    for rows in (None, torch.tensor([7, 0, 3])):
+        got = ops.stream_norm(x.cuda(), w.cuda(), 1e-3, 1.0, dtype, rows=None if rows is None else rows.cuda())
+        want = oracle.rms_norm_zero_centred((x if rows is None else x[rows]).double().numpy(), w.double().numpy(), 1e-3)
+        tol = 1e-5 if dtype == torch.float32 else 8e-3
+        np.testing.assert_allclose(got.double().cpu().numpy(), want, atol=tol, rtol=tol)
+
+
+@BOTH
+def test_embedding_rows_widen_exactly(ops, dtype):
+    table = torch.randn((50, 37)).to(dtype).cuda()
+    ids = torch.tensor([0, 49, 7, 7], dtype=torch.int32, device="cuda")
+    assert torch.equal(ops.embed_rows(ids, table), table[ids.long()].float())
+
+
+@BOTH
+@pytest.mark.parametrize("inner,group", [(96, 24), (1200, 600), (40, 40), (2304, 2304), (9000, 4500), (35, 7)])
+def test_gate_norm_gate_and_activation(ops, dtype, inner, group):
+    rows, act = 5, 77
+    g = torch.Generator().manual_seed(inner)
+    y, z, p = (torch.randn((rows, inner), generator=g).to(dtype) for _ in range(3))
+    a = torch.randn((rows, act), generator=g).to(dtype)
+    w = torch.randn(inner, generator=g)
+    offset = -(-inner // 8) * 8
+    out = torch.full((rows, offset + 80), float("nan"), dtype=dtype, device="cuda")
+    ops.mixer_finish(out, inner, a.cuda(), offset, y=y.cuda(), pre_gate=z.cuda(), post_gate=p.cuda(), weight=w.cuda(),
+                     group_size=group, eps=1e-5)
+    d = lambda t: t.double().numpy()  # noqa: E731
+    v = (d(y) * oracle.silu(d(z))).reshape(rows, inner // group, group)
+    want = oracle.over_rms(v, 1e-5).reshape(rows, inner) * d(w) * oracle.sigmoid(d(p))
+    got = out.double().cpu().numpy()
+    tol = 2e-5 if dtype == torch.float32 else 1.5e-2
+    np.testing.assert_allclose(got[:, :inner], want, atol=tol, rtol=tol)
+    np.testing.assert_allclose(got[:, offset:offset + act], oracle.gelu_erf(d(a)), atol=tol, rtol=tol)
+    assert (got[:, inner:offset] == 0).all() and (got[:, offset + act:] == 0).all()
+
+
+# -- the model through the engine's step -----------------------------------------------------------------------
+
+def rounding_error(config, tensors, tokens, want):
+    """How far 16-bit rounding of every product's operands and result alone moves each position's logits: positions
+    where a head's output nearly vanishes before its norm are far more sensitive than others."""
+    def rounded(x):
+        return torch.from_numpy(np.ascontiguousarray(x)).bfloat16().double().numpy()
+
+    exact = oracle.linear
+    oracle.linear = lambda x, w: rounded(exact(rounded(x), w))
+    try:
+        got = oracle.forward(config, tensors, tokens)
+    finally:
+        oracle.linear = exact
+    return np.sqrt(((got - want) ** 2).mean(1)) / max(1.0, want.std())
+
+
+class Harness:
+    """Feeds whole token lists in portions and compares the logits of every position with the oracle's."""
+
+    def __init__(self, config, dtype, seed=0, scale=None, **kw):
+        self.config, self.dtype = config, dtype
+        self.tensors = random_checkpoint(config, seed)
+        if scale:
+            scale(self.tensors)
+        self.oracle_tensors = to_oracle(self.tensors)
+        self.engine = make_engine(config, self.tensors, dtype, **kw)
+        self.tokens, self.want, self.at, self.limit = {}, {}, {}, {}
+        self.positions = self.over = 0
+
+    def request(self, req_id, n, seed=0):
+        rng = np.random.default_rng(seed + 100)
+        self.tokens[req_id] = rng.integers(0, self.config["vocab"], n).tolist()
+        self.want[req_id] = oracle.forward(self.config, self.oracle_tensors, self.tokens[req_id])
+        self.at[req_id] = 0
+        self.limit[req_id] = np.full(n, 4e-5)
+        if self.dtype == torch.bfloat16:
+            self.limit[req_id] = 1.5e-2 + 3 * rounding_error(self.config, self.oracle_tensors, self.tokens[req_id],
+                                                             self.want[req_id])
+
+    def step(self, portions):
+        from vllm_metal_b200.v1.engine import StepEntry
+
+        entries, rows, limits = [], [], []
+        for req_id, n in portions.items():
+            lo = self.at[req_id]
+            n = min(n, len(self.tokens[req_id]) - lo)
+            if n <= 0:
+                continue
+            entries.append(StepEntry(req_id, self.tokens[req_id][lo:lo + n], range(n)))
+            rows.append(self.want[req_id][lo:lo + n])
+            limits.append(self.limit[req_id][lo:lo + n])
+            self.at[req_id] += n
+        got = self.engine.advance(entries).double().cpu().numpy()
+        want = np.concatenate(rows)
+        err = np.sqrt(((got - want) ** 2).mean(1)) / max(1.0, want.std())
+        ratio = err / np.concatenate(limits)
+        # a sensitive position may land on either side of its own estimate; a wrong key or state moves whole stretches
+        self.positions += len(ratio)
+        self.over += int((ratio > 1).sum())
+        allowed = 0 if self.dtype == torch.float32 else max(2, 0.02 * self.positions)
+        assert self.over <= allowed and ratio.max() <= 4, (portions, int(ratio.argmax()), float(ratio.max()), self.over)
+        for req_id in portions:
+            if self.at[req_id] == len(self.tokens[req_id]):
+                self.engine.finish(req_id)
+
+    def drain(self, req_id, portions):
+        i = 0
+        while self.at[req_id] < len(self.tokens[req_id]):
+            self.step({req_id: portions[i % len(portions)]})
+            i += 1
+
+
+def configs():
+    odd = [layer("mlstm", ff=19, heads=2, dim=11, vdim=13, gate_cap=3.5), layer("mamba2", ff=None, heads=3, groups=1, state=9,
+           vdim=7, conv=2, norm_groups=7), layer("latent_attention", ff=33, heads=3, dim=9, rot_dim=6, vdim=5, kv_rank=21,
+           rot={"base": 77.0, "dims": 6}, mask={"size": 11})]
+    wide = [layer("latent_attention", heads=2, dim=96, rot_dim=64, vdim=144, kv_rank=176, rot={"base": 1e5, "dims": 64},
+                  mask={"size": 200}), layer("mamba2", heads=2, groups=2, state=136, vdim=72, conv=5, norm_groups=1),
+            layer("mlstm", heads=2, dim=136, vdim=72, gate_cap=15.0)]
+    ones = [layer("mamba2", heads=1, groups=1, state=8, vdim=8, conv=1, norm_groups=1),
+            layer("latent_attention", heads=1, mask={"size": 1}), layer("mlstm", heads=1)]
+    open_mask = [layer("latent_attention", mask=None), layer("latent_attention", mask={"size": 300}, scale=0.5)]
+    return {"default": default_config(), "odd": make_config(odd, vocab=61, width=37, eps=1e-3),
+            "wide": make_config(wide, vocab=130, width=160), "ones": make_config(ones, vocab=33, width=24),
+            "open_mask": make_config(open_mask)}
+
+
+@BOTH
+@pytest.mark.parametrize("name", list(configs()))
+def test_prompts_portions_and_decoding_agree_with_the_oracle(name, dtype):
+    h = Harness(configs()[name], dtype)
+    for i, portions in enumerate(([400], [150, 1, 1, 2], [64], [16, 3], [2], [1, 7, 90])):
+        n = 230 if i < 4 else 70
+        h.request(str(i), n, seed=i)
+        h.drain(str(i), portions)
+    h.request("one", 1)
+    h.drain("one", [1])
+
+
+@BOTH
+def test_token_by_token_from_the_first_token(dtype):
+    h = Harness(default_config(), dtype)
+    h.request("a", 90)
+    h.drain("a", [1])
+
+
+@BOTH
+def test_batches_of_unequal_requests_with_reused_pages_and_slots(dtype):
+    """Four slots and pages for little more than four requests; eleven requests come and go, each in its own rhythm."""
+    h = Harness(default_config(), dtype, max_tokens=640, max_num_seqs=4)
+    rng = np.random.default_rng(5)
+    lengths = [150, 33, 97, 5, 160, 16, 2, 120, 64, 1, 75]
+    for i, n in enumerate(lengths):
+        h.request(str(i), n, seed=i)
+    waiting, live = [str(i) for i in range(len(lengths))], []
+    while waiting or live:
+        while waiting and len(live) < 4:
+            live.append(waiting.pop(0))
+        chosen = [r for r in live if rng.random() < 0.8] or live[:1]
+        h.step({r: int(rng.choice([1, 1, 2, 5, 17, 40, 64])) for r in chosen})
+        live = [r for r in live if h.at[r] < len(h.tokens[r])]
+    assert h.engine.pool.num_free == h.engine.pool.num_blocks and h.engine.slots.num_free == 4
+
+
+@BOTH
+def test_a_request_alone_and_in_a_batch(dtype):
+    cfg = default_config()
+    tensors = random_checkpoint(cfg)
+    from vllm_metal_b200.v1.engine import StepEntry
+
+    rng = np.random.default_rng(0)
+    toks = [rng.integers(0, cfg["vocab"], n).tolist() for n in (90, 41, 7)]
+    alone = make_engine(cfg, tensors, dtype)
+    first = [alone.advance([StepEntry(str(i), t, [len(t) - 1])]).clone() for i, t in enumerate(toks)]
+    second = [alone.advance([StepEntry(str(i), [3], [0])]).clone() for i in range(3)]
+    together = make_engine(cfg, tensors, dtype)
+    a = together.advance([StepEntry(str(i), t, [len(t) - 1]) for i, t in enumerate(toks)])
+    tol = 2e-5 if dtype == torch.float32 else 4e-2
+    torch.testing.assert_close(a, torch.cat(first), atol=tol * float(a.abs().max()), rtol=0)
+    b = together.advance([StepEntry(str(i), [3], [0]) for i in (2, 0, 1)])
+    torch.testing.assert_close(b, torch.cat([second[i] for i in (2, 0, 1)]), atol=tol * float(b.abs().max()), rtol=0)
+
+
+@BOTH
+def test_long_decoding_past_windows_pages_and_graph_buckets(dtype):
+    h = Harness(make_config([layer("latent_attention"), layer("mamba2"), layer("mlstm", gate_cap=15.0)]), dtype)
+    h.request("long", 620, seed=2)
+    h.drain("long", [300] + [1] * 400)
+
+
+@BOTH
+@pytest.mark.parametrize("long_prompt", [True, False])
+@pytest.mark.parametrize("window", [53, 64, None])
+def test_one_outstanding_key_counts_up_to_the_windows_edge(dtype, long_prompt, window):
+    """The weights are made so that every query asks for token 7's key: it outweighs all others as long as the window
+    holds it, and the logits of exactly those positions depend on it."""
+    cfg = make_config([layer("latent_attention", mask=window and {"size": window}, dim=32, kv_rank=64)])
+    dq = 32 + LATENT["rot_dim"]
+
+    def shape(t):
+        t["embed"][:, 0], t["embed"][:, 1] = 0.0, 2.0
+        t["embed"][7, 0] = 6.0
+        q = t["l0.mix.q"].view(LATENT["heads"], dq, -1)
+        q.zero_()
+        q[:, 0, 1] = 6.0
+        t["l0.mix.dkv"][0] = 0.0
+        t["l0.mix.dkv"][0, 0] = 3.0
+        t["l0.mix.uk"].view(LATENT["heads"], 32, 64)[:, 0] = 0.0
+        t["l0.mix.uk"].view(LATENT["heads"], 32, 64)[:, 0, 0] = 3.0
+
+    h = Harness(cfg, dtype, scale=shape)
+    n, at = 240, 100
+    h.request("a", n)
+    toks = [t if t != 7 else 8 for t in h.tokens["a"]]
+    plain = oracle.forward(cfg, h.oracle_tensors, toks)
+    toks[at] = 7
+    h.tokens["a"], h.want["a"] = toks, oracle.forward(cfg, h.oracle_tensors, toks)
+    h.limit["a"][:] = 4e-5 if dtype == torch.float32 else 4e-2
+    moved = np.sqrt(((plain - h.want["a"]) ** 2).mean(1)) / h.want["a"].std()
+    end = n if window is None else at + window
+    assert (moved[at:end] > 0.15).all() and (moved[:at] == 0).all() and (moved[end:] == 0).all()
+    h.drain("a", [n] if long_prompt else [at + 20] + [1] * n)
+
+
+def test_layers_share_weights_but_not_state():
+    ls = [layer("mlstm"), layer("mamba2"), layer("latent_attention")]
+    ls += [shared(ls, 0), shared(ls, 1), shared(ls, 2)]
+    h = Harness(make_config(ls), torch.float32)
+    m = h.engine.model
+    assert m.layers[3] is m.layers[0] and m.layers[5] is m.layers[2]
+    c = h.engine.cache
+    assert c.states[3].matrix.data_ptr() != c.states[0].matrix.data_ptr() and c.latent[5].data_ptr() != c.latent[2].data_ptr()
+    h.request("a", 60)
+    h.drain("a", [31, 1])
+
+
+@BOTH
+def test_residual_stream_after_every_layer(dtype):
+    from vllm_metal_b200.v1.engine import StepEntry
+
+    cfg = default_config()
+    tensors = random_checkpoint(cfg)
+    e = make_engine(cfg, tensors, dtype)
+    got, want, toks = [], [], list(range(40))
+    e.model.residual_hook = lambda i, x: got.append(x.double().cpu().numpy())
+    e.advance([StepEntry("a", toks)])
+    oracle.forward(cfg, to_oracle(tensors), toks, want)
+    assert len(got) == len(want) == len(cfg["layers"])
+    for i, (a, b) in enumerate(zip(got, want)):
+        assert np.abs(a - b).max() <= (2e-5 if dtype == torch.float32 else 4e-2) * np.abs(b).max(), i
+
+
+# -- the framework's entry points --------------------------------------------------------------------------------
+
+def _greedy_oracle(cfg, tensors, prompt, n):
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(oracle.forward(cfg, tensors, toks)[-1].argmax()))
+    return toks[len(prompt):]
+
+
+def test_greedy_generation_through_scheduler_and_command_line(tmp_path):
+    from vllm_metal_b200.v1.engine import Engine
+
+    cfg = default_config()
+    tensors = random_checkpoint(cfg, seed=3)
+    folder = write_folder(tmp_path / "model", cfg, tensors)
+    rng = np.random.default_rng(1)
+    prompts = [rng.integers(0, cfg["vocab"], n).tolist() for n in (70, 1, 18, 33, 9, 50)]
+    want = [_greedy_oracle(cfg, to_oracle(tensors), p, 12) for p in prompts]
+    # three slots, a budget smaller than the prompts and a pool for about three requests: portions, waiting, reuse
+    e = Engine.from_folder(folder, dtype="float32", max_tokens=256, max_num_seqs=3, max_batched_tokens=32)
+    assert e.generate(prompts, 12) == want
+    assert e.pool.num_free == e.pool.num_blocks and not e.live
+    (tmp_path / "p.jsonl").write_text("\n".join(json.dumps(p) for p in prompts))
+    r = subprocess.run([sys.executable, "-m", "vllm_metal_b200", "generate", "--model", folder, "--prompts",
+                        str(tmp_path / "p.jsonl"), "--max-new-tokens", "12", "--dtype", "float32", "--max-tokens", "512"],
+                       cwd=ROOT, capture_output=True, text=True, timeout=240)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [json.loads(x) for x in r.stdout.splitlines() if x.startswith("[")] == want
+
+
+def test_trace_replay_program(tmp_path):
+    cfg = make_config([layer("mamba2"), layer("latent_attention"), layer("mlstm")])
+    tensors = random_checkpoint(cfg, seed=4)
+    folder = write_folder(tmp_path / "model", cfg, tensors)
+    toks = {k: np.random.default_rng(i).integers(0, cfg["vocab"], 50).tolist() for i, k in enumerate("ab")}
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": toks["a"][:20], "want": [19, 3]},
+                                      {"id": "b", "tokens": toks["b"][:1], "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "b", "tokens": toks["b"][1:49], "want": [0]},
+                                      {"id": "a", "tokens": toks["a"][20:21], "want": [0]}], "end": ["a"]},
+             {"step": 2, "entries": [{"id": "b", "tokens": toks["b"][49:], "want": []}], "end": ["b"]}]
+    out = tmp_path / "out"
+    out.mkdir()
+    r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", folder, "--dtype", "float32", "--out", str(out),
+                        "--max-tokens", "128"], input="\n".join(map(json.dumps, steps)) + "\n", capture_output=True,
+                       text=True, timeout=240)
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == ["done 0", "done 1", "done 2"]
+    w = {k: oracle.forward(cfg, to_oracle(tensors), t) for k, t in toks.items()}
+    for n, rows in ((0, [w["a"][19], w["a"][3]]), (1, [w["b"][1], w["a"][20]])):
+        got = np.fromfile(out / f"{n}.f32", "<f4").reshape(len(rows), -1)
+        np.testing.assert_allclose(got, np.stack(rows), atol=1e-3)
+    assert not (out / "2.f32").exists()
+
+
+def test_worker_drives_a_hybrid_model_from_scheduler_outputs(tmp_path):
+    """The vLLM worker: loading by architecture, cache from the KV config, chunked prefill beside decoding, a finished
+    request's slot going to the next one."""
+    pytest.importorskip("vllm")
+    import types
+
+    from vllm.v1.core.sched.output import CachedRequestData, NewRequestData, SchedulerOutput
+
+    from vllm_metal_b200.v1.worker import B200Worker
+
+    cfg = default_config()
+    tensors = random_checkpoint(cfg, seed=6)
+    folder = write_folder(tmp_path / "model", cfg, tensors)
+    w = object.__new__(B200Worker)
+    w._requests, w._pending, w._drafts, w._drafter, w._pipeline = {}, None, {}, None, None
+    w.device, w.model = torch.device("cuda", 0), None
+    w.parallel_config = types.SimpleNamespace(tensor_parallel_size=1)
+    w.model_config = types.SimpleNamespace(hf_config=types.SimpleNamespace(**cfg), model=folder, seed=0, max_model_len=256,
+                                           enforce_eager=False, dtype=torch.float32)
+    w.scheduler_config = types.SimpleNamespace(max_num_seqs=2)
+    w.cache_config = types.SimpleNamespace(block_size=16, gpu_memory_utilization=0.5)
+    w.vllm_config = types.SimpleNamespace(load_config=types.SimpleNamespace(load_format="auto"))
+    w.load_model()
+    specs = w.get_kv_cache_spec()
+    assert sorted(specs) == sorted(f"layers.{i}.self_attn" for i in (0, 3, 5))
+    assert w.get_cache_block_size_bytes() == 16 * 3 * (48 + 8) * 4 and w.determine_available_memory() > 0
+    w.initialize_from_config(types.SimpleNamespace(num_blocks=40, kv_cache_groups=[object()]))
+    w.compile_or_warm_up_model()
+
+    rng = np.random.default_rng(2)
+    prompts = {r: rng.integers(0, cfg["vocab"], n).tolist() for r, n in (("A", 37), ("B", 9), ("C", 21))}
+    blocks = {"A": [5, 9, 2, 17], "B": [3, 20], "C": [5, 7, 1]}
+    computed, out = dict.fromkeys(prompts, 0), {r: [] for r in prompts}
+
+    def run(num, new=(), finished=()):
+        new_reqs = [NewRequestData(req_id=r, prompt_token_ids=prompts[r], mm_features=[], sampling_params=None,
+                                   pooling_params=None, block_ids=(blocks[r],), num_computed_tokens=0,
+                                   lora_request=None) for r in new]
+        old = [r for r in num if r not in new]
+        cached = CachedRequestData(req_ids=old, resumed_req_ids=set(), new_token_ids=[[] for _ in old], all_token_ids={},
+                                   new_block_ids=[None] * len(old), num_computed_tokens=[computed[r] for r in old],
+                                   num_output_tokens=[1] * len(old))
+        w.execute_model(SchedulerOutput(
+            scheduled_new_reqs=new_reqs, scheduled_cached_reqs=cached, num_scheduled_tokens=num,
+            total_num_scheduled_tokens=sum(num.values()), scheduled_spec_decode_tokens={}, scheduled_encoder_inputs={},
+            num_common_prefix_blocks=[0], finished_req_ids=set(finished), free_encoder_mm_hashes=[]))
+        got = w.sample_tokens(None)
+        for r, t in zip(got.req_ids, got.sampled_token_ids, strict=True):
+            computed[r] += num[r]
+            out[r] += t
+
+    run({"A": 20, "B": 9}, new=["A", "B"])
+    run({"A": 17, "B": 1})
+    for _ in range(3):
+        run({"A": 1, "B": 1})
+    run({"B": 1, "C": 21}, new=["C"], finished=["A"])  # C takes A's slot and one of its pages
+    for _ in range(3):
+        run({"B": 1, "C": 1})
+    for r in prompts:
+        assert out[r] == _greedy_oracle(cfg, to_oracle(tensors), prompts[r], len(out[r])), r

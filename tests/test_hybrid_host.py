@@ -1,0 +1,338 @@
+"""Host side of the hybrid decoders (no GPU): configuration, checkpoint container, registry, slots and pages, the batch
+plans, scheduling -- and the oracle's own mechanisms against closed forms."""
+
+from __future__ import annotations
+
+import copy
+
+import numpy as np
+import pytest
+import torch
+
+from oracle import hybrid as oracle
+
+from .hybrid_helpers import default_config, layer, make_config, random_checkpoint, segments, shared, write_folder
+
+
+# -- configuration, registry, checkpoints ---------------------------------------------------------------------
+
+def test_configuration_reads_every_size_and_follows_shared_weights():
+    from vllm_metal_b200.lm.hybrid_config import HybridArgs
+    from vllm_metal_b200.lm.hybrid_random import tensor_shapes
+
+    ls = [layer("mamba2"), layer("mlstm", ff=None), layer("latent_attention", mask=None)]
+    ls += [shared(ls, 1)]
+    ls += [shared(ls, 3)]  # a shared layer may name another shared one
+    a = HybridArgs.parse(make_config(ls, vocab=99, width=40, eps=1e-3))
+    assert (a.vocab, a.width, a.eps, a.num_layers) == (99, 40, 1e-3, 5)
+    assert [x.weights for x in a.layers] == [0, 1, 2, 1, 1] and [x.ff for x in a.layers] == [56, 0, 56, 0, 0]
+    assert a.layers[2].mixer.window == 0 and a.layers_of("mlstm") == [1, 3, 4]
+    assert a.layers[0].mixer.conv_channels == 6 * 16 + 2 * 3 * 24
+    shapes = tensor_shapes(a)
+    assert "l3.mix.q" not in shapes and "l1.mlp.up" not in shapes and shapes["l2.mix.dkv"] == (56, 40)
+
+
+@pytest.mark.parametrize("edit,message", [
+    (lambda c: c["layers"][0].update(type="conv"), "unknown mixer"),
+    (lambda c: c["layers"][0]["mixer"].pop("heads"), "'heads' is missing"),
+    (lambda c: c["layers"][0]["mixer"].update(groups=4), "groups"),
+    (lambda c: c["layers"][0]["mlp"].update(kind="moe"), "feed-forward kind"),
+    (lambda c: c["layers"][1].update(weights_of=0), "names a layer of type"),
+    (lambda c: c["layers"][1].update(weights_of=9), "is not a layer"),
+    (lambda c: c["layers"][1]["mixer"].update(gate_cap=0), "gate_cap"),
+    (lambda c: c.update(layers=[]), "no layers"),
+    (lambda c: c.pop("norm"), "'norm' is missing"),
+])
+def test_configuration_errors_name_the_entry(edit, message):
+    from vllm_metal_b200.lm.hybrid_config import ConfigError, HybridArgs
+
+    c = make_config([layer("mamba2"), layer("mlstm")])
+    edit(c)
+    with pytest.raises(ConfigError, match=message):
+        HybridArgs.parse(c)
+
+
+def test_registry_chooses_by_architecture():
+    from vllm_metal_b200.lm.registry import DecoderFamily, HybridFamily, family_of
+
+    assert isinstance(family_of(default_config()), HybridFamily)
+    assert isinstance(family_of({"architectures": ["Qwen3ForCausalLM"]}), DecoderFamily)
+    for bad in ({}, {"architecture": "Nobody"}):
+        with pytest.raises(ValueError, match="architecture"):
+            family_of(bad)
+
+
+def test_safetensors_round_trip_and_damage(tmp_path):
+    from vllm_metal_b200.lm.safetensors_io import SafetensorsFile, SafetensorsFolder, save_safetensors
+
+    t = {"a.b": torch.randn(3, 5).bfloat16(), "n": torch.arange(4, dtype=torch.int32), "e": torch.zeros(0, 2),
+         "f": torch.randn(7)}
+    path = str(tmp_path / "x.safetensors")
+    save_safetensors(path, t)
+    f = SafetensorsFile(path)
+    assert list(f.keys()) == list(t)
+    for k, v in t.items():
+        assert f.shape(k) == tuple(v.shape) and f.tensor(k).dtype == v.dtype and torch.equal(f.tensor(k), v)
+    save_safetensors(str(tmp_path / "y.safetensors"), {"z": torch.ones(2)})
+    both = SafetensorsFolder(str(tmp_path))
+    assert "z" in both and torch.equal(both.tensor("n"), t["n"])
+    with pytest.raises(KeyError, match="nothing"):
+        both.tensor("nothing")
+    save_safetensors(str(tmp_path / "w.safetensors"), {"z": torch.ones(2)})
+    with pytest.raises(ValueError, match="two files"):
+        SafetensorsFolder(str(tmp_path))
+    raw = open(path, "rb").read()
+    open(path, "wb").write(raw[:len(raw) - 8])
+    with pytest.raises(ValueError):
+        SafetensorsFile(path)
+
+
+def test_a_checkpoint_of_the_wrong_shape_is_refused(tmp_path):
+    from vllm_metal_b200.lm.hybrid import HybridModel
+    from vllm_metal_b200.lm.hybrid_config import HybridArgs
+
+    cfg = make_config([layer("mlstm")])
+    t = random_checkpoint(cfg)
+    t["l0.mix.v"] = t["l0.mix.v"][:-1]
+    folder = write_folder(tmp_path / "m", cfg, t)
+    with pytest.raises(ValueError, match="l0.mix.v"):
+        HybridModel.from_folder(HybridArgs.parse(cfg), folder, torch.float32, "cpu")
+
+
+def test_stacked_and_side_by_side_products_equal_the_separate_ones():
+    from vllm_metal_b200.lm.dense import SideBySideLinear, StackedLinear
+
+    g = torch.Generator().manual_seed(0)
+    w = {"a": torch.randn((5, 12), generator=g), "b": torch.randn((9, 12), generator=g), "c": torch.randn((8, 12), generator=g)}
+    st = StackedLinear(w, torch.float32, "cpu")
+    x = torch.randn((4, 12), generator=g)
+    for name, part in st.split(st(x)).items():
+        torch.testing.assert_close(part, x @ w[name].t())
+        assert st.slices[name][0] % 8 == 0
+    o = {"p": torch.randn((6, 5), generator=g), "q": torch.randn((6, 3), generator=g)}
+    sb = SideBySideLinear(o, torch.float32, "cpu")
+    y = sb.operand(4).zero_()
+    p, q = torch.randn((4, 5), generator=g), torch.randn((4, 3), generator=g)
+    y[:, :5], y[:, sb.offsets["q"]:sb.offsets["q"] + 3] = p, q
+    r = torch.randn((4, 6), generator=g)
+    want = r + p @ o["p"].t() + q @ o["q"].t()
+    sb.add_into(r, y)
+    torch.testing.assert_close(r, want)
+
+
+# -- slots, pages, plans -----------------------------------------------------------------------------------------
+
+def test_state_slots_and_pages_go_round():
+    from vllm_metal_b200.attention.caches.state_cache import StateSlots
+    from vllm_metal_b200.v1.engine import BlockPool
+
+    s = StateSlots(2)
+    a, b = s.acquire("a"), s.acquire("b")
+    assert {a, b} == {1, 2} and s.acquire("a") == a
+    with pytest.raises(RuntimeError, match="in use"):
+        s.acquire("c")
+    s.release("a")
+    s.release("nobody")
+    assert s.acquire("c") == a and s.num_free == 0
+
+    p = BlockPool(5, 16)
+    x, y = [], []
+    p.extend(x, 17)
+    p.extend(x, 32)
+    p.extend(y, 48)
+    assert len(x) == 2 and len(y) == 3 and sorted(x + y) == [1, 2, 3, 4, 5] and p.num_free == 0
+    with pytest.raises(RuntimeError, match="pages"):
+        p.extend(x, 33)
+    p.release(y)
+    p.extend(x, 33)
+    assert p.num_free == 2 and y == []
+
+
+def test_hybrid_cache_sizes_follow_the_layers():
+    from vllm_metal_b200.attention.caches.hybrid_cache import HybridCache, latent_bytes_per_token
+    from vllm_metal_b200.lm.hybrid_config import HybridArgs
+
+    a = HybridArgs.parse(default_config())
+    c = HybridCache(a, 3, 16, 2, torch.bfloat16, "cpu")
+    assert sorted(c.latent) == [0, 3, 5] and sorted(c.states) == [1, 2, 4, 6]
+    assert c.latent[0].shape == (48, 56) and latent_bytes_per_token(a, torch.bfloat16) == 3 * 56 * 2
+    assert c.states[1].matrix.shape == (3, 3, 40, 24) and c.states[1].normaliser.shape == (3, 3, 1, 40)
+    assert c.states[2].conv.shape == (3, 3, 240) and c.states[2].normaliser is None
+    assert c.nbytes == 48 * 3 * 56 * 2 + 3 * HybridCache.state_bytes_per_slot(a, torch.bfloat16)
+    pages = c.latent[3].view(3, 16, 56)
+    pages[1] = 1.0
+    pages[2] = 2.0
+    c.copy_blocks([(1, 2), (2, 1)])  # sources are read before any destination is written
+    assert float(pages[1, 0, 0]) == 2.0 and float(pages[2, 0, 0]) == 1.0
+    with pytest.raises(RuntimeError):
+        c.copy_blocks([(0, 3)])
+
+
+def test_segment_metadata_lists_chunks_and_splits_the_batch():
+    m = segments([1, 3, 70, 130], [40, 3, 71, 400], block_size=16, device="cpu")
+    assert m.max_q_len == 130 and m.num_chunks == 5 and m.has_short
+    assert m.chunk_seq.tolist() == [2, 2, 3, 3, 3] and m.chunk_row.tolist() == [4, 68, 74, 138, 202]
+    assert m.seq_chunk0.tolist()[2:] == [0, 2]
+    assert m.split(64) == (2, 4, 3) and m.split(100) == (3, 74, 70) and m.split(1000) == (4, 204, 130)
+    assert m.expand_plan(1000, 0) is None
+    p = m.expand_plan(64, 50)
+    assert p.first_row == 4 and p.first.tolist() == [0, 221] and p.count.tolist() == [71, 179]
+    assert p.out_row.tolist() == [0, 96] and p.rows_total == 96 + 192 and p.max_count == 179
+    assert p.block_tables.tolist() == [[0, 1, 2, 0, 0, 0], [3, 4, 5, 6, 7, 8]] and p.cu_seqlens_q.tolist() == [0, 70, 200]
+    assert m.expand_plan(64, 0).first.tolist() == [0, 0] and m.expand_plan(64, 50) is p
+    # a long segment in front of a short one stays with the latent-space rows
+    assert segments([70, 2, 90], [70, 2, 90], device="cpu").split(64) == (2, 72, 70)
+
+
+def test_runner_packs_short_prompts_first_and_keeps_the_callers_rows():
+    from vllm_metal_b200.v1.model_runner import PagedModelRunner
+
+    r = object.__new__(PagedModelRunner)
+    ids = [10, 20, 21, 22, 23, 24, 30, 40, 41, 42]
+    dec, pre = [([1], 5)], [([2], 5, 0), ([3], 1, 0), ([4], 3, 0)]
+    got, order, rows, slots = r._short_first(ids, dec, pre, [0, 3, 9, 6, 5], [7, 1, 2, 3])
+    assert got == [10, 30, 40, 41, 42, 20, 21, 22, 23, 24] and [p[1] for p in order] == [1, 3, 5] and slots == [7, 2, 3, 1]
+    assert [got[i] for i in rows] == [ids[i] for i in (0, 3, 9, 6, 5)]
+    got, _, rows, _ = r._short_first(ids, dec, pre, None, [7, 1, 2, 3])
+    assert [got[i] for i in rows] == [10, 24, 30, 42]  # every segment's last row, in the caller's order
+
+
+class _FakeRunner:
+    """Stands in for the device: 'logits' whose argmax is the row's token plus one."""
+
+    stateful, use_cuda_graph, max_batch = True, False, 8
+
+    def __init__(self, vocab):
+        self.vocab, self.steps = vocab, []
+
+    def forward_rows(self, ids, dec, pre, rows, slots):
+        assert len(slots) == len(dec) + len(pre) == len(set(slots))
+        used = [b for r in dec for b in r[0]] + [b for r in pre for b in r[0]]
+        assert len(used) == len(set(used))
+        self.steps.append((len(dec), [p[1] for p in pre]))
+        out = torch.zeros((len(rows), self.vocab))
+        for i, r in enumerate(rows):
+            out[i, (ids[r] + 1) % self.vocab] = 1.0
+        return out
+
+    def _greedy(self, logits):
+        return logits.argmax(1)
+
+
+def _fake_engine(**kw):
+    import types
+
+    from vllm_metal_b200.attention.caches.state_cache import StateSlots
+    from vllm_metal_b200.v1 import engine as mod
+
+    cache = types.SimpleNamespace(num_blocks=kw.pop("blocks") + 1, block_size=16, device="cpu")
+    real = mod.PagedModelRunner
+    mod.PagedModelRunner = lambda *a, **k: _FakeRunner(100)
+    try:
+        e = mod.Engine(None, cache, vocab=100, max_model_len=1000, **kw)
+    finally:
+        mod.PagedModelRunner = real
+    assert isinstance(e.slots, StateSlots)
+    return e
+
+
+def test_scheduler_mixes_portions_with_decoding_and_waits_for_pages():
+    e = _fake_engine(blocks=8, max_num_seqs=3, max_batched_tokens=20)
+    prompts = [list(range(5, 5 + n)) for n in (50, 3, 30, 17)]
+    out = e.generate(prompts, 6)
+    assert out == [[(p[-1] + 1 + i) % 100 for i in range(6)] for p in prompts]
+    steps = e.runner.steps
+    assert any(d > 0 and pre for d, pre in steps)                       # portions beside decoding rows
+    assert all(d + sum(pre) <= 20 for d, pre in steps)
+    assert e.pool.num_free == 8 and e.slots.num_free == 3 and not e.live
+    with pytest.raises(ValueError, match="never fit"):
+        e.add_request("big", [1] * 130, 1)
+    with pytest.raises(ValueError, match="vocabulary"):
+        e.add_request("bad", [100], 1)
+
+
+def test_step_interface_checks_its_entries():
+    from vllm_metal_b200.v1.engine import StepEntry
+
+    e = _fake_engine(blocks=8, max_num_seqs=2)
+    got = e.advance([StepEntry("a", [1, 2, 3], [2, 0]), StepEntry("b", [9], [])])
+    assert got.argmax(1).tolist() == [4, 2]
+    assert e.advance([StepEntry("b", [50], [0]), StepEntry("a", [7], [0])]).argmax(1).tolist() == [51, 8]
+    for bad, message in (([StepEntry("a", [])], "no tokens"), ([StepEntry("a", [1], [1])], "outside"),
+                         ([StepEntry("a", [1]), StepEntry("a", [2])], "twice"), ([StepEntry("a", [-1])], "vocabulary")):
+        with pytest.raises(ValueError, match=message):
+            e.advance(bad)
+    with pytest.raises(RuntimeError, match="live already"):
+        e.advance([StepEntry("c", [1])])
+    e.finish("a")
+    e.advance([StepEntry("c", [1])])
+    assert e.advance([]).shape == (0, 100)
+
+
+# -- the oracle's mechanisms ------------------------------------------------------------------------------------
+
+def test_oracle_mlstm_equals_the_unstabilised_form():
+    rng = np.random.default_rng(0)
+    t, h, k, v = 30, 2, 5, 4
+    q, kk, vv = rng.standard_normal((t, h, k)), rng.standard_normal((t, h, k)), rng.standard_normal((t, h, v))
+    li, lf = rng.standard_normal((t, h)), oracle.log_sigmoid(rng.standard_normal((t, h)))
+    got = oracle.mlstm_recurrence(q, kk, vv, li, lf)
+    for head in range(h):
+        s, n = np.zeros((k, v)), np.zeros(k)
+        for i in range(t):
+            s = np.exp(lf[i, head]) * s + np.exp(li[i, head]) * np.outer(kk[i, head], vv[i, head])
+            n = np.exp(lf[i, head]) * n + np.exp(li[i, head]) * kk[i, head]
+            # max(|n q|, 1) without the running maximum; the 1e-6 only matters relative to it
+            np.testing.assert_allclose(got[i, head], s.T @ q[i, head] / max(abs(n @ q[i, head]), 1.0), rtol=1e-4, atol=1e-6)
+
+
+def test_oracle_mamba2_equals_the_quadratic_form():
+    rng = np.random.default_rng(1)
+    t, h, g, n, v = 20, 4, 2, 3, 5
+    x, b, c = rng.standard_normal((t, h, v)), rng.standard_normal((t, g, n)), rng.standard_normal((t, g, n))
+    dt, a, d = oracle.softplus(rng.standard_normal((t, h))), rng.standard_normal(h), rng.standard_normal(h)
+    got = oracle.mamba2_recurrence(x, b, c, dt, a, d)
+    for head in range(h):
+        cum = np.cumsum(-np.exp(a[head]) * dt[:, head])
+        w = np.tril(np.exp(cum[:, None] - cum[None]) * dt[None, :, head] * (c[:, head // 2] @ b[:, head // 2].T))
+        np.testing.assert_allclose(got[:, head], w @ x[:, head] + d[head] * x[:, head], rtol=1e-10, atol=1e-12)
+
+
+def test_oracle_rotation_keeps_relative_positions_and_the_window_is_exact():
+    rng = np.random.default_rng(2)
+    q, k = rng.standard_normal((1, 1, 8)), rng.standard_normal((1, 1, 8))
+    dot = lambda i, j: float((oracle.rotate_interleaved(q, [i], 8, 100.0) * oracle.rotate_interleaved(k, [j], 8, 100.0)).sum())  # noqa: E731
+    assert abs(dot(7, 3) - dot(104, 100)) < 1e-9 and abs(dot(7, 3) - dot(7, 4)) > 1e-3
+    assert np.array_equal(oracle.rotate_interleaved(q, [5], 4, 100.0)[:, :, 4:], q[:, :, 4:])
+    assert [j for j in range(10) if oracle.visible(6, j, 3)] == [4, 5, 6]
+
+
+@pytest.mark.parametrize("edit", ["window", "gate", "rot", "conv", "skip", "norm_groups", "cap", "shared", "forget"])
+def test_a_planted_mistake_in_the_oracle_shows(edit):
+    """Every mechanism moves the logits of a small model: an oracle that gets one wrong is told apart."""
+    cfg = make_config([layer("mamba2"), layer("mlstm"), layer("latent_attention", mask={"size": 9})])
+    cfg["layers"].append(shared(cfg["layers"], 0))
+    t = {k: v.double().numpy() for k, v in random_checkpoint(cfg).items()}
+    toks = np.random.default_rng(0).integers(0, cfg["vocab"], 40).tolist()
+    right = oracle.forward(cfg, t, toks)
+    bad_cfg, bad = copy.deepcopy(cfg), dict(t)
+    if edit == "window":
+        bad_cfg["layers"][2]["mixer"]["mask"]["size"] = 10
+    elif edit == "gate":
+        bad["l2.mix.g"] = np.zeros_like(t["l2.mix.g"])
+    elif edit == "rot":
+        bad_cfg["layers"][2]["mixer"]["rot"]["base"] = 50.0
+    elif edit == "conv":
+        bad["l0.mix.conv"] = t["l0.mix.conv"][:, ::-1]
+    elif edit == "skip":
+        bad["l0.mix.D"] = np.zeros_like(t["l0.mix.D"])
+    elif edit == "norm_groups":
+        bad_cfg["layers"][0]["mixer"]["norm_groups"] = 1
+    elif edit == "cap":
+        bad_cfg["layers"][1]["mixer"]["gate_cap"] = 1.5
+    elif edit == "shared":
+        bad_cfg["layers"].pop()
+    elif edit == "forget":
+        bad["l1.mix.f.b"] = t["l1.mix.f.b"] - 3.0
+    err = np.sqrt(((oracle.forward(bad_cfg, bad, toks) - right) ** 2).mean(1)) / right.std()
+    assert err[12:].max() > 2e-2, err.max()

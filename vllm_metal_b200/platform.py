@@ -126,6 +126,10 @@ class B200Platform(Platform):
         cache = vllm_config.cache_config
         if cache is not None and getattr(cache, "block_size", None) is None:
             cache.block_size = 16
+        hf = getattr(getattr(vllm_config, "model_config", None), "hf_config", None)
+        if cache is not None and getattr(hf, "architecture", None) is not None and \
+                getattr(cache, "enable_prefix_caching", False):
+            cache.enable_prefix_caching = False  # hybrid decoders: a recurrent state has no prefix to reuse
         comp = getattr(vllm_config, "compilation_config", None)
         if comp is not None and hasattr(comp, "custom_ops") and not comp.custom_ops:
             comp.custom_ops = ["none"]  # no torch.compile / inductor on this path (CUDA graphs are ours)

@@ -18,12 +18,16 @@ from typing import Any
 
 import torch
 
-from vllm.v1.kv_cache_interface import FullAttentionSpec, KVCacheConfig, KVCacheSpec, SlidingWindowSpec
+from vllm.v1.kv_cache_interface import (FullAttentionSpec, KVCacheConfig, KVCacheSpec, MLAAttentionSpec,
+                                        SlidingWindowSpec)
 from vllm.v1.worker.worker_base import WorkerBase
 
+from ..attention.caches.hybrid_cache import HybridCache, latent_bytes_per_token
 from ..attention.caches.kv_cache import B200PagedKVCache
+from ..attention.caches.state_cache import StateSlots
 from ..lm.decoder import Model
-from ..lm.registry import FAMILIES, HybridFamily, model_args_from_hf_config
+from ..lm.hybrid_config import HybridArgs
+from ..lm.registry import FAMILIES, HybridFamily, model_args_from_hf_config, read_config
 from .model_runner import PagedModelRunner
 
 logger = logging.getLogger(__name__)
@@ -98,10 +102,14 @@ class B200Worker(WorkerBase):
 
     def load_model(self) -> None:
         """Builds the decoder for the HF config with RANDOM-INITIALISED affine-quantized weights (``seed``):
-        the BASELINE configs are all random-init and no checkpoint reader is wired (the AWQ repack path is
-        ``quant/awq_loader.py``; safetensors loading is out of scope).  ``load_format`` other than
+        the BASELINE configs are all random-init and no checkpoint reader is wired for these families (the AWQ repack
+        path is ``quant/awq_loader.py``; hybrid decoders do load safetensors).  ``load_format`` other than
         "dummy"/"auto" therefore raises instead of silently ignoring a checkpoint."""
         lf = str(getattr(getattr(self.vllm_config, "load_config", None), "load_format", "dummy"))
+        hybrid = self._hybrid_config()
+        if hybrid is not None:
+            self._load_hybrid(hybrid, lf)
+            return
         if lf not in ("dummy", "auto", "LoadFormat.DUMMY", "LoadFormat.AUTO"):
             raise NotImplementedError(f"load_format={lf}: only random-init ('dummy') weights are wired on this path")
         args = model_args_from_hf_config(self.model_config.hf_config)
@@ -109,12 +117,41 @@ class B200Worker(WorkerBase):
         self.model = Model(args, torch.bfloat16, self.device, seed=int(self.model_config.seed or 0),
                            rank=self.rank, world=world, allreduce=self._allreduce)
 
+    def _hybrid_config(self) -> dict | None:
+        """The configuration of a hybrid decoder (lm/registry.py), or None for the transformer decoders."""
+        hf = self.model_config.hf_config
+        config = hf.to_dict() if hasattr(hf, "to_dict") else dict(vars(hf))
+        name = config.get("architecture") or next(iter(config.get("architectures") or []), None)
+        return config if isinstance(FAMILIES.get(name), HybridFamily) else None
+
+    def _load_hybrid(self, config: dict, load_format: str) -> None:
+        """Weights from the model folder's safetensors files, or random ones for the "dummy" format."""
+        if self.parallel_config.tensor_parallel_size != 1:
+            raise NotImplementedError("hybrid decoders run on one GPU (no tensor-parallel form of their mixers)")
+        if self._drafter is not None:
+            raise NotImplementedError("a recurrent state cannot be rolled back: no speculative decoding with such layers")
+        fmt = load_format.rsplit(".", 1)[-1].lower()
+        if fmt not in ("dummy", "auto", "safetensors"):
+            raise NotImplementedError(f"load_format={load_format}: hybrid decoders load safetensors or random weights")
+        folder = None if fmt == "dummy" else str(self.model_config.model)
+        family = FAMILIES[config.get("architecture") or config["architectures"][0]]
+        args = family.parse(config if "layers" in config else read_config(str(self.model_config.model)))
+        dtype = getattr(self.model_config, "dtype", torch.bfloat16)
+        dtype = dtype if dtype in family.dtypes else torch.bfloat16
+        self.model = family.load(args, folder, dtype, self.device, seed=int(self.model_config.seed or 0))
+
+    @property
+    def _is_hybrid(self) -> bool:
+        return isinstance(getattr(self.model, "args", None), HybridArgs)
+
     def get_model(self) -> Any:
         return self.model
 
     # ---- KV cache (worker.py:199-250; cache_policy.py:383-411) ----------------
     def get_cache_block_size_bytes(self) -> int:
         a = self.model.args
+        if self._is_hybrid:
+            return latent_bytes_per_token(a, self.model.dtype) * self.cache_config.block_size
         world = self.parallel_config.tensor_parallel_size
         return 2 * a.num_layers * self.cache_config.block_size * (a.n_kv_heads // world) * a.head_dim * 2
 
@@ -127,10 +164,23 @@ class B200Worker(WorkerBase):
         torch.cuda.synchronize(self.device)
         free, total = torch.cuda.mem_get_info(self.device)
         budget = int(total * self.cache_config.gpu_memory_utilization) - (total - free) - (1 << 30)
+        if self._is_hybrid:  # the state slots come out of the same budget
+            slots = int(self.scheduler_config.max_num_seqs) + 1
+            budget -= slots * HybridCache.state_bytes_per_slot(self.model.args, self.model.dtype)
         return max(budget, 0)
 
     def get_kv_cache_spec(self) -> dict[str, KVCacheSpec]:
         a = self.model.args
+        if self._is_hybrid:
+            # one latent row per token and layer; all latent layers share the request's pages (a window is applied by
+            # the kernels).  Recurrent state lives in slots of this worker, outside vLLM's pools.
+            rows = [a.layers[i].mixer for i in a.layers_of("latent_attention")]
+            if not rows:
+                raise NotImplementedError("a hybrid decoder without any latent-attention layer has no paged cache")
+            width = max(m.kv_rank + m.rot_dim for m in rows)
+            return {f"layers.{i}.self_attn": MLAAttentionSpec(block_size=self.cache_config.block_size, num_kv_heads=1,
+                                                              head_size=width, dtype=self.model.dtype)
+                    for i in a.layers_of("latent_attention")}
         world = self.parallel_config.tensor_parallel_size
         windows = a.sliding_window_per_layer()
         specs: dict[str, KVCacheSpec] = {}
@@ -152,7 +202,14 @@ class B200Worker(WorkerBase):
         groups = getattr(kv_cache_config, "kv_cache_groups", None) or []
         self._num_kv_groups = max(1, len(groups))
         group_sizes = None
-        if len(groups) > 1:
+        if self._is_hybrid:
+            if len(groups) > 1:
+                raise NotImplementedError("hybrid decoders keep their latent layers in one KV-cache group")
+            slots = int(self.scheduler_config.max_num_seqs)
+            self.kv_cache = HybridCache(a, int(kv_cache_config.num_blocks), self.cache_config.block_size, slots,
+                                        self.model.dtype, self.device)
+            self._state_slots = StateSlots(slots)
+        elif len(groups) > 1:
             # vLLM grouped the layers (full + sliding-window specs): adopt its layout as is -- per-layer page size,
             # window and the scheduler group whose block ids the layer reads (reference adopt_layout, runtime/mha.py:74)
             from ..attention.caches.mha_layout import MHAKVCacheLayout
@@ -180,7 +237,7 @@ class B200Worker(WorkerBase):
         r = self.model_runner
         if r is not None and r.use_cuda_graph:
             for b in sorted({1, min(8, r.max_batch), r.max_batch}):
-                r.decode_step([0] * b, [[0]] * b, [1] * b)  # block 0 is the reserved padding block
+                r.decode_step([0] * b, [[0]] * b, [1] * b, state_slots=[0] * b)  # block 0 is the reserved padding block
         torch.cuda.synchronize(self.device)
         return time.perf_counter() - start
 
@@ -197,15 +254,21 @@ class B200Worker(WorkerBase):
                 raise NotImplementedError(
                     f"execute_model expects vllm.v1.core.sched.output.SchedulerOutput; {type(so).__name__} has no "
                     f"'{field}'")
+        state_slots = getattr(self, "_state_slots", None)  # recurrent layers: one slot per live request
         spec_tokens = dict(so.scheduled_spec_decode_tokens or {})  # req_id -> scheduled draft token ids
         for rid in list(so.finished_req_ids) + list(so.preempted_req_ids or ()):
             self._requests.pop(rid, None)
+            if state_slots is not None:
+                state_slots.release(rid)
         for nr in so.scheduled_new_reqs:
             if nr.prompt_token_ids is None:
                 raise NotImplementedError("prompt embeddings are outside the B200 decode hot path")
             if len(nr.block_ids) != getattr(self, "_num_kv_groups", 1):
                 raise RuntimeError(f"request {nr.req_id}: {len(nr.block_ids)} block-id lists for "
                                    f"{getattr(self, '_num_kv_groups', 1)} KV-cache groups")
+            if state_slots is not None and int(nr.num_computed_tokens):
+                raise RuntimeError(f"request {nr.req_id} starts at token {nr.num_computed_tokens}: a recurrent state has "
+                                   "no prefix to reuse (prefix caching must be off)")
             self._requests[nr.req_id] = _RequestState(list(nr.prompt_token_ids), [list(b) for b in nr.block_ids],
                                                       int(nr.num_computed_tokens))
         cached = so.scheduled_cached_reqs
@@ -251,6 +314,8 @@ class B200Worker(WorkerBase):
             tokens.extend(st.tokens[st.num_computed:st.num_computed + n])
             pre_rows.append((st.block_ids if grouped else st.block_ids[0], n, st.num_computed))
         order = decodes + prefills
+        # keyword for the runner calls below; models without recurrent layers are called as ever
+        state = {} if state_slots is None else {"state_slots": [state_slots.acquire(rid) for rid, _, _ in order]}
         r = self.model_runner
         pipe = getattr(self, "_pipeline", None)
         if pipe is not None:
@@ -263,7 +328,7 @@ class B200Worker(WorkerBase):
                 rows = [pipe.pending_row(rid) if st.tokens[st.num_computed] < 0 else -1 for rid, st, _ in decodes]
                 if any(row < 0 and st.tokens[st.num_computed] < 0 for row, (_, st, _) in zip(rows, decodes, strict=True)):
                     raise RuntimeError("decode pipeline: a placeholder token has no pending row")
-                handle = r.submit_decode(tokens, [b for b, _ in dec_rows], [n for _, n in dec_rows], rows)
+                handle = r.submit_decode(tokens, [b for b, _ in dec_rows], [n for _, n in dec_rows], rows, **state)
                 self._pending = (order, handle, "deferred")
                 return
             pipe.begin_step()  # synchronous step: the pending tokens land before any state is read
@@ -284,9 +349,9 @@ class B200Worker(WorkerBase):
             sampled.extend(flat[at:])
         elif not pre_rows and r.use_cuda_graph and len(dec_rows) <= r.max_batch:
             # pure decode: the CUDA-graph path (pinned staging -> one H2D -> graph replay -> D2H token ids)
-            sampled = r.decode_step(tokens, [b for b, _ in dec_rows], [n for _, n in dec_rows])
+            sampled = r.decode_step(tokens, [b for b, _ in dec_rows], [n for _, n in dec_rows], **state)
         else:
-            sampled = r.execute(tokens, dec_rows, pre_rows)
+            sampled = r.execute(tokens, dec_rows, pre_rows, **state)
         self._pending = (order, sampled, spec_tokens)
 
     def sample_tokens(self, grammar_output: Any = None):
