@@ -143,7 +143,8 @@ int b200_head_linear(const b200_head_linear_args* a, void* stream);
 
 /* Latent attention in the latent space: every query head attends over the same cached rows
  * [latent kv_rank | key part rot_dim]; values are the latents.  q [T, heads, kv_rank + rot_dim], out
- * [T, heads, kv_rank].  Only segments of at most max_q_len rows are computed.  window <= 0: none. */
+ * [T, heads, kv_rank].  Only segments of at most max_q_len rows are computed.  window <= 0: none.
+ * kernel: 0 auto, 1 any type and size, 2 warp-level tensor cores, 3 tcgen05. */
 typedef struct b200_latent_attn_args {
   const void* q;
   const void* cache;
@@ -163,6 +164,8 @@ typedef struct b200_latent_attn_args {
 size_t b200_latent_attention_workspace_bytes(const b200_latent_attn_args* a);
 int b200_latent_attention_num_launches(const b200_latent_attn_args* a);
 int b200_latent_attention(const b200_latent_attn_args* a, void* stream);
+/* Synchronises.  1 if a bounded wait inside the kernel ever ran out (that launch wrote no results), else 0. */
+int b200_latent_attention_failed(void);
 
 /* Rows [first[i], first[i] + count[i]) of request i's cached latents, gathered from the pages into consecutive rows
  * of out [rows, kv_rank + rot_dim] starting at out_row[i] (the operand of the products that expand keys and values);

@@ -47,9 +47,10 @@ class Pool:
 
 
 @pytest.mark.parametrize("dtype,kernel,splits", [(torch.float32, 1, 0), (torch.bfloat16, 1, 0), (torch.bfloat16, 2, 0),
-                                                  (torch.bfloat16, 2, 3), (torch.bfloat16, 2, 7)])
+                                                  (torch.bfloat16, 2, 3), (torch.bfloat16, 2, 7), (torch.bfloat16, 3, 0),
+                                                  (torch.bfloat16, 3, 1), (torch.bfloat16, 3, 4)])
 @pytest.mark.parametrize("heads,rank,rot,window,bs", [(5, 48, 16, 0, 16), (32, 512, 64, 96, 16), (3, 64, 16, 33, 8),
-                                                       (40, 80, 32, 7, 32)])
+                                                       (40, 80, 32, 7, 32), (16, 320, 64, 0, 64)])
 def test_latent_space_attention(ops, dtype, kernel, splits, heads, rank, rot, window, bs):
     ctx, q_lens = [301, 1, 64, 97, 33], [1, 1, 3, 9, 33]
     pool = Pool(ctx, rank + rot, dtype, bs)
@@ -65,9 +66,10 @@ def test_latent_space_attention(ops, dtype, kernel, splits, heads, rank, rot, wi
         tol = 3e-5 if dtype == torch.float32 else 1e-2
         assert np.abs(got[at:at + n] - want).max() <= tol * np.abs(want).max(), (i, n)
         at += n
+    assert not ops.latent_attention_failed()
 
 
-@pytest.mark.parametrize("dtype,kernel", [(torch.float32, 1), (torch.bfloat16, 2)])
+@pytest.mark.parametrize("dtype,kernel", [(torch.float32, 1), (torch.bfloat16, 2), (torch.bfloat16, 3)])
 def test_one_key_just_inside_and_just_outside_the_window(ops, dtype, kernel):
     """One key outweighs all others; it must count for the last position that sees it and for none after."""
     rank, rot, heads, bs, window = 32, 16, 2, 16, 45

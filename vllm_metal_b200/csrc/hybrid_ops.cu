@@ -156,6 +156,120 @@ mixer_finish_kernel(const b200_mixer_finish_args a, int norm_blocks) {
   }
 }
 
+// The same for 16-bit types whose rows, groups and offsets are whole 16-byte units: 8 columns a thread and step, the
+// group held in registers between its norm and its store.  LANES threads share a group (a warp or the CTA).
+template <typename T>
+struct alignas(16) Vec8 {
+  T e[8];
+};
+__device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
+template <typename T, int LANES, int VPL>
+__global__ void __launch_bounds__(256)
+mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks, int act_vecs) {
+  pdl_trigger();
+  pdl_wait();
+  const int64_t r = blockIdx.y;
+  T* o = reinterpret_cast<T*>(a.out) + r * a.out_stride;
+  if ((int)blockIdx.x < norm_blocks) {
+    __shared__ float red[8];
+    const T* y = reinterpret_cast<const T*>(a.y) + r * a.y_stride;
+    const T* pre = a.pre_gate ? reinterpret_cast<const T*>(a.pre_gate) + r * a.pre_stride : nullptr;
+    const T* post = a.post_gate ? reinterpret_cast<const T*>(a.post_gate) + r * a.post_stride : nullptr;
+    const int gs = a.group_size > 0 ? a.group_size : LANES * VPL * 8;
+    const int group = LANES == 32 ? blockIdx.x * 8 + (threadIdx.x >> 5) : blockIdx.x;
+    const int c0 = group * gs, c1 = min(c0 + gs, a.inner), first = c0 + (threadIdx.x % LANES) * 8;
+    Vec8<T> vy[VPL], vg[VPL];
+#pragma unroll
+    for (int j = 0; j < VPL; ++j) {
+      const int c = first + j * LANES * 8;
+      if (c < c1) {
+        const int yc = a.y_head_dim > 0 ? c / a.y_head_dim * a.y_head_stride + c % a.y_head_dim : c;
+        vy[j] = *reinterpret_cast<const Vec8<T>*>(y + yc);
+        if (pre) vg[j] = *reinterpret_cast<const Vec8<T>*>(pre + c);
+      }
+    }
+    float v[VPL][8], ss = 0.f, inv = 1.f;
+#pragma unroll
+    for (int j = 0; j < VPL; ++j) {
+      const bool live = first + j * LANES * 8 < c1;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        v[j][e] = live ? to_float(vy[j].e[e]) : 0.f;
+        if (pre && live) {
+          const float z = to_float(vg[j].e[e]);
+          v[j][e] *= z * fast_sigmoid(z);
+        }
+        ss += v[j][e] * v[j][e];
+      }
+    }
+    if (a.group_size > 0) {
+      ss = LANES == 32 ? warp_sum(ss) : block_sum<256>(ss, red);
+      inv = 1.f / sqrtf(ss / (float)gs + a.eps);
+    }
+#pragma unroll
+    for (int j = 0; j < VPL; ++j) {
+      const int c = first + j * LANES * 8;
+      if (c >= c1) continue;
+      float w[8];
+      if (a.weight) {
+        *reinterpret_cast<float4*>(w) = *reinterpret_cast<const float4*>(a.weight + c);
+        *reinterpret_cast<float4*>(w + 4) = *reinterpret_cast<const float4*>(a.weight + c + 4);
+      }
+      if (post) vg[j] = *reinterpret_cast<const Vec8<T>*>(post + c);
+      Vec8<T> res;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        float x = v[j][e] * inv;
+        if (a.weight) x *= w[e];
+        if (post) x *= fast_sigmoid(to_float(vg[j].e[e]));
+        res.e[e] = from_float<T>(x);
+      }
+      *reinterpret_cast<Vec8<T>*>(o + c) = res;
+    }
+  } else {
+    const T* in = reinterpret_cast<const T*>(a.act_in) + r * a.act_stride;
+    const int base = ((int)blockIdx.x - norm_blocks) * act_vecs * 2048 + threadIdx.x * 8;
+    for (int j = 0; j < act_vecs; ++j) {
+      const int i = base + j * 2048;
+      if (i >= a.act_dim) break;
+      Vec8<T> x = *reinterpret_cast<const Vec8<T>*>(in + i);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x.e[e] = from_float<T>(gelu_erf_f(to_float(x.e[e])));
+      *reinterpret_cast<Vec8<T>*>(o + a.act_offset + i) = x;
+    }
+  }
+  if (blockIdx.x == 0 && a.act_dim > 0)
+    for (int c = a.act_offset + a.act_dim + threadIdx.x; c < a.out_cols; c += 256) o[c] = from_float<T>(0.f);
+}
+
+template <typename T>
+bool finish_vec_ok(const b200_mixer_finish_args& a) {
+  auto ok = [](const void* p, int64_t stride) { return !p || (((uintptr_t)p & 15) == 0 && stride % 8 == 0); };
+  const int gs = a.group_size > 0 ? a.group_size : 1024;
+  return sizeof(T) == 2 && ok(a.y, a.y_stride) && ok(a.pre_gate, a.pre_stride) && ok(a.post_gate, a.post_stride) &&
+         ok(a.act_in, a.act_stride) && ok(a.out, a.out_stride) && ((uintptr_t)a.weight & 15) == 0 && a.inner % 8 == 0 &&
+         gs % 8 == 0 && gs <= 8192 && a.act_dim % 8 == 0 && a.act_offset % 8 == 0 && a.y_head_dim % 8 == 0 &&
+         a.y_head_stride % 8 == 0 && (a.act_dim > 0 ? a.act_offset : a.out_cols) == a.inner;
+}
+
+template <typename T>
+int launch_finish_vec(const b200_mixer_finish_args& a, cudaStream_t st) {
+  const int gs = a.group_size > 0 ? a.group_size : 1024, groups = a.y ? (a.inner + gs - 1) / gs : 0;
+  const bool warp = gs <= 1024;
+  const int vpl = warp ? (gs + 255) / 256 : (gs + 2047) / 2048;
+  const int nb = warp ? (groups + 7) / 8 : groups, vecs = a.rows >= 256 ? 4 : 1;
+  const int ab = (a.act_dim + vecs * 2048 - 1) / (vecs * 2048);
+  auto* kern = warp ? (vpl == 1   ? mixer_finish_vec_kernel<T, 32, 1>
+                       : vpl == 2 ? mixer_finish_vec_kernel<T, 32, 2>
+                                  : mixer_finish_vec_kernel<T, 32, 4>)
+                    : (vpl == 1   ? mixer_finish_vec_kernel<T, 256, 1>
+                       : vpl == 2 ? mixer_finish_vec_kernel<T, 256, 2>
+                                  : mixer_finish_vec_kernel<T, 256, 4>);
+  B200_CUDA_OK(launch_pdl(kern, dim3(nb + ab > 0 ? nb + ab : 1, a.rows), dim3(256), 0, st, a, nb, vecs));
+  return check_launch("mixer_finish");
+}
+
 // ---- causal depthwise convolution -----------------------------------------------------------
 // One thread per channel walks kConvTile rows with the taps in registers.  Only the first tile of a segment touches
 // the carried inputs, and it takes the new ones straight from the input rows, so the tiles never race.
@@ -233,6 +347,78 @@ causal_conv_kernel(const T* __restrict__ in, const float* __restrict__ weight, c
   }
 }
 
+// 16-bit types with whole 16-byte units: 8 channels a thread.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+causal_conv_vec_kernel(const T* __restrict__ in, const float* __restrict__ weight, const float* __restrict__ bias,
+                       T* __restrict__ state, const int32_t* __restrict__ cu, const int32_t* __restrict__ seq_lens,
+                       const int32_t* __restrict__ slots, T* __restrict__ out, int channels, int64_t in_stride,
+                       int64_t out_stride, int activation) {
+  pdl_trigger();
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
+  float w[TAPS][8], b[8];
+  if (c < channels) {  // the weights do not depend on earlier kernels
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) {
+      *reinterpret_cast<float4*>(w[k]) = *reinterpret_cast<const float4*>(weight + (int64_t)k * channels + c);
+      *reinterpret_cast<float4*>(w[k] + 4) = *reinterpret_cast<const float4*>(weight + (int64_t)k * channels + c + 4);
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) b[e] = bias ? bias[c + e] : 0.f;
+  }
+  pdl_wait();
+  const int s = blockIdx.y;
+  const int row0 = cu[s], len = cu[s + 1] - row0;
+  const int t0 = blockIdx.z * kConvTile;
+  if (t0 >= len || c >= channels) return;
+  const bool fresh = seq_lens[s] == len;
+  T* st = state + (int64_t)slots[s] * (TAPS - 1) * channels + c;
+  const T* x = in + (int64_t)row0 * in_stride + c;
+  auto zero = [] {
+    Vec8<T> z;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) z.e[e] = from_float<T>(0.f);
+    return z;
+  };
+  auto at = [&](int t) {  // input of position t of the segment, carried or new
+    if (t >= 0) return *reinterpret_cast<const Vec8<T>*>(x + (int64_t)t * in_stride);
+    return fresh ? zero() : *reinterpret_cast<const Vec8<T>*>(st + (int64_t)(TAPS - 1 + t) * channels);
+  };
+  Vec8<T> win[TAPS > 1 ? TAPS - 1 : 1];
+#pragma unroll
+  for (int k = 0; k < TAPS - 1; ++k) win[k] = at(t0 - (TAPS - 1) + k);
+  if (t0 == 0 && TAPS > 1) {
+    Vec8<T> nv[TAPS > 1 ? TAPS - 1 : 1];
+#pragma unroll
+    for (int k = 0; k < TAPS - 1; ++k) nv[k] = at(len - (TAPS - 1) + k);
+#pragma unroll
+    for (int k = 0; k < TAPS - 1; ++k) *reinterpret_cast<Vec8<T>*>(st + (int64_t)k * channels) = nv[k];
+  }
+  const int t1 = min(t0 + kConvTile, len);
+#pragma unroll 4
+  for (int t = t0; t < t1; ++t) {
+    const Vec8<T> cur = *reinterpret_cast<const Vec8<T>*>(x + (int64_t)t * in_stride);
+    Vec8<T> res;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      float acc = b[e];
+#pragma unroll
+      for (int k = 0; k < TAPS - 1; ++k) acc += w[k][e] * to_float(win[k].e[e]);
+      acc += w[TAPS - 1][e] * to_float(cur.e[e]);
+      if (activation) acc *= fast_sigmoid(acc);
+      res.e[e] = from_float<T>(acc);
+    }
+    *reinterpret_cast<Vec8<T>*>(out + (int64_t)(row0 + t) * out_stride + c) = res;
+#pragma unroll
+    for (int k = 0; k < TAPS - 1; ++k) {
+      if (k == TAPS - 2)
+        win[k] = cur;
+      else
+        win[k] = win[k + 1];
+    }
+  }
+}
+
 }  // namespace
 }  // namespace b200
 
@@ -283,6 +469,7 @@ int b200_mixer_finish(const b200_mixer_finish_args* a, void* stream) {
   const int ab = (a->act_dim + 1023) / 1024;
   const int grid = nb + ab > 0 ? nb + ab : 1;
   return B200_DISPATCH_DTYPE(a->dtype, T, [&]() -> int {
+    if (finish_vec_ok<T>(*a)) return launch_finish_vec<T>(*a, (cudaStream_t)stream);
     B200_CUDA_OK(launch_pdl(warp ? mixer_finish_kernel<T, true> : mixer_finish_kernel<T, false>,
                             dim3(grid, a->rows), dim3(256), 0, (cudaStream_t)stream, *a, nb));
     return check_launch("mixer_finish");
@@ -300,6 +487,16 @@ int b200_causal_conv(const void* in, const float* weight, const float* bias, voi
   B200_CHECK_ARG(num_seqs <= 65535 && (max_q_len + kConvTile - 1) / kConvTile <= 65535, "causal_conv: batch too large");
   const dim3 grid((channels + 127) / 128, num_seqs, (max_q_len + kConvTile - 1) / kConvTile);
   return B200_DISPATCH_DTYPE(dtype, T, [&]() -> int {
+    if (sizeof(T) == 2 && taps >= 2 && taps <= 4 && channels % 8 == 0 && in_stride % 8 == 0 && out_stride % 8 == 0 &&
+        (((uintptr_t)in | (uintptr_t)out | (uintptr_t)state | (uintptr_t)weight) & 15) == 0) {
+      auto* kern = taps == 4   ? causal_conv_vec_kernel<T, 4>
+                   : taps == 3 ? causal_conv_vec_kernel<T, 3>
+                               : causal_conv_vec_kernel<T, 2>;
+      B200_CUDA_OK(launch_pdl(kern, dim3((channels + 1023) / 1024, grid.y, grid.z), dim3(128), 0, (cudaStream_t)stream,
+                              (const T*)in, weight, bias, (T*)state, cu_seqlens, seq_lens, slots, (T*)out, channels,
+                              in_stride, out_stride, activation));
+      return check_launch("causal_conv");
+    }
     auto* kern = taps == 4   ? causal_conv_kernel<T, 4>
                  : taps == 3 ? causal_conv_kernel<T, 3>
                  : taps == 2 ? causal_conv_kernel<T, 2>

@@ -5,8 +5,10 @@
 //  * latent_mma_kernel (bf16): 32 (token, head) rows per CTA against 32-key tiles on m16n8k16 tensor cores, split over
 //    the keys when the batch alone does not fill the GPU; softmax in fp32, the weights enter the value product as a
 //    two-term bf16 split (16 significant bits).
+//  * latent_tc_kernel (latent_attention_tc.cuh): the same on tcgen05, the default wherever pages and sizes allow TMA.
 //  * latent_simt_kernel: any type and size; one CTA per (token, head).
 #include "../../include/b200_hybrid_ops.h"
+#include "latent_attention_tc.cuh"
 #include "mma_sync.cuh"
 
 namespace b200 {
@@ -91,7 +93,7 @@ latent_simt_kernel(const b200_latent_attn_args a) {
 constexpr int kThreads = 256;
 constexpr int kRows = 32, kKeys = 32;
 constexpr int kPPitch = 40;
-constexpr int kMaxRank = 512, kMaxWidth = 640;
+constexpr int kMaxRank = 512, kMaxWidth = 640, kMaxSplits = 64;
 
 struct Smem {
   int pitch;
@@ -297,32 +299,40 @@ latent_mma_kernel(const b200_latent_attn_args a, int splits) {
   }
 }
 
-// One warp per (token, head) row of the computed segments: the partial outputs of the splits become one.
-__global__ void __launch_bounds__(256)
+// One CTA per (token, head) row of the computed segments, 4 columns a thread: the splits' partial outputs become one.
+__global__ void __launch_bounds__(128)
 latent_merge_kernel(const b200_latent_attn_args a, int splits) {
   pdl_trigger();
   pdl_wait();
+  __shared__ float weight[kMaxSplits];
   const int s = blockIdx.y, row0 = a.cu_seqlens[s], len = a.cu_seqlens[s + 1] - row0;
-  const int rr = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int rr = blockIdx.x;
   if (len <= 0 || len > a.max_q_len || rr >= len * a.heads) return;
   const int rank = a.kv_rank;
   const size_t all_rows = (size_t)a.num_tokens * a.heads, row = (size_t)row0 * a.heads + rr;
   const float* wo = reinterpret_cast<const float*>(a.workspace);
   const float* wml = wo + (size_t)splits * all_rows * rank;
-  float m = -INFINITY, l = 0.f;
-  for (int p = 0; p < splits; ++p) m = fmaxf(m, wml[2 * (p * all_rows + row)]);
-  for (int p = 0; p < splits; ++p) {
-    const float mp = wml[2 * (p * all_rows + row)];
-    if (mp > -INFINITY) l += exp2f(mp - m) * wml[2 * (p * all_rows + row) + 1];
-  }
-  bf16* out = reinterpret_cast<bf16*>(a.out) + (int64_t)(row0 + rr / a.heads) * a.out_stride + (int64_t)(rr % a.heads) * rank;
-  const float inv = 1.f / l;
-  for (int d = lane * 4; d < rank; d += 128) {
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int p = 0; p < splits; ++p) {
+  if (threadIdx.x < 32) {
+    float m = -INFINITY, l = 0.f;
+    for (int p = threadIdx.x; p < splits; p += 32) m = fmaxf(m, wml[2 * (p * all_rows + row)]);
+    m = warp_max(m);
+    for (int p = threadIdx.x; p < splits; p += 32) {
       const float mp = wml[2 * (p * all_rows + row)];
-      if (mp == -INFINITY) continue;
-      const float w = exp2f(mp - m) * inv;
+      const float w = mp == -INFINITY ? 0.f : exp2f(mp - m);
+      weight[p] = w;
+      l += w * wml[2 * (p * all_rows + row) + 1];
+    }
+    l = warp_sum(l);
+    __syncwarp();
+    for (int p = threadIdx.x; p < splits; p += 32) weight[p] /= l;
+  }
+  __syncthreads();
+  bf16* out = reinterpret_cast<bf16*>(a.out) + (int64_t)(row0 + rr / a.heads) * a.out_stride + (int64_t)(rr % a.heads) * rank;
+  for (int d = threadIdx.x * 4; d < rank; d += 512) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int p = 0; p < splits; ++p) {
+      const float w = weight[p];
       const float4 v = *reinterpret_cast<const float4*>(wo + (p * all_rows + row) * rank + d);
       acc.x += w * v.x, acc.y += w * v.y, acc.z += w * v.z, acc.w += w * v.w;
     }
@@ -331,35 +341,81 @@ latent_merge_kernel(const b200_latent_attn_args a, int splits) {
   }
 }
 
+enum Kind { kSimt = 1, kMma = 2, kTc = 3 };
 struct Plan {
-  bool mma;
+  Kind kind;
   int splits;
 };
 
-Plan plan(const b200_latent_attn_args& a) {
-  Plan p{false, 1};
+bool tc_supported(const b200_latent_attn_args& a) {
   const int width = a.kv_rank + a.rot_dim;
-  p.mma = a.kernel != 1 && a.dtype == B200_BF16 && a.kv_rank % 16 == 0 && width % 16 == 0 && a.kv_rank <= kMaxRank &&
-          width <= kMaxWidth && a.q_stride % 8 == 0 && a.out_stride % 8 == 0 &&
-          (((uintptr_t)a.q | (uintptr_t)a.cache | (uintptr_t)a.out) & 15) == 0;
-  if (!p.mma) return p;
+  return a.dtype == B200_BF16 && a.scale > 0.f && width % 8 == 0 && a.kv_rank % 8 == 0 && a.kv_rank <= kMaxRank &&
+         width <= 64 * latent_tc::kMaxSlices && a.q_stride == (int64_t)a.heads * width && a.block_size >= 8 &&
+         latent_tc::kKeys % a.block_size == 0 && a.num_slots < (1LL << 31) &&
+         (((uintptr_t)a.q | (uintptr_t)a.cache) & 15) == 0 && tc::encode_fn() != nullptr;
+}
+
+bool mma_supported(const b200_latent_attn_args& a) {
+  const int width = a.kv_rank + a.rot_dim;
+  return a.dtype == B200_BF16 && a.kv_rank % 16 == 0 && width % 16 == 0 && a.kv_rank <= kMaxRank && width <= kMaxWidth &&
+         a.q_stride % 8 == 0 && a.out_stride % 8 == 0 &&
+         (((uintptr_t)a.q | (uintptr_t)a.cache | (uintptr_t)a.out) & 15) == 0;
+}
+
+Plan plan(const b200_latent_attn_args& a) {
+  Plan p{kSimt, 1};
+  if ((a.kernel == 0 || a.kernel == kTc) && tc_supported(a))
+    p.kind = kTc;
+  else if ((a.kernel == 0 || a.kernel == kMma) && mma_supported(a))
+    p.kind = kMma;
+  if (p.kind == kSimt) return p;
   const int64_t items = (int64_t)a.num_seqs * ((a.max_q_len * a.heads + kRows - 1) / kRows);
   int keys = a.max_seq_len;
   if (a.window > 0 && a.window + a.max_q_len < keys) keys = a.window + a.max_q_len;
-  const int tiles = (keys + kKeys - 1) / kKeys;
+  const int tile = p.kind == kTc ? latent_tc::kKeys : kKeys;
+  const int tiles = (keys + tile - 1) / tile;
   if (a.force_splits > 0) {
     p.splits = a.force_splits < tiles ? a.force_splits : (tiles > 0 ? tiles : 1);
+    if (p.splits > kMaxSplits) p.splits = kMaxSplits;
     return p;
   }
-  // waves of 2 CTAs per SM; a wave costs its tiles plus a fill / drain of about 3, a split adds the merge launch
-  const int64_t resident = 2 * (int64_t)(sm_count() > 0 ? sm_count() : 148);
+  // waves of resident CTAs; a wave costs its tiles plus a fill / drain of about 3, a split adds the merge launch
+  const int64_t resident = (p.kind == kTc ? 1 : 2) * (int64_t)(sm_count() > 0 ? sm_count() : 148);
   double best = 1e30;
-  for (int s = 1; s <= 64 && s * 4 <= (tiles > 4 ? tiles : 4); ++s) {
+  for (int s = 1; s <= kMaxSplits && s * 2 <= (tiles > 2 ? tiles : 2); ++s) {
     const double waves = (double)((items * s + resident - 1) / resident);
-    const double cost = waves * ((tiles + s - 1) / s + 3.0) + (s > 1 ? 4.0 + 0.15 * s : 0.0);
+    const double cost = waves * ((tiles + s - 1) / s + 3.0) + (s > 1 ? 3.0 + 0.1 * s : 0.0);
     if (cost < best) best = cost, p.splits = s;
   }
   return p;
+}
+
+int launch_tc(const b200_latent_attn_args& a, int splits, cudaStream_t st) {
+  using namespace latent_tc;
+  Params p;
+  p.block_tables = a.block_tables, p.seq_lens = a.seq_lens, p.cu = a.cu_seqlens, p.out = a.out;
+  p.wo = reinterpret_cast<float*>(a.workspace);
+  p.out_stride = a.out_stride, p.num_tokens = a.num_tokens, p.heads = a.heads, p.rank = a.kv_rank;
+  p.width = a.kv_rank + a.rot_dim, p.slices = (p.width + 63) / 64, p.mtiles = (a.kv_rank + 127) / 128;
+  p.block_size = a.block_size, p.max_blocks = a.max_blocks_per_seq, p.window = a.window, p.max_q_len = a.max_q_len;
+  p.splits = splits, p.scale2 = a.scale * kLog2e;
+  CUtensorMap q_map, c_map;
+  int rc = tc::make_map_2d(&q_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, a.q, p.width, (uint64_t)a.num_tokens * a.heads,
+                           (uint64_t)p.width * 2, 64, latent_tc::kRows, CU_TENSOR_MAP_L2_PROMOTION_L2_128B);
+  if (rc != B200_OK) return rc;
+  rc = tc::make_map_2d(&c_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, a.cache, p.width, (uint64_t)a.num_slots,
+                       (uint64_t)p.width * 2, 64, a.block_size, CU_TENSOR_MAP_L2_PROMOTION_L2_128B);
+  if (rc != B200_OK) return rc;
+  static bool attr = false;
+  if (!attr) {
+    B200_CUDA_OK(cudaFuncSetAttribute(latent_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                      latent_tc::smem_bytes(latent_tc::kMaxSlices)));
+    attr = true;
+  }
+  const int rows = a.max_q_len * a.heads;
+  B200_CUDA_OK(launch_pdl(latent_tc_kernel, dim3((rows + latent_tc::kRows - 1) / latent_tc::kRows, a.num_seqs, splits),
+                          dim3(latent_tc::kThreads), latent_tc::smem_bytes(p.slices), st, q_map, c_map, p));
+  return B200_OK;
 }
 
 }  // namespace
@@ -388,8 +444,8 @@ int b200_latent_attention(const b200_latent_attn_args* a, void* stream) {
   B200_CHECK_ARG(a->num_seqs <= 65535, "latent_attention: batch too large");
   cudaStream_t st = (cudaStream_t)stream;
   const Plan p = plan(*a);
-  if (!p.mma) {
-    B200_CHECK_ARG(a->kernel != 2, "latent_attention: this type or these sizes have no tensor-core form");
+  if (p.kind == kSimt) {
+    B200_CHECK_ARG(a->kernel <= 1, "latent_attention: this type or these sizes have no tensor-core form");
     B200_CHECK_ARG(a->kv_rank <= kSimtThreads * kSimtRegs, "latent_attention: kv_rank %d above %d", a->kv_rank,
                    kSimtThreads * kSimtRegs);
     B200_CHECK_ARG(a->heads <= 65535 && a->num_slots < (1LL << 31), "latent_attention: batch too large");
@@ -401,18 +457,29 @@ int b200_latent_attention(const b200_latent_attn_args* a, void* stream) {
     });
   }
   B200_CHECK_ARG(b200_latent_attention_workspace_bytes(a) <= a->workspace_bytes, "latent_attention: workspace too small");
+  const int rows = a->max_q_len * a->heads;
   static bool attr = false;
-  if (!attr) {
+  if (p.kind == kTc) {
+    const int rc = launch_tc(*a, p.splits, st);
+    if (rc != B200_OK) return rc;
+  } else if (!attr) {
     B200_CUDA_OK(cudaFuncSetAttribute(latent_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                       (int)Smem(kMaxWidth).total));
     attr = true;
   }
-  const int rows = a->max_q_len * a->heads;
-  B200_CUDA_OK(launch_pdl(latent_mma_kernel, dim3((rows + kRows - 1) / kRows, a->num_seqs, p.splits), dim3(kThreads),
+  if (p.kind == kMma)
+    B200_CUDA_OK(launch_pdl(latent_mma_kernel, dim3((rows + kRows - 1) / kRows, a->num_seqs, p.splits), dim3(kThreads),
                           Smem(a->kv_rank + a->rot_dim).total, st, *a, p.splits));
   if (p.splits > 1)
-    B200_CUDA_OK(launch_pdl(latent_merge_kernel, dim3((rows + 7) / 8, a->num_seqs), dim3(256), 0, st, *a, p.splits));
+    B200_CUDA_OK(launch_pdl(latent_merge_kernel, dim3(rows, a->num_seqs), dim3(128), 0, st, *a, p.splits));
   return check_launch("latent_attention");
+}
+
+// 1 if a bounded wait of the tcgen05 kernel ever ran out in this process (its results were then not written).
+int b200_latent_attention_failed(void) {
+  int v = 0;
+  if (cudaMemcpyFromSymbol(&v, latent_tc::g_failed, sizeof(v)) != cudaSuccess) return -1;
+  return v;
 }
 
 }  // extern "C"

@@ -58,6 +58,79 @@ latent_prep_kernel(const b200_latent_prep_args a) {
   }
 }
 
+// 16-bit types with whole 16-byte units everywhere: 8 columns a thread and step, whole rotation pairs.
+template <typename T>
+struct alignas(16) Vec8 {
+  T e[8];
+};
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_prep_vec_kernel(const b200_latent_prep_args a) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float red[8];
+  extern __shared__ float cs[];
+  const int64_t t = blockIdx.x;
+  const int half = a.rot_dims >> 1, tid = threadIdx.x;
+  const float pos = (float)a.positions[t];
+  for (int i = tid; i < half; i += 256) sincosf(pos * a.inv_freq[i], &cs[half + i], &cs[i]);
+  const T* down = reinterpret_cast<const T*>(a.down) + t * a.down_stride;
+  const int64_t slot = a.slot_mapping[t];
+  const bool cached = slot >= 0 && slot < a.num_slots;
+  Vec8<T> c;
+  float ss = 0.f;
+  if (tid * 8 < a.kv_rank) {  // kv_rank <= 2048
+    c = *reinterpret_cast<const Vec8<T>*>(down + tid * 8);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += to_float(c.e[e]) * to_float(c.e[e]);
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  auto rotate = [&](Vec8<T> x, int d) {  // columns d .. d + 7 of the rotated part
+#pragma unroll
+    for (int e = 0; e < 8; e += 2) {
+      if (d + e >= a.rot_dims) break;
+      const int i = (d + e) >> 1;
+      const float u = to_float(x.e[e]), v = to_float(x.e[e + 1]), co = cs[i], si = cs[half + i];
+      x.e[e] = from_float<T>(u * co - v * si);
+      x.e[e + 1] = from_float<T>(v * co + u * si);
+    }
+    return x;
+  };
+  if (cached) {
+    T* row = reinterpret_cast<T*>(a.cache) + slot * (a.kv_rank + a.rot_dim);
+    float total = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) total += red[i];
+    const float inv = 1.f / sqrtf(total / (float)a.kv_rank + a.eps);
+    if (tid * 8 < a.kv_rank) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) c.e[e] = from_float<T>(to_float(c.e[e]) * inv * a.norm_weight[tid * 8 + e]);
+      *reinterpret_cast<Vec8<T>*>(row + tid * 8) = c;
+    }
+    for (int d = tid * 8; d < a.rot_dim; d += 2048)
+      *reinterpret_cast<Vec8<T>*>(row + a.kv_rank + d) =
+          rotate(*reinterpret_cast<const Vec8<T>*>(down + a.kv_rank + d), d);
+  }
+  const T* q = reinterpret_cast<const T*>(a.q) + t * a.q_stride;
+  T* o = reinterpret_cast<T*>(a.q_out) + t * a.q_out_stride;
+  const int first = (a.copy_nope ? 0 : a.rot_offset) >> 3, span = (a.q_cols >> 3) - first, dh = a.dim + a.rot_dim;
+  for (int i = tid; i < a.heads * span; i += 256) {
+    const int h = i / span, col = (first + i - h * span) * 8;
+    const T* qh = q + h * dh;
+    Vec8<T> v;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v.e[e] = from_float<T>(0.f);
+    if (col < a.rot_offset) {
+      if (col < a.dim) v = *reinterpret_cast<const Vec8<T>*>(qh + col);
+    } else if (col < a.rot_offset + a.rot_dim) {
+      v = rotate(*reinterpret_cast<const Vec8<T>*>(qh + a.dim + col - a.rot_offset), col - a.rot_offset);
+    }
+    *reinterpret_cast<Vec8<T>*>(o + (int64_t)h * a.q_cols + col) = v;
+  }
+}
+
 __device__ __forceinline__ float gate_value(const void* gate, int64_t off, int is_f32, int is_half) {
   const float z = is_f32    ? reinterpret_cast<const float*>(gate)[off]
                   : is_half ? to_float(reinterpret_cast<const __half*>(gate)[off])
@@ -206,7 +279,16 @@ int b200_latent_prep(const b200_latent_prep_args* a, void* stream) {
   B200_CHECK_ARG(a->q_cols >= a->rot_offset + a->rot_dim && (!a->copy_nope || a->rot_offset >= a->dim),
                  "latent_prep: query columns overlap");
   if (a->num_tokens <= 0) return B200_OK;
+  auto ok = [](const void* p, int64_t stride) { return ((uintptr_t)p & 15) == 0 && stride % 8 == 0; };
+  const bool vec = ok(a->q, a->q_stride) && ok(a->down, a->down_stride) && ok(a->cache, 0) && ok(a->q_out, a->q_out_stride) &&
+                   a->dim % 8 == 0 && a->rot_dim % 8 == 0 && a->kv_rank % 8 == 0 && a->kv_rank <= 2048 &&
+                   a->q_cols % 8 == 0 && a->rot_offset % 8 == 0;
   return B200_DISPATCH_DTYPE(a->dtype, T, [&]() -> int {
+    if (vec && sizeof(T) == 2) {
+      B200_CUDA_OK(launch_pdl(latent_prep_vec_kernel<T>, dim3(a->num_tokens), dim3(256), a->rot_dims * sizeof(float),
+                              (cudaStream_t)stream, *a));
+      return check_launch("latent_prep");
+    }
     B200_CUDA_OK(launch_pdl(latent_prep_kernel<T>, dim3(a->num_tokens), dim3(128), a->rot_dims * sizeof(float),
                             (cudaStream_t)stream, *a));
     return check_launch("latent_prep");

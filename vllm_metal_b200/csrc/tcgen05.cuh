@@ -23,10 +23,9 @@ __device__ __forceinline__ void mbar_expect_tx(uint32_t bar, uint32_t bytes) {
   asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes)
                : "memory");
 }
-// try_wait WITHOUT a suspend-time hint.  With a hint ptxas emits TRYWAIT + NANOSLEEP.SYNCS <hint>, and the
-// wake-up out of that sleep costs ~0.5-1 us per hand-off (measured: a pipeline doing nothing but mbarrier
-// hand-offs ran at 0.78 us per stage, profiles/r02_qstream_ablation.txt); the bare form spins on the
-// hardware's own short bounded wait.
+// try_wait WITHOUT a suspend-time hint: with one, the wake-up costs ~0.5-1 us per hand-off (measured: a pipeline doing
+// nothing but mbarrier hand-offs ran at 0.78 us per stage, profiles/r02_qstream_ablation.txt); the bare form spins on
+// the hardware's own short bounded wait.
 __device__ __forceinline__ bool mbar_try_wait(uint32_t bar, uint32_t parity) {
   uint32_t ok;
   asm volatile(
@@ -45,8 +44,8 @@ __device__ __forceinline__ void mbar_wait(uint32_t bar, uint32_t parity) {
     if (++spins > (1u << 26)) __trap();  // a protocol bug must fault, not hang the box
   }
 }
-// For warps that wait LONG (producers a ring ahead, epilogue warps a tile ahead): the suspend-time hint makes
-// ptxas emit TRYWAIT + NANOSLEEP.SYNCS, so the waiter stays out of the issue slots the working warps need.
+// For warps that wait LONG (producers a ring ahead, epilogue warps a tile ahead): the suspend-time hint keeps the
+// waiter out of the issue slots the working warps need.
 __device__ __forceinline__ void mbar_wait_parked(uint32_t bar, uint32_t parity) {
   uint32_t spins = 0;
   for (;;) {
@@ -61,6 +60,24 @@ __device__ __forceinline__ void mbar_wait_parked(uint32_t bar, uint32_t parity) 
     if (ok) return;
     if (++spins > (1u << 24)) __trap();
   }
+}
+// One look, no wait (for a warp that watches two barriers).
+__device__ __forceinline__ bool mbar_test(uint32_t bar, uint32_t parity) {
+  uint32_t ok;
+  asm volatile(
+      "{\n\t.reg .pred p;\n\t"
+      "mbarrier.test_wait.parity.shared::cta.b64 p, [%1], %2;\n\t"
+      "selp.u32 %0, 1, 0, p;\n\t}"
+      : "=r"(ok)
+      : "r"(bar), "r"(parity)
+      : "memory");
+  return ok != 0;
+}
+// Bounded wait that reports instead of trapping: the caller abandons its loop, the kernel drains and returns.
+__device__ __forceinline__ bool mbar_wait_or_fail(uint32_t bar, uint32_t parity) {
+  for (uint32_t spins = 0; spins < (1u << 22); ++spins)
+    if (mbar_try_wait(bar, parity)) return true;
+  return false;
 }
 __device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap* map, uint32_t bar,
                                             int c0, int c1) {
@@ -138,6 +155,16 @@ __device__ __forceinline__ uint64_t make_smem_desc(uint32_t addr) {
   uint64_t d = (uint64_t)((addr & 0x3FFFFu) >> 4);
   d |= (uint64_t)1 << 16;
   d |= (uint64_t)(1024 >> 4) << 32;
+  d |= (uint64_t)1 << 46;
+  d |= (uint64_t)2 << 61;
+  return d;
+}
+// MN-major SWIZZLE_128B operand (cute::UMMA canonical layout ((8,n),(8,k)):((1,LBO),(8,SBO)) in 16-byte units):
+// 64 elements of N contiguous in a 128-byte row, rows = k, 8-row groups SBO apart, 64-wide N chunks LBO apart.
+__device__ __forceinline__ uint64_t make_smem_desc_mn(uint32_t addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
+  uint64_t d = (uint64_t)((addr & 0x3FFFFu) >> 4);
+  d |= (uint64_t)(lbo_bytes >> 4) << 16;
+  d |= (uint64_t)(sbo_bytes >> 4) << 32;
   d |= (uint64_t)1 << 46;
   d |= (uint64_t)2 << 61;
   return d;

@@ -27,6 +27,7 @@ HYBRID_SYMBOLS = (
     "b200_latent_attention",
     "b200_latent_attention_workspace_bytes",
     "b200_latent_attention_num_launches",
+    "b200_latent_attention_failed",
     "b200_latent_gather",
 )
 
@@ -278,7 +279,7 @@ class HybridOps:
                          num_seqs: int | None = None, *, kernel: int = 0, force_splits: int = 0) -> torch.Tensor:
         """Attention of ``q [T, H, kv_rank + rot]`` over the paged latent rows; returns ``[T, H, kv_rank]``.  The
         first ``num_seqs`` segments of ``meta`` cover q's rows; ``window <= 0``: causal only.  ``kernel``: 0 auto,
-        1 any-size, 2 tensor cores (raises where it does not apply)."""
+        1 any-size, 2 warp-level tensor cores, 3 tcgen05 (2 and 3 raise where they do not apply)."""
         t, heads, width = q.shape
         if not q.is_contiguous() or not q.is_cuda or cache.dtype != q.dtype or cache.shape[1] != width:
             raise ValueError("latent_attention: q must be contiguous and match the cache rows")
@@ -299,6 +300,10 @@ class HybridOps:
         self._check(self._lib.b200_latent_attention(ctypes.byref(a), _stream()))
         self.launches += self._lib.b200_latent_attention_num_launches(ctypes.byref(a))
         return out
+
+    def latent_attention_failed(self) -> bool:
+        """Whether a wait inside the tcgen05 kernel ever ran out (synchronises)."""
+        return self._lib.b200_latent_attention_failed() != 0
 
     def latent_gather(self, cache, block_tables, first, count, out_row, out, max_count: int, block_size: int,
                       pad: int) -> None:
