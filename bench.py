@@ -663,6 +663,23 @@ def run_b200(args) -> None:
         os._exit(0)
 
 
+def run_hybrid(args) -> None:
+    """--hybrid: one JSON line with prefill / decode throughput and every kernel's roofline, per size."""
+    if args.impl == "reference" or args.gpus != 1:
+        _emit(json.dumps({"impl": args.impl, "unavailable": "hybrid decoders: one GPU, no reference arm"}))
+        return
+    sys.path.insert(0, os.path.join(ROOT, "profiles"))
+    import bench_hybrid
+
+    clocks = ClockSampler(0)
+    clocks.start()
+    clocks.mark()
+    line = bench_hybrid.main(tuple(args.hybrid_sizes.split(",")), steps=min(args.steps, 64), warmup=max(3, args.warmup))
+    clocks.window()
+    line["clocks"] = clocks.stop()
+    _emit(json.dumps(line))
+
+
 _REAL_STDOUT = None
 
 
@@ -689,7 +706,13 @@ def main() -> None:
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--config", default="b", choices=sorted(CONFIGS), help="BASELINE.json config (default b = headline)")
+    ap.add_argument("--hybrid", action="store_true",
+                    help="hybrid decoders (latent attention / Mamba-2 / mLSTM) beside the closest transformer of this framework")
+    ap.add_argument("--hybrid-sizes", default="s,m", help="sizes of profiles/bench_hybrid.py")
     args = ap.parse_args()
+    if args.hybrid:
+        run_hybrid(args)
+        return
     select_config(args.config)
     if args.gpus < CONFIGS[args.config][6] and args.impl == "b200":
         _emit(json.dumps({"config": args.config, "unavailable": f"config {args.config} needs --gpus >= {CONFIGS[args.config][6]}"}))

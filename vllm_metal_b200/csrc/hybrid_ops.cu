@@ -3,6 +3,8 @@
 #include "../../include/b200_hybrid_ops.h"
 #include "common.cuh"
 
+#include <type_traits>
+
 namespace b200 {
 namespace {
 
@@ -157,16 +159,17 @@ mixer_finish_kernel(const b200_mixer_finish_args a, int norm_blocks) {
 }
 
 // The same for 16-bit types whose rows, groups and offsets are whole 16-byte units: 8 columns a thread and step, the
-// group held in registers between its norm and its store.  LANES threads share a group (a warp or the CTA).
+// group held in registers between its norm and its store.  LANES threads share a group, VPL units each; the activation
+// half takes ACT units a thread.
 template <typename T>
 struct alignas(16) Vec8 {
   T e[8];
 };
 __device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 
-template <typename T, int LANES, int VPL>
+template <typename T, int LANES, int VPL, int ACT>
 __global__ void __launch_bounds__(256)
-mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks, int act_vecs) {
+mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks) {
   pdl_trigger();
   pdl_wait();
   const int64_t r = blockIdx.y;
@@ -177,7 +180,7 @@ mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks, int act
     const T* pre = a.pre_gate ? reinterpret_cast<const T*>(a.pre_gate) + r * a.pre_stride : nullptr;
     const T* post = a.post_gate ? reinterpret_cast<const T*>(a.post_gate) + r * a.post_stride : nullptr;
     const int gs = a.group_size > 0 ? a.group_size : LANES * VPL * 8;
-    const int group = LANES == 32 ? blockIdx.x * 8 + (threadIdx.x >> 5) : blockIdx.x;
+    const int group = blockIdx.x * (256 / LANES) + threadIdx.x / LANES;
     const int c0 = group * gs, c1 = min(c0 + gs, a.inner), first = c0 + (threadIdx.x % LANES) * 8;
     Vec8<T> vy[VPL], vg[VPL];
 #pragma unroll
@@ -204,7 +207,14 @@ mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks, int act
       }
     }
     if (a.group_size > 0) {
-      ss = LANES == 32 ? warp_sum(ss) : block_sum<256>(ss, red);
+      ss = warp_sum(ss);
+      if (LANES > 32) {
+        if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+        __syncthreads();
+        ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < LANES / 32; ++i) ss += red[threadIdx.x / LANES * (LANES / 32) + i];
+      }
       inv = 1.f / sqrtf(ss / (float)gs + a.eps);
     }
 #pragma unroll
@@ -229,14 +239,18 @@ mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks, int act
     }
   } else {
     const T* in = reinterpret_cast<const T*>(a.act_in) + r * a.act_stride;
-    const int base = ((int)blockIdx.x - norm_blocks) * act_vecs * 2048 + threadIdx.x * 8;
-    for (int j = 0; j < act_vecs; ++j) {
+    const int base = ((int)blockIdx.x - norm_blocks) * ACT * 2048 + threadIdx.x * 8;
+    Vec8<T> x[ACT];
+#pragma unroll
+    for (int j = 0; j < ACT; ++j)
+      if (base + j * 2048 < a.act_dim) x[j] = *reinterpret_cast<const Vec8<T>*>(in + base + j * 2048);
+#pragma unroll
+    for (int j = 0; j < ACT; ++j) {
       const int i = base + j * 2048;
       if (i >= a.act_dim) break;
-      Vec8<T> x = *reinterpret_cast<const Vec8<T>*>(in + i);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x.e[e] = from_float<T>(gelu_erf_f(to_float(x.e[e])));
-      *reinterpret_cast<Vec8<T>*>(o + a.act_offset + i) = x;
+      for (int e = 0; e < 8; ++e) x[j].e[e] = from_float<T>(gelu_erf_f(to_float(x[j].e[e])));
+      *reinterpret_cast<Vec8<T>*>(o + a.act_offset + i) = x[j];
     }
   }
   if (blockIdx.x == 0 && a.act_dim > 0)
@@ -246,7 +260,7 @@ mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks, int act
 template <typename T>
 bool finish_vec_ok(const b200_mixer_finish_args& a) {
   auto ok = [](const void* p, int64_t stride) { return !p || (((uintptr_t)p & 15) == 0 && stride % 8 == 0); };
-  const int gs = a.group_size > 0 ? a.group_size : 1024;
+  const int gs = a.group_size > 0 ? a.group_size : 2048;
   return sizeof(T) == 2 && ok(a.y, a.y_stride) && ok(a.pre_gate, a.pre_stride) && ok(a.post_gate, a.post_stride) &&
          ok(a.act_in, a.act_stride) && ok(a.out, a.out_stride) && ((uintptr_t)a.weight & 15) == 0 && a.inner % 8 == 0 &&
          gs % 8 == 0 && gs <= 8192 && a.act_dim % 8 == 0 && a.act_offset % 8 == 0 && a.y_head_dim % 8 == 0 &&
@@ -255,18 +269,21 @@ bool finish_vec_ok(const b200_mixer_finish_args& a) {
 
 template <typename T>
 int launch_finish_vec(const b200_mixer_finish_args& a, cudaStream_t st) {
-  const int gs = a.group_size > 0 ? a.group_size : 1024, groups = a.y ? (a.inner + gs - 1) / gs : 0;
-  const bool warp = gs <= 1024;
-  const int vpl = warp ? (gs + 255) / 256 : (gs + 2047) / 2048;
-  const int nb = warp ? (groups + 7) / 8 : groups, vecs = a.rows >= 256 ? 4 : 1;
-  const int ab = (a.act_dim + vecs * 2048 - 1) / (vecs * 2048);
-  auto* kern = warp ? (vpl == 1   ? mixer_finish_vec_kernel<T, 32, 1>
-                       : vpl == 2 ? mixer_finish_vec_kernel<T, 32, 2>
-                                  : mixer_finish_vec_kernel<T, 32, 4>)
-                    : (vpl == 1   ? mixer_finish_vec_kernel<T, 256, 1>
-                       : vpl == 2 ? mixer_finish_vec_kernel<T, 256, 2>
-                                  : mixer_finish_vec_kernel<T, 256, 4>);
-  B200_CUDA_OK(launch_pdl(kern, dim3(nb + ab > 0 ? nb + ab : 1, a.rows), dim3(256), 0, st, a, nb, vecs));
+  const int gs = a.group_size > 0 ? a.group_size : 2048, groups = a.y ? (a.inner + gs - 1) / gs : 0;
+  const int lanes = gs <= 256 ? 32 : gs <= 512 ? 64 : gs <= 1024 ? 128 : 256;
+  const int vpl = gs <= 2048 ? 1 : gs <= 4096 ? 2 : 4, act = a.rows >= 256 ? 2 : 1;
+  const int nb = (groups * lanes + 255) / 256, ab = (a.act_dim + act * 2048 - 1) / (act * 2048);
+  auto pick = [&](auto act_tag) {
+    constexpr int A = decltype(act_tag)::value;
+    return vpl == 4      ? mixer_finish_vec_kernel<T, 256, 4, A>
+           : vpl == 2    ? mixer_finish_vec_kernel<T, 256, 2, A>
+           : lanes == 32 ? mixer_finish_vec_kernel<T, 32, 1, A>
+           : lanes == 64 ? mixer_finish_vec_kernel<T, 64, 1, A>
+           : lanes == 128 ? mixer_finish_vec_kernel<T, 128, 1, A>
+                          : mixer_finish_vec_kernel<T, 256, 1, A>;
+  };
+  auto* kern = act == 2 ? pick(std::integral_constant<int, 2>()) : pick(std::integral_constant<int, 1>());
+  B200_CUDA_OK(launch_pdl(kern, dim3(nb + ab > 0 ? nb + ab : 1, a.rows), dim3(256), 0, st, a, nb));
   return check_launch("mixer_finish");
 }
 
