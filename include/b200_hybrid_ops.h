@@ -68,11 +68,12 @@ int b200_causal_conv(const void* in, const float* weight, const float* bias, voi
  * state [slots, heads, key_dim, value_dim]; mLSTM also norm_state [slots, heads, vtiles, key_dim] and max_state
  * [slots, heads, vtiles] with vtiles = ceil(value_dim / 64): one copy per 64-wide value tile, so that the tiles of a
  * head never wait for one another.
- * Segments of at most seq_limit rows run token by token; longer ones (16-bit types only) in chunks of
- * B200_RECURRENCE_CHUNK rows listed by chunk_seq / chunk_row (segment and first row of every chunk of every longer
+ * Segments of at most seq_limit rows run token by token; longer ones (bf16 only) in chunks of `chunk` rows (what
+ * b200_recurrence_chunk says) listed by chunk_seq / chunk_row (segment and first row of every chunk of every longer
  * segment, in order; seq_chunk0[s] = index of segment s's first chunk).  workspace: see
  * b200_recurrence_workspace_bytes. */
-#define B200_RECURRENCE_CHUNK 64
+#define B200_RECURRENCE_CHUNK 64     /* warp-level tensor cores */
+#define B200_RECURRENCE_CHUNK_TC 128 /* tcgen05: key_dim a multiple of 64, at most 512 */
 typedef struct b200_recurrence_args {
   const void* q;
   const void* k;
@@ -97,12 +98,14 @@ typedef struct b200_recurrence_args {
   size_t workspace_bytes;
   int64_t q_stride, k_stride, v_stride, gate_stride, out_stride;
   int32_t kind, dtype, num_tokens, num_seqs, num_heads, num_groups, key_dim, value_dim;
-  int32_t num_chunks, seq_limit;
+  int32_t num_chunks, chunk, seq_limit;
   float q_scale, gate_cap;
 } b200_recurrence_args;
 size_t b200_recurrence_workspace_bytes(const b200_recurrence_args* a);
-/* 1 if the chunked form covers this call's type and sizes (it needs 16-bit operands and 16-multiples). */
-int b200_recurrence_can_chunk(const b200_recurrence_args* a);
+/* Rows per chunk of the form that covers this call's type and sizes; 0: token by token only. */
+int b200_recurrence_chunk(const b200_recurrence_args* a);
+/* Synchronises.  1 if a bounded wait inside a tcgen05 kernel ever ran out (that launch wrote no results), else 0. */
+int b200_recurrence_failed(void);
 int b200_recurrence(const b200_recurrence_args* a, void* stream);
 int b200_recurrence_num_launches(const b200_recurrence_args* a);
 

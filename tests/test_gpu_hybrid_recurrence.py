@@ -73,30 +73,35 @@ class Case:
 
 
 SHAPES = [("ssd", 6, 3, 24, 16), ("ssd", 4, 1, 128, 64), ("ssd", 2, 2, 72, 136), ("mlstm", 3, 3, 40, 24),
-          ("mlstm", 2, 2, 128, 200), ("ssd", 3, 3, 5, 7), ("mlstm", 1, 1, 9, 65)]
+          ("mlstm", 2, 2, 128, 200), ("ssd", 4, 2, 64, 64), ("mlstm", 2, 2, 192, 72), ("mlstm", 1, 1, 256, 64),
+          ("ssd", 1, 1, 320, 8), ("ssd", 3, 3, 5, 7), ("mlstm", 1, 1, 9, 65)]
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("kind,heads,groups,k,v", SHAPES)
 def test_whole_sequences_portions_and_single_rows_agree_with_the_oracle(ops, kind, heads, groups, k, v, dtype):
-    c = Case(kind, heads, groups, k, v, [200, 131, 70, 3], dtype)
+    c = Case(kind, heads, groups, k, v, [300, 231, 70, 3], dtype)
     slots = {0: 4, 1: 2, 2: 1, 3: 3}
-    c.step(ops, {0: 130, 1: 1, 2: 64, 3: 2}, slots)      # chunk edges, a fresh single row, a portion of two
-    c.step(ops, {2: 1, 0: 1, 1: 65}, slots)
+    c.step(ops, {0: 230, 1: 1, 2: 64, 3: 2}, slots)      # chunk edges, a fresh single row, a portion of two
+    c.step(ops, {2: 1, 0: 1, 1: 165}, slots)
     c.step(ops, {3: 1, 1: 5, 0: 4, 2: 5}, slots)          # on both sides of the token-by-token limit
     c.step(ops, {0: 65, 1: 60}, slots)
 
 
-@pytest.mark.parametrize("kind,heads,groups,k,v", SHAPES[:5])
-def test_chunked_and_sequential_forms_leave_the_same_state(ops, kind, heads, groups, k, v):
-    a, b = (Case(kind, heads, groups, k, v, [190], torch.bfloat16) for _ in range(2))
-    for n in (150, 40):
-        a.step(ops, {0: n}, {0: 1})
+@pytest.mark.parametrize("kind,heads,groups,k,v", SHAPES[:9])
+@pytest.mark.parametrize("chunk", [64, 128])
+def test_chunked_and_sequential_forms_leave_the_same_state(ops, kind, heads, groups, k, v, chunk):
+    if chunk == 128 and k % 64:
+        pytest.skip("the tcgen05 form takes whole 64-wide slices of the key")
+    a, b = (Case(kind, heads, groups, k, v, [390], torch.bfloat16) for _ in range(2))
+    for n in (350, 40):
+        a.step(ops, {0: n}, {0: 1}, chunk=chunk)
         b.step(ops, {0: n}, {0: 1}, force_sequential=True)
     torch.testing.assert_close(a.state[1], b.state[1], rtol=2e-4, atol=2e-5 * float(b.state[1].abs().max()))
     if kind == "mlstm":
         torch.testing.assert_close(a.norm[1], b.norm[1], rtol=2e-4, atol=2e-5 * float(b.norm[1].abs().max()))
         torch.testing.assert_close(a.max[1], b.max[1], rtol=1e-4, atol=1e-3)
+    assert not ops.recurrence_failed()
 
 
 @pytest.mark.parametrize("kind", ["ssd", "mlstm"])

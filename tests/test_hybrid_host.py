@@ -170,9 +170,13 @@ def test_hybrid_cache_sizes_follow_the_layers():
 
 def test_segment_metadata_lists_chunks_and_splits_the_batch():
     m = segments([1, 3, 70, 130], [40, 3, 71, 400], block_size=16, device="cpu")
-    assert m.max_q_len == 130 and m.num_chunks == 5 and m.has_short
-    assert m.chunk_seq.tolist() == [2, 2, 3, 3, 3] and m.chunk_row.tolist() == [4, 68, 74, 138, 202]
-    assert m.seq_chunk0.tolist()[2:] == [0, 2]
+    assert m.max_q_len == 130 and m.has_short
+    c = m.chunks[64]
+    assert c.num == 5 and c.seq.tolist() == [2, 2, 3, 3, 3] and c.row.tolist() == [4, 68, 74, 138, 202]
+    assert c.seq0.tolist()[2:] == [0, 2]
+    c = m.chunks[128]
+    assert c.seq.tolist() == [2, 3, 3] and c.row.tolist() == [4, 74, 202] and c.seq0.tolist()[2:] == [0, 1]
+    assert not segments([1, 4], [9, 4], device="cpu").chunks
     assert m.split(64) == (2, 4, 3) and m.split(100) == (3, 74, 70) and m.split(1000) == (4, 204, 130)
     assert m.expand_plan(1000, 0) is None
     p = m.expand_plan(64, 50)

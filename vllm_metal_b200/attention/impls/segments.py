@@ -10,7 +10,7 @@ from dataclasses import dataclass, field
 import numpy as np
 import torch
 
-from ...metal.hybrid_ops import RECURRENCE_CHUNK
+from ...metal.hybrid_ops import RECURRENCE_CHUNKS
 from .sdpa import _KernelMetadata, _positions, _to_device
 
 # Segments of at most this many rows go through the recurrences token by token (their state is streamed once per row);
@@ -35,15 +35,22 @@ class ExpandPlan:
 
 
 @dataclass(frozen=True, eq=False)
+class ChunkList:
+    """The chunks of the segments longer than ``CHUNK_LIMIT``, for one chunk size."""
+
+    num: int
+    seq: torch.Tensor   # int32 [num] segment of every chunk
+    row: torch.Tensor   # int32 [num] its first row
+    seq0: torch.Tensor  # int32 [S] index of a segment's first chunk
+
+
+@dataclass(frozen=True, eq=False)
 class SegmentMetadata(_KernelMetadata):
     state_slots: torch.Tensor = None  # int32 [S]
     max_q_len: int = 1
-    num_chunks: int = 0
     has_short: bool = True
     chunk_limit: int = CHUNK_LIMIT
-    chunk_seq: torch.Tensor | None = None
-    chunk_row: torch.Tensor | None = None
-    seq_chunk0: torch.Tensor | None = None
+    chunks: dict[int, ChunkList] = field(default_factory=dict)  # by rows per chunk; empty: no long segment
     # host copies the expansion plans are made from (None on the all-decode path, which never expands)
     q_lens: np.ndarray | None = None
     context_lens: np.ndarray | None = None
@@ -101,21 +108,22 @@ def segment_metadata(ctx, block_size: int, device) -> SegmentMetadata:
         table[i, :len(row)] = row
     slots = ctx.state_slots if ctx.state_slots is not None else [0] * n
     long = np.nonzero(q > CHUNK_LIMIT)[0]
-    chunk_seq, chunk_row = [], []
-    seq_chunk0 = np.zeros(n, dtype=np.int32)
-    for s in long:
-        seq_chunk0[s] = len(chunk_seq)
-        rows = range(int(cu[s]), int(cu[s + 1]), RECURRENCE_CHUNK)
-        chunk_seq += [int(s)] * len(rows)
-        chunk_row += list(rows)
     dev = lambda x, t=torch.int32: _to_device(np.asarray(x), t, device)  # noqa: E731
+    chunks = {}
+    for size in RECURRENCE_CHUNKS if len(long) else ():
+        seq, row, seq0 = [], [], np.zeros(n, dtype=np.int32)
+        for s in long:
+            seq0[s] = len(seq)
+            starts = range(int(cu[s]), int(cu[s + 1]), size)
+            seq += [int(s)] * len(starts)
+            row += list(starts)
+        chunks[size] = ChunkList(len(seq), dev(np.asarray(seq, dtype=np.int32)), dev(np.asarray(row, dtype=np.int32)),
+                                 dev(seq0))
     meta = SegmentMetadata(
         slot_mapping=dev(np.asarray(ctx.slot_mapping, dtype=np.int64), torch.int64),
         seq_lens=dev(np.asarray(ctx.context_lens, dtype=np.int32)), cu_seqlens_q=dev(cu.astype(np.int32)),
         block_tables=dev(table), block_size=block_size, max_seq_len=max(ctx.context_lens), positions=dev(_positions(ctx)),
-        state_slots=dev(np.asarray(slots, dtype=np.int32)), max_q_len=int(q.max()), num_chunks=len(chunk_seq),
-        has_short=len(long) < n, chunk_seq=dev(np.asarray(chunk_seq, dtype=np.int32)) if chunk_seq else None,
-        chunk_row=dev(np.asarray(chunk_row, dtype=np.int32)) if chunk_seq else None,
-        seq_chunk0=dev(seq_chunk0) if chunk_seq else None, q_lens=q, context_lens=np.asarray(ctx.context_lens))
+        state_slots=dev(np.asarray(slots, dtype=np.int32)), max_q_len=int(q.max()),
+        has_short=len(long) < n, chunks=chunks, q_lens=q, context_lens=np.asarray(ctx.context_lens))
     ctx.kernel_metadata_cache[key] = meta
     return meta

@@ -4,8 +4,9 @@
 //
 //  * sequential form: one CTA per (64-wide value tile, head, segment); the fp32 state is streamed once per token
 //    (decode: HBM-bound at 2 * key_dim * value_dim * 4 bytes per head), any type and any size.
-//  * chunked form (16-bit operands): recurrence_chunk.cuh, tensor cores over 64-row chunks, all chunks in parallel.
-#include "recurrence_chunk.cuh"
+//  * chunked forms (bf16 operands), all chunks in parallel: recurrence_tc.cuh (tcgen05, 128 rows) where the key size is
+//    whole 64-wide slices, else recurrence_chunk.cuh (warp-level tensor cores, 64 rows).
+#include "recurrence_tc.cuh"
 
 namespace b200 {
 namespace rec {
@@ -168,7 +169,16 @@ size_t b200_recurrence_workspace_bytes(const b200_recurrence_args* a) {
   return a && a->num_chunks > 0 ? rec::Workspace::bytes(*a) : 0;
 }
 
-int b200_recurrence_can_chunk(const b200_recurrence_args* a) { return a && rec::can_chunk(*a) ? 1 : 0; }
+int b200_recurrence_chunk(const b200_recurrence_args* a) {
+  if (!a) return 0;
+  return rec::tcr::supported(*a) ? B200_RECURRENCE_CHUNK_TC : rec::can_chunk(*a) ? B200_RECURRENCE_CHUNK : 0;
+}
+
+int b200_recurrence_failed(void) {
+  int v = 0;
+  if (cudaMemcpyFromSymbol(&v, rec::tcr::g_failed, sizeof(v)) != cudaSuccess) return -1;
+  return v;
+}
 
 int b200_recurrence_num_launches(const b200_recurrence_args* a) {
   return (a->seq_limit > 0 ? 1 : 0) + (a->num_chunks > 0 ? 3 : 0);
@@ -194,7 +204,12 @@ int b200_recurrence(const b200_recurrence_args* a, void* stream) {
     if (rc != B200_OK) return rc;
   }
   if (a->num_chunks > 0) {
-    B200_CHECK_ARG(rec::can_chunk(*a), "recurrence: this type or these sizes have no chunked form");
+    if (a->chunk == B200_RECURRENCE_CHUNK_TC) {
+      B200_CHECK_ARG(rec::tcr::supported(*a), "recurrence: this type or these sizes have no tcgen05 form");
+      return a->kind == rec::kSsd ? rec::tcr::launch<rec::kSsd>(*a, st) : rec::tcr::launch<rec::kMlstm>(*a, st);
+    }
+    B200_CHECK_ARG(a->chunk == B200_RECURRENCE_CHUNK && rec::can_chunk(*a),
+                   "recurrence: this type or these sizes have no chunked form of %d rows", a->chunk);
     return a->kind == rec::kSsd ? rec::launch_chunked<rec::kSsd>(*a, st) : rec::launch_chunked<rec::kMlstm>(*a, st);
   }
   return B200_OK;

@@ -36,13 +36,14 @@ struct Workspace {
   }
 };
 
-// The gates of a chunk's rows.  cum[t]: cumulative log decay; SSD: src[t] = step size dt, mLSTM: src[t] = log input
-// weight minus cum[t], top[t] = running maximum of src.  Rows past the end contribute nothing.  All 128 threads call.
-template <int KIND>
+// The gates of a chunk's ROWS rows.  cum[t]: cumulative log decay; SSD: src[t] = step size dt, mLSTM: src[t] = log input
+// weight minus cum[t], top[t] = running maximum of src.  Rows past the end contribute nothing.  All threads call.
+template <int KIND, int ROWS = kChunk>
 __device__ __forceinline__ void chunk_gates(const b200_recurrence_args& a, int row0, int rows, int h, float* cum,
                                             float* src, float* top) {
   const int tid = threadIdx.x;
-  if (tid < kChunk) {
+  constexpr int E = ROWS / 32;
+  if (tid < ROWS) {
     float decay = 0.f, in = KIND == kSsd ? 0.f : -INFINITY;
     if (tid < rows) {
       const int64_t off = (int64_t)(row0 + tid) * a.gate_stride + h;
@@ -61,8 +62,12 @@ __device__ __forceinline__ void chunk_gates(const b200_recurrence_args& a, int r
   }
   __syncthreads();
   if (tid < 32) {
-    float x0 = cum[2 * tid], x1 = cum[2 * tid + 1];
-    float run = x0 + x1;
+    float x[E], run = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      run += cum[E * tid + e];
+      x[e] = run;
+    }
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
       const float y = __shfl_up_sync(0xffffffffu, run, o);
@@ -70,15 +75,17 @@ __device__ __forceinline__ void chunk_gates(const b200_recurrence_args& a, int r
     }
     float excl = __shfl_up_sync(0xffffffffu, run, 1);
     if (tid == 0) excl = 0.f;
-    x0 += excl;
-    x1 += x0;
-    cum[2 * tid] = x0;
-    cum[2 * tid + 1] = x1;
+#pragma unroll
+    for (int e = 0; e < E; ++e) cum[E * tid + e] = x[e] + excl;
     if (KIND == kMlstm) {
-      const float s0 = src[2 * tid] - x0, s1 = src[2 * tid + 1] - x1;
-      src[2 * tid] = s0;
-      src[2 * tid + 1] = s1;
-      float mx = fmaxf(s0, s1);
+      float mx = -INFINITY, m[E];
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const float v = src[E * tid + e] - (x[e] + excl);
+        src[E * tid + e] = v;
+        mx = fmaxf(mx, v);
+        m[e] = mx;
+      }
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const float y = __shfl_up_sync(0xffffffffu, mx, o);
@@ -86,8 +93,8 @@ __device__ __forceinline__ void chunk_gates(const b200_recurrence_args& a, int r
       }
       float below = __shfl_up_sync(0xffffffffu, mx, 1);
       if (tid == 0) below = -INFINITY;
-      top[2 * tid] = fmaxf(below, s0);
-      top[2 * tid + 1] = mx;
+#pragma unroll
+      for (int e = 0; e < E; ++e) top[E * tid + e] = fmaxf(below, m[e]);
     }
   }
   __syncthreads();
@@ -105,7 +112,7 @@ __device__ __forceinline__ void load_tile(bf16* dst, const bf16* src, int64_t st
 __device__ __forceinline__ int chunk_rows(const b200_recurrence_args& a, int c, int* row0) {
   const int s = a.chunk_seq[c];
   *row0 = a.chunk_row[c];
-  return min(kChunk, a.cu_seqlens[s + 1] - *row0);
+  return min(a.chunk, a.cu_seqlens[s + 1] - *row0);
 }
 
 // ---- 1: the chunk's own contribution -----------------------------------------------------------
@@ -226,7 +233,7 @@ chunk_scan_kernel(const b200_recurrence_args a, int state_blocks) {
   const int s = blockIdx.z, h = blockIdx.y;
   const int len = a.cu_seqlens[s + 1] - a.cu_seqlens[s];
   if (len <= a.seq_limit) return;
-  const int nc = (len + kChunk - 1) / kChunk, cfirst = a.seq_chunk0[s];
+  const int nc = (len + a.chunk - 1) / a.chunk, cfirst = a.seq_chunk0[s];
   const bool fresh = a.seq_lens[s] == len;
   const int K = a.key_dim, V = a.value_dim;
   const Workspace ws(a);

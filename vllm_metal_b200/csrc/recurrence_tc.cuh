@@ -1,0 +1,434 @@
+// The chunked recurrence of recurrence_chunk.cuh on tcgen05, 128 rows a chunk: steps 1 (a chunk's own contribution) and 3
+// (its outputs) as M = 128 products with fp32 accumulators in tensor memory; step 2 (the scan) is shared.  q, k, v tiles
+// arrive by TMA; every 32-bit factor enters as three bf16 terms (24 significant bits), one product per term into the
+// same accumulator.
+#pragma once
+
+#include "recurrence_chunk.cuh"
+#include "tcgen05.cuh"
+
+namespace b200 {
+namespace rec {
+namespace tcr {
+using namespace tc;
+
+constexpr int C = B200_RECURRENCE_CHUNK_TC, kThreads = 256;
+constexpr int kTile = C * 128;  // bytes of a [128 rows x 64 bf16] tile, 128-byte rows, swizzled
+constexpr int kMaxKey = 512;
+
+__device__ int g_failed = 0;
+
+__device__ __forceinline__ uint32_t swz(int row, int chunk) { return row * 128 + ((chunk ^ (row & 7)) << 4); }
+__device__ __forceinline__ void st16(uint32_t addr, const uint32_t* v) {
+  asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]) : "memory");
+}
+// 8 fp32 values as three 16-byte units of bf16, one per term tile at `addr` + j * kTile.
+__device__ __forceinline__ void split8(uint32_t addr, const float* x) {
+  uint32_t t[kTerms][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    uint32_t p[kTerms];
+    mma::split_pair<kTerms>(x[2 * i], x[2 * i + 1], p);
+#pragma unroll
+    for (int j = 0; j < kTerms; ++j) t[j][i] = p[j];
+  }
+#pragma unroll
+  for (int j = 0; j < kTerms; ++j) st16(addr + j * kTile, t[j]);
+}
+__device__ __forceinline__ float ld_bf16(const uint8_t* tile, int row, int col) {
+  return to_float(*reinterpret_cast<const bf16*>(tile + swz(row, col >> 3) + (col & 7) * 2));
+}
+
+inline int state_smem(int key_dim) { return ((key_dim + 63) / 64 + kTerms) * kTile + 4096 + 1024; }
+constexpr int kOutputSmem = (2 + 2 + 1 + kTerms) * kTile + 8192 + 1024;
+
+// ---- 1: U [key_dim x 64] = K^T (w V), A = K^T (MN-major), B = the weighted values' terms (MN-major) ----------
+template <int KIND>
+__global__ void __launch_bounds__(kThreads)
+state_kernel(const __grid_constant__ CUtensorMap k_map, const b200_recurrence_args a) {
+  extern __shared__ __align__(1024) uint8_t raw[];
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
+  const int K = a.key_dim, V = a.value_dim, c0 = tile * kTileV, slices = (K + 63) / 64, mtiles = (K + 127) / 128;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = h / (a.num_heads / a.num_groups);
+  const uint32_t base = (smem_u32(raw) + 1023u) & ~1023u;
+  uint8_t* gen = raw + (base - smem_u32(raw));
+  const uint32_t sk = base, sv = sk + slices * kTile, sb = sv + kTerms * kTile;
+  float* cum = reinterpret_cast<float*>(gen + (sb - base) + 64);
+  float *src = cum + C, *top = src + C, *wgt = top + C;
+  volatile uint32_t* tmem_gen = reinterpret_cast<volatile uint32_t*>(gen + (sb - base) + 32);
+  const uint32_t bar_load = sb, bar_mma = sb + 8;
+  int row0;
+  const int rows = chunk_rows(a, c, &row0);
+  if (tid == 0) {
+    mbar_init(bar_load, 1);
+    mbar_init(bar_mma, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == 1) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(sb + 32), "n"(256) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_gen;
+  if (warp == 0 && elect_one()) {
+    mbar_expect_tx(bar_load, slices * kTile);
+    for (int i = 0; i < slices; ++i) tma_load_2d(sk + i * kTile, &k_map, bar_load, g * K + i * 64, row0);
+  }
+  __syncwarp();
+  chunk_gates<KIND, C>(a, row0, rows, h, cum, src, top);
+  const float total = cum[C - 1];
+  if (tid < C) {
+    float w = 0.f;
+    if (tid < rows) w = KIND == kSsd ? src[tid] * expf(total - cum[tid]) : expf(src[tid] - top[C - 1]);
+    wgt[tid] = w;
+  }
+  __syncthreads();
+  const Workspace ws(a);
+  float* scal = ws.scal + 4 * ((size_t)c * a.num_heads + h);
+  if (tile == 0 && tid == 0) {
+    scal[0] = total;
+    if (KIND == kMlstm) {
+      scal[1] = top[C - 1];
+      const int s = a.chunk_seq[c];
+      if (row0 == a.cu_seqlens[s]) {
+        const bool fresh = a.seq_lens[s] == a.cu_seqlens[s + 1] - row0;
+        scal[2] = fresh ? 0.f : a.max_state[((int64_t)a.slots[s] * a.num_heads + h) * gridDim.x];
+      }
+    }
+  }
+  {  // weighted values: two threads a row, 32 columns each
+    const int r = tid >> 1, cc0 = (tid & 1) * 32;
+    const bf16* vr = reinterpret_cast<const bf16*>(a.v) + (int64_t)(row0 + r) * a.v_stride + (int64_t)h * V + c0;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int cc = cc0 + i * 8;
+      uint4 x4 = make_uint4(0, 0, 0, 0);
+      if (r < rows && c0 + cc < V) x4 = *reinterpret_cast<const uint4*>(vr + cc);
+      const bf16* xe = reinterpret_cast<const bf16*>(&x4);
+      float x[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = wgt[r] * to_float(xe[e]);
+      split8(sv + swz(r, cc >> 3), x);
+    }
+  }
+  fence_proxy_async();
+  __syncthreads();
+  bool ok = mbar_wait_or_fail(bar_load, 0);
+  if (warp == 0) {
+    tc_fence_after();
+    if (ok && elect_one()) {
+      const uint32_t idesc = make_idesc(1, 128, 64) | (1u << 15) | (1u << 16);
+      const uint64_t da = make_smem_desc_mn(sk, kTile, 1024), db = make_smem_desc_mn(sv, kTile, 1024);
+      for (int m = 0; m < mtiles; ++m)
+#pragma unroll
+        for (int k = 0; k < C / 16; ++k)
+#pragma unroll
+          for (int j = 0; j < kTerms; ++j)
+            tc_mma_f16(tmem + m * 64, da + 2 * m * (kTile >> 4) + k * (2048 >> 4), db + j * (kTile >> 4) + k * (2048 >> 4),
+                       idesc, (k | j) != 0 ? 1u : 0u);
+      tc_commit(bar_mma);
+    }
+    __syncwarp();
+  }
+  if (KIND == kMlstm && tile == 0 && ok) {  // the key sum beside the products
+    for (int kd = tid; kd < K; kd += kThreads) {
+      const uint8_t* t = gen + (sk - base) + (kd >> 6) * kTile;
+      float n = 0.f;
+      for (int r = 0; r < rows; ++r) n += wgt[r] * ld_bf16(t, r, kd & 63);
+      ws.keysum[((size_t)c * a.num_heads + h) * K + kd] = n;
+    }
+  }
+  ok = ok && mbar_wait_or_fail(bar_mma, 0);
+  tc_fence_after();
+  if (ok) {
+    float* U = ws.state + ((size_t)c * a.num_heads + h) * K * V;
+    const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
+    const int half = (warp >> 2) * 32;
+    for (int m = 0; m < mtiles; ++m) {
+      uint32_t u[32];
+      tmem_ld<32>(tmem + lane_addr + m * 64 + half, u);
+      const int kd = m * 128 + (warp & 3) * 32 + lane;
+      if (kd < K)
+#pragma unroll
+        for (int i = 0; i < 32; i += 4)
+          if (c0 + half + i < V)
+            *reinterpret_cast<uint4*>(U + (size_t)kd * V + c0 + half + i) = make_uint4(u[i], u[i + 1], u[i + 2], u[i + 3]);
+    }
+  } else if (lane == 0) {
+    atomicExch(&g_failed, 1);
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "n"(256) : "memory");
+  }
+}
+
+// ---- 3: outputs.  Tensor memory: scores [0,128) | q S_in [128,192) | (weights scores) v [192,256) | the weighted scores'
+// terms, 64 columns of bf16 pairs each [256,448) -----------------------------------------------------------------
+constexpr int TM_SC = 0, TM_O1 = 128, TM_O2 = 192, TM_P = 256;
+
+template <int KIND>
+__global__ void __launch_bounds__(kThreads)
+output_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
+              const __grid_constant__ CUtensorMap v_map, const b200_recurrence_args a) {
+  extern __shared__ __align__(1024) uint8_t raw[];
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
+  const int K = a.key_dim, V = a.value_dim, c0 = tile * kTileV;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = h / (a.num_heads / a.num_groups);
+  const uint32_t base = (smem_u32(raw) + 1023u) & ~1023u;
+  uint8_t* gen = raw + (base - smem_u32(raw));
+  const uint32_t sq = base, sk = sq + 2 * kTile, sv = sk + 2 * kTile, ss = sv + kTile, sb = ss + kTerms * kTile;
+  float* cum = reinterpret_cast<float*>(gen + (sb - base) + 64);
+  float *src = cum + C, *top = src + C, *scale = top + C, *part = scale + C /* [2][C] */, *nin = part + 2 * C /* [128] */;
+  volatile uint32_t* tmem_gen = reinterpret_cast<volatile uint32_t*>(gen + (sb - base) + 48);
+  const uint32_t bar_load = sb, bar_v = sb + 8, bar_mma = sb + 16;
+  int row0;
+  const int rows = chunk_rows(a, c, &row0);
+  if (tid == 0) {
+    mbar_init(bar_load, 1);
+    mbar_init(bar_v, 1);
+    mbar_init(bar_mma, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == 1) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(sb + 48), "n"(512) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_gen;
+  const Workspace ws(a);
+  const float* S = ws.state + ((size_t)c * a.num_heads + h) * K * V;
+  const float* keysum = ws.keysum + ((size_t)c * a.num_heads + h) * K;
+  const int slabs = (K + 127) / 128;
+  auto load = [&](int slab) {  // the slab's 64-wide slices of q and k
+    const int n = min(2, (K - slab * 128 + 63) / 64);
+    if (warp == 0 && elect_one()) {
+      mbar_expect_tx(bar_load, 2 * n * kTile);
+      for (int i = 0; i < n; ++i) {
+        tma_load_2d(sq + i * kTile, &q_map, bar_load, g * K + slab * 128 + i * 64, row0);
+        tma_load_2d(sk + i * kTile, &k_map, bar_load, g * K + slab * 128 + i * 64, row0);
+      }
+    }
+    __syncwarp();
+  };
+  load(0);
+  if (warp == 0 && elect_one()) {
+    mbar_expect_tx(bar_v, kTile);
+    tma_load_2d(sv, &v_map, bar_v, h * V + c0, row0);
+  }
+  __syncwarp();
+  chunk_gates<KIND, C>(a, row0, rows, h, cum, src, top);
+  const float m_in = KIND == kMlstm ? ws.scal[4 * ((size_t)c * a.num_heads + h) + 3] : 0.f;
+  if (tid < C) {
+    if (KIND == kMlstm) top[tid] = fmaxf(m_in, top[tid]);
+    scale[tid] = KIND == kSsd ? expf(cum[tid]) : expf(m_in - top[tid]);
+  }
+  bool ok = true;
+  float dot = 0.f;  // mLSTM: q . normaliser-on-entry, row tid / 2, alternate 16-byte units
+  for (int slab = 0; slab < slabs; ++slab) {
+    const int dims = min(128, K - slab * 128);
+    {  // the state on entry, split: two threads a key row, 32 columns each
+      const int r = tid >> 1, cc0 = (tid & 1) * 32;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int cc = cc0 + i * 8;
+        float x[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] = 0.f;
+        if (r < dims && c0 + cc < V) {
+          const float* p = S + (size_t)(slab * 128 + r) * V + c0 + cc;
+          *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(p);
+          *reinterpret_cast<float4*>(x + 4) = *reinterpret_cast<const float4*>(p + 4);
+        }
+        split8(ss + swz(r, cc >> 3), x);
+      }
+      if (KIND == kMlstm && tid < 128) nin[tid] = tid < dims ? keysum[slab * 128 + tid] : 0.f;
+    }
+    fence_proxy_async();
+    __syncthreads();
+    ok = ok && mbar_wait_or_fail(bar_load, slab & 1);
+    if (warp == 0) {
+      tc_fence_after();
+      if (ok && elect_one()) {
+        const uint32_t idesc_qk = make_idesc(1, 128, 128), idesc_qs = make_idesc(1, 128, 64) | (1u << 16);
+        const uint64_t dq = make_smem_desc(sq), dk = make_smem_desc(sk), ds = make_smem_desc_mn(ss, kTile, 1024);
+        for (int k = 0; k < dims / 16; ++k) {
+          const uint64_t off = (uint64_t)((k >> 2) * (kTile >> 4) + (k & 3) * 2);
+          tc_mma_f16(tmem + TM_SC, dq + off, dk + off, idesc_qk, (slab | k) != 0 ? 1u : 0u);
+#pragma unroll
+          for (int j = 0; j < kTerms; ++j)
+            tc_mma_f16(tmem + TM_O1, dq + off, ds + j * (kTile >> 4) + k * (2048 >> 4), idesc_qs,
+                       (slab | k | j) != 0 ? 1u : 0u);
+        }
+        tc_commit(bar_mma);
+      }
+      __syncwarp();
+    }
+    if (KIND == kMlstm && ok) {
+      const int r = tid >> 1;
+      for (int u = tid & 1; u < dims / 8; u += 2) {
+        const uint4 x4 = *reinterpret_cast<const uint4*>(gen + (u >> 3) * kTile + swz(r, u & 7));
+        const bf16* x = reinterpret_cast<const bf16*>(&x4);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) dot += to_float(x[e]) * nin[u * 8 + e];
+      }
+    }
+    ok = ok && mbar_wait_or_fail(bar_mma, slab & 1);
+    tc_fence_after();
+    __syncthreads();  // everybody is done with the slab's tiles
+    if (slab + 1 < slabs) load(slab + 1);
+  }
+  if (KIND == kMlstm) dot += __shfl_xor_sync(0xffffffffu, dot, 1);
+  // scores -> weights x scores; thread = row, 64 columns
+  const int t = (warp & 3) * 32 + lane, half = warp >> 2;
+  const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
+  {
+    float sum = 0.f;
+    const float ct = cum[t], tt = KIND == kMlstm ? top[t] : 0.f;
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int s0 = half * 64 + q * 32;
+      uint32_t terms[kTerms][16];
+      if (s0 <= (warp & 3) * 32 + 31) {  // some column is on or below the diagonal for some lane of the warp
+        uint32_t u[32];
+        tmem_ld<32>(tmem + lane_addr + TM_SC + s0, u);
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) {
+          float x[2];
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int s = s0 + i + e;
+            float w = 0.f;
+            if (s <= t && s < rows) w = KIND == kSsd ? __expf(ct - cum[s]) * src[s] : __expf(src[s] - tt);
+            x[e] = __uint_as_float(u[i + e]) * w * a.q_scale;
+            if (w == 0.f) x[e] = 0.f;
+            sum += x[e];
+          }
+          uint32_t p[kTerms];
+          mma::split_pair<kTerms>(x[0], x[1], p);
+#pragma unroll
+          for (int j = 0; j < kTerms; ++j) terms[j][i >> 1] = p[j];
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < kTerms; ++j)
+#pragma unroll
+          for (int i = 0; i < 16; ++i) terms[j][i] = 0u;
+      }
+#pragma unroll
+      for (int j = 0; j < kTerms; ++j) tmem_st16(tmem + lane_addr + TM_P + j * 64 + s0 / 2, terms[j]);
+    }
+    if (KIND == kMlstm) part[half * C + t] = sum;
+  }
+  if (KIND == kMlstm && (tid & 1) == 0) nin[tid >> 1] = dot;  // row tid / 2; nin is free after the last slab
+  tc_fence_before();
+  __syncthreads();
+  ok = ok && mbar_wait_or_fail(bar_v, 0);
+  if (warp == 0) {
+    tc_fence_after();
+    if (ok && elect_one()) {
+      const uint32_t idesc = make_idesc(1, 128, 64) | (1u << 16);
+      const uint64_t dv = make_smem_desc_mn(sv, kTile, 1024);
+#pragma unroll
+      for (int k = 0; k < C / 16; ++k)
+#pragma unroll
+        for (int j = 0; j < kTerms; ++j)
+          tc_mma_f16_ts(tmem + TM_O2, tmem + TM_P + j * 64 + k * 8, dv + k * (2048 >> 4), idesc, (k | j) != 0 ? 1u : 0u);
+      tc_commit(bar_mma);
+    }
+    __syncwarp();
+  }
+  ok = ok && mbar_wait_or_fail(bar_mma, slabs & 1);
+  tc_fence_after();
+  if (!ok) {
+    if (lane == 0) atomicExch(&g_failed, 1);
+  } else {
+    uint32_t u1[32], u2[32];
+    tmem_ld<32>(tmem + lane_addr + TM_O1 + half * 32, u1);
+    tmem_ld<32>(tmem + lane_addr + TM_O2 + half * 32, u2);
+    const float f = scale[t] * a.q_scale, skip = KIND == kSsd ? a.skip[h] : 0.f;
+    float div = 1.f;
+    if (KIND == kMlstm)
+      div = 1.f / (fmaxf(fabsf(part[t] + part[C + t] + nin[t] * f), expf(-(cum[t] + top[t]))) + 1e-6f);
+    if (t < rows) {
+      bf16* out = reinterpret_cast<bf16*>(a.out) + (int64_t)(row0 + t) * a.out_stride + (int64_t)h * V + c0;
+#pragma unroll
+      for (int i = 0; i < 32; i += 8) {
+        const int col = half * 32 + i;
+        if (c0 + col >= V) break;
+        const uint4 v4 = *reinterpret_cast<const uint4*>(gen + (sv - base) + swz(t, col >> 3));
+        const bf16* v = reinterpret_cast<const bf16*>(&v4);
+        uint4 r4;
+        bf16* r = reinterpret_cast<bf16*>(&r4);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          float y = (__uint_as_float(u1[i + e]) * f + __uint_as_float(u2[i + e])) * div;
+          if (KIND == kSsd) y += skip * to_float(v[e]);
+          r[e] = __float2bfloat16_rn(y);
+        }
+        *reinterpret_cast<uint4*>(out + col) = r4;
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "n"(512) : "memory");
+  }
+}
+
+inline bool supported(const b200_recurrence_args& a) {
+  return can_chunk(a) && a.key_dim % 64 == 0 && a.key_dim <= kMaxKey && ((uintptr_t)a.out & 15) == 0 && a.out_stride % 8 == 0 &&
+         state_smem(a.key_dim) <= 227 * 1024 && encode_fn() != nullptr;
+}
+
+template <int KIND>
+int launch(const b200_recurrence_args& a, cudaStream_t st) {
+  B200_CHECK_ARG(a.workspace && a.workspace_bytes >= Workspace::bytes(a), "recurrence: workspace too small");
+  B200_CHECK_ARG(a.chunk_seq && a.chunk_row && a.seq_chunk0, "recurrence: no chunk list");
+  B200_CHECK_ARG(a.num_chunks <= 65535, "recurrence: more than 65535 chunks");
+  CUtensorMap q_map, k_map, v_map;
+  const struct {
+    CUtensorMap* map;
+    const void* ptr;
+    uint64_t cols;
+    int64_t stride;
+  } maps[3] = {{&q_map, a.q, (uint64_t)a.num_groups * a.key_dim, a.q_stride},
+               {&k_map, a.k, (uint64_t)a.num_groups * a.key_dim, a.k_stride},
+               {&v_map, a.v, (uint64_t)a.num_heads * a.value_dim, a.v_stride}};
+  for (const auto& m : maps) {
+    const int rc = make_map_2d(m.map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, m.ptr, m.cols, (uint64_t)a.num_tokens,
+                               (uint64_t)m.stride * 2, 64, C, CU_TENSOR_MAP_L2_PROMOTION_L2_128B);
+    if (rc != B200_OK) return rc;
+  }
+  static bool attr = false;  // per instantiation
+  if (!attr) {
+    B200_CUDA_OK(cudaFuncSetAttribute(state_kernel<KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, state_smem(kMaxKey)));
+    B200_CUDA_OK(cudaFuncSetAttribute(output_kernel<KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, kOutputSmem));
+    attr = true;
+  }
+  const dim3 grid((a.value_dim + kTileV - 1) / kTileV, a.num_heads, a.num_chunks);
+  B200_CUDA_OK(launch_pdl(state_kernel<KIND>, grid, dim3(kThreads), state_smem(a.key_dim), st, k_map, a));
+  const int blocks = (a.key_dim * a.value_dim / 4 + kScanThreads - 1) / kScanThreads;
+  B200_CUDA_OK(launch_pdl(chunk_scan_kernel<KIND>, dim3(blocks + (KIND == kMlstm ? 1 : 0), a.num_heads, a.num_seqs),
+                          dim3(kScanThreads), 0, st, a, blocks));
+  B200_CUDA_OK(launch_pdl(output_kernel<KIND>, grid, dim3(kThreads), kOutputSmem, st, q_map, k_map, v_map, a));
+  return check_launch("recurrence (tcgen05)");
+}
+
+}  // namespace tcr
+}  // namespace rec
+}  // namespace b200

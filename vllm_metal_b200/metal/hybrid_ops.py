@@ -20,7 +20,8 @@ HYBRID_SYMBOLS = (
     "b200_causal_conv",
     "b200_recurrence",
     "b200_recurrence_workspace_bytes",
-    "b200_recurrence_can_chunk",
+    "b200_recurrence_chunk",
+    "b200_recurrence_failed",
     "b200_recurrence_num_launches",
     "b200_latent_prep",
     "b200_head_linear",
@@ -31,7 +32,7 @@ HYBRID_SYMBOLS = (
     "b200_latent_gather",
 )
 
-RECURRENCE_CHUNK = 64
+RECURRENCE_CHUNKS = (64, 128)  # rows per chunk of the two chunked forms
 RECURRENCE_TILE_V = 64
 
 
@@ -54,7 +55,7 @@ RecurrenceArgs = _struct(
       "chunk_row seq_chunk0 out workspace",
     Z="workspace_bytes",
     L="q_stride k_stride v_stride gate_stride out_stride",
-    I="kind dtype num_tokens num_seqs num_heads num_groups key_dim value_dim num_chunks seq_limit",
+    I="kind dtype num_tokens num_seqs num_heads num_groups key_dim value_dim num_chunks chunk seq_limit",
     F="q_scale gate_cap")
 LatentPrepArgs = _struct(
     "LatentPrepArgs", "b200_latent_prep_args",
@@ -88,7 +89,7 @@ def bind_hybrid(lib: ctypes.CDLL) -> None:
         getattr(lib, f"b200_{name}_workspace_bytes").argtypes = [ctypes.POINTER(struct)]
         getattr(lib, f"b200_{name}_workspace_bytes").restype = ctypes.c_size_t
         getattr(lib, f"b200_{name}_num_launches").argtypes = [ctypes.POINTER(struct)]
-    lib.b200_recurrence_can_chunk.argtypes = [ctypes.POINTER(RecurrenceArgs)]
+    lib.b200_recurrence_chunk.argtypes = [ctypes.POINTER(RecurrenceArgs)]
 
 
 def _rows(name: str, t: torch.Tensor, dtype: torch.dtype | None = None) -> torch.Tensor:
@@ -166,6 +167,10 @@ class HybridOps:
         self._check(self._lib.b200_mixer_finish(ctypes.byref(a), _stream()))
         self.launches += 1
 
+    def recurrence_failed(self) -> bool:
+        """Whether a wait inside a tcgen05 kernel of the recurrences ever ran out (synchronises)."""
+        return self._lib.b200_recurrence_failed() != 0
+
     def causal_conv(self, x, weight, bias, state, seg, silu: bool = True) -> torch.Tensor:
         """Depthwise causal convolution of ``x [T, C]`` over the segments of ``seg`` (carried inputs in
         ``state [slots, taps-1, C]``); ``weight`` fp32 ``[taps, C]``, ``bias`` fp32 ``[C]``."""
@@ -184,10 +189,11 @@ class HybridOps:
 
     def recurrence(self, kind: str, q, k, v, gate_a, gate_b, seg, state, *, heads: int, groups: int, key_dim: int,
                    value_dim: int, bias_a, bias_b=None, rate=None, skip=None, norm_state=None, max_state=None,
-                   q_scale: float = 1.0, gate_cap: float = 0.0, force_sequential: bool = False) -> torch.Tensor:
+                   q_scale: float = 1.0, gate_cap: float = 0.0, force_sequential: bool = False,
+                   chunk: int = 0) -> torch.Tensor:
         """Gated linear recurrence (``kind`` "ssd" / "mlstm") over the segments of ``seg``: outputs ``[T, heads *
         value_dim]``, the slots' fp32 states updated in place.  Segments longer than ``seg.chunk_limit`` rows run in
-        chunks on tensor cores where type and sizes allow."""
+        chunks on tensor cores where type and sizes allow (``chunk``: a form by its rows per chunk, 0 = auto)."""
         a = RecurrenceArgs()
         for name, t in (("q", q), ("k", k), ("v", v), ("gate_a", gate_a), ("gate_b", gate_b)):
             if t is not None:
@@ -216,12 +222,16 @@ class HybridOps:
         a.num_heads, a.num_groups, a.key_dim, a.value_dim = heads, groups, key_dim, value_dim
         a.q_scale, a.gate_cap = float(q_scale), float(gate_cap)
         a.seq_limit = 0x7FFFFFFF
-        if seg.num_chunks > 0 and not force_sequential and self._lib.b200_recurrence_can_chunk(ctypes.byref(a)):
-            a.num_chunks = seg.num_chunks
+        a.chunk = 0
+        if seg.chunks and not force_sequential:
+            a.chunk = chunk or self._lib.b200_recurrence_chunk(ctypes.byref(a))
+        if a.chunk:
+            plan = seg.chunks[a.chunk]
+            a.num_chunks = plan.num
             # the sequential launch only exists for the segments that need it
             a.seq_limit = seg.chunk_limit if seg.has_short else 0
-            a.chunk_seq, a.chunk_row = seg.chunk_seq.data_ptr(), seg.chunk_row.data_ptr()
-            a.seq_chunk0 = seg.seq_chunk0.data_ptr()
+            a.chunk_seq, a.chunk_row = plan.seq.data_ptr(), plan.row.data_ptr()
+            a.seq_chunk0 = plan.seq0.data_ptr()
             need = self._lib.b200_recurrence_workspace_bytes(ctypes.byref(a))
             ws = self._workspace(v.device, need)
             a.workspace, a.workspace_bytes = ws.data_ptr(), ws.numel()
