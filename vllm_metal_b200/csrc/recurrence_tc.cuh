@@ -22,7 +22,14 @@ __device__ __forceinline__ uint32_t swz(int row, int chunk) { return row * 128 +
 __device__ __forceinline__ void st16(uint32_t addr, const uint32_t* v) {
   asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(addr), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]) : "memory");
 }
-// 8 fp32 values as three 16-byte units of bf16, one per term tile at `addr` + j * kTile.
+__device__ __forceinline__ void tmem_st8(uint32_t taddr, const uint32_t* v) {  // tmem_st_wait() before the next use
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};" ::"r"(taddr), "r"(v[0]), "r"(v[1]),
+               "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7])
+               : "memory");
+}
+__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+// 8 fp32 values as three 16-byte units of bf16, one per term tile at `addr` + j * STRIDE.
+template <int STRIDE = kTile>
 __device__ __forceinline__ void split8(uint32_t addr, const float* x) {
   uint32_t t[kTerms][4];
 #pragma unroll
@@ -33,14 +40,15 @@ __device__ __forceinline__ void split8(uint32_t addr, const float* x) {
     for (int j = 0; j < kTerms; ++j) t[j][i] = p[j];
   }
 #pragma unroll
-  for (int j = 0; j < kTerms; ++j) st16(addr + j * kTile, t[j]);
+  for (int j = 0; j < kTerms; ++j) st16(addr + j * STRIDE, t[j]);
 }
 __device__ __forceinline__ float ld_bf16(const uint8_t* tile, int row, int col) {
   return to_float(*reinterpret_cast<const bf16*>(tile + swz(row, col >> 3) + (col & 7) * 2));
 }
 
 inline int state_smem(int key_dim) { return ((key_dim + 63) / 64 + kTerms) * kTile + 4096 + 1024; }
-constexpr int kOutputSmem = (2 + 2 + 1 + kTerms) * kTile + 8192 + 1024;
+constexpr int kHalfTile = 64 * 128;  // 64 key dimensions of the state, one term
+constexpr int kOutputSmem = (2 + 2 + 1) * kTile + kTerms * kHalfTile + 4608 + 1024;  // two CTAs an SM
 
 // ---- 1: U [key_dim x 64] = K^T (w V), A = K^T (MN-major), B = the weighted values' terms (MN-major) ----------
 template <int KIND>
@@ -170,12 +178,13 @@ state_kernel(const __grid_constant__ CUtensorMap k_map, const b200_recurrence_ar
   }
 }
 
-// ---- 3: outputs.  Tensor memory: scores [0,128) | q S_in [128,192) | (weights scores) v [192,256) | the weighted scores'
-// terms, 64 columns of bf16 pairs each [256,448) -----------------------------------------------------------------
-constexpr int TM_SC = 0, TM_O1 = 128, TM_O2 = 192, TM_P = 256;
+// ---- 3: outputs.  Tensor memory, 256 columns so that two CTAs share an SM: scores [0,128), over them later two terms of
+// the weighted scores (64 columns of bf16 pairs each; the third follows in a second pass over the first one's columns)
+// | q S_in [128,192) | (weighted scores) v [192,256) -----------------------------------------------------------
+constexpr int TM_SC = 0, TM_O1 = 128, TM_O2 = 192;
 
 template <int KIND>
-__global__ void __launch_bounds__(kThreads)
+__global__ void __launch_bounds__(kThreads, 2)
 output_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
               const __grid_constant__ CUtensorMap v_map, const b200_recurrence_args a) {
   extern __shared__ __align__(1024) uint8_t raw[];
@@ -187,7 +196,7 @@ output_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
   const int g = h / (a.num_heads / a.num_groups);
   const uint32_t base = (smem_u32(raw) + 1023u) & ~1023u;
   uint8_t* gen = raw + (base - smem_u32(raw));
-  const uint32_t sq = base, sk = sq + 2 * kTile, sv = sk + 2 * kTile, ss = sv + kTile, sb = ss + kTerms * kTile;
+  const uint32_t sq = base, sk = sq + 2 * kTile, sv = sk + 2 * kTile, ss = sv + kTile, sb = ss + kTerms * kHalfTile;
   float* cum = reinterpret_cast<float*>(gen + (sb - base) + 64);
   float *src = cum + C, *top = src + C, *scale = top + C, *part = scale + C /* [2][C] */, *nin = part + 2 * C /* [128] */;
   volatile uint32_t* tmem_gen = reinterpret_cast<volatile uint32_t*>(gen + (sb - base) + 48);
@@ -201,7 +210,7 @@ output_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (warp == 1) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(sb + 48), "n"(512) : "memory");
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(sb + 48), "n"(256) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
   tc_fence_before();
@@ -237,121 +246,148 @@ output_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
   }
   bool ok = true;
   float dot = 0.f;  // mLSTM: q . normaliser-on-entry, row tid / 2, alternate 16-byte units
+  // the state on entry goes through shared memory 64 key dimensions at a time: four threads a key row, 16 columns each
+  const int sr = tid >> 2, sc0 = (tid & 3) * 16;
+  float x[16];
+  auto fetch_state = [&](int k0) {
+#pragma unroll
+    for (int i = 0; i < 16; i += 4)
+      *reinterpret_cast<float4*>(x + i) = k0 + sr < K && c0 + sc0 + i < V
+                                              ? *reinterpret_cast<const float4*>(S + (size_t)(k0 + sr) * V + c0 + sc0 + i)
+                                              : make_float4(0.f, 0.f, 0.f, 0.f);
+  };
+  fetch_state(0);
+  int passes = 0;  // completed phases of bar_mma
   for (int slab = 0; slab < slabs; ++slab) {
     const int dims = min(128, K - slab * 128);
-    {  // the state on entry, split: two threads a key row, 32 columns each
-      const int r = tid >> 1, cc0 = (tid & 1) * 32;
+    for (int part64 = 0; part64 * 64 < dims; ++part64) {
+      split8<kHalfTile>(ss + swz(sr, sc0 >> 3), x);
+      split8<kHalfTile>(ss + swz(sr, (sc0 >> 3) + 1), x + 8);
+      if (KIND == kMlstm && part64 == 0 && tid < 128) nin[tid] = tid < dims ? keysum[slab * 128 + tid] : 0.f;
+      fence_proxy_async();
+      __syncthreads();
+      if (part64 == 0) ok = ok && mbar_wait_or_fail(bar_load, slab & 1);
+      if (warp == 0) {
+        tc_fence_after();
+        if (ok && elect_one()) {
+          const uint32_t idesc_qk = make_idesc(1, 128, 128), idesc_qs = make_idesc(1, 128, 64) | (1u << 16);
+          const uint64_t dq = make_smem_desc(sq) + part64 * (kTile >> 4), dk = make_smem_desc(sk) + part64 * (kTile >> 4);
+          const uint64_t ds = make_smem_desc_mn(ss, kHalfTile, 1024);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int cc = cc0 + i * 8;
-        float x[8];
+          for (int k = 0; k < 4; ++k) {
+            const uint32_t more = (slab | part64 | k) != 0 ? 1u : 0u;
+            tc_mma_f16(tmem + TM_SC, dq + 2 * k, dk + 2 * k, idesc_qk, more);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = 0.f;
-        if (r < dims && c0 + cc < V) {
-          const float* p = S + (size_t)(slab * 128 + r) * V + c0 + cc;
-          *reinterpret_cast<float4*>(x) = *reinterpret_cast<const float4*>(p);
-          *reinterpret_cast<float4*>(x + 4) = *reinterpret_cast<const float4*>(p + 4);
+            for (int j = 0; j < kTerms; ++j)
+              tc_mma_f16(tmem + TM_O1, dq + 2 * k, ds + j * (kHalfTile >> 4) + k * (2048 >> 4), idesc_qs, more | (j != 0 ? 1u : 0u));
+          }
+          tc_commit(bar_mma);
         }
-        split8(ss + swz(r, cc >> 3), x);
+        __syncwarp();
       }
-      if (KIND == kMlstm && tid < 128) nin[tid] = tid < dims ? keysum[slab * 128 + tid] : 0.f;
-    }
-    fence_proxy_async();
-    __syncthreads();
-    ok = ok && mbar_wait_or_fail(bar_load, slab & 1);
-    if (warp == 0) {
+      fetch_state(slab * 128 + part64 * 64 + 64);
+      if (KIND == kMlstm && ok) {
+        const int r = tid >> 1;
+        for (int u = part64 * 8 + (tid & 1); u < part64 * 8 + 8; u += 2) {
+          const uint4 x4 = *reinterpret_cast<const uint4*>(gen + (u >> 3) * kTile + swz(r, u & 7));
+          const bf16* qx = reinterpret_cast<const bf16*>(&x4);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) dot += to_float(qx[e]) * nin[u * 8 + e];
+        }
+      }
+      ok = ok && mbar_wait_or_fail(bar_mma, passes & 1);
+      ++passes;
       tc_fence_after();
-      if (ok && elect_one()) {
-        const uint32_t idesc_qk = make_idesc(1, 128, 128), idesc_qs = make_idesc(1, 128, 64) | (1u << 16);
-        const uint64_t dq = make_smem_desc(sq), dk = make_smem_desc(sk), ds = make_smem_desc_mn(ss, kTile, 1024);
-        for (int k = 0; k < dims / 16; ++k) {
-          const uint64_t off = (uint64_t)((k >> 2) * (kTile >> 4) + (k & 3) * 2);
-          tc_mma_f16(tmem + TM_SC, dq + off, dk + off, idesc_qk, (slab | k) != 0 ? 1u : 0u);
-#pragma unroll
-          for (int j = 0; j < kTerms; ++j)
-            tc_mma_f16(tmem + TM_O1, dq + off, ds + j * (kTile >> 4) + k * (2048 >> 4), idesc_qs,
-                       (slab | k | j) != 0 ? 1u : 0u);
-        }
-        tc_commit(bar_mma);
-      }
-      __syncwarp();
     }
-    if (KIND == kMlstm && ok) {
-      const int r = tid >> 1;
-      for (int u = tid & 1; u < dims / 8; u += 2) {
-        const uint4 x4 = *reinterpret_cast<const uint4*>(gen + (u >> 3) * kTile + swz(r, u & 7));
-        const bf16* x = reinterpret_cast<const bf16*>(&x4);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) dot += to_float(x[e]) * nin[u * 8 + e];
-      }
-    }
-    ok = ok && mbar_wait_or_fail(bar_mma, slab & 1);
-    tc_fence_after();
     __syncthreads();  // everybody is done with the slab's tiles
     if (slab + 1 < slabs) load(slab + 1);
   }
   if (KIND == kMlstm) dot += __shfl_xor_sync(0xffffffffu, dot, 1);
-  // scores -> weights x scores; thread = row, 64 columns
+  // scores -> weights x scores; thread = row, 64 columns.  Both column halves are read before either is overwritten.
   const int t = (warp & 3) * 32 + lane, half = warp >> 2;
   const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
+  uint32_t third[32];
   {
     float sum = 0.f;
     const float ct = cum[t], tt = KIND == kMlstm ? top[t] : 0.f;
+    const int s0 = half * 64;
+    const bool any = s0 <= (warp & 3) * 32 + 31;  // some column is on or below the diagonal for some lane of the warp
+    uint32_t u[64];
+    if (any) {
 #pragma unroll
-    for (int q = 0; q < 2; ++q) {
-      const int s0 = half * 64 + q * 32;
-      uint32_t terms[kTerms][16];
-      if (s0 <= (warp & 3) * 32 + 31) {  // some column is on or below the diagonal for some lane of the warp
-        uint32_t u[32];
-        tmem_ld<32>(tmem + lane_addr + TM_SC + s0, u);
+      for (int q = 0; q < 2; ++q) {
+        uint32_t w[32];
+        tmem_ld<32>(tmem + lane_addr + TM_SC + s0 + q * 32, w);
 #pragma unroll
-        for (int i = 0; i < 32; i += 2) {
-          float x[2];
+        for (int i = 0; i < 32; ++i) u[q * 32 + i] = w[i];
+      }
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      uint32_t t0[16], t1[16];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+        t0[i] = t1[i] = 0u;
+        third[q * 8 + i] = 0u;
+        if (any) {
+          float y[2];
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            const int s = s0 + i + e;
-            float w = 0.f;
-            if (s <= t && s < rows) w = KIND == kSsd ? __expf(ct - cum[s]) * src[s] : __expf(src[s] - tt);
-            x[e] = __uint_as_float(u[i + e]) * w * a.q_scale;
-            if (w == 0.f) x[e] = 0.f;
-            sum += x[e];
+            const int s = s0 + q * 16 + 2 * i + e;
+            const bool see = s <= t && s < rows;
+            const float w = KIND == kSsd ? __expf(ct - cum[s]) * src[s] : __expf(src[s] - tt);
+            y[e] = see ? __uint_as_float(u[q * 16 + 2 * i + e]) * w * a.q_scale : 0.f;
+            sum += y[e];
           }
           uint32_t p[kTerms];
-          mma::split_pair<kTerms>(x[0], x[1], p);
-#pragma unroll
-          for (int j = 0; j < kTerms; ++j) terms[j][i >> 1] = p[j];
+          mma::split_pair<kTerms>(y[0], y[1], p);
+          t0[i] = p[0], t1[i] = p[1], third[q * 8 + i] = p[2];
         }
-      } else {
-#pragma unroll
-        for (int j = 0; j < kTerms; ++j)
-#pragma unroll
-          for (int i = 0; i < 16; ++i) terms[j][i] = 0u;
       }
-#pragma unroll
-      for (int j = 0; j < kTerms; ++j) tmem_st16(tmem + lane_addr + TM_P + j * 64 + s0 / 2, terms[j]);
+      tmem_st8(tmem + lane_addr + TM_SC + half * 32 + q * 8, t0);
+      tmem_st8(tmem + lane_addr + TM_SC + 64 + half * 32 + q * 8, t1);
     }
     if (KIND == kMlstm) part[half * C + t] = sum;
   }
   if (KIND == kMlstm && (tid & 1) == 0) nin[tid >> 1] = dot;  // row tid / 2; nin is free after the last slab
+  tmem_st_wait();
   tc_fence_before();
   __syncthreads();
   ok = ok && mbar_wait_or_fail(bar_v, 0);
-  if (warp == 0) {
-    tc_fence_after();
-    if (ok && elect_one()) {
-      const uint32_t idesc = make_idesc(1, 128, 64) | (1u << 16);
-      const uint64_t dv = make_smem_desc_mn(sv, kTile, 1024);
+  const uint32_t idesc_pv = make_idesc(1, 128, 64) | (1u << 16);
+  const uint64_t dv = make_smem_desc_mn(sv, kTile, 1024);
+  auto product = [&](int terms, uint32_t first) {
+    if (warp == 0) {
+      tc_fence_after();
+      if (ok && elect_one()) {
 #pragma unroll
-      for (int k = 0; k < C / 16; ++k)
-#pragma unroll
-        for (int j = 0; j < kTerms; ++j)
-          tc_mma_f16_ts(tmem + TM_O2, tmem + TM_P + j * 64 + k * 8, dv + k * (2048 >> 4), idesc, (k | j) != 0 ? 1u : 0u);
-      tc_commit(bar_mma);
+        for (int k = 0; k < C / 16; ++k)
+          for (int j = 0; j < terms; ++j)
+            tc_mma_f16_ts(tmem + TM_O2, tmem + TM_SC + j * 64 + k * 8, dv + k * (2048 >> 4), idesc_pv,
+                          first | ((k | j) != 0 ? 1u : 0u));
+        tc_commit(bar_mma);
+      }
+      __syncwarp();
     }
-    __syncwarp();
+    ok = ok && mbar_wait_or_fail(bar_mma, passes & 1);
+    ++passes;
+    tc_fence_after();
+  };
+  product(2, 0u);
+#pragma unroll
+  for (int q = 0; q < 4; ++q) {
+    uint32_t w[16];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) w[i] = third[q * 8 + i];
+    tmem_st8(tmem + lane_addr + TM_SC + half * 32 + q * 8, w);
   }
-  ok = ok && mbar_wait_or_fail(bar_mma, slabs & 1);
-  tc_fence_after();
+  tmem_st_wait();
+  tc_fence_before();
+  __syncthreads();
+  product(1, 1u);
   if (!ok) {
     if (lane == 0) atomicExch(&g_failed, 1);
   } else {
@@ -386,7 +422,7 @@ output_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "n"(512) : "memory");
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "n"(256) : "memory");
   }
 }
 
