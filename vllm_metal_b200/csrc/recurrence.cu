@@ -181,7 +181,7 @@ int b200_recurrence_failed(void) {
 }
 
 int b200_recurrence_num_launches(const b200_recurrence_args* a) {
-  return (a->seq_limit > 0 ? 1 : 0) + (a->num_chunks > 0 ? 3 : 0);
+  return (a->seq_limit > 0 ? 1 : 0) + (a->num_chunks > 0 ? (a->chunk == B200_RECURRENCE_CHUNK_TC ? 4 : 3) : 0);
 }
 
 int b200_recurrence(const b200_recurrence_args* a, void* stream) {

@@ -23,16 +23,18 @@ constexpr int kTileElems = 64 * kPad;
 
 // workspace: U / S_in [chunks][heads][K][V], then per (chunk, head): key-sum [K], then {total, amax, m_in, first_m}
 struct Workspace {
-  float *state, *keysum, *scal;
+  float *state, *keysum, *scal, *gates;  // gates (128-row form): per (chunk, head) {cum, src, top, weight}[128]
   __host__ __device__ Workspace(const b200_recurrence_args& a) {
     const size_t ch = (size_t)a.num_chunks * a.num_heads;
     state = reinterpret_cast<float*>(a.workspace);
     keysum = state + ch * a.key_dim * a.value_dim;
     scal = keysum + (a.kind == kMlstm ? ch * a.key_dim : 0);
+    gates = scal + 4 * ch;
   }
   static size_t bytes(const b200_recurrence_args& a) {
     const size_t ch = (size_t)a.num_chunks * a.num_heads;
-    return (ch * a.key_dim * a.value_dim + (a.kind == kMlstm ? ch * a.key_dim : 0) + 4 * ch) * sizeof(float);
+    return (ch * a.key_dim * a.value_dim + (a.kind == kMlstm ? ch * a.key_dim : 0) + 4 * ch +
+            (a.chunk == B200_RECURRENCE_CHUNK_TC ? ch * 4 * B200_RECURRENCE_CHUNK_TC : 0)) * sizeof(float);
   }
 };
 

@@ -1,4 +1,4 @@
-// The chunked recurrence of recurrence_chunk.cuh on tcgen05, 128 rows a chunk: steps 1 (a chunk's own contribution) and 3
+// The chunked recurrence of recurrence_chunk.cuh on tcgen05, 128 rows a chunk: the gates once per (chunk, head), steps 1 (a chunk's own contribution) and 3
 // (its outputs) as M = 128 products with fp32 accumulators in tensor memory; step 2 (the scan) is shared.  q, k, v tiles
 // arrive by TMA; every 32-bit factor enters as three bf16 terms (24 significant bits), one product per term into the
 // same accumulator.
@@ -46,9 +46,91 @@ __device__ __forceinline__ float ld_bf16(const uint8_t* tile, int row, int col) 
   return to_float(*reinterpret_cast<const bf16*>(tile + swz(row, col >> 3) + (col & 7) * 2));
 }
 
-inline int state_smem(int key_dim) { return ((key_dim + 63) / 64 + kTerms) * kTile + 4096 + 1024; }
+inline int state_smem(int key_dim) { return ((key_dim + 63) / 64 + kTerms) * kTile + 1024 + 1024; }
 constexpr int kHalfTile = 64 * 128;  // 64 key dimensions of the state, one term
 constexpr int kOutputSmem = (2 + 2 + 1) * kTile + kTerms * kHalfTile + 4608 + 1024;  // two CTAs an SM
+
+// ---- 0: gates.  One warp per (chunk, head), 4 consecutive rows a lane; what steps 1 and 3 need of them -----------
+template <int KIND>
+__global__ void __launch_bounds__(kThreads)
+gates_kernel(const b200_recurrence_args a) {
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.y, h = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= a.num_heads) return;
+  int row0;
+  const int rows = chunk_rows(a, c, &row0);
+  float cum[4], src[4], top[4], run = 0.f;
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const int t = lane * 4 + e;
+    float decay = 0.f;
+    src[e] = KIND == kSsd ? 0.f : -INFINITY;
+    if (t < rows) {
+      const int64_t off = (int64_t)(row0 + t) * a.gate_stride + h;
+      const float ga = to_float(reinterpret_cast<const bf16*>(a.gate_a)[off]);
+      if (KIND == kSsd) {
+        src[e] = softplus_f(ga + a.bias_a[h]);
+        decay = -a.rate[h] * src[e];
+      } else {
+        const float gb = to_float(reinterpret_cast<const bf16*>(a.gate_b)[off]);
+        src[e] = a.gate_cap * tanhf((ga + a.bias_a[h]) / a.gate_cap);
+        decay = -softplus_f(-a.gate_cap * tanhf((gb + a.bias_b[h]) / a.gate_cap));
+      }
+    }
+    run += decay;
+    cum[e] = run;
+  }
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float y = __shfl_up_sync(0xffffffffu, run, o);
+    if (lane >= o) run += y;
+  }
+  float excl = __shfl_up_sync(0xffffffffu, run, 1);
+  if (lane == 0) excl = 0.f;
+  const float total = __shfl_sync(0xffffffffu, run, 31);
+  float mx = -INFINITY;
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    cum[e] += excl;
+    if (KIND == kMlstm) src[e] -= cum[e];
+    mx = fmaxf(mx, src[e]);
+    top[e] = mx;
+  }
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float y = __shfl_up_sync(0xffffffffu, mx, o);
+    if (lane >= o) mx = fmaxf(mx, y);
+  }
+  float below = __shfl_up_sync(0xffffffffu, mx, 1);
+  if (lane == 0) below = -INFINITY;
+  const float amax = __shfl_sync(0xffffffffu, mx, 31);
+  const Workspace ws(a);
+  float4* g = reinterpret_cast<float4*>(ws.gates + ((size_t)c * a.num_heads + h) * 4 * C) + lane;
+  float w[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    top[e] = fmaxf(top[e], below);
+    w[e] = lane * 4 + e >= rows ? 0.f : KIND == kSsd ? src[e] * expf(total - cum[e]) : expf(src[e] - amax);
+  }
+  g[0] = make_float4(cum[0], cum[1], cum[2], cum[3]);
+  g[C / 4] = make_float4(src[0], src[1], src[2], src[3]);
+  g[C / 2] = make_float4(top[0], top[1], top[2], top[3]);
+  g[3 * C / 4] = make_float4(w[0], w[1], w[2], w[3]);
+  if (lane == 0) {
+    float* scal = ws.scal + 4 * ((size_t)c * a.num_heads + h);
+    scal[0] = total;
+    if (KIND == kMlstm) {
+      scal[1] = amax;
+      const int s = a.chunk_seq[c];
+      if (row0 == a.cu_seqlens[s]) {
+        const bool fresh = a.seq_lens[s] == a.cu_seqlens[s + 1] - row0;
+        const int tiles = (a.value_dim + kTileV - 1) / kTileV;
+        scal[2] = fresh ? 0.f : a.max_state[((int64_t)a.slots[s] * a.num_heads + h) * tiles];
+      }
+    }
+  }
+}
 
 // ---- 1: U [key_dim x 64] = K^T (w V), A = K^T (MN-major), B = the weighted values' terms (MN-major) ----------
 template <int KIND>
@@ -64,8 +146,7 @@ state_kernel(const __grid_constant__ CUtensorMap k_map, const b200_recurrence_ar
   const uint32_t base = (smem_u32(raw) + 1023u) & ~1023u;
   uint8_t* gen = raw + (base - smem_u32(raw));
   const uint32_t sk = base, sv = sk + slices * kTile, sb = sv + kTerms * kTile;
-  float* cum = reinterpret_cast<float*>(gen + (sb - base) + 64);
-  float *src = cum + C, *top = src + C, *wgt = top + C;
+  float* wgt = reinterpret_cast<float*>(gen + (sb - base) + 64);
   volatile uint32_t* tmem_gen = reinterpret_cast<volatile uint32_t*>(gen + (sb - base) + 32);
   const uint32_t bar_load = sb, bar_mma = sb + 8;
   int row0;
@@ -88,29 +169,12 @@ state_kernel(const __grid_constant__ CUtensorMap k_map, const b200_recurrence_ar
     for (int i = 0; i < slices; ++i) tma_load_2d(sk + i * kTile, &k_map, bar_load, g * K + i * 64, row0);
   }
   __syncwarp();
-  chunk_gates<KIND, C>(a, row0, rows, h, cum, src, top);
-  const float total = cum[C - 1];
-  if (tid < C) {
-    float w = 0.f;
-    if (tid < rows) w = KIND == kSsd ? src[tid] * expf(total - cum[tid]) : expf(src[tid] - top[C - 1]);
-    wgt[tid] = w;
-  }
-  __syncthreads();
   const Workspace ws(a);
-  float* scal = ws.scal + 4 * ((size_t)c * a.num_heads + h);
-  if (tile == 0 && tid == 0) {
-    scal[0] = total;
-    if (KIND == kMlstm) {
-      scal[1] = top[C - 1];
-      const int s = a.chunk_seq[c];
-      if (row0 == a.cu_seqlens[s]) {
-        const bool fresh = a.seq_lens[s] == a.cu_seqlens[s + 1] - row0;
-        scal[2] = fresh ? 0.f : a.max_state[((int64_t)a.slots[s] * a.num_heads + h) * gridDim.x];
-      }
-    }
-  }
+  const float* wgt_g = ws.gates + ((size_t)c * a.num_heads + h) * 4 * C + 3 * C;
+  if (KIND == kMlstm && tid < C) wgt[tid] = wgt_g[tid];
   {  // weighted values: two threads a row, 32 columns each
     const int r = tid >> 1, cc0 = (tid & 1) * 32;
+    const float wr = wgt_g[r];
     const bf16* vr = reinterpret_cast<const bf16*>(a.v) + (int64_t)(row0 + r) * a.v_stride + (int64_t)h * V + c0;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
@@ -120,7 +184,7 @@ state_kernel(const __grid_constant__ CUtensorMap k_map, const b200_recurrence_ar
       const bf16* xe = reinterpret_cast<const bf16*>(&x4);
       float x[8];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] = wgt[r] * to_float(xe[e]);
+      for (int e = 0; e < 8; ++e) x[e] = wr * to_float(xe[e]);
       split8(sv + swz(r, cc >> 3), x);
     }
   }
@@ -238,10 +302,12 @@ output_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__
     tma_load_2d(sv, &v_map, bar_v, h * V + c0, row0);
   }
   __syncwarp();
-  chunk_gates<KIND, C>(a, row0, rows, h, cum, src, top);
   const float m_in = KIND == kMlstm ? ws.scal[4 * ((size_t)c * a.num_heads + h) + 3] : 0.f;
   if (tid < C) {
-    if (KIND == kMlstm) top[tid] = fmaxf(m_in, top[tid]);
+    const float* gates = ws.gates + ((size_t)c * a.num_heads + h) * 4 * C;
+    cum[tid] = gates[tid];
+    src[tid] = gates[C + tid];
+    if (KIND == kMlstm) top[tid] = fmaxf(m_in, gates[2 * C + tid]);
     scale[tid] = KIND == kSsd ? expf(cum[tid]) : expf(m_in - top[tid]);
   }
   bool ok = true;
@@ -457,6 +523,7 @@ int launch(const b200_recurrence_args& a, cudaStream_t st) {
     attr = true;
   }
   const dim3 grid((a.value_dim + kTileV - 1) / kTileV, a.num_heads, a.num_chunks);
+  B200_CUDA_OK(launch_pdl(gates_kernel<KIND>, dim3((a.num_heads + 7) / 8, a.num_chunks), dim3(kThreads), 0, st, a));
   B200_CUDA_OK(launch_pdl(state_kernel<KIND>, grid, dim3(kThreads), state_smem(a.key_dim), st, k_map, a));
   const int blocks = (a.key_dim * a.value_dim / 4 + kScanThreads - 1) / kScanThreads;
   B200_CUDA_OK(launch_pdl(chunk_scan_kernel<KIND>, dim3(blocks + (KIND == kMlstm ? 1 : 0), a.num_heads, a.num_seqs),
