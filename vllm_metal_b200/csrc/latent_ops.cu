@@ -160,81 +160,91 @@ head_linear_kernel(const b200_head_linear_args a) {
   }
 }
 
-// bf16 on tensor cores: 64 rows x 64 outputs of one head per CTA, 64-wide k slabs, double-buffered.
-constexpr int kPad = 72;
+// bf16 on tensor cores: 64 rows x 32 outputs of one head per CTA, 64-wide k slabs in a ring of four.
+constexpr int kPad = 72, kCols = 32, kRing = 4;
+constexpr int kHeadLinearSmem = kRing * (64 + kCols) * kPad * 2;
 __global__ void __launch_bounds__(128)
-head_linear_mma_kernel(const b200_head_linear_args a) {
-  __shared__ __align__(16) bf16 sx[2][64 * kPad];
-  __shared__ __align__(16) bf16 sw[2][64 * kPad];
+head_linear_mma_kernel(const b200_head_linear_args a, int pairs) {
+  extern __shared__ __align__(16) uint8_t hl_raw[];
+  bf16* sx = reinterpret_cast<bf16*>(hl_raw);
+  bf16* sw = sx + kRing * 64 * kPad;
   pdl_trigger();
-  const int h = blockIdx.y, n0 = blockIdx.x * 64, r0 = blockIdx.z * 64;
+  const int h = blockIdx.y, n0 = blockIdx.x * kCols, r0 = blockIdx.z * 64;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const bf16* x = reinterpret_cast<const bf16*>(a.x) + (int64_t)r0 * a.x_stride + h * a.x_head_stride;
   const bf16* w = reinterpret_cast<const bf16*>(a.w) + ((int64_t)h * a.n + n0) * a.k;
-  const int rows = min(64, a.rows - r0), cols = min(64, a.n - n0);
-  auto load_w = [&](int buf, int k0) {
-    for (int i = tid; i < 512; i += 128) {
+  const int rows = min(64, a.rows - r0), cols = min(kCols, a.n - n0), slabs = (a.k + 63) / 64;
+  auto load_w = [&](int s) {
+    for (int i = tid; i < kCols * 8; i += 128) {
       const int r = i >> 3, c = (i & 7) * 8;
-      const bool live = r < cols && k0 + c < a.k;
-      mma::cp_async16(&sw[buf][r * kPad + c], live ? w + (int64_t)r * a.k + k0 + c : w, live);
+      const bool live = r < cols && s * 64 + c < a.k;
+      mma::cp_async16(&sw[((s % kRing) * kCols + r) * kPad + c], live ? w + (int64_t)r * a.k + s * 64 + c : w, live);
     }
   };
-  auto load_x = [&](int buf, int k0) {
+  auto load_x = [&](int s) {
     for (int i = tid; i < 512; i += 128) {
       const int r = i >> 3, c = (i & 7) * 8;
-      const bool live = r < rows && k0 + c < a.k;
-      mma::cp_async16(&sx[buf][r * kPad + c], live ? x + (int64_t)r * a.x_stride + k0 + c : x, live);
+      const bool live = r < rows && s * 64 + c < a.k;
+      mma::cp_async16(&sx[((s % kRing) * 64 + r) * kPad + c], live ? x + (int64_t)r * a.x_stride + s * 64 + c : x, live);
     }
   };
-  load_w(0, 0);  // weights do not depend on the previous kernel
+  for (int s = 0; s < kRing - 1 && s < slabs; ++s) load_w(s);  // weights do not depend on the previous kernel
   pdl_wait();
-  load_x(0, 0);
-  mma::cp_commit();
-  float acc[8][4];
+  for (int s = 0; s < kRing - 1; ++s) {
+    if (s < slabs) load_x(s);
+    mma::cp_commit();  // the weights ride in the first group: waiting for it means waiting for all of them
+  }
+  float acc[4][4];
 #pragma unroll
-  for (int n = 0; n < 8; ++n)
+  for (int n = 0; n < 4; ++n)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[n][e] = 0.f;
-  const int slabs = (a.k + 63) / 64;
   for (int s = 0; s < slabs; ++s) {
-    if (s + 1 < slabs) {
-      load_w((s + 1) & 1, (s + 1) * 64);
-      load_x((s + 1) & 1, (s + 1) * 64);
+    mma::cp_wait<kRing - 2>();
+    __syncthreads();
+    if (s + kRing - 1 < slabs) {
+      load_w(s + kRing - 1);
+      load_x(s + kRing - 1);
     }
     mma::cp_commit();
-    mma::cp_wait<1>();
-    __syncthreads();
-    const bf16 *xs = sx[s & 1], *wsm = sw[s & 1];
+    const bf16 *xs = sx + (s % kRing) * 64 * kPad, *wsm = sw + (s % kRing) * kCols * kPad;
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks) {
       uint32_t fa[4];
       mma::ldsm4(fa, &xs[(warp * 16 + (lane & 15)) * kPad + ks * 16 + (lane >> 4) * 8]);
 #pragma unroll
-      for (int n2 = 0; n2 < 4; ++n2) {
+      for (int n2 = 0; n2 < 2; ++n2) {
         uint32_t fb[4];
         mma::ldsm4(fb, &wsm[(n2 * 16 + (lane >> 4) * 8 + (lane & 7)) * kPad + ks * 16 + ((lane >> 3) & 1) * 8]);
         mma::mma16816(acc[2 * n2], fa, fb[0], fb[1]);
         mma::mma16816(acc[2 * n2 + 1], fa, fb[2], fb[3]);
       }
     }
-    __syncthreads();
   }
 #pragma unroll
-  for (int n = 0; n < 8; ++n)
+  for (int n = 0; n < 4; ++n)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int r = warp * 16 + (lane >> 2) + e * 8, c = n0 + n * 8 + (lane & 3) * 2;
       if (r >= rows || c >= a.n) continue;
-      const int64_t t = r0 + r;
+      const int64_t t = r0 + r, off = t * a.gate_stride + (int64_t)h * a.n + c;
       float u = acc[n][2 * e], v = acc[n][2 * e + 1];
-      if (a.gate) {
-        const int64_t off = t * a.gate_stride + (int64_t)h * a.n + c;
-        u *= gate_value(a.gate, off, 0, 0);
-        if (c + 1 < a.n) v *= gate_value(a.gate, off + 1, 0, 0);
-      }
       bf16* y = reinterpret_cast<bf16*>(a.y) + t * a.y_stride + h * a.y_head_stride + c;
-      y[0] = __float2bfloat16_rn(u);
-      if (c + 1 < a.n) y[1] = __float2bfloat16_rn(v);
+      if (pairs) {  // whole aligned pairs
+        if (a.gate) {
+          const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(reinterpret_cast<const bf16*>(a.gate) + off));
+          u *= 1.f / (1.f + expf(-z.x));
+          v *= 1.f / (1.f + expf(-z.y));
+        }
+        *reinterpret_cast<__nv_bfloat162*>(y) = __floats2bfloat162_rn(u, v);
+      } else {
+        if (a.gate) u *= gate_value(a.gate, off, 0, 0);
+        y[0] = __float2bfloat16_rn(u);
+        if (c + 1 < a.n) {
+          if (a.gate) v *= gate_value(a.gate, off + 1, 0, 0);
+          y[1] = __float2bfloat16_rn(v);
+        }
+      }
     }
 }
 
@@ -300,8 +310,15 @@ int b200_head_linear(const b200_head_linear_args* a, void* stream) {
   if (a->rows <= 0) return B200_OK;
   auto ok = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
   if (a->dtype == B200_BF16 && a->k % 8 == 0 && a->x_stride % 8 == 0 && a->x_head_stride % 8 == 0 && ok(a->x) && ok(a->w)) {
-    const dim3 grid((a->n + 63) / 64, a->heads, (a->rows + 63) / 64);
-    B200_CUDA_OK(launch_pdl(head_linear_mma_kernel, grid, dim3(128), 0, (cudaStream_t)stream, *a));
+    const dim3 grid((a->n + kCols - 1) / kCols, a->heads, (a->rows + 63) / 64);
+    const int pairs = a->n % 2 == 0 && a->y_stride % 2 == 0 && a->y_head_stride % 2 == 0 && a->gate_stride % 2 == 0 &&
+                      (((uintptr_t)a->y | (uintptr_t)a->gate) & 3) == 0;
+    static bool attr = false;
+    if (!attr) {
+      B200_CUDA_OK(cudaFuncSetAttribute(head_linear_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kHeadLinearSmem));
+      attr = true;
+    }
+    B200_CUDA_OK(launch_pdl(head_linear_mma_kernel, grid, dim3(128), kHeadLinearSmem, (cudaStream_t)stream, *a, pairs));
     return check_launch("head_linear (mma)");
   }
   B200_CHECK_ARG(a->rows <= 65535, "head_linear: more than 65535 rows");
