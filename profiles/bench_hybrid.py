@@ -189,6 +189,47 @@ def kernel_table(size: str, batch: int = 64, ctx: int = 4096, chunk: int = 2048)
     return rows
 
 
+def like_table(size: str, batch: int = 64, ctx: int = 4096, chunk: int = 2048) -> list[dict]:
+    """The closest transformer's kernels of the same kinds at the same sizes: what the table above is held against."""
+    import torch
+
+    from vllm_metal_b200.metal import get_ops
+
+    ops, hbm, tf, _ = get_ops(), *peaks()
+    a, bf, rows = transformer_args(size, 1), torch.bfloat16, []
+    H, Hk, D = a.n_heads, a.n_kv_heads, a.head_dim
+
+    def add(phase, name, us, nbytes=0.0, flops=0.0):
+        bound = max(nbytes / (hbm * 1e3), flops / (tf * 1e6))
+        rows.append({"phase": phase, "kernel": "like: " + name, "us": round(us, 2), "roofline_us": round(bound, 2),
+                     "bound": "hbm" if nbytes / (hbm * 1e3) >= flops / (tf * 1e6) else "tensor", "frac": round(bound / us, 3)})
+
+    for phase, q_lens, ctxs in (("decode", [1] * batch, [ctx] * batch), ("prefill", [chunk], [ctx + chunk])):
+        meta, blocks = _segments(q_lens, ctxs)
+        T = sum(q_lens)
+        sets = max(2, min(32, L2_BYTES // (T * a.hidden * 4)))
+        r = lambda *s: torch.randn(s, device="cuda").to(bf)  # noqa: E731
+        w = torch.ones(a.hidden, dtype=bf, device="cuda")
+        xs, res = [r(T, a.hidden) for _ in range(sets)], [r(T, a.hidden) for _ in range(sets)]
+        add(phase, "rms_norm + residual", graph_us([lambda x=x, y=y: ops.rms_norm(x, w, 1e-5, residual=y)
+                                                     for x, y in zip(xs, res)]), T * a.hidden * 8)
+        gu = [r(T, 2 * a.intermediate) for _ in range(max(2, min(16, L2_BYTES // (T * a.intermediate * 4))))]
+        add(phase, "silu_mul", graph_us([lambda g=g: ops.silu_mul(g) for g in gu]), T * a.intermediate * 6)
+        kc, vc = r(blocks, 16, Hk, D), r(blocks, 16, Hk, D)
+        qkv = [r(T, (H + 2 * Hk) * D) for _ in range(max(2, min(16, L2_BYTES // (T * (H + 2 * Hk) * D * 2))))]
+        parts = [[z.reshape(T, -1, D) for z in t.split([H * D, Hk * D, Hk * D], 1)] for t in qkv]
+        add(phase, "norm_rope_cache", graph_us([lambda p=p: ops.norm_rope_cache(
+            *p, kc, vc, meta.slot_mapping, positions=meta.positions, rot_dim=D, base=1e4) for p in parts]),
+            T * ((2 * H + Hk) * D * 2 + 4 * Hk * D * 2))
+        q, out = r(T, H, D), torch.empty((T, H, D), dtype=bf, device="cuda")
+        caches = [(kc, vc), (kc.clone(), vc.clone())]
+        pairs = sum(c - n + i + 1 for n, c in zip(q_lens, ctxs) for i in range(n))
+        add(phase, "paged attention", graph_us([lambda c=c: ops.paged_attention_primitive(
+            q, c[0], c[1], Hk, D ** -0.5, 0.0, meta.block_tables, meta.seq_lens, meta.cu_seqlens_q, 16, max(ctxs), -1, out)
+            for c in caches]), sum(ctxs) * Hk * D * 4 + T * H * D * 4, 4.0 * pairs * H * D)
+    return rows
+
+
 def _latent_rows(ops, add, phase, m, lay, ps, meta, pool, y, T, q_lens, ctxs, act) -> None:
     import torch
 
@@ -235,6 +276,10 @@ def _latent_rows(ops, add, phase, m, lay, ps, meta, pool, y, T, q_lens, ctxs, ac
     add(phase, "latent: attention over expanded keys", graph_us([lambda kv=kv: ops.paged_attention_primitive(
         q_full, kv[:, :, 0], kv[:, :, 1], H, m.scale, 0.0, plan.block_tables, plan.count, plan.cu_seqlens_q, EXPAND_PAGE,
         plan.max_count, m.window if m.window > 0 else -1, out, wide_weights=True, _kernel=3) for kv in kvs]),
+        2 * (2 * kvs[0].numel() // 2 + 2 * q_full.numel()), 2.0 * pairs * H * (m.dim + m.rot_dim + m.vdim))
+    add(phase, "latent: the same, weights rounded to 16 bits", graph_us([lambda kv=kv: ops.paged_attention_primitive(
+        q_full, kv[:, :, 0], kv[:, :, 1], H, m.scale, 0.0, plan.block_tables, plan.count, plan.cu_seqlens_q, EXPAND_PAGE,
+        plan.max_count, m.window if m.window > 0 else -1, out, _kernel=3) for kv in kvs]),
         2 * (2 * kvs[0].numel() // 2 + 2 * q_full.numel()), 2.0 * pairs * H * (m.dim + m.rot_dim + m.vdim))
     o = out.view(T, -1)
     add(phase, "latent: gate, gelu", graph_us([lambda p=p: ops.mixer_finish(
@@ -341,7 +386,7 @@ def main(sizes=("s", "m"), kernels: bool = True, steps: int = 32, warmup: int = 
             entry["models"].append(whole_model(size, kind, batch, ctx, chunk, steps, warmup))
             torch.cuda.empty_cache()
         if kernels:
-            entry["kernels"] = kernel_table(size, batch, ctx, chunk)
+            entry["kernels"] = kernel_table(size, batch, ctx, chunk) + like_table(size, batch, ctx, chunk)
             torch.cuda.empty_cache()
         result["sizes"][size] = entry
     return result

@@ -290,7 +290,7 @@ int launch_finish_vec(const b200_mixer_finish_args& a, cudaStream_t st) {
 // ---- causal depthwise convolution -----------------------------------------------------------
 // One thread per channel walks kConvTile rows with the taps in registers.  Only the first tile of a segment touches
 // the carried inputs, and it takes the new ones straight from the input rows, so the tiles never race.
-constexpr int kConvTile = 16;
+constexpr int kConvTile = 8;
 constexpr int kConvMaxTaps = 16;
 
 template <typename T, int TAPS>
@@ -411,10 +411,16 @@ causal_conv_vec_kernel(const T* __restrict__ in, const float* __restrict__ weigh
 #pragma unroll
     for (int k = 0; k < TAPS - 1; ++k) *reinterpret_cast<Vec8<T>*>(st + (int64_t)k * channels) = nv[k];
   }
-  const int t1 = min(t0 + kConvTile, len);
-#pragma unroll 4
-  for (int t = t0; t < t1; ++t) {
-    const Vec8<T> cur = *reinterpret_cast<const Vec8<T>*>(x + (int64_t)t * in_stride);
+  const int n = min(kConvTile, len - t0);
+  Vec8<T> rows[kConvTile];
+#pragma unroll
+  for (int i = 0; i < kConvTile; ++i)
+    if (i < n) rows[i] = *reinterpret_cast<const Vec8<T>*>(x + (int64_t)(t0 + i) * in_stride);
+#pragma unroll
+  for (int i = 0; i < kConvTile; ++i) {
+    if (i >= n) break;
+    const int t = t0 + i;
+    const Vec8<T> cur = rows[i];
     Vec8<T> res;
 #pragma unroll
     for (int e = 0; e < 8; ++e) {

@@ -350,7 +350,8 @@ struct Plan {
 bool tc_supported(const b200_latent_attn_args& a) {
   const int width = a.kv_rank + a.rot_dim;
   return a.dtype == B200_BF16 && a.scale > 0.f && width % 8 == 0 && a.kv_rank % 8 == 0 && a.kv_rank <= kMaxRank &&
-         width <= 64 * latent_tc::kMaxSlices && a.q_stride == (int64_t)a.heads * width && a.block_size >= 8 &&
+         width <= 64 * latent_tc::kMaxSlices && a.q_stride == (int64_t)a.heads * width &&
+         a.out_stride == (int64_t)a.heads * a.kv_rank && a.block_size >= 8 &&
          latent_tc::kKeys % a.block_size == 0 && a.num_slots < (1LL << 31) &&
          (((uintptr_t)a.q | (uintptr_t)a.cache) & 15) == 0 && tc::encode_fn() != nullptr;
 }
@@ -395,7 +396,7 @@ int launch_tc(const b200_latent_attn_args& a, int splits, cudaStream_t st) {
   Params p;
   p.block_tables = a.block_tables, p.seq_lens = a.seq_lens, p.cu = a.cu_seqlens, p.out = a.out;
   p.wo = reinterpret_cast<float*>(a.workspace);
-  p.out_stride = a.out_stride, p.num_tokens = a.num_tokens, p.heads = a.heads, p.rank = a.kv_rank;
+  p.num_tokens = a.num_tokens, p.heads = a.heads, p.rank = a.kv_rank;
   p.width = a.kv_rank + a.rot_dim, p.slices = (p.width + 63) / 64, p.mtiles = (a.kv_rank + 127) / 128;
   p.block_size = a.block_size, p.max_blocks = a.max_blocks_per_seq, p.window = a.window, p.max_q_len = a.max_q_len;
   p.splits = splits, p.scale2 = a.scale * kLog2e;

@@ -37,7 +37,6 @@ struct Params {
   const int32_t* cu;
   void* out;
   float* wo;
-  int64_t out_stride;
   int num_tokens, heads, rank, width, slices, mtiles, block_size, max_blocks, window, max_q_len, splits;
   float scale2;  // scale * log2(e)
 };
@@ -358,9 +357,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constan
         if (rbase + r >= nrows || dim >= p.rank) continue;
         const float x = nt > 0 ? (__uint_as_float(a[r]) + __uint_as_float(b[r])) * inv[r] : 0.f;
         if (p.splits == 1) {
-          const int rr = r_first + rbase + r;
-          reinterpret_cast<__nv_bfloat16*>(p.out)[(int64_t)(row0 + rr / p.heads) * p.out_stride +
-                                                  (int64_t)(rr % p.heads) * p.rank + dim] = __float2bfloat16_rn(x);
+          reinterpret_cast<__nv_bfloat16*>(p.out)[(first + rbase + r) * p.rank + dim] = __float2bfloat16_rn(x);
         } else {
           p.wo[((size_t)split * all_rows + first + rbase + r) * p.rank + dim] = x;
         }
