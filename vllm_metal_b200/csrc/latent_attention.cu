@@ -299,45 +299,45 @@ latent_mma_kernel(const b200_latent_attn_args a, int splits) {
   }
 }
 
-// One CTA per (token, head) row of the computed segments, 4 columns a thread: the splits' partial outputs become one.
-__global__ void __launch_bounds__(128)
-latent_merge_kernel(const b200_latent_attn_args a, int splits) {
+// The splits' partial outputs of a (token, head) row become one: `wpr` warps a row, 4 columns a lane and step.
+__global__ void __launch_bounds__(256)
+latent_merge_kernel(const b200_latent_attn_args a, int splits, int wpr) {
   pdl_trigger();
   pdl_wait();
-  __shared__ float weight[kMaxSplits];
+  __shared__ float weights[8][kMaxSplits];
   const int s = blockIdx.y, row0 = a.cu_seqlens[s], len = a.cu_seqlens[s + 1] - row0;
-  const int rr = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int rr = blockIdx.x * (8 / wpr) + warp / wpr;
   if (len <= 0 || len > a.max_q_len || rr >= len * a.heads) return;
   const int rank = a.kv_rank;
   const size_t all_rows = (size_t)a.num_tokens * a.heads, row = (size_t)row0 * a.heads + rr;
   const float* wo = reinterpret_cast<const float*>(a.workspace);
-  const float* wml = wo + (size_t)splits * all_rows * rank;
-  if (threadIdx.x < 32) {
-    float m = -INFINITY, l = 0.f;
-    for (int p = threadIdx.x; p < splits; p += 32) m = fmaxf(m, wml[2 * (p * all_rows + row)]);
-    m = warp_max(m);
-    for (int p = threadIdx.x; p < splits; p += 32) {
-      const float mp = wml[2 * (p * all_rows + row)];
-      const float w = mp == -INFINITY ? 0.f : exp2f(mp - m);
-      weight[p] = w;
-      l += w * wml[2 * (p * all_rows + row) + 1];
-    }
-    l = warp_sum(l);
-    __syncwarp();
-    for (int p = threadIdx.x; p < splits; p += 32) weight[p] /= l;
+  const float2* wml = reinterpret_cast<const float2*>(wo + (size_t)splits * all_rows * rank);
+  float* weight = weights[warp];
+  float m = -INFINITY, l = 0.f;
+  for (int p = lane; p < splits; p += 32) m = fmaxf(m, wml[p * all_rows + row].x);
+  m = warp_max(m);
+  for (int p = lane; p < splits; p += 32) {
+    const float2 ml = wml[p * all_rows + row];
+    const float w = ml.x == -INFINITY ? 0.f : exp2f(ml.x - m);
+    weight[p] = w;
+    l += w * ml.y;
   }
-  __syncthreads();
+  l = warp_sum(l);
+  __syncwarp();
+  const float inv = 1.f / l;
   bf16* out = reinterpret_cast<bf16*>(a.out) + (int64_t)(row0 + rr / a.heads) * a.out_stride + (int64_t)(rr % a.heads) * rank;
-  for (int d = threadIdx.x * 4; d < rank; d += 512) {
-    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 4
+  for (int d = (warp % wpr) * 128 + lane * 4; d < rank; d += wpr * 128) {
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 2
     for (int p = 0; p < splits; ++p) {
       const float w = weight[p];
       const float4 v = *reinterpret_cast<const float4*>(wo + (p * all_rows + row) * rank + d);
       acc.x += w * v.x, acc.y += w * v.y, acc.z += w * v.z, acc.w += w * v.w;
     }
-    reinterpret_cast<__nv_bfloat162*>(out + d)[0] = __floats2bfloat162_rn(acc.x, acc.y);
-    reinterpret_cast<__nv_bfloat162*>(out + d)[1] = __floats2bfloat162_rn(acc.z, acc.w);
+    reinterpret_cast<__nv_bfloat162*>(out + d)[0] = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
+    reinterpret_cast<__nv_bfloat162*>(out + d)[1] = __floats2bfloat162_rn(acc.z * inv, acc.w * inv);
   }
 }
 
@@ -471,8 +471,10 @@ int b200_latent_attention(const b200_latent_attn_args* a, void* stream) {
   if (p.kind == kMma)
     B200_CUDA_OK(launch_pdl(latent_mma_kernel, dim3((rows + kRows - 1) / kRows, a->num_seqs, p.splits), dim3(kThreads),
                           Smem(a->kv_rank + a->rot_dim).total, st, *a, p.splits));
-  if (p.splits > 1)
-    B200_CUDA_OK(launch_pdl(latent_merge_kernel, dim3(rows, a->num_seqs), dim3(128), 0, st, *a, p.splits));
+  if (p.splits > 1) {
+    const int wpr = (int64_t)rows * a->num_seqs >= 1024 ? 1 : 4;
+    B200_CUDA_OK(launch_pdl(latent_merge_kernel, dim3((rows * wpr + 7) / 8, a->num_seqs), dim3(256), 0, st, *a, p.splits, wpr));
+  }
   return check_launch("latent_attention");
 }
 
