@@ -340,3 +340,18 @@ def test_a_planted_mistake_in_the_oracle_shows(edit):
         bad["l1.mix.f.b"] = t["l1.mix.f.b"] - 3.0
     err = np.sqrt(((oracle.forward(bad_cfg, bad, toks) - right) ** 2).mean(1)) / right.std()
     assert err[12:].max() > 2e-2, err.max()
+
+
+def test_the_hybrid_component_is_a_library_of_its_own():
+    """The sources listed for the component cover every symbol the hybrid operators bind and exist in the tree."""
+    import re
+
+    from vllm_metal_b200.metal import EXPORTED_SYMBOLS
+    from vllm_metal_b200.metal.build import COMPONENTS, output_path, sources
+    from vllm_metal_b200.metal.hybrid_ops import HYBRID_SYMBOLS
+
+    files = sources("hybrid")
+    assert all(f.exists() for f in files) and output_path("hybrid") != output_path() and len(files) == len(COMPONENTS["hybrid"])
+    text = "\n".join(f.read_text() for f in files)
+    for name in (*HYBRID_SYMBOLS, "b200_paged_attention", "b200_argmax", "b200_advance_decode", "b200_last_error"):
+        assert name in EXPORTED_SYMBOLS and re.search(rf"\b{name}\s*\(", text), name

@@ -21,10 +21,9 @@ def _generate(argv: list[str]) -> int:
     args = ap.parse_args(argv)
 
     from .lm.registry import family_of, read_config
-    from .metal.build import build, ensure
+    from .metal.build import ensure
 
-    component = family_of(read_config(args.model)).component
-    build() if component is None else ensure(component)
+    ensure(family_of(read_config(args.model)).component)
 
     from .v1.engine import Engine
 

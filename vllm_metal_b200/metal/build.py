@@ -96,8 +96,9 @@ def _file_hash(src: Path, extra: list[str]) -> str:
     return h.hexdigest()
 
 
-def ensure(component: str) -> Path:
-    """The full library if it is there and fresh, else the component's, compiled now if need be."""
+def ensure(component: str | None = None) -> Path:
+    """The full library if it is there and fresh, else the component's (``None``: the full one), compiled now if need
+    be."""
     if not stale_artifacts():
         return output_path()
     return build(component=component)

@@ -35,10 +35,9 @@ def main(argv: list[str] | None = None) -> int:
     if DTYPES[args.dtype] not in family.dtypes:
         print(f"model family '{family.name}' does not run in {args.dtype}", file=sys.stderr)
         return EXIT_UNSUPPORTED_DTYPE
-    if family.component is not None:
-        from ..metal.build import ensure
+    from ..metal.build import ensure
 
-        ensure(family.component)
+    ensure(family.component)
 
     import torch
 
