@@ -162,6 +162,73 @@ typedef struct b200_stream_step_args {
 #define B200_MAX_STREAMS 16
 int b200_stream_step(const b200_stream_step_args* a, void* stream);
 
+/* What lies between two sublayers that stand between norms of their own, one launch, fp32 stream x [rows, dim]:
+ *   r = y, or with parts > 0 sum_j part_weight[row, j] y[row * parts + j] (+ sigmoid(extra_gate[row]) extra[row]);
+ *   x += r / rms(r) * out_norm        (y NULL: x is read only)
+ *   h = x / rms(x) * in_norm          (h NULL: nothing follows)
+ *   h += conv(h) with taps weights [taps, dim] if conv_weight: the earlier inputs come from state[slots[row], taps - 1, dim]
+ *   (oldest first; zeros for a request's first tokens, seq_lens[row] counts this one), which takes h in; for batches of
+ *   one row a request.
+ * row_ids: the stream rows to work on (h is packed, the result is indexed like the stream), x is not written then.
+ * Norm, gate and convolution weights fp32; y, extra, h and state of dtype. */
+typedef struct b200_residual_step_args {
+  float* x;
+  const void* y;
+  const float* part_weight;
+  const void* extra;
+  const float* extra_gate;
+  const float* out_norm;
+  const float* in_norm;
+  void* h;
+  const float* conv_weight;
+  void* state;
+  const int32_t* slots;
+  const int32_t* seq_lens;
+  const int64_t* row_ids;
+  int64_t y_stride, extra_stride, gate_stride, h_stride;
+  int32_t rows, dim, parts, taps;
+  float eps;
+  int32_t dtype;
+} b200_residual_step_args;
+int b200_residual_step(const b200_residual_step_args* a, void* stream);
+
+#define B200_MAX_EXPERTS 1024
+/* Routed experts.  b200_expert_route, per row: s = softmax(logits[row, 0:experts]); the `top` experts with the largest
+ * s + correction (fp32, NULL: 0; ties to the lower number), best first, go to chosen [rows, top] and their s * scale to
+ * weights [rows, top]. */
+int b200_expert_route(const float* logits, int64_t logits_stride, const float* correction, int32_t* chosen, float* weights,
+                      int rows, int experts, int top, float scale, void* stream);
+
+/* The (row, place) pairs p = row * top + place sorted by expert: pairs [rows * top], first [experts + 1] the start of each
+ * expert's stretch, tiles [experts + 1] the running count of the stretches' tiles of tile_rows pairs. */
+int b200_expert_plan(const int32_t* chosen, int32_t* pairs, int32_t* first, int32_t* tiles, int rows, int experts, int top,
+                     int tile_rows, void* stream);
+
+/* Products of all experts at once.  `gated` = 1, the way in:
+ *   out[i, n] = silu(w[e, n] . x[pairs[i] / top]) * (w[e, inter + n] . x[pairs[i] / top])   i in e's stretch, n < n_out
+ * (w [experts, 2 n_out, k], out [pairs, n_out] in sorted order); 0, the way out:
+ *   out[pairs[i], n] = w[e, n] . x[i]                                            (w [experts, n_out, k], x in sorted order).
+ * A shared expert that every row takes runs in the same launch (shared_w not NULL): its rows are x (gated) or shared_x, its
+ * results shared_out [rows, shared_n_out].  Element strides; rows of w and shared_w are w_stride and shared_w_stride apart.
+ * kernel: 0 auto, 1 any type and size, 2 tcgen05 (bf16, whole 8-element units).  tile_rows as given to the plan (32, 64 or
+ * 128); max_tiles bounds tiles[experts]. */
+typedef struct b200_expert_product_args {
+  const void* x;
+  const void* w;
+  void* out;
+  const void* shared_x;
+  const void* shared_w;
+  void* shared_out;
+  const int32_t* pairs;
+  const int32_t* first;
+  const int32_t* tiles;
+  int64_t x_stride, w_stride, out_stride, shared_x_stride, shared_w_stride, shared_out_stride;
+  int32_t rows, experts, top, n_out, k, shared_n_out, shared_k, tile_rows, max_tiles, gated, dtype, kernel;
+} b200_expert_product_args;
+int b200_expert_product(const b200_expert_product_args* a, void* stream);
+/* Synchronises.  1 if a bounded wait inside the tcgen05 kernel ever ran out (that launch's results are invalid), else 0. */
+int b200_expert_product_failed(void);
+
 /* Before latent attention, per row: the latent is normed (weight fp32, plain), the shared key part is rotated
  * (interleaved pairs), both go to the latent cache row slot_mapping[t]:
  * [latent kv_rank | key part rot_dim]; the rotated part of every query head goes to
@@ -184,6 +251,29 @@ typedef struct b200_latent_prep_args {
   int32_t dtype;
 } b200_latent_prep_args;
 int b200_latent_prep(const b200_latent_prep_args* a, void* stream);
+
+/* Before attention with rotated, then normed heads, per row: the interleaved pairs (2i, 2i + 1) of the first rot_dims
+ * dimensions of every query and key head are turned by positions[t] * f_i and scaled by rot_factor, with f_i = freq[2i] +
+ * freq[2i + 1] as a high and a low part; the head is divided by its root mean square; a query head also takes
+ * q_weight[h] (fp32, NULL: 1).  Queries are updated in place, keys and values go to cache row slot_mapping[t] (negative or out of
+ * range: padding, nothing is cached). */
+typedef struct b200_rope_norm_cache_args {
+  void* q;
+  const void* k;
+  const void* v;
+  const float* q_weight;
+  const float* freq; /* [rot_dims / 2][2] */
+  const int32_t* positions;
+  const int64_t* slot_mapping;
+  void* key_cache; /* [num_blocks, block_size, kv_heads, dim], rows contiguous */
+  void* value_cache;
+  int64_t q_stride, k_stride, v_stride;
+  int64_t k_block_stride, k_token_stride, v_block_stride, v_token_stride, num_blocks;
+  int32_t num_tokens, heads, kv_heads, dim, vdim, rot_dims, block_size;
+  float rot_factor, eps;
+  int32_t dtype;
+} b200_rope_norm_cache_args;
+int b200_rope_norm_cache(const b200_rope_norm_cache_args* a, void* stream);
 
 /* y[t, h, n] = sum_k w[h, n, k] x[t, h, k], times sigmoid(gate[t, h * n_dim + n]) if gate: the per-head products of
  * latent attention (queries into the latent space, latent outputs into value space). */

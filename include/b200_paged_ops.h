@@ -25,7 +25,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 5
+#define B200_ABI_VERSION 6
 
 /* Element types of activations / caches (reference: dtype_to_metal,
  * paged_ops.cpp:185-196 -- float, half, bfloat16 are the supported set). */
@@ -113,7 +113,7 @@ int b200_copy_blocks(void* key_cache, void* value_cache, const int32_t* src,
  *
  * Row r = (sequence s, position q_pos of q_len) attends KV positions
  * [max(0, eff - W), eff) with eff = seq_len - q_len + q_pos + 1
- * (pagedattention.metal:913, :1129-1133); W = sliding_window, < 0 disables.
+ * (pagedattention.metal:913, :1129-1133); W = sliding_window, < 0 disables; with a window also [0, min(keep_first, eff)).
  * Softmax in the log2 domain with fp32 accumulation, optional softcap
  * tanh(s/c)*c, sink folded once per row, out = O / (l + 1e-6)
  * (pagedattention.metal:1138, :1318-1328, :1383).  Rows with eff <= 0 are left
@@ -175,6 +175,7 @@ typedef struct b200_paged_attn_args {
   int32_t plain_softmax; /* 1: out = O / l, without the reference's 1e-6 in the denominator */
   int32_t min_q_len;     /* rows of the shortest sequence of the batch if the caller knows it, else 0: where all of them are
                           * the tile kernel's, the per-row kernels are not launched */
+  int32_t keep_first;    /* with a window: positions below this stay visible to every later row */
 } b200_paged_attn_args;
 
 size_t b200_paged_attention_workspace_bytes(const b200_paged_attn_args* args);

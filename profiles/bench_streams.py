@@ -98,7 +98,7 @@ def kernel_table(size: str, batch: int = 64, ctx: int = 4096, chunk: int = 2048)
             T * (row + W * 2 + (W * 6 if decode else 0)))
         if not decode:
             hs = [rnd(T, W) for _ in range(n_sets(T * W * 2))]
-            add(phase, "token shift", graph_us([lambda h=h: ops.causal_conv(h, lay.shift_taps, None, cache.previous[0].unsqueeze(1),
+            add(phase, "token shift", graph_us([lambda h=h: ops.causal_conv(h, lay.shift_taps, None, cache.previous[0],
                                                                             meta, silu=False) for h in hs]), T * W * 4)
         ids = torch.randint(0, VOCAB, (T,), device="cuda", dtype=torch.int32)
         add(phase, "embedding + positions", graph_us([lambda: ops.embed_streams(ids, model.embed, S, meta.positions, model.freq)] * 4),

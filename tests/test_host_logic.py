@@ -169,13 +169,15 @@ def test_library_exports_every_declared_symbol():
     assert declared == set(EXPORTED_SYMBOLS)
     for name in sorted(declared):
         assert hasattr(lib, name), f"{name} declared in include/*.h but not exported"
-    assert lib.b200_abi_version() == 5  # args.out_dtype .. args.plain_softmax
+    assert lib.b200_abi_version() == 6  # args.out_dtype .. args.keep_first
     assert lib.b200_partition_size() == 512
 
 
 def test_args_struct_matches_header_layout():
-    # 10 pointers/size_t + 12 int32 + 6 int64 + 2 float + 3 int32 (out_dtype, window_seqlen_q, wide_weights), padded to 8
-    assert ctypes.sizeof(PagedAttnArgs) == 10 * 8 + 12 * 4 + 6 * 8 + 2 * 4 + 4 * 4 + 3 * 8 + 8
+    # 10 pointers/size_t + 12 int32 + 6 int64 + 2 float + 4 int32 (out_dtype .. value_dim) + 3 int64 (value strides) + 3 int32
+    # (plain_softmax, min_q_len, keep_first), padded to 8
+    assert ctypes.sizeof(PagedAttnArgs) == 10 * 8 + 12 * 4 + 6 * 8 + 2 * 4 + 4 * 4 + 3 * 8 + 4 * 4
+    assert PagedAttnArgs.keep_first.offset == ctypes.sizeof(PagedAttnArgs) - 8
     assert PagedAttnArgs.out_dtype.offset == 10 * 8 + 12 * 4 + 6 * 8 + 2 * 4
     assert PagedAttnArgs.window_seqlen_q.offset == PagedAttnArgs.out_dtype.offset + 4
     assert PagedAttnArgs.q_stride.offset == 10 * 8 + 12 * 4

@@ -88,7 +88,7 @@ def test_registry_model_class_and_cache():
     c = HybridCache(a, 5, 16, 2, torch.bfloat16, "cpu")
     assert sorted(c.kv) == [1, 3, 5] and sorted(c.states) == sorted(c.previous) == list(range(6)) and not c.latent
     assert [t.shape for t in c.kv[3]] == [(5, 16, 2, 24), (5, 16, 2, 40)] and c.states[1].matrix.shape == (3, 2, 16, 56)
-    assert c.previous[4].shape == (3, 88) and c.previous[4].dtype == torch.bfloat16
+    assert c.previous[4].shape == (3, 1, 88) and c.previous[4].dtype == torch.bfloat16
     assert c.kv[1][0].data_ptr() != c.kv[3][0].data_ptr()
     assert paged_bytes_per_token(a, torch.bfloat16) == 3 * 2 * (24 + 40) * 2
     assert c.nbytes == 5 * 16 * paged_bytes_per_token(a, torch.bfloat16) + 3 * HybridCache.state_bytes_per_slot(a, torch.bfloat16)

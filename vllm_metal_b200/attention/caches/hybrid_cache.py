@@ -1,7 +1,7 @@
 """What a hybrid decoder keeps between steps: one paged pool of latent rows per latent-attention layer (one row
 ``[latent | rotated key part]`` per token instead of keys and values per head), paged keys and values per layer with
-softmax attention, one set of state slots per recurrent layer and, where tokens are shifted, the last input of every
-layer per slot.  Layers that share weights still have a pool or slots of their own."""
+softmax attention, one set of state slots per recurrent layer and, where a convolution or a token shift stands before
+the mixer, the last inputs of every layer per slot.  Layers that share weights still have a pool or slots of their own."""
 
 from __future__ import annotations
 
@@ -10,7 +10,7 @@ from collections.abc import Sequence
 import torch
 
 from ...lm.hybrid_config import (HybridArgs, LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs,
-                                SideBySideArgs)
+                                SideBySideArgs, cached_heads)
 from .state_cache import RecurrentState
 
 
@@ -30,7 +30,7 @@ class HybridCache:
         self.latent: dict[int, torch.Tensor] = {}
         self.kv: dict[int, tuple[torch.Tensor, torch.Tensor]] = {}  # [blocks, block_size, kv heads, dim / vdim]
         self.states: dict[int, RecurrentState] = {}
-        self.previous: dict[int, torch.Tensor] = {}                 # [slots, width], the activation type
+        self.previous: dict[int, torch.Tensor] = {}                 # [slots, taps - 1, width], the activation type
         for i, layer in enumerate(args.layers):
             m = layer.mixer
             if isinstance(m, LatentAttentionArgs):
@@ -45,11 +45,13 @@ class HybridCache:
             elif isinstance(m, (LightningArgs, SideBySideArgs)):
                 r = m.right if isinstance(m, SideBySideArgs) else m
                 self.states[i] = RecurrentState.allocate(num_slots, r.heads, r.dim, r.vdim, self.device)
-            if isinstance(m, SideBySideArgs):
-                self.kv[i] = tuple(torch.zeros((num_blocks, block_size, m.left.kv_heads, d), dtype=dtype,
-                                               device=self.device) for d in (m.left.dim, m.left.vdim))
-            if args.design.hyper_connected:
-                self.previous[i] = torch.zeros((num_slots + 1, args.width), dtype=dtype, device=self.device)
+            a = cached_heads(m)
+            if a is not None:
+                self.kv[i] = tuple(torch.zeros((num_blocks, block_size, a.kv_heads, d), dtype=dtype, device=self.device)
+                                   for d in (a.dim, a.vdim))
+            if args.input_taps:
+                self.previous[i] = torch.zeros((num_slots + 1, args.input_taps - 1, args.width), dtype=dtype,
+                                               device=self.device)
 
     @staticmethod
     def state_bytes_per_slot(args: HybridArgs, dtype: torch.dtype) -> int:

@@ -29,6 +29,10 @@ inline ValueStrides value_strides(const b200_paged_attn_args& a) {
   if (a.v_token_stride > 0) return {a.v_block_stride, a.v_token_stride, a.v_head_stride};
   return {a.kv_block_stride, a.kv_token_stride, a.kv_head_stride};
 }
+// Kept first positions matter beside a window only; no row has more than max_seq_len.
+inline int keep_first(const b200_paged_attn_args& a) {
+  return a.sliding_window < 0 ? 0 : a.keep_first < a.max_seq_len ? a.keep_first : a.max_seq_len;
+}
 inline float denom_eps(const b200_paged_attn_args& a) { return a.plain_softmax ? 0.f : 1e-6f; }
 
 // One output element: rounded to the call's dtype T; with out_f16 (T = bf16) that value is stored as fp16 -- exact
@@ -75,12 +79,20 @@ __device__ __forceinline__ int find_seq_idx(const int32_t* __restrict__ cu, int 
 // rounded down to a 16-token tile), so windowed rows need ceil((W+15)/psize)
 // partitions instead of ceil(max_seq_len/psize): pages wholly outside the window
 // are never touched (the reference iterates and masks them).
+//
+// Kept first positions [0, keep_first) come ahead of the window: the 16-token tiles that hold them and lie wholly before
+// `base` are `kept` tiles.  A row's tiles are then numbered 0 .. without the gap between the two stretches; `gap` is
+// what a token counted that way has to be moved by once it is past the kept tiles (token_at), and partitions are laid
+// out over these numbers.
 struct RowInfo {
   int seq, eff, beg, base;
+  int kept, gap;
+  __device__ __forceinline__ int span() const { return eff - base + kept * 16; }
+  __device__ __forceinline__ int token_at(int v) const { return v < kept * 16 ? v : v + gap; }
 };
 __device__ __forceinline__ RowInfo row_info(const int32_t* __restrict__ cu,
                                             const int32_t* __restrict__ seq_lens, int num_seqs,
-                                            int t, int sliding_window, int skip_qlen = 0) {
+                                            int t, int sliding_window, int keep_first, int skip_qlen = 0) {
   RowInfo r;
   r.seq = find_seq_idx(cu, num_seqs, t);
   const int q_start = cu[r.seq];
@@ -89,10 +101,13 @@ __device__ __forceinline__ RowInfo row_info(const int32_t* __restrict__ cu,
   if (skip_qlen > 0 && q_len >= skip_qlen) r.eff = 0;  // mixed batch: the tile kernel owns this sequence
   r.beg = 0;
   r.base = 0;
+  r.kept = 0;
   if (sliding_window >= 0) {
     r.beg = max(0, r.eff - sliding_window);
     r.base = r.beg & ~15;
+    r.kept = min((keep_first + 15) >> 4, r.base >> 4);
   }
+  r.gap = r.base - r.kept * 16;
   return r;
 }
 

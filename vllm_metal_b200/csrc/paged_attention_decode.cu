@@ -23,6 +23,7 @@ bool decode_mma_supported(const b200_paged_attn_args& a) {
     if (a.dtype != B200_BF16 && !same) return false;
     if (dk % 8 || dv % 8 || dk > 256 || dv > 256 || (a.window_seqlen_q > 1 && !same)) return false;
   }
+  if (a.window_seqlen_q > 1 && keep_first(a) > 0) return false;  // window batches know one visible stretch a row
   const int G = a.num_q_heads / a.num_kv_heads;
   if (G < 1 || G > 16) return false;
   if (log2_exact_i(a.block_size) < 0) return false;
@@ -76,6 +77,7 @@ int launch_decode_mma(const b200_paged_attn_args& a, const SplitWorkspace* ws, c
   p.block_shift = log2_exact_i(a.block_size);
   p.max_blocks_per_seq = a.max_blocks_per_seq;
   p.sliding_window = a.sliding_window;
+  p.keep_first = keep_first(a);
   p.q_stride = a.q_stride;
   p.out_stride = a.out_stride;
   p.block_stride16 = (uint32_t)(a.kv_block_stride / 8);

@@ -25,6 +25,8 @@
 // time against a V fragment zeroed outside that row's range, so a non-finite V at a position only later rows may see
 // cannot reach earlier rows through 0 * inf (test_windowed_skips_masked_inf_v).
 //
+// Kept first positions (per-row mode): the tiles that hold them precede the window's, see RowInfo.
+//
 // DK / DV: compile-time widths of the products over keys and values.  WIDE forms take any size up to that, the columns past
 // it zero-filled (a run-time width, whose every step is a branch, ran 1.6 times slower).  WIDE: the softmax weights enter P.V
 // as two terms of the operand type; with PACK (at most 8 heads a group) the second terms are the MMA rows the group leaves
@@ -116,7 +118,7 @@ struct DecodeParams {
   const int32_t* cu_seqlens_q;
   const float* sinks;
   int num_seqs, num_q_heads, num_kv_heads, group;
-  int block_shift, max_blocks_per_seq, sliding_window;
+  int block_shift, max_blocks_per_seq, sliding_window, keep_first;
   int64_t q_stride, out_stride;
   uint32_t block_stride16, token_stride16;      // cache strides in 16-byte units
   uint32_t v_block_stride16, v_token_stride16;
@@ -164,6 +166,7 @@ paged_decode_mma_kernel(const DecodeParams p) {
 
   // ---- the CTA's query rows: one (t0), or in window mode nrows consecutive rows of sequence s ----
   int s, t0, nrows, eff0;  // eff0 = KV positions row t0 may see (pagedattention.metal:913); row t0+i sees eff0+i
+  RowInfo ri{};
   if constexpr (WIN) {
     s = blockIdx.y / p.win_subs;
     const int r0 = (blockIdx.y - s * p.win_subs) * p.win_rows;
@@ -175,7 +178,7 @@ paged_decode_mma_kernel(const DecodeParams p) {
     eff0 = p.seq_lens[s] - q_len + r0 + 1;
   } else {
     t0 = blockIdx.y;
-    const RowInfo ri = row_info(p.cu_seqlens_q, p.seq_lens, p.num_seqs, t0, p.sliding_window, p.ws.skip_qlen);
+    ri = row_info(p.cu_seqlens_q, p.seq_lens, p.num_seqs, t0, p.sliding_window, p.keep_first, p.ws.skip_qlen);
     s = ri.seq;
     nrows = 1;
     eff0 = ri.eff;
@@ -202,9 +205,15 @@ paged_decode_mma_kernel(const DecodeParams p) {
     hi = max(end, beg);
     return 2;
   };
+  const bool kept = !WIN && p.keep_first > 0;  // two stretches: the range below counts tokens without the gap between them
   // union of the rows' ranges (what is streamed) and their intersection (where no row masks anything)
   int beg, end, ulo = 0, uhi = 0x7fffffff;
-  {
+  if (kept) {
+    beg = p.partitioned ? part * p.ws.partition_size : 0;
+    end = ri.span();
+    if (beg >= end) return;
+    if (p.partitioned) end = min(end, beg + p.ws.partition_size);
+  } else {
     int umin = 0x7fffffff, umax = 0, live = 0;
     for (int qi = 0; qi < nrows; ++qi) {
       int lo, hi;
@@ -268,14 +277,16 @@ paged_decode_mma_kernel(const DecodeParams p) {
 
   auto issue_tile = [&](int j, int stage) {
     if (j < n_tiles) {
-      const int tok = (first_tile + j) * kTileTokens + (lane & 15);
+      const int at = (first_tile + j) * kTileTokens + (lane & 15);
+      const int tok = kept ? ri.token_at(at) : at;
       int page = tok >> p.block_shift;
       page = min(page, p.max_blocks_per_seq - 1);
       int64_t blk = table[page];
       if (blk < 0 || blk >= p.num_blocks) blk = 0;
       uint32_t koff = (uint32_t)blk * p.block_stride16 + (uint32_t)(tok & block_mask) * p.token_stride16;
       uint32_t voff = (uint32_t)blk * p.v_block_stride16 + (uint32_t)(tok & block_mask) * p.v_token_stride16;
-      if (tok < beg || tok >= end) koff = voff = 0xFFFFFFFFu;  // zero-fill rows outside the range
+      // zero-fill rows outside the range
+      if (at < beg || at >= end || (kept && tok < ri.beg && tok >= p.keep_first)) koff = voff = 0xFFFFFFFFu;
       const uint32_t sbase = warp_smem + stage * STAGE_BYTES;
       if constexpr (!WIDE) {  // one layout for both: one row lookup serves K and V
         constexpr int CHUNKS = DK / 8;       // 16-byte chunks per row
@@ -350,6 +361,7 @@ paged_decode_mma_kernel(const DecodeParams p) {
     }
     // ---- scale, softcap, log2 domain, range mask -------------------------------
     const int tok0 = (first_tile + j) * kTileTokens + 2 * tq;
+    const int moved = kept && first_tile + j >= ri.kept ? ri.gap : 0;
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
@@ -357,7 +369,8 @@ paged_decode_mma_kernel(const DecodeParams p) {
         float v = sacc[nt][e] * sc_mul;
         if (p.softcap > 0.f) v = tanhf(v / p.softcap) * p.softcap * kLog2e;  // :1120-1122,1138
         const int tok = tok0 + nt * 8 + (e & 1);
-        const bool in = e < 2 ? (tok >= lo0 && tok < hi0) : (tok >= lo1 && tok < hi1);
+        bool in = e < 2 ? (tok >= lo0 && tok < hi0) : (tok >= lo1 && tok < hi1);
+        if (kept) in = in && (tok + moved >= ri.beg || tok + moved < p.keep_first);
         sacc[nt][e] = in ? v : -INFINITY;
       }
     }

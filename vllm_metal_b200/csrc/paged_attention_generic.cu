@@ -24,7 +24,7 @@ paged_attention_generic_kernel(T* __restrict__ out, const T* __restrict__ query,
                                const int32_t* __restrict__ cu_seqlens_q,
                                const float* __restrict__ sinks, int num_seqs, int num_q_heads,
                                int num_kv_heads, int head_dim, int v_dim, int block_shift,
-                               int max_blocks_per_seq, int sliding_window, int64_t q_stride,
+                               int max_blocks_per_seq, int sliding_window, int keep_first, int64_t q_stride,
                                int64_t out_stride, int64_t kv_block_stride,
                                int64_t kv_token_stride, int64_t kv_head_stride, ValueStrides vs, int64_t num_blocks,
                                float scale, float softcap, SplitWorkspace ws, bool partitioned) {
@@ -35,14 +35,14 @@ paged_attention_generic_kernel(T* __restrict__ out, const T* __restrict__ query,
   const int part = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 
-  const RowInfo ri = row_info(cu_seqlens_q, seq_lens, num_seqs, t, sliding_window, ws.skip_qlen);
+  const RowInfo ri = row_info(cu_seqlens_q, seq_lens, num_seqs, t, sliding_window, keep_first, ws.skip_qlen);
   const int s = ri.seq, eff = ri.eff;  // eff: pagedattention.metal:913
   if (eff <= 0) return;                // :917-920 (row left untouched)
 
-  int lo = ri.beg, hi = eff;  // window: :1129-1133
+  int lo = keep_first > 0 ? 0 : ri.beg - ri.gap, hi = ri.span();  // window: :1129-1133; counted without the gap
   if (partitioned) {
-    const int p0 = ri.base + part * ws.partition_size;
-    if (p0 >= eff) return;  // :922-926 empty partition: nothing written, reduce skips it
+    const int p0 = part * ws.partition_size;
+    if (p0 >= hi) return;  // :922-926 empty partition: nothing written, reduce skips it
     lo = max(lo, p0);
     hi = min(hi, p0 + ws.partition_size);
   }
@@ -64,7 +64,9 @@ paged_attention_generic_kernel(T* __restrict__ out, const T* __restrict__ query,
 #pragma unroll
   for (int i = 0; i < kMaxEpl; ++i) o[i] = 0.f;
 
-  for (int tok = lo + warp; tok < hi; tok += kGenericWarps) {
+  for (int v = lo + warp; v < hi; v += kGenericWarps) {
+    const int tok = ri.token_at(v);
+    if (tok < ri.beg && tok >= keep_first) continue;  // between the kept positions and the window
     int64_t blk = table[tok >> block_shift];
     if (blk < 0 || blk >= num_blocks) blk = 0;  // padded / corrupt entry: stay in bounds
     const int64_t base = blk * kv_block_stride + (int64_t)(tok & block_mask) * kv_token_stride +
@@ -157,15 +159,14 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 split_reduce_kernel(T* __restrict__ out, const int32_t* __restrict__ seq_lens,
                     const int32_t* __restrict__ cu_seqlens_q, const float* __restrict__ sinks,
-                    int num_seqs, int num_q_heads, int head_dim, int sliding_window,
+                    int num_seqs, int num_q_heads, int head_dim, int sliding_window, int keep_first,
                     int64_t out_stride, SplitWorkspace ws) {
   pdl_trigger();
   pdl_wait();
   const int h = blockIdx.x, t = blockIdx.y;
-  const RowInfo ri = row_info(cu_seqlens_q, seq_lens, num_seqs, t, sliding_window, ws.skip_qlen);
-  const int eff = ri.eff;
-  if (eff <= 0) return;
-  int np = (eff - ri.base + ws.partition_size - 1) / ws.partition_size;  // :1946
+  const RowInfo ri = row_info(cu_seqlens_q, seq_lens, num_seqs, t, sliding_window, keep_first, ws.skip_qlen);
+  if (ri.eff <= 0) return;
+  int np = (ri.span() + ws.partition_size - 1) / ws.partition_size;  // :1946
   np = min(np, ws.num_partitions);
   const int64_t row = ((int64_t)t * num_q_heads + h) * ws.num_partitions;
 
@@ -214,7 +215,7 @@ int launch_generic(const b200_paged_attn_args& a, const SplitWorkspace* ws, cuda
     launch_pdl(paged_attention_generic_kernel<T>, dim3(grid), dim3(kGenericWarps * 32), smem, st, 
         (T*)a.out, (const T*)a.query, (const T*)a.key_cache, (const T*)a.value_cache,
         a.block_tables, a.seq_lens, a.cu_seqlens_q, a.sinks, a.num_seqs, a.num_q_heads,
-        a.num_kv_heads, a.head_dim, value_dim(a), shift, a.max_blocks_per_seq, a.sliding_window, a.q_stride,
+        a.num_kv_heads, a.head_dim, value_dim(a), shift, a.max_blocks_per_seq, a.sliding_window, keep_first(a), a.q_stride,
         a.out_stride, a.kv_block_stride, a.kv_token_stride, a.kv_head_stride, value_strides(a), a.num_blocks,
         a.scale, a.softcap, w, ws != nullptr);
     return check_launch("paged_attention_generic_kernel");
@@ -226,7 +227,7 @@ int launch_split_reduce(const b200_paged_attn_args& a, const SplitWorkspace& ws,
   return B200_DISPATCH_DTYPE(a.dtype, T, [&]() -> int {
     launch_pdl(split_reduce_kernel<T>, dim3(grid), dim3(128), 0, st, (T*)a.out, a.seq_lens, a.cu_seqlens_q, a.sinks,
                                                  a.num_seqs, a.num_q_heads, value_dim(a),
-                                                 a.sliding_window, a.out_stride, ws);
+                                                 a.sliding_window, keep_first(a), a.out_stride, ws);
     return check_launch("split_reduce_kernel");
   });
 }
@@ -256,6 +257,7 @@ static int validate(const b200_paged_attn_args* a) {
   B200_CHECK_ARG(a->dtype == B200_F32 || a->dtype == B200_F16 || a->dtype == B200_BF16,
                  "paged_attention: unsupported dtype code %d", a->dtype);
   B200_CHECK_ARG(a->num_blocks > 0, "paged_attention: num_blocks must be > 0");
+  B200_CHECK_ARG(a->keep_first >= 0, "paged_attention: keep_first must not be negative, got %d", a->keep_first);
   B200_CHECK_ARG(a->window_seqlen_q >= 0, "paged_attention: window_seqlen_q must be >= 1 (1 = per-token decode), got %d",
                  a->window_seqlen_q);
   B200_CHECK_ARG(a->out_dtype == 0 || a->out_dtype == a->dtype || (a->out_dtype == B200_F16 && a->dtype == B200_BF16),
@@ -264,10 +266,11 @@ static int validate(const b200_paged_attn_args* a) {
 }
 
 // Longest KV span any row can cover: a windowed row only walks [eff-W, eff)
-// rounded out to 16-token tiles (see RowInfo).
+// and the kept first positions, rounded out to 16-token tiles (see RowInfo).
 static int effective_span(const b200_paged_attn_args& a) {
   int L = a.max_seq_len;
-  if (a.sliding_window >= 0 && a.sliding_window + 15 < L) L = a.sliding_window + 15;
+  const int seen = a.sliding_window + 15 + (keep_first(a) + 15) / 16 * 16;
+  if (a.sliding_window >= 0 && seen < L) L = seen;
   return L < 1 ? 1 : L;
 }
 

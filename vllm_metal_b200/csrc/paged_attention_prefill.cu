@@ -24,6 +24,8 @@
 // out of the products.  Values of up to 192 columns fit beside 64-token score tiles (KV = 64); wider ones are cut into slices
 // of at most 128, one CTA each (blockIdx.z), which repeat the scores.
 //
+// Kept first positions beside a window: their blocks are walked ahead of the window's, masked by position.
+//
 // Flops per launch: 4 * D * sum_i q_i * (ctx_i + (q_i + 1) / 2) per q head (causal).
 #include "paged_attention.cuh"
 #include "tcgen05.cuh"
@@ -44,7 +46,7 @@ struct Params {
   const int32_t* cu;
   const float* sinks;
   int num_seqs, num_q_tokens, num_kv_heads, group;
-  int block_size, pages_per_tile, max_blocks_per_seq, sliding_window, min_qlen;
+  int block_size, pages_per_tile, max_blocks_per_seq, sliding_window, keep_first, min_qlen;
   int64_t out_stride;
   float scale, softcap, denom_eps;
   int head_dim, value_dim, slice;  // slice: value columns per CTA
@@ -142,7 +144,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   if (kv_hi <= 0) return;
   const int kv_lo = p.sliding_window >= 0 ? max(0, qabs0 + 1 - p.sliding_window) : 0;
   const int j0 = kv_lo / BK, j1 = (kv_hi - 1) / BK;   // KV blocks j0..j1
-  const int nblk = j1 - j0 + 1;
+  // kept first positions: the blocks that hold them and precede the window's come first
+  const int kept = min((p.keep_first + BK - 1) / BK, j0);
+  const int nblk = j1 - j0 + 1 + kept;
+  auto block_at = [&](int it) { return it < kept ? it : j0 + it - kept; };
 
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -202,7 +207,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
     int st = 0;
     uint32_t ph = 1;
     for (int it = 0; it < nblk; ++it) {
-      const int tok0 = (j0 + it) * BK;
+      const int tok0 = block_at(it) * BK;
       // block ids of this tile's pages: lane l holds page l (pages wholly past seq_len read block 0 and are masked)
       int bid_l = 0;
       if (lane < p.pages_per_tile) {
@@ -274,7 +279,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           mbar_wait(bar_v_full + 8 * st, (it / STAGES) & 1);
           // V rows at positions >= seq_len are whatever the pool holds (another sequence's page, never-written
           // memory): their P is 0, but 0 * NaN would poison O, so those rows are zeroed before the product
-          const int nvalid = seq_len - (j0 + it) * BK;
+          const int nvalid = seq_len - block_at(it) * BK;
           if (nvalid < BK) {
             for (int idx = lane; idx < (BK - nvalid) * 8 * SM::V_HALVES; idx += 32) {
               const int row = nvalid + idx / (8 * SM::V_HALVES), rem = idx % (8 * SM::V_HALVES);
@@ -311,6 +316,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       // this row sees KV positions [row_lo, row_hi); rows past the tile's valid rows see nothing
       const int row_hi = r < nrows ? min(seq_len, qabs + 1) : 0;
       const int row_lo = p.sliding_window >= 0 ? max(0, qabs + 1 - p.sliding_window) : 0;
+      const int row_keep = min(p.keep_first, row_hi);
       const float sc = p.scale * kLog2e;
       const float cap_in = SOFTCAP ? p.scale / p.softcap : 0.f, cap_out = SOFTCAP ? p.softcap * kLog2e : 0.f;  // tanh(s*scale/c)*c
       const float inv_sc = SOFTCAP ? 1.f / sc : 0.f;
@@ -332,7 +338,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 #pragma unroll
             for (int q = 0; q < 32; ++q) s[g * 32 + q] = __uint_as_float(v[g][q]);
         }
-        const int kv0 = (j0 + it) * BK;
+        const int kv0 = block_at(it) * BK;
         // The softmax threads are instruction-issue bound (a polynomial ex2 on the FMA pipe made the kernel 20% SLOWER),
         // so the row is touched as little as possible: the max is taken over the RAW scores (scale > 0 commutes with
         // max), the scale and the max subtraction are one packed fma per column pair, the row sum one packed add.
@@ -345,7 +351,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           for (int c = 0; c < BK; ++c) {
             float x = SOFTCAP ? tanh_approx(s[c] * cap_in) * cap_out * inv_sc : s[c];  // back in raw-score units
             const int kv = kv0 + c;
-            x = (kv >= row_lo && kv < row_hi) ? x : -INFINITY;
+            x = (kv >= row_lo && kv < row_hi) || kv < row_keep ? x : -INFINITY;
             s[c] = x;
             m_raw = fmaxf(m_raw, x);
           }
@@ -521,6 +527,7 @@ static int launch(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) 
   p.pages_per_tile = KV / a.block_size;
   p.max_blocks_per_seq = a.max_blocks_per_seq;
   p.sliding_window = a.sliding_window;
+  p.keep_first = keep_first(a);
   p.min_qlen = min_qlen;
   p.out_stride = a.out_stride;
   p.scale = a.scale;

@@ -16,6 +16,7 @@
 // 2*Hkv*D*esize cache write.
 #include "common.cuh"
 #include "../../include/b200_decoder_ops.h"
+#include "../../include/b200_hybrid_ops.h"
 
 namespace b200 {
 
@@ -111,7 +112,136 @@ norm_rope_cache_kernel(T* __restrict__ q, T* __restrict__ k, const T* __restrict
   }
 }
 
+// ---- the other order: RoPE -> per-head norm without a weight -> cache --------------------------------
+// Angles from a frequency table (scaled rotations), once per token and CTA.  One CTA per token, a warp per head, a lane
+// holds the pairs lane, lane + 32, ... of the head in registers from load to store.
+template <typename T>
+struct alignas(2 * sizeof(T)) Pair {
+  T a, b;
+};
+template <typename T, int NP, bool VEC>
+__device__ __forceinline__ void load_pairs(const T* src, int dim, float2 (&v)[NP]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {
+    const int e = 2 * (lane + 32 * j);
+    v[j] = make_float2(0.f, 0.f);
+    if (VEC) {
+      if (e < dim) {
+        const Pair<T> p = *reinterpret_cast<const Pair<T>*>(src + e);
+        v[j] = make_float2(to_float(p.a), to_float(p.b));
+      }
+    } else {
+      if (e < dim) v[j].x = to_float(src[e]);
+      if (e + 1 < dim) v[j].y = to_float(src[e + 1]);
+    }
+  }
+}
+
+template <typename T, int NP, bool VEC>
+__global__ void __launch_bounds__(RC_WARPS * 32)
+rope_norm_cache_kernel(const b200_rope_norm_cache_args a) {
+  __shared__ float2 turn[RC_MAX_D / 2];  // factor * (cos, sin)
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const float pos = (float)a.positions[t];
+  for (int i = threadIdx.x; 2 * i < a.rot_dims; i += RC_WARPS * 32) {
+    // what the rounded product and the frequency's low part leave of the angle, r, turns it by a Taylor step
+    const float hi = a.freq[2 * i], ang = pos * hi, r = fmaf(pos, a.freq[2 * i + 1], fmaf(pos, hi, -ang));
+    float sn, cs;
+    sincosf(ang, &sn, &cs);
+    const float s1 = fmaf(-r * r, r * (1.f / 6.f), r), c1 = -0.5f * r * r;  // sin r, cos r - 1
+    turn[i] = make_float2(a.rot_factor * (cs + fmaf(-s1, sn, c1 * cs)), a.rot_factor * (sn + fmaf(s1, cs, c1 * sn)));
+  }
+  __syncthreads();
+  const int64_t slot = a.slot_mapping[t];
+  const bool cached = slot >= 0 && slot < a.num_blocks * a.block_size;
+  const int64_t blk = cached ? slot / a.block_size : 0, off = cached ? slot - blk * a.block_size : 0;
+  T* krow = reinterpret_cast<T*>(a.key_cache) + blk * a.k_block_stride + off * a.k_token_stride;
+  T* vrow = reinterpret_cast<T*>(a.value_cache) + blk * a.v_block_stride + off * a.v_token_stride;
+  for (int h = blockIdx.y * RC_WARPS + warp; h < a.heads + 2 * a.kv_heads; h += RC_WARPS * gridDim.y) {
+    if (h >= a.heads + a.kv_heads) {
+      const int hv = h - a.heads - a.kv_heads;
+      const T* src = reinterpret_cast<const T*>(a.v) + (int64_t)t * a.v_stride + (int64_t)hv * a.vdim;
+      T* dst = vrow + (int64_t)hv * a.vdim;
+      if (!cached) continue;
+      if (a.vdim % (16 / sizeof(T)) == 0 && (((uintptr_t)src | (uintptr_t)dst) & 15) == 0) {
+        for (int i = lane; i < a.vdim / (int)(16 / sizeof(T)); i += 32)
+          reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+      } else {
+        for (int i = lane; i < a.vdim; i += 32) dst[i] = src[i];
+      }
+      continue;
+    }
+    const bool is_q = h < a.heads;
+    if (!is_q && !cached) continue;
+    T* qrow = reinterpret_cast<T*>(a.q) + (int64_t)t * a.q_stride + (int64_t)h * a.dim;
+    const T* src = is_q ? qrow : reinterpret_cast<const T*>(a.k) + (int64_t)t * a.k_stride + (int64_t)(h - a.heads) * a.dim;
+    T* dst = is_q ? qrow : krow + (int64_t)(h - a.heads) * a.dim;
+    float2 v[NP];
+    load_pairs<T, NP, VEC>(src, a.dim, v);
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < NP; ++j) {
+      const int i = lane + 32 * j;
+      if (2 * i < a.rot_dims) {
+        const float2 w = turn[i];
+        v[j] = make_float2(v[j].x * w.x - v[j].y * w.y, v[j].y * w.x + v[j].x * w.y);
+      }
+      ss += v[j].x * v[j].x + v[j].y * v[j].y;
+    }
+    float f = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
+    if (is_q && a.q_weight) f *= a.q_weight[h];
+#pragma unroll
+    for (int j = 0; j < NP; ++j) {
+      const int e = 2 * (lane + 32 * j);
+      if (VEC) {
+        if (e < a.dim) *reinterpret_cast<Pair<T>*>(dst + e) = Pair<T>{from_float<T>(v[j].x * f), from_float<T>(v[j].y * f)};
+      } else {
+        if (e < a.dim) dst[e] = from_float<T>(v[j].x * f);
+        if (e + 1 < a.dim) dst[e + 1] = from_float<T>(v[j].y * f);
+      }
+    }
+  }
+}
+
+template <typename T, bool VEC>
+int launch_rope_norm_cache(const b200_rope_norm_cache_args& a, cudaStream_t st) {
+  const int total = a.heads + 2 * a.kv_heads, need = (total + RC_WARPS - 1) / RC_WARPS;
+  const dim3 grid(a.num_tokens, a.num_tokens >= 1024 ? 1 : need);
+  auto* kern = a.dim <= 64    ? rope_norm_cache_kernel<T, 1, VEC>
+               : a.dim <= 128 ? rope_norm_cache_kernel<T, 2, VEC>
+               : a.dim <= 256 ? rope_norm_cache_kernel<T, 4, VEC>
+                              : rope_norm_cache_kernel<T, 8, VEC>;
+  B200_CUDA_OK(launch_pdl(kern, grid, dim3(RC_WARPS * 32), 0, st, a));
+  return check_launch("rope_norm_cache");
+}
+
 }  // namespace b200
+
+extern "C" int b200_rope_norm_cache(const b200_rope_norm_cache_args* a, void* stream) {
+  using namespace b200;
+  B200_CHECK_ARG(a && a->q && a->k && a->v && a->key_cache && a->value_cache && a->positions && a->slot_mapping,
+                 "rope_norm_cache: null pointer argument");
+  B200_CHECK_ARG(a->heads > 0 && a->kv_heads > 0 && a->vdim > 0 && a->dim > 0 && a->dim <= RC_MAX_D,
+                 "rope_norm_cache: head size must be in [1, %d], got %d (heads %d/%d)", RC_MAX_D, a->dim, a->heads, a->kv_heads);
+  B200_CHECK_ARG(a->rot_dims >= 0 && a->rot_dims % 2 == 0 && a->rot_dims <= a->dim && (a->rot_dims == 0 || a->freq),
+                 "rope_norm_cache: %d rotated of %d dimensions", a->rot_dims, a->dim);
+  B200_CHECK_ARG(a->block_size > 0 && a->num_blocks > 0 && a->k_token_stride >= (int64_t)a->kv_heads * a->dim &&
+                     a->v_token_stride >= (int64_t)a->kv_heads * a->vdim,
+                 "rope_norm_cache: bad cache geometry");
+  if (a->num_tokens <= 0) return B200_OK;
+  return B200_DISPATCH_DTYPE(a->dtype, T, [&]() -> int {
+    auto ok = [](const void* p, int64_t s0, int64_t s1) {
+      return (uintptr_t)p % (2 * sizeof(T)) == 0 && s0 % 2 == 0 && s1 % 2 == 0;
+    };
+    const bool vec = a->dim % 2 == 0 && ok(a->q, a->q_stride, 0) && ok(a->k, a->k_stride, 0) &&
+                     ok(a->key_cache, a->k_block_stride, a->k_token_stride);
+    return vec ? launch_rope_norm_cache<T, true>(*a, (cudaStream_t)stream)
+               : launch_rope_norm_cache<T, false>(*a, (cudaStream_t)stream);
+  });
+}
 
 extern "C" int b200_norm_rope_cache(void* q, void* k, const void* v, const void* q_norm_weight,
                                     const void* k_norm_weight, const int32_t* positions,

@@ -40,6 +40,12 @@ class StackedLinear:
     def __call__(self, x: torch.Tensor) -> torch.Tensor:
         return torch.mm(x, self.weight.t())
 
+    def wide(self, x: torch.Tensor) -> torch.Tensor:
+        """The product kept in fp32."""
+        if x.dtype == torch.float32:
+            return torch.mm(x, self.weight.t())
+        return torch.mm(x, self.weight.t(), out_dtype=torch.float32)
+
     def split(self, y: torch.Tensor) -> dict[str, torch.Tensor]:
         return {name: y[:, lo:hi] for name, (lo, hi) in self.slices.items()}
 

@@ -4,8 +4,12 @@ sees typed records only.  What a design fixes -- how a layer is arranged, its no
 
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass
 from typing import Any
+
+MAX_EXPERTS = 1024    # what the routing kernels take (B200_MAX_EXPERTS)
+MAX_INPUT_TAPS = 16
 
 
 class ConfigError(ValueError):
@@ -160,17 +164,118 @@ class SideBySideArgs:
                    LightningArgs.parse(_take(m, "right", where, dict), f"{where}.right"))
 
 
-MixerArgs = LatentAttentionArgs | Mamba2Args | MLSTMArgs | LightningArgs | SideBySideArgs
-MIXER_ARGS = {c.kind: c for c in (LatentAttentionArgs, Mamba2Args, MLSTMArgs, LightningArgs, SideBySideArgs)}
+@dataclass(frozen=True)
+class RotaryArgs:
+    """Rotation of the first ``dims`` dimensions of a head; with ``factor`` > 0 the frequencies are scaled (YaRN)."""
+
+    dims: int
+    base: float
+    factor: float = 0.0
+    original: float = 0.0
+    fast: float = 0.0
+    slow: float = 0.0
+
+    @classmethod
+    def parse(cls, rot: dict | None, where: str) -> RotaryArgs:
+        if not rot:
+            return cls(0, 1.0)
+        where = f"{where}.rot"
+        s = rot.get("scaling")
+        a = cls(_take(rot, "dims", where), _take(rot, "base", where, float),
+                **({} if not s else {k: _take(s, k, f"{where}.scaling", float) for k in ("factor", "original", "fast", "slow")}))
+        if a.dims < 0 or a.dims % 2 or (a.dims and not a.base > 1):
+            raise ConfigError(f"{where}: dims {a.dims} must be even, base {a.base} above 1")
+        if s and not (a.factor > 0 and a.original > 0 and a.fast > 0 and a.slow > 0):
+            raise ConfigError(f"{where}.scaling: factor, original, fast and slow must be positive")
+        return a
+
+    def frequencies(self) -> list[float]:
+        """Angle per position of every pair."""
+        plain = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if not self.factor or not self.dims:
+            return plain
+        # the pair (a real number) that turns `t` times over the original length
+        pair = lambda t: self.dims * math.log(self.original / (2 * math.pi * t)) / (2 * math.log(self.base))  # noqa: E731
+        lo, hi = max(math.floor(pair(self.fast)), 0), min(math.ceil(pair(self.slow)), self.dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(len(plain))]
+        return [f / self.factor * r + f * (1.0 - r) for f, r in zip(plain, ramp)]
+
+    @property
+    def amplitude(self) -> float:
+        """What cosine and sine are multiplied by."""
+        return 0.1 * math.log(self.factor) + 1.0 if self.factor else 1.0
+
+
+@dataclass(frozen=True)
+class RotaryAttentionArgs:
+    """Softmax attention with rotated, then normed heads; a window and the first tokens kept beside it."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotaryArgs
+    window: int      # 0: every earlier token is visible
+    keep_first: int  # of the first tokens, visible whatever the window
+
+    kind = "attention"
+
+    @classmethod
+    def parse(cls, m: dict, where: str) -> RotaryAttentionArgs:
+        a = SoftmaxAttentionArgs.parse(m, where)
+        mask = m.get("mask") or {}
+        b = cls(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, RotaryArgs.parse(m.get("rot"), where),
+                int(mask.get("size") or 0), int(mask.get("keep_first") or 0))
+        if b.rot.dims > b.dim or b.window < 0 or b.keep_first < 0:
+            raise ConfigError(f"{where}: rot.dims {b.rot.dims} of dim {b.dim}, mask.size {b.window}, mask.keep_first {b.keep_first}")
+        return b
+
+
+MixerArgs = LatentAttentionArgs | Mamba2Args | MLSTMArgs | LightningArgs | SideBySideArgs | RotaryAttentionArgs
+MIXER_ARGS = {c.kind: c for c in (LatentAttentionArgs, Mamba2Args, MLSTMArgs, LightningArgs, SideBySideArgs,
+                                  RotaryAttentionArgs)}
+
+
+@dataclass(frozen=True)
+class RoutedArgs:
+    """Feed-forward of routed experts, with a gated shared one beside them."""
+
+    experts: int
+    top: int
+    ff: int
+    scale: float
+    shared_ff: int  # 0: none
+
+    @classmethod
+    def parse(cls, mlp: dict, where: str) -> RoutedArgs:
+        where = f"{where}.mlp"
+        router = _take(mlp, "router", where, dict)
+        shared = mlp.get("shared")
+        a = cls(_take(router, "experts", f"{where}.router"), _take(router, "top", f"{where}.router"),
+                _take(_take(mlp, "expert", where, dict), "ff", f"{where}.expert"),
+                _take(router, "scale", f"{where}.router", float), _take(shared, "ff", f"{where}.shared") if shared else 0)
+        _positive(a, where, "experts", "top", "ff")
+        if a.top > a.experts or a.experts > MAX_EXPERTS:
+            raise ConfigError(f"{where}: {a.top} of {a.experts} experts (at most {MAX_EXPERTS})")
+        if shared and a.shared_ff < 1:
+            raise ConfigError(f"{where}.shared: ff must be at least 1")
+        return a
 
 
 def paged_row(mixer: MixerArgs) -> int:
     """Elements a layer with this mixer caches per token."""
     if isinstance(mixer, LatentAttentionArgs):
         return mixer.kv_rank + mixer.rot_dim
+    a = cached_heads(mixer)
+    return a.kv_heads * (a.dim + a.vdim) if a is not None else 0
+
+
+def cached_heads(mixer: MixerArgs) -> SoftmaxAttentionArgs | RotaryAttentionArgs | None:
+    """The attention whose keys and values (of ``kv_heads``) a layer with this mixer caches, if any."""
     if isinstance(mixer, SideBySideArgs):
-        return mixer.left.kv_heads * (mixer.left.dim + mixer.left.vdim)
-    return 0
+        return mixer.left
+    return mixer if isinstance(mixer, RotaryAttentionArgs) else None
 
 
 @dataclass(frozen=True)
@@ -178,20 +283,29 @@ class Design:
     """What the architecture fixes."""
 
     mixers: tuple[str, ...]
-    hyper_connected: bool = False  # sublayers around several streams (lm/streams.py), else parallel layers (lm/hybrid.py)
+    # "parallel": mixer and feed-forward from one norm (lm/hybrid.py); "hyper": sublayers around several streams
+    # (lm/streams.py); "sandwich": sublayers between two norms, a short convolution on the mixer's input (lm/sandwich.py)
+    layout: str = "parallel"
+    feed_forward: str = "dense"
+
+    @property
+    def hyper_connected(self) -> bool:
+        return self.layout == "hyper"
 
 
 DESIGNS = {
     "Mapuvik": Design(("latent_attention", "mamba2", "mlstm")),
-    "Tatazen": Design(("lightning", "parallel"), hyper_connected=True),
+    "Tatazen": Design(("lightning", "parallel"), "hyper"),
+    "Kerolorn": Design(("attention",), "sandwich", "moe"),
 }
 
 
 @dataclass(frozen=True)
 class LayerArgs:
     mixer: MixerArgs
-    ff: int       # 0: no feed-forward
+    ff: int       # dense feed-forward; 0: none
     weights: int  # the layer whose tensors this one uses (itself unless shared)
+    routed: RoutedArgs | None = None
 
 
 @dataclass(frozen=True)
@@ -202,6 +316,8 @@ class HybridArgs:
     eps: float
     layers: tuple[LayerArgs, ...]  # in the order they run: a looped layer is there once a pass
     streams: int = 1               # copies of the residual stream (hyper-connected designs)
+    input_taps: int = 0            # of the convolution on a mixer's input (2: token shift); 0: none
+    logit_scale: float = 1.0
 
     @property
     def design(self) -> Design:
@@ -237,14 +353,17 @@ class HybridArgs:
             if kind not in design.mixers:
                 raise ConfigError(f"{where}: unknown mixer '{kind}' (known: {', '.join(sorted(design.mixers))})")
             mixer = MIXER_ARGS[kind].parse(_take(entry, "mixer", where, dict), where)
-            ff = 0
+            ff, routed = 0, None
             if entry.get("mlp") is not None:
                 mlp = entry["mlp"]
-                if mlp.get("kind", "dense") != "dense":
-                    raise ConfigError(f"{where}: feed-forward kind '{mlp.get('kind')}' is not supported (dense only)")
-                ff = _take(mlp, "ff", where)
-                if ff < 1:
-                    raise ConfigError(f"{where}: ff must be at least 1")
+                if mlp.get("kind", "dense") != design.feed_forward:
+                    raise ConfigError(f"{where}: feed-forward kind '{mlp.get('kind')}' is not supported ({design.feed_forward} only)")
+                if design.feed_forward == "moe":
+                    routed = RoutedArgs.parse(mlp, where)
+                else:
+                    ff = _take(mlp, "ff", where)
+                    if ff < 1:
+                        raise ConfigError(f"{where}: ff must be at least 1")
             src = entry.get("weights_of")
             src = i if src is None else int(src)
             if src != i:
@@ -259,14 +378,21 @@ class HybridArgs:
                     src = int(entry_list[src]["weights_of"])
                 if entry_list[src]["type"] != kind:
                     raise ConfigError(f"{where}: weights_of {src} names a layer of type {entry_list[src]['type']}")
-            layers.append(LayerArgs(mixer, ff, src))
+            layers.append(LayerArgs(mixer, ff, src, routed))
         if not layers:
             raise ConfigError(f"{name}: no layers")
         if config.get("loop") is not None:
             layers = cls._unroll(layers, config["loop"], name)
+        extra: dict[str, Any] = {}
+        if design.layout == "hyper":
+            extra = dict(streams=_take(config, "streams", name), input_taps=2)
+        elif design.layout == "sandwich":
+            extra = dict(input_taps=_take(_take(config, "canon", name, dict), "taps", f"{name}: canon"),
+                         logit_scale=_take(config, "logit_scale", name, float))
+            if not 1 <= extra["input_taps"] <= MAX_INPUT_TAPS:
+                raise ConfigError(f"{name}: canon.taps {extra['input_taps']} outside 1..{MAX_INPUT_TAPS}")
         a = cls(name=name, vocab=_take(config, "vocab", name), width=_take(config, "width", name),
-                eps=_take(_take(config, "norm", name, dict), "eps", name, float), layers=tuple(layers),
-                streams=_take(config, "streams", name) if design.hyper_connected else 1)
+                eps=_take(_take(config, "norm", name, dict), "eps", name, float), layers=tuple(layers), **extra)
         _positive(a, name, "vocab", "width", "streams")
         return a
 

@@ -5,7 +5,8 @@ from __future__ import annotations
 
 import torch
 
-from .hybrid_config import HybridArgs, LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs, SideBySideArgs
+from .hybrid_config import (HybridArgs, LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs, RotaryAttentionArgs,
+                            SideBySideArgs)
 
 
 def tensor_shapes(args: HybridArgs) -> dict[str, tuple[int, ...]]:
@@ -37,8 +38,23 @@ def tensor_shapes(args: HybridArgs) -> dict[str, tuple[int, ...]]:
                        p + "left.v": (a.kv_heads * a.vdim, w), p + "left.q.norm": (a.dim,), p + "left.k.norm": (a.dim,),
                        p + "left.o": (w, a.heads * a.vdim), **_lightning_shapes(m.right, p + "right.", w),
                        p + "left.out": (w,), p + "right.out": (w,)}
+        elif isinstance(m, RotaryAttentionArgs):
+            shapes |= {p + "q": (m.heads * m.dim, w), p + "k": (m.kv_heads * m.dim, w), p + "v": (m.kv_heads * m.vdim, w),
+                       p + "temp": (m.heads,), p + "o": (w, m.heads * m.vdim)}
         if layer.ff:
             shapes |= {f"l{i}.mlp.up": (layer.ff, w), f"l{i}.mlp.down": (w, layer.ff)}
+        if layer.routed is not None:
+            r, p = layer.routed, f"l{i}.mlp."
+            units = [(f"e{e}.", r.ff) for e in range(r.experts)] + ([("shared.", r.shared_ff)] if r.shared_ff else [])
+            for name, ff in units:
+                shapes |= {p + name + "gate": (ff, w), p + name + "up": (ff, w), p + name + "down": (w, ff)}
+            shapes |= {p + "router": (r.experts, w), p + "correction": (r.experts,)}
+            if r.shared_ff:
+                shapes |= {p + "shared.sg": (1, w)}
+        if args.design.layout == "sandwich":
+            shapes |= {f"l{i}.norm1b": (w,), f"l{i}.canon1": (w, args.input_taps)}
+            if layer.routed is not None:
+                shapes |= {f"l{i}.norm2": (w,), f"l{i}.norm2b": (w,)}
         if args.design.hyper_connected:
             s = args.streams
             shapes |= {f"l{i}.shift": (w,)}
@@ -58,15 +74,19 @@ def _lightning_shapes(m: LightningArgs, p: str, w: int) -> dict[str, tuple[int, 
 def random_tensors(args: HybridArgs, device="cpu", seed: int = 0):
     """A ``get(name, shape)`` for ``HybridModel`` whose tensors are drawn when asked for."""
     shapes = tensor_shapes(args)
+    number = {name: i for i, name in enumerate(shapes)}
 
     def get(name: str, shape: tuple[int, ...]) -> torch.Tensor:
         if shapes[name] != tuple(shape):
             raise ValueError(f"tensor '{name}': asked for {shape}, the configuration says {shapes[name]}")
-        gen = torch.Generator(device=device).manual_seed(seed * 1000003 + list(shapes).index(name))
+        gen = torch.Generator(device=device).manual_seed(seed * 1000003 + number[name])
         t = torch.empty(shape, dtype=torch.float32, device=device).normal_(0.0, 1.0, generator=gen)
         leaf = name.split(".", 1)[-1]
-        plain_norm = args.design.hyper_connected and len(shape) == 1 and leaf.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2")
-        if leaf in ("mix.dkv.norm", "mix.norm", "mix.left.out", "mix.right.out") or plain_norm:
+        plain_norm = args.design.layout != "parallel" and len(shape) == 1 and leaf.rsplit(".", 1)[-1] in (
+            "norm", "norm1", "norm2", "norm1b", "norm2b", "temp")
+        if leaf == "mlp.correction":          # of the size of the scores it is added to
+            t = 0.5 * t / shape[0]
+        elif leaf in ("mix.dkv.norm", "mix.norm", "mix.left.out", "mix.right.out") or plain_norm:
             t = 1.0 + 0.1 * t
         elif leaf in ("hc1.in", "hc2.in"):     # about the mean of the streams
             t = (1.0 + 0.3 * t) / shape[0]

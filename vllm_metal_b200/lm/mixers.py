@@ -13,7 +13,8 @@ import torch
 
 from ..attention.impls.segments import EXPAND_PAGE
 from ..metal import get_ops
-from .hybrid_config import LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs, SoftmaxAttentionArgs
+from .hybrid_config import (LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs, RotaryAttentionArgs,
+                            SoftmaxAttentionArgs)
 
 Get = Callable[[str, tuple[int, ...]], torch.Tensor]
 
@@ -131,6 +132,35 @@ class SoftmaxAttentionMixer(Mixer):
             ops.mixer_finish(y, inner, up, act_offset)
 
 
+class RotaryAttentionMixer(Mixer):
+    """Causal attention over paged keys and values: heads rotated, then normed, scores scaled per head; a sliding window
+    and the first tokens kept beside it."""
+
+    def __init__(self, m: RotaryAttentionArgs, width: int, eps: float, get: Get, dtype, device) -> None:
+        self.m, self.eps = m, eps
+        self.weights = {"q": get("q", (m.heads * m.dim, width)), "k": get("k", (m.kv_heads * m.dim, width)),
+                        "v": get("v", (m.kv_heads * m.vdim, width))}
+        self.out_weight = get("o", (width, m.heads * m.vdim))
+        self.temperature = get("temp", (m.heads,)).to(device=device, dtype=torch.float32)
+        f = torch.tensor(m.rot.frequencies(), dtype=torch.float64)
+        self.freq = torch.stack([f.float(), (f - f.float().double()).float()], dim=1).contiguous().to(device)
+
+    def run(self, parts, up, meta, cache, layer: int, y: torch.Tensor, act_offset: int) -> None:
+        m, ops = self.m, get_ops()
+        keys, values = cache.kv[layer]
+        q, k, v = (parts[n].unflatten(1, (h, d)) for n, h, d in (("q", m.heads, m.dim), ("k", m.kv_heads, m.dim),
+                                                                  ("v", m.kv_heads, m.vdim)))
+        ops.rope_norm_cache(q, k, v, keys, values, meta.slot_mapping, meta.positions, self.freq, m.rot.amplitude, self.eps,
+                            self.temperature)
+        inner = m.heads * m.vdim
+        ops.paged_attention_primitive(q, keys, values, m.kv_heads, m.scale, 0.0, meta.block_tables, meta.seq_lens,
+                                      meta.cu_seqlens_q, meta.block_size, meta.max_seq_len, m.window if m.window > 0 else -1,
+                                      y[:, :inner].unflatten(1, (m.heads, m.vdim)), wide_weights=True, plain_softmax=True,
+                                      min_q_len=meta.min_q_len, keep_first=m.keep_first)
+        if up is not None or y.shape[1] > inner:
+            ops.mixer_finish(y, inner, up, act_offset)
+
+
 class LatentAttentionMixer(Mixer):
     """Latent attention: short segments attend in the latent space (queries are taken there by the keys' up-projection),
     long ones get their visible keys and values expanded first, whichever is the smaller work."""
@@ -221,4 +251,4 @@ class LatentAttentionMixer(Mixer):
 
 MIXERS = {c: k for c, k in ((LatentAttentionArgs, LatentAttentionMixer), (Mamba2Args, Mamba2Mixer),
                             (MLSTMArgs, MLSTMMixer), (LightningArgs, LightningMixer),
-                            (SoftmaxAttentionArgs, SoftmaxAttentionMixer))}
+                            (SoftmaxAttentionArgs, SoftmaxAttentionMixer), (RotaryAttentionArgs, RotaryAttentionMixer))}

@@ -57,9 +57,10 @@ class HybridFamily(ModelFamily):
     @staticmethod
     def model_class(args: HybridArgs) -> type:
         from .hybrid import HybridModel
+        from .sandwich import SandwichModel
         from .streams import StreamModel
 
-        return StreamModel if args.design.hyper_connected else HybridModel
+        return {"parallel": HybridModel, "hyper": StreamModel, "sandwich": SandwichModel}[args.design.layout]
 
     def make_cache(self, args, num_blocks, block_size, num_slots, dtype, device):
         from ..attention.caches.hybrid_cache import HybridCache
@@ -92,6 +93,7 @@ _DECODER = DecoderFamily()
 FAMILIES: dict[str, ModelFamily] = {
     "Mapuvik": HybridFamily("hybrid"),
     "Tatazen": HybridFamily("streams"),
+    "Kerolorn": HybridFamily("sandwich"),
     **dict.fromkeys(("LlamaForCausalLM", "MistralForCausalLM", "Qwen3ForCausalLM", "GptOssForCausalLM"), _DECODER),
 }
 

@@ -92,7 +92,7 @@ class StreamLayer:
                                          **step)
         else:
             h, _ = ops.stream_step(streams, result, self.mix.reader, **step)
-            shifted = ops.causal_conv(h, self.shift_taps, None, previous.unsqueeze(1), meta, silu=False)
+            shifted = ops.causal_conv(h, self.shift_taps, None, previous, meta, silu=False)
         stacked = self.input(shifted)
         parts = self.input.split(stacked)
         out = dict(self.mix.writer, gate=self.gate.split(self.gate(h))["gate"])

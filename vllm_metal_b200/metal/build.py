@@ -29,6 +29,9 @@ COMPONENTS: dict[str, tuple[str, ...]] = {
                "paged_attention_decode_packed", "paged_attention_decode_wide", "paged_attention_generic", "paged_attention_prefill", "recurrence"),
     "streams": ("c_abi", "decoder_ops", "hybrid_ops", "paged_attention_decode", "paged_attention_decode_packed",
                 "paged_attention_decode_wide", "paged_attention_generic", "paged_attention_prefill", "recurrence", "rope_cache", "stream_ops"),
+    "sandwich": ("c_abi", "decoder_ops", "experts", "hybrid_ops", "paged_attention_decode", "paged_attention_decode_packed",
+                 "paged_attention_decode_wide", "paged_attention_generic", "paged_attention_prefill", "residual_step",
+                 "rope_cache"),
 }
 _wanted: list[str] = []  # the component this process asked for last
 

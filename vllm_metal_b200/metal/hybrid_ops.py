@@ -1,5 +1,5 @@
 """Operator surface of ``include/b200_hybrid_ops.h``: the mixers of hybrid decoders (latent attention, gated linear
-recurrences), the norms / gates either side of them and the hyper-connected residual.  ``HybridOps`` is mixed into the object ``get_ops()`` returns;
+recurrences), the norms / gates either side of them, the residual steps and the routed experts.  ``HybridOps`` is mixed into the object ``get_ops()`` returns;
 like there, a CPU tensor or an unsupported size raises and nothing falls back."""
 
 from __future__ import annotations
@@ -33,6 +33,17 @@ HYBRID_SYMBOLS = (
 )
 
 STREAM_SYMBOLS = ("b200_embed_streams", "b200_stream_step")
+
+SANDWICH_SYMBOLS = (
+    "b200_residual_step",
+    "b200_rope_norm_cache",
+    "b200_expert_route",
+    "b200_expert_plan",
+    "b200_expert_product",
+    "b200_expert_product_failed",
+)
+
+EXPERT_TILES = (32, 64, 128)  # pairs per tile of the expert products
 
 RECURRENCE_CHUNKS = (64, 128)  # rows per chunk of the two chunked forms
 RECURRENCE_TILE_V = 64
@@ -72,6 +83,20 @@ LatentPrepArgs = _struct(
     L="q_stride down_stride q_out_stride num_slots",
     I="num_tokens heads dim rot_dim rot_dims kv_rank q_cols rot_offset copy_nope",
     F="eps", I2="dtype")
+ResidualStepArgs = _struct(
+    "ResidualStepArgs", "b200_residual_step_args",
+    P="x y part_weight extra extra_gate out_norm in_norm h conv_weight state slots seq_lens row_ids",
+    L="y_stride extra_stride gate_stride h_stride", I="rows dim parts taps", F="eps", I2="dtype")
+RopeNormCacheArgs = _struct(
+    "RopeNormCacheArgs", "b200_rope_norm_cache_args",
+    P="q k v q_weight freq positions slot_mapping key_cache value_cache",
+    L="q_stride k_stride v_stride k_block_stride k_token_stride v_block_stride v_token_stride num_blocks",
+    I="num_tokens heads kv_heads dim vdim rot_dims block_size", F="rot_factor eps", I2="dtype")
+ExpertProductArgs = _struct(
+    "ExpertProductArgs", "b200_expert_product_args",
+    P="x w out shared_x shared_w shared_out pairs first tiles",
+    L="x_stride w_stride out_stride shared_x_stride shared_w_stride shared_out_stride",
+    I="rows experts top n_out k shared_n_out shared_k tile_rows max_tiles gated dtype kernel")
 HeadLinearArgs = _struct(
     "HeadLinearArgs", "b200_head_linear_args",
     P="x w gate y", L="x_stride x_head_stride y_stride y_head_stride gate_stride", I="rows heads n k dtype")
@@ -93,12 +118,16 @@ def bind_hybrid(lib: ctypes.CDLL) -> None:
     lib.b200_embed_streams.argtypes = [vp] * 5 + [i32] * 5 + [vp]
     for name, struct in (("mixer_finish", MixerFinishArgs), ("stream_step", StreamStepArgs), ("recurrence", RecurrenceArgs),
                          ("latent_prep", LatentPrepArgs), ("head_linear", HeadLinearArgs),
+                         ("residual_step", ResidualStepArgs), ("rope_norm_cache", RopeNormCacheArgs),
+                         ("expert_product", ExpertProductArgs),
                          ("latent_attention", LatentAttnArgs)):
         getattr(lib, "b200_" + name).argtypes = [ctypes.POINTER(struct), vp]
     for name, struct in (("recurrence", RecurrenceArgs), ("latent_attention", LatentAttnArgs)):
         getattr(lib, f"b200_{name}_workspace_bytes").argtypes = [ctypes.POINTER(struct)]
         getattr(lib, f"b200_{name}_workspace_bytes").restype = ctypes.c_size_t
         getattr(lib, f"b200_{name}_num_launches").argtypes = [ctypes.POINTER(struct)]
+    lib.b200_expert_route.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, f32, vp]
+    lib.b200_expert_plan.argtypes = [vp] * 4 + [i32] * 4 + [vp]
     lib.b200_recurrence_chunk.argtypes = [ctypes.POINTER(RecurrenceArgs)]
 
 
@@ -237,8 +266,8 @@ class HybridOps:
             a.h, a.h_stride = h.data_ptr(), h.stride(0)
             a.in_weight, a.norm_weight = _f32("in_weight", reader[0], s), _f32("norm_weight", reader[1], dim)
         if shift is not None:
-            if previous.dtype != dtype or previous.shape[1:] != (dim,) or not previous.is_contiguous():
-                raise ValueError("previous must be contiguous [slots, dim] of the activation type")
+            if previous.dtype != dtype or previous.shape[1:].numel() != dim or not previous.is_contiguous():
+                raise ValueError("previous must be contiguous [slots, (1,) dim] of the activation type")
             if seg.cu_seqlens_q.shape[0] - 1 != t:
                 raise ValueError("the fused token shift takes one row per request")
             shifted = torch.empty_like(h)
@@ -248,6 +277,154 @@ class HybridOps:
         self._check(self._lib.b200_stream_step(ctypes.byref(a), _stream()))
         self.launches += 1
         return h, shifted
+
+    def residual_step(self, x, result=None, in_norm=None, *, eps: float, dtype, rows=None, conv=None, seg=None):
+        """What lies between two sublayers that stand between norms (one launch).  ``result``: what the last one left --
+        ``y [T, dim]`` (or, with ``part_weight [T, parts]``, ``[T * parts, dim]``), optionally ``extra`` with
+        ``extra_gate [T]``, and its ``norm`` -- is added to the fp32 stream ``x [T, dim]``; ``in_norm`` of the next one
+        gives its input, returned.  ``conv`` = (weights [taps, dim], state) with ``seg``: the input plus its convolution, for
+        a batch of single rows.  ``rows`` (int64): only these rows are worked on, the input is packed, ``x`` stays."""
+        _rows("x", x, torch.float32)
+        t, dim = x.shape
+        if not x.is_contiguous():
+            raise ValueError("x must be contiguous")
+        a = ResidualStepArgs()
+        a.x, a.dim, a.eps, a.dtype = x.data_ptr(), dim, float(eps), _DTYPE[dtype]
+        a.rows = t if rows is None else rows.shape[0]
+        if rows is not None:
+            if rows.dtype != torch.int64 or not rows.is_cuda:
+                raise ValueError("rows must be int64 on the device")
+            a.row_ids = rows.data_ptr()
+        if result is not None:
+            y, pw, extra = _rows("y", result["y"], dtype), result.get("part_weight"), result.get("extra")
+            a.parts = 0 if pw is None else pw.shape[1]
+            if y.shape != (t * max(1, a.parts), dim):
+                raise ValueError(f"y is {tuple(y.shape)}, the stream has {t} rows of {dim}")
+            a.y, a.y_stride, a.out_norm = y.data_ptr(), y.stride(0), _f32("norm", result["norm"], dim)
+            if pw is not None:
+                a.part_weight = _f32("part_weight", pw, t * a.parts)
+            if extra is not None:
+                gate = result["extra_gate"]
+                if _rows("extra", extra, dtype).shape != (t, dim) or gate.dtype != torch.float32 or gate.shape != (t,):
+                    raise ValueError("extra must be [T, dim] and its gate float32 [T]")
+                a.extra, a.extra_stride = extra.data_ptr(), extra.stride(0)
+                a.extra_gate, a.gate_stride = gate.data_ptr(), gate.stride(0)
+        h = None
+        if in_norm is not None:
+            h = torch.empty((a.rows, dim), dtype=dtype, device=x.device)
+            a.h, a.h_stride, a.in_norm = h.data_ptr(), h.stride(0), _f32("in_norm", in_norm, dim)
+        if conv is not None:
+            weight, state = conv
+            taps = weight.shape[0]
+            if state.dtype != dtype or tuple(state.shape[1:]) != (taps - 1, dim) or not state.is_contiguous():
+                raise ValueError(f"state must be contiguous [slots, {taps - 1}, {dim}] of the activation type")
+            if seg.cu_seqlens_q.shape[0] - 1 != t:
+                raise ValueError("the fused convolution takes one row per request")
+            a.conv_weight, a.taps = _f32("conv weight", weight, taps * dim), taps
+            a.state = state.data_ptr() if state.numel() else None
+            a.slots, a.seq_lens = seg.state_slots.data_ptr(), seg.seq_lens.data_ptr()
+        self._check(self._lib.b200_residual_step(ctypes.byref(a), _stream()))
+        self.launches += 1
+        return h
+
+    def rope_norm_cache(self, q, k, v, key_cache, value_cache, slot_mapping, positions, freq, factor: float, eps: float,
+                        q_weight=None) -> None:
+        """Heads rotated (interleaved pairs, ``freq [pairs, 2]`` high and low parts, times ``factor``), then divided by
+        their root mean square, queries times ``q_weight [H]``: ``q [T, H, D]`` in place, ``k [T, G, D]`` and
+        ``v [T, G, V]`` into the paged caches."""
+        t, heads, dim = q.shape
+        groups, vdim = v.shape[1:]
+        for name, x in (("q", q), ("k", k), ("v", v)):
+            if not x.is_cuda or x.stride(2) != 1 or x.stride(1) != x.shape[2] or x.dtype != key_cache.dtype or x.shape[0] != t:
+                raise ValueError(f"{name}: [T, heads, size] rows of the cache's type with contiguous heads, got {tuple(x.shape)}")
+        if k.shape[1:] != (groups, dim) or key_cache.shape[2:] != (groups, dim) or value_cache.shape[2:] != (groups, vdim) or \
+                key_cache.shape[:2] != value_cache.shape[:2] or key_cache.stride()[2:] != (dim, 1) or \
+                value_cache.stride()[2:] != (vdim, 1) or value_cache.dtype != key_cache.dtype:
+            raise ValueError("caches must be [num_blocks, block_size, G, D / V] with contiguous rows")
+        if positions.dtype != torch.int32 or slot_mapping.dtype != torch.int64 or positions.shape != (t,) or \
+                slot_mapping.shape != (t,):
+            raise ValueError("positions must be int32 [T] and slot_mapping int64 [T]")
+        a = RopeNormCacheArgs()
+        a.q, a.k, a.v, a.key_cache, a.value_cache = (x.data_ptr() for x in (q, k, v, key_cache, value_cache))
+        a.q_weight = _f32("q_weight", q_weight, heads)
+        a.rot_dims = freq.numel()
+        a.freq = _f32("freq", freq, freq.numel()) if freq.numel() else None
+        a.positions, a.slot_mapping = positions.data_ptr(), slot_mapping.data_ptr()
+        a.q_stride, a.k_stride, a.v_stride = q.stride(0), k.stride(0), v.stride(0)
+        a.k_block_stride, a.k_token_stride = key_cache.stride()[:2]
+        a.v_block_stride, a.v_token_stride = value_cache.stride()[:2]
+        a.num_blocks, a.block_size = key_cache.shape[:2]
+        a.num_tokens, a.heads, a.kv_heads, a.dim, a.vdim = t, heads, groups, dim, vdim
+        a.rot_factor, a.eps, a.dtype = float(factor), float(eps), _DTYPE[q.dtype]
+        self._check(self._lib.b200_rope_norm_cache(ctypes.byref(a), _stream()))
+        self.launches += 1
+
+    def expert_route(self, logits, correction, experts: int, top: int, scale: float):
+        """``(chosen int32 [T, top], weights fp32 [T, top])`` of fp32 router logits (their first ``experts`` columns)."""
+        _rows("logits", logits, torch.float32)
+        t = logits.shape[0]
+        if logits.shape[1] < experts:
+            raise ValueError(f"logits have {logits.shape[1]} columns for {experts} experts")
+        chosen = torch.empty((t, top), dtype=torch.int32, device=logits.device)
+        weights = torch.empty((t, top), dtype=torch.float32, device=logits.device)
+        self._check(self._lib.b200_expert_route(
+            logits.data_ptr(), logits.stride(0), _f32("correction", correction, experts), chosen.data_ptr(),
+            weights.data_ptr(), t, experts, top, float(scale), _stream()))
+        self.launches += 1
+        return chosen, weights
+
+    def expert_plan(self, chosen, experts: int, tile_rows: int):
+        """The (row, place) pairs of ``chosen`` sorted by expert: ``(pairs, first, tiles, tile_rows)``."""
+        if chosen.dtype != torch.int32 or not chosen.is_cuda or not chosen.is_contiguous():
+            raise ValueError("chosen must be contiguous int32 on the device")
+        t, top = chosen.shape
+        buf = torch.empty((t * top + 2 * (experts + 1),), dtype=torch.int32, device=chosen.device)
+        pairs, first, tiles = buf.split([t * top, experts + 1, experts + 1])
+        self._check(self._lib.b200_expert_plan(chosen.data_ptr(), pairs.data_ptr(), first.data_ptr(), tiles.data_ptr(), t,
+                                               experts, top, tile_rows, _stream()))
+        self.launches += 1
+        return pairs, first, tiles, tile_rows
+
+    def expert_product(self, x, weight, plan, top: int, rows: int, *, gated: bool, shared_x=None, shared_weight=None,
+                       k: int = 0, shared_k: int = 0, kernel: int = 0):
+        """Products of all experts: ``weight [E, n, columns]`` of which ``k`` columns count (0: all).  ``gated``: ``x [rows,
+        k]`` through the gate and up halves of ``n``, sorted by expert; else ``x`` sorted, results by pair.  A shared expert's
+        ``shared_weight [n', columns]`` runs along (on ``shared_x``, or on ``x`` when gated).  ``(out, shared out or None)``;
+        results have whole 8-column rows, of which the last may be padding."""
+        pairs, first, tiles, tile_rows = plan
+        experts, n, cols = weight.shape
+        half = 2 if gated else 1
+        _rows("x", x, weight.dtype)
+        if not weight.is_contiguous() or x.shape[0] != (rows if gated else rows * top) or x.shape[1] < (k or cols):
+            raise ValueError(f"expert_product: x {tuple(x.shape)} and weight {tuple(weight.shape)} disagree")
+        up8 = lambda c: -(-c // 8) * 8  # noqa: E731
+        empty = lambda r, c: torch.empty((r, up8(c)), dtype=x.dtype, device=x.device)[:, :c]  # noqa: E731
+        a = ExpertProductArgs()
+        a.x, a.x_stride, a.w, a.w_stride = x.data_ptr(), x.stride(0), weight.data_ptr(), cols
+        a.rows, a.experts, a.top, a.n_out, a.k = rows, experts, top, n // half, k or cols
+        out = empty(rows * top, n // half)
+        a.out, a.out_stride = out.data_ptr(), out.stride(0)
+        shared_out = None
+        if shared_weight is not None:
+            sn, scols = shared_weight.shape
+            sx = x if gated else _rows("shared_x", shared_x, x.dtype)
+            if sx.shape[0] != rows or not shared_weight.is_contiguous() or sx.shape[1] < (shared_k or scols):
+                raise ValueError("expert_product: the shared expert's operands disagree")
+            shared_out = empty(rows, sn // half)
+            a.shared_x, a.shared_x_stride = sx.data_ptr(), sx.stride(0)
+            a.shared_w, a.shared_w_stride = shared_weight.data_ptr(), scols
+            a.shared_out, a.shared_out_stride = shared_out.data_ptr(), shared_out.stride(0)
+            a.shared_n_out, a.shared_k = sn // half, shared_k or scols
+        a.pairs, a.first, a.tiles = pairs.data_ptr(), first.data_ptr(), tiles.data_ptr()
+        a.tile_rows, a.max_tiles = tile_rows, rows * top // tile_rows + min(experts, rows * top)
+        a.gated, a.dtype, a.kernel = int(gated), _DTYPE[x.dtype], kernel
+        self._check(self._lib.b200_expert_product(ctypes.byref(a), _stream()))
+        self.launches += 1
+        return out, shared_out
+
+    def expert_product_failed(self) -> bool:
+        """Whether a wait inside the tcgen05 kernel of the expert products ever ran out (synchronises)."""
+        return self._lib.b200_expert_product_failed() != 0
 
     def causal_conv(self, x, weight, bias, state, seg, silu: bool = True) -> torch.Tensor:
         """Depthwise causal convolution of ``x [T, C]`` over the segments of ``seg`` (carried inputs in
