@@ -665,7 +665,7 @@ def run_b200(args) -> None:
 
 
 def run_design(args, module: str, sizes: str) -> None:
-    """--hybrid / --streams: one JSON line with prefill / decode throughput and every kernel's roofline, per size."""
+    """--hybrid / --streams / --sandwich: one JSON line with prefill / decode throughput and every kernel's roofline, per size."""
     if args.impl == "reference" or args.gpus != 1:
         _emit(json.dumps({"impl": args.impl, "unavailable": "these decoders: one GPU, no reference arm"}))
         return
@@ -712,12 +712,18 @@ def main() -> None:
     ap.add_argument("--streams", action="store_true",
                     help="hyper-connected decoders (lightning attention, softmax attention beside it) and the closest transformer")
     ap.add_argument("--stream-sizes", default="s,m,w", help="sizes of profiles/bench_streams.py")
+    ap.add_argument("--sandwich", action="store_true",
+                    help="sandwich-norm decoders with routed experts and the closest transformer with routed experts")
+    ap.add_argument("--sandwich-sizes", default="s,m,w", help="sizes of profiles/bench_sandwich.py")
     args = ap.parse_args()
     if args.hybrid:
         run_design(args, "bench_hybrid", args.hybrid_sizes)
         return
     if args.streams:
         run_design(args, "bench_streams", args.stream_sizes)
+        return
+    if args.sandwich:
+        run_design(args, "bench_sandwich", args.sandwich_sizes)
         return
     select_config(args.config)
     if args.gpus < CONFIGS[args.config][6] and args.impl == "b200":

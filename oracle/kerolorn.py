@@ -72,6 +72,8 @@ def frequencies(rot):
 def rotate(x, positions, rot):
     """``x`` [T, H, D]: the neighbouring pairs of the first ``dims`` dimensions are turned."""
     y = np.array(x, F)
+    if not rot:
+        return y
     freq, factor = frequencies(rot)
     for i, f in enumerate(freq):
         a = np.asarray(positions, F) * f
@@ -82,18 +84,18 @@ def rotate(x, positions, rot):
 
 
 def visible(i, j, mask):
-    """Whether position ``i`` sees position ``j``."""
-    if j > i:
-        return False
+    """Whether position ``i`` sees position ``j`` (numbers or arrays)."""
     size = (mask or {}).get("size")
-    return not size or i - j < size or j < ((mask or {}).get("keep_first") or 0)
+    if not size:
+        return j <= i
+    return (j <= i) & ((i - j < size) | (j < (mask.get("keep_first") or 0)))
 
 
 def softmax_attention(q, k, v, scale, mask):
     """``q`` [T, H, D], ``k`` [T, G, D], ``v`` [T, G, V], ``scale`` [H]: [T, H, V]."""
     t, heads, _ = q.shape
     per = heads // k.shape[1]
-    seen = np.array([[visible(i, j, mask) for j in range(t)] for i in range(t)])
+    seen = visible(np.arange(t)[:, None], np.arange(t), mask)
     out = np.zeros((t, heads, v.shape[2]), F)
     for h in range(heads):
         s = np.where(seen, q[:, h] @ k[:, h // per].T * scale[h], -np.inf)
@@ -104,9 +106,9 @@ def softmax_attention(q, k, v, scale, mask):
 
 def attention_mixer(h, m, p, eps):
     t, heads, groups, dim, vdim = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    pos = np.arange(t)
-    q = over_rms(rotate(linear(h, p["q"]).reshape(t, heads, dim), pos, m["rot"]), eps)
-    k = over_rms(rotate(linear(h, p["k"]).reshape(t, groups, dim), pos, m["rot"]), eps)
+    pos, rot = np.arange(t), m.get("rot")
+    q = over_rms(rotate(linear(h, p["q"]).reshape(t, heads, dim), pos, rot), eps)
+    k = over_rms(rotate(linear(h, p["k"]).reshape(t, groups, dim), pos, rot), eps)
     v = linear(h, p["v"]).reshape(t, groups, vdim)
     scale = m["scale"] * np.asarray(p["temp"], F)
     return linear(softmax_attention(q, k, v, scale, m.get("mask")).reshape(t, heads * vdim), p["o"])
