@@ -210,7 +210,7 @@ int b200_expert_plan(const int32_t* chosen, int32_t* pairs, int32_t* first, int3
  *   out[pairs[i], n] = w[e, n] . x[i]                                            (w [experts, n_out, k], x in sorted order).
  * A shared expert that every row takes runs in the same launch (shared_w not NULL): its rows are x (gated) or shared_x, its
  * results shared_out [rows, shared_n_out].  Element strides; rows of w and shared_w are w_stride and shared_w_stride apart.
- * kernel: 0 auto, 1 any type and size, 2 tcgen05 (bf16, whole 8-element units).  tile_rows as given to the plan (32, 64 or
+ * kernel: 0 auto, 1 any type and size, 2 tcgen05 (bf16, whole 8-element units; an odd n_out also writes the column after it).  tile_rows as given to the plan (32, 64 or
  * 128); max_tiles bounds tiles[experts]. */
 typedef struct b200_expert_product_args {
   const void* x;
@@ -226,7 +226,8 @@ typedef struct b200_expert_product_args {
   int32_t rows, experts, top, n_out, k, shared_n_out, shared_k, tile_rows, max_tiles, gated, dtype, kernel;
 } b200_expert_product_args;
 int b200_expert_product(const b200_expert_product_args* a, void* stream);
-/* Synchronises.  1 if a bounded wait inside the tcgen05 kernel ever ran out (that launch's results are invalid), else 0. */
+/* Synchronises.  1 if the tcgen05 kernel ever found a plan that does not fit together or a bounded wait inside it ran out (that
+ * launch's results are invalid), else 0. */
 int b200_expert_product_failed(void);
 
 /* Before latent attention, per row: the latent is normed (weight fp32, plain), the shared key part is rotated

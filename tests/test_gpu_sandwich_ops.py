@@ -266,6 +266,22 @@ def test_plan(ops, t, n, top, tile):
         assert sorted(pairs[first[e]:first[e + 1]]) == np.nonzero(chosen.ravel() == e)[0].tolist()
 
 
+def test_the_sort_sees_the_choices_of_the_launch_before_it(ops):
+    """Routing and sorting back to back into memory that still holds other choices, as a step of the model runs them."""
+    rng = np.random.default_rng(0)
+    zs = [f32(rng.standard_normal((200, 48))) for _ in range(6)]
+    stale = [torch.randint(0, 48, (200, 5), dtype=torch.int32, device="cuda") for _ in range(4)]
+    del stale
+    got = []
+    for z in zs * 5:
+        chosen, _ = ops.expert_route(z @ torch.eye(48, device="cuda"), None, 48, 5, 1.0)
+        pairs, first, _, _ = ops.expert_plan(chosen, 48, 32)
+        got.append((chosen.clone(), pairs.clone(), first.clone()))
+    for chosen, pairs, first in got:
+        assert torch.equal(first.diff(), torch.bincount(chosen.flatten(), minlength=48).int())
+        assert torch.equal(chosen.flatten()[pairs.long()], torch.arange(48, device="cuda").repeat_interleave(first.diff()).int())
+
+
 def products(ops, t, width, ff, n, top, shared, dtype, tile, kernel, seed=0):
     """Both products of random experts against one matrix product per pair."""
     rng = np.random.default_rng(seed)

@@ -8,12 +8,15 @@
 namespace b200 {
 namespace {
 
+// No __restrict__ on what an earlier launch writes: it would make the loads read-only ones, which are not held back by
+// the wait for that launch.
+
 // ---- routing: a warp per row ------------------------------------------------------------------------
 constexpr int kRouteWarps = 4;
 
 __global__ void __launch_bounds__(kRouteWarps * 32)
-expert_route_kernel(const float* __restrict__ logits, int64_t stride, const float* __restrict__ correction,
-                    int32_t* __restrict__ chosen, float* __restrict__ weights, int rows, int experts, int top, float scale) {
+expert_route_kernel(const float* logits, int64_t stride, const float* correction, int32_t* chosen, float* weights, int rows,
+                    int experts, int top, float scale) {
   extern __shared__ float sm[];  // per warp: scores [experts], choice scores [experts]
   pdl_trigger();
   pdl_wait();
@@ -48,14 +51,9 @@ expert_route_kernel(const float* __restrict__ logits, int64_t stride, const floa
   }
   look();
   for (int j = 0; j < top; ++j) {
-    float b = best;
-    int i = at;
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, b, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, i, o);
-      if (ob > b || (ob == b && oi < i)) b = ob, i = oi;
-    }
+    const uint32_t bits = __float_as_uint(best), key = bits ^ ((int32_t)bits < 0 ? 0xffffffffu : 0x80000000u);  // same order
+    const uint32_t top_key = __reduce_max_sync(0xffffffffu, key);
+    int i = __reduce_min_sync(0xffffffffu, key == top_key ? at : 0x7fffffff);
     if (i >= experts) i = j % experts;  // scores that compare with nothing (NaN): any expert, in bounds
     if (lane == i % 32) {
       chosen[r * top + j] = i;
@@ -67,11 +65,10 @@ expert_route_kernel(const float* __restrict__ logits, int64_t stride, const floa
 }
 
 // ---- plan: pairs sorted by expert, one CTA ----------------------------------------------------------
-constexpr int kPlanThreads = 1024;
+constexpr int kPlanThreads = 1024, kPlanKeep = 16;
 
 __global__ void __launch_bounds__(kPlanThreads)
-expert_plan_kernel(const int32_t* __restrict__ chosen, int32_t* __restrict__ pairs, int32_t* __restrict__ first,
-                   int32_t* __restrict__ tiles, int total, int experts, int tile_rows) {
+expert_plan_kernel(const int32_t* chosen, int32_t* pairs, int32_t* first, int32_t* tiles, int total, int experts, int tile_rows) {
   extern __shared__ int count[];  // [experts] counts, then next free places
   __shared__ int warp_pairs[32], warp_tiles[32], base_pairs, base_tiles;
   pdl_trigger();
@@ -80,7 +77,18 @@ expert_plan_kernel(const int32_t* __restrict__ chosen, int32_t* __restrict__ pai
   if (tid == 0) base_pairs = base_tiles = 0;
   pdl_wait();
   __syncthreads();
-  for (int p = tid; p < total; p += kPlanThreads) atomicAdd(&count[chosen[p]], 1);
+  auto expert_of = [&](int p) { return min((uint32_t)chosen[p], (uint32_t)experts - 1); };  // in bounds whatever it holds
+  // up to kPlanKeep pairs a thread stay in registers for the second pass
+  int keep[kPlanKeep];
+#pragma unroll
+  for (int j = 0; j < kPlanKeep; ++j) {
+    const int p = tid + j * kPlanThreads;
+    keep[j] = p < total ? (int)expert_of(p) : -1;
+  }
+#pragma unroll
+  for (int j = 0; j < kPlanKeep; ++j)
+    if (keep[j] >= 0) atomicAdd(&count[keep[j]], 1);
+  for (int p = tid + kPlanKeep * kPlanThreads; p < total; p += kPlanThreads) atomicAdd(&count[expert_of(p)], 1);
   __syncthreads();
   for (int e0 = 0; e0 < experts; e0 += kPlanThreads) {  // running sums, kPlanThreads experts at a time
     const int e = e0 + tid, n = e < experts ? count[e] : 0, nt = (n + tile_rows - 1) / tile_rows;
@@ -104,7 +112,10 @@ expert_plan_kernel(const int32_t* __restrict__ chosen, int32_t* __restrict__ pai
   }
   if (tid == 0) first[experts] = base_pairs, tiles[experts] = base_tiles;
   // places inside a stretch are taken as they come: a pair's results do not depend on its place
-  for (int p = tid; p < total; p += kPlanThreads) pairs[atomicAdd(&count[chosen[p]], 1)] = p;
+#pragma unroll
+  for (int j = 0; j < kPlanKeep; ++j)
+    if (keep[j] >= 0) pairs[atomicAdd(&count[keep[j]], 1)] = tid + j * kPlanThreads;
+  for (int p = tid + kPlanKeep * kPlanThreads; p < total; p += kPlanThreads) pairs[atomicAdd(&count[expert_of(p)], 1)] = p;
 }
 
 // ---- products, any type and size ----------------------------------------------------------------------

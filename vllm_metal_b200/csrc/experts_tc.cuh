@@ -8,9 +8,10 @@
 //
 //   warp 0     TMA producer: weight tiles (straight: also the token tile, consecutive rows of the sorted activations)
 //   warp 1     MMA issuer: D_h[128 features x TOKENS] += W_h[128 x 64] X[TOKENS x 64]^T per 64-column step, h = 0, 1
-//   warps 2-5  epilogue, thread = feature; two accumulator pairs, so the next item's products overlap it
+//   warps 2-5  epilogue, thread = feature, stores in pairs; two pairs of accumulators, so the next item's products
+//              overlap it
 //   warps 6-9  (gated) the token tile: rows gathered by pair with 16-byte asynchronous copies into the swizzled layout
-// Rows past a stretch's end hold whatever is there: their columns of the product go nowhere.
+// Products are as wide as the tile has rows, in steps of 16; the columns of rows past a stretch's end go nowhere.
 #pragma once
 
 #include "../../include/b200_hybrid_ops.h"
@@ -21,7 +22,7 @@
 namespace b200 {
 
 // The stretch that holds tile `i`: the last one whose running count is not past it (empty ones are stepped over).
-__device__ __forceinline__ int find_stretch(const int32_t* __restrict__ tiles, int n, int i) {
+__device__ __forceinline__ int find_stretch(const int32_t* tiles, int n, int i) {
   int lo = 0, hi = n;
   while (hi - lo > 1) {
     const int mid = (lo + hi) >> 1;
@@ -37,7 +38,7 @@ constexpr int kSlab = 64;                 // columns of K per stage
 constexpr int kHalfBytes = 128 * 128;     // 128 weight rows x 64 columns
 constexpr int kGatherLag = 3;             // stages of gathered rows in flight
 
-__device__ int g_failed = 0;  // a wait ran out: results of the launch are invalid
+__device__ int g_failed = 0;  // a wait ran out or the plan was not sound: results of the launch are invalid
 
 struct Params {
   const int32_t* pairs;
@@ -47,14 +48,15 @@ struct Params {
   __nv_bfloat16* out;
   __nv_bfloat16* shared_out;
   int64_t x_stride, out_stride, shared_out_stride;
-  int rows, experts, top, n_out, k, shared_n_out, shared_k, shared_tiles;
+  int rows, experts, top, n_out, k, shared_n_out, shared_k, shared_tiles, max_tiles;
 };
 
 template <int TOKENS>
 struct Shape {
   static constexpr int X_BYTES = TOKENS * 128, STAGE_BYTES = 2 * kHalfBytes + X_BYTES;
   static constexpr int STAGES = TOKENS <= 64 ? 5 : 4;
-  static constexpr int TMEM_COLS = 4 * TOKENS;
+  static constexpr int TMEM_COLS = 4 * TOKENS;            // two accumulator pairs
+  static constexpr int BOX = TOKENS < 64 ? TOKENS : 64;   // rows of a token tile per copy
 };
 inline int smem_bytes(int stages, int stage_bytes, int experts) { return stages * stage_bytes + 1024 + 256 + 8 * (experts + 1); }
 
@@ -102,6 +104,14 @@ struct Work {
   }
 };
 
+// Lane l holds columns c0 and c1 of feature l: an even lane gets (l, l + 1) of c0, an odd one (l - 1, l) of c1.
+__device__ __forceinline__ uint32_t swap_pack(uint32_t c0, uint32_t c1) {
+  const bool odd = threadIdx.x & 1;
+  const uint32_t other = __shfl_xor_sync(0xffffffffu, odd ? c0 : c1, 1);
+  const __nv_bfloat162 v = __floats2bfloat162_rn(__uint_as_float(odd ? other : c0), __uint_as_float(odd ? c1 : other));
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
 template <int TOKENS, bool GATED>
 __global__ void __launch_bounds__(GATED ? 320 : 192, 1)
 expert_product_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map,
@@ -137,15 +147,27 @@ expert_product_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
   pdl_wait();
+  // The plan is checked on the way in: running counts that fit together, so that whatever they hold, every row below is
+  // a row of the operands.
+  const int pairs_total = p.rows * p.top;
   for (int i = threadIdx.x; i <= p.experts; i += blockDim.x) {
-    tiles[i] = p.tiles[i];
-    first[i] = p.first[i];
+    const int t = p.tiles[i], f = p.first[i];
+    tiles[i] = t;
+    first[i] = f;
+    const int tn = i < p.experts ? p.tiles[i + 1] : t, fn = i < p.experts ? p.first[i + 1] : pairs_total;
+    if (t < 0 || f < 0 || t > p.max_tiles || f > pairs_total || (i < p.experts && (fn < f || tn - t != (fn - f + TOKENS - 1) / TOKENS)))
+      *sfail = 1;
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_gen;
-  const Work<TOKENS, GATED> work(p, tiles);
+  const bool sound = *sfail == 0;
+  __syncthreads();
+  Work<TOKENS, GATED> work(p, tiles);
+  if (!sound) work.total = 0;
+
+  auto pair_at = [&](int i) { return (int)min((uint32_t)p.pairs[i], (uint32_t)pairs_total - 1); };
 
   if (warp == 0) {
     // ===== TMA producer =====
@@ -163,14 +185,18 @@ expert_product_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid
         const uint32_t dst = base + st * SH::STAGE_BYTES, bar = bar_full + 8 * st;
         if (!(ok = mbar_wait_or_fail(bar_empty + 8 * st, ((n / STAGES) & 1) ^ 1))) break;
         if (elect_one()) {
-          mbar_expect_tx(bar, (both ? 2 : 1) * kHalfBytes + (GATED ? 0 : SH::X_BYTES));
+          const int boxes = GATED ? 0 : (w.nrows + SH::BOX - 1) / SH::BOX;
+          mbar_expect_tx(bar, (both ? 2 : 1) * kHalfBytes + boxes * SH::BOX * 128);
           tma_load_2d(dst, wm, bar, s * kSlab, r0);
           if (both) tma_load_2d(dst + kHalfBytes, wm, bar, s * kSlab, r1);
-          if (!GATED) tma_load_2d(dst + 2 * kHalfBytes, xm, bar, s * kSlab, w.row0);
+          for (int j = 0; j < boxes; ++j)
+            tma_load_2d(dst + 2 * kHalfBytes + j * SH::BOX * 128, xm, bar, s * kSlab, w.row0 + j * SH::BOX);
         }
         __syncwarp();
       }
     }
+    // the last products' arrivals find the CTA still there
+    for (int s = max(0, n - STAGES); ok && s < n; ++s) ok = mbar_wait_or_fail(bar_empty + 8 * (s % STAGES), (s / STAGES) & 1);
     if (!ok) {
       if (lane == 0) *sfail = 1;
       // the copies in flight land before the CTA's memory goes away
@@ -178,7 +204,6 @@ expert_product_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid
     }
   } else if (warp == 1) {
     // ===== MMA issuer =====
-    const uint32_t idesc = make_idesc(1, 128, TOKENS);
     const uint32_t tb = __shfl_sync(0xffffffffu, tmem, 0);
     int n = 0, it = 0;
     bool ok = true;
@@ -186,6 +211,7 @@ expert_product_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid
       const Item w = work.at(p, tiles, first, i);
       const int slabs = (w.k + kSlab - 1) / kSlab, b = it & 1;
       const bool both = GATED || w.feature + 128 < w.n_out;
+      const uint32_t idesc = make_idesc(1, 128, (w.nrows + 15) & ~15);
       if (!(ok = mbar_wait_or_fail(bar_free + 8 * b, ((it >> 1) & 1) ^ 1))) break;
       const uint32_t d0 = tb + b * 2 * TOKENS, d1 = d0 + TOKENS;
       for (int s = 0; s < slabs; ++s, ++n) {
@@ -219,27 +245,34 @@ expert_product_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid
       if (!(ok = mbar_wait_or_fail(bar_acc + 8 * b, (it >> 1) & 1))) break;
       tc_fence_after();
       const uint32_t d0 = tmem + lane_addr + b * 2 * TOKENS, d1 = d0 + TOKENS;
-      const int feature = w.feature + q * 32 + lane;
-      __nv_bfloat16* out = w.shared ? p.shared_out : p.out;
+      const int feature = w.feature + q * 32 + (lane & ~1);  // of the pair a lane stores
+      __nv_bfloat16* out = (w.shared ? p.shared_out : p.out) + feature;
       const int64_t ost = w.shared ? p.shared_out_stride : p.out_stride;
-      const bool live0 = feature < w.n_out, live1 = !GATED && feature + 128 < w.n_out;
-      const bool both = GATED || w.feature + 128 < w.n_out;
+      const bool live0 = feature < w.n_out, live1 = !GATED && feature + 128 < w.n_out, both = GATED || w.feature + 128 < w.n_out;
       for (int c0 = 0; c0 < w.nrows; c0 += 16) {
         uint32_t u[16], v[16];
         tmem_ld<16>(d0 + c0, u);
         if (both) tmem_ld<16>(d1 + c0, v);
+        const int mine = w.row0 + min(c0 + (lane & 15), w.nrows - 1);
+        const int place = GATED || w.shared ? mine : pair_at(mine);
+        if (GATED) {
 #pragma unroll
-        for (int c = 0; c < 16; ++c) {
-          if (c0 + c >= w.nrows) break;
-          const int row = w.row0 + c0 + c;
-          if (GATED) {
+          for (int c = 0; c < 16; ++c) {
             const float z = __uint_as_float(u[c]);
-            const float y = z * __fdividef(1.f, 1.f + __expf(-z)) * __uint_as_float(v[c]);
-            if (live0) out[row * ost + feature] = __float2bfloat16_rn(y);
-          } else {
-            __nv_bfloat16* o = out + (w.shared ? row : p.pairs[row]) * ost + feature;
-            if (live0) o[0] = __float2bfloat16_rn(__uint_as_float(u[c]));
-            if (live1) o[128] = __float2bfloat16_rn(__uint_as_float(v[c]));
+            u[c] = __float_as_uint(z * __fdividef(1.f, 1.f + __expf(-z)) * __uint_as_float(v[c]));
+          }
+        }
+        // neighbouring lanes swap a column each: one 4-byte store of two features a lane for two columns
+#pragma unroll
+        for (int c = 0; c < 16; c += 2) {
+          const int col = c + (lane & 1), row = __shfl_sync(0xffffffffu, place, col);
+          const bool live = c0 + col < w.nrows;
+          __nv_bfloat16* o = out + row * ost;
+          const uint32_t x = swap_pack(u[c], u[c + 1]);
+          if (live && live0) *reinterpret_cast<uint32_t*>(o) = x;
+          if (!GATED && both) {
+            const uint32_t y = swap_pack(v[c], v[c + 1]);
+            if (live && live1) *reinterpret_cast<uint32_t*>(o + 128) = y;
           }
         }
       }
@@ -267,7 +300,7 @@ expert_product_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid
 #pragma unroll
       for (int m = 0; m < PER; ++m) {
         const int r = r_first + 16 * m, row = w.row0 + min(r, w.nrows - 1);
-        src[m] = p.x + (int64_t)(w.shared ? row : p.pairs[row] / p.top) * p.x_stride + c * 8;
+        src[m] = p.x + (int64_t)(w.shared ? row : pair_at(row) / p.top) * p.x_stride + c * 8;
       }
       for (int s = 0; s < slabs; ++s) {
         const int st = n % STAGES;
@@ -305,7 +338,7 @@ expert_product_tc_kernel(const __grid_constant__ CUtensorMap w_map, const __grid
 inline bool supported(const b200_expert_product_args& a) {
   auto ok = [](const void* p, int64_t stride) { return !p || (((uintptr_t)p & 15) == 0 && stride % 8 == 0 && stride < (1ll << 36)); };
   return a.dtype == B200_BF16 && (a.tile_rows == 32 || a.tile_rows == 64 || a.tile_rows == 128) && a.k % 8 == 0 &&
-         ok(a.x, a.x_stride) && ok(a.w, a.w_stride) &&
+         ok(a.x, a.x_stride) && ok(a.w, a.w_stride) && ok(a.out, a.out_stride) && ok(a.shared_out, a.shared_out_stride) &&
          (!a.shared_w || (a.shared_k % 8 == 0 && ok(a.shared_w, a.shared_w_stride) && ok(a.shared_x, a.shared_x_stride))) &&
          (int64_t)a.experts * a.n_out * 2 < (1ll << 31) && encode_fn() != nullptr;
 }
@@ -327,11 +360,11 @@ int launch_form(const b200_expert_product_args& a, cudaStream_t st) {
   CUtensorMap w, x, sw, sx;
   const int64_t w_rows = (int64_t)a.experts * a.n_out * (GATED ? 2 : 1);
   int rc = make_map_2d(&w, bf, a.w, a.k, w_rows, a.w_stride * 2, kSlab, 128, promo);
-  if (rc == B200_OK && !GATED) rc = make_map_2d(&x, bf, a.x, a.k, (uint64_t)a.rows * a.top, a.x_stride * 2, kSlab, TOKENS, promo);
+  if (rc == B200_OK && !GATED) rc = make_map_2d(&x, bf, a.x, a.k, (uint64_t)a.rows * a.top, a.x_stride * 2, kSlab, SH::BOX, promo);
   if (rc == B200_OK && a.shared_w) rc = make_map_2d(&sw, bf, a.shared_w, a.shared_k, (uint64_t)a.shared_n_out * (GATED ? 2 : 1),
                                                     a.shared_w_stride * 2, kSlab, 128, promo);
   if (rc == B200_OK && a.shared_w && !GATED)
-    rc = make_map_2d(&sx, bf, a.shared_x, a.shared_k, a.rows, a.shared_x_stride * 2, kSlab, TOKENS, promo);
+    rc = make_map_2d(&sx, bf, a.shared_x, a.shared_k, a.rows, a.shared_x_stride * 2, kSlab, SH::BOX, promo);
   if (rc != B200_OK) return rc;
   if (GATED) x = sx = w;  // not read
   if (!a.shared_w) sw = w, sx = x;
@@ -352,6 +385,7 @@ int launch_form(const b200_expert_product_args& a, cudaStream_t st) {
   p.k = a.k;
   p.shared_n_out = a.shared_n_out;
   p.shared_k = a.shared_k;
+  p.max_tiles = a.max_tiles;
   p.shared_tiles = a.shared_w ? (a.rows + TOKENS - 1) / TOKENS : 0;
   constexpr int FEATURES = GATED ? 128 : 256;
   const int64_t items = (int64_t)a.max_tiles * ((a.n_out + FEATURES - 1) / FEATURES) +

@@ -43,7 +43,7 @@ class RoutedExperts:
         way_out[:, :ff].copy_(get(name + "down", (self.width, ff)))
 
     def tile_rows(self, rows: int) -> int:
-        """Pairs per tile: few experts should need a second pass over their weights, prompts should fill the tensor cores."""
+        """Pairs per tile: few experts should need a second pass over their weights."""
         if self.any_size:
             return EXPERT_TILES[0]
         per_expert = rows * self.r.top / self.r.experts
