@@ -11,7 +11,7 @@ static int log2_exact_i(int v) {
 
 // The forms that were there for keys and values of one size; everything else (and 16-bit-wide weights) is bf16 only.
 static bool plain_form(const b200_paged_attn_args& a) {
-  return (a.head_dim == 64 || a.head_dim == 128) && value_dim(a) == a.head_dim && !a.wide_weights;
+  return (a.head_dim == 64 || a.head_dim == 128) && value_dim(a) == a.head_dim && !a.wide_weights && keep_first(a) == 0;
 }
 
 bool decode_mma_supported(const b200_paged_attn_args& a) {
@@ -23,7 +23,8 @@ bool decode_mma_supported(const b200_paged_attn_args& a) {
     if (a.dtype != B200_BF16 && !same) return false;
     if (dk % 8 || dv % 8 || dk > 256 || dv > 256 || (a.window_seqlen_q > 1 && !same)) return false;
   }
-  if (a.window_seqlen_q > 1 && keep_first(a) > 0) return false;  // window batches know one visible stretch a row
+  // kept first positions: bf16, one row a CTA (window batches know one visible stretch a row)
+  if (keep_first(a) > 0 && (a.dtype != B200_BF16 || a.window_seqlen_q > 1)) return false;
   const int G = a.num_q_heads / a.num_kv_heads;
   if (G < 1 || G > 16) return false;
   if (log2_exact_i(a.block_size) < 0) return false;
@@ -105,6 +106,7 @@ int launch_decode_mma(const b200_paged_attn_args& a, const SplitWorkspace* ws, c
     p.win_subs = (a.window_seqlen_q + p.win_rows - 1) / p.win_rows;
     grid.y = (unsigned)(a.num_seqs * p.win_subs);
   }
+  if (p.keep_first > 0) return p.group <= 8 ? launch_decode_kept_packed(p, grid, st) : launch_decode_kept(p, grid, st);
   if (wide_form(a)) return p.group <= 8 ? launch_decode_wide_packed(p, grid, st) : launch_decode_wide(p, grid, st);
   if (a.dtype == B200_BF16) {
     if (a.head_dim == 128) return launch_one<__nv_bfloat16, 128, 3>(p, grid, st);

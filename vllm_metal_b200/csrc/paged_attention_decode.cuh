@@ -25,7 +25,7 @@
 // time against a V fragment zeroed outside that row's range, so a non-finite V at a position only later rows may see
 // cannot reach earlier rows through 0 * inf (test_windowed_skips_masked_inf_v).
 //
-// Kept first positions (per-row mode): the tiles that hold them precede the window's, see RowInfo.
+// KEEP: first positions kept beside a window (WIDE, per-row mode); the tiles that hold them precede the window's, see RowInfo.
 //
 // DK / DV: compile-time widths of the products over keys and values.  WIDE forms take any size up to that, the columns past
 // it zero-filled (a run-time width, whose every step is a branch, ran 1.6 times slower).  WIDE: the softmax weights enter P.V
@@ -142,7 +142,7 @@ constexpr int decode_wide_stages(int dk, int dv) {
   return fit < 2 ? 2 : fit > 4 ? 4 : fit;
 }
 
-template <typename T, int DK, int DV, int STAGES, bool WIN, bool WIDE, bool PACK>
+template <typename T, int DK, int DV, int STAGES, bool WIN, bool WIDE, bool PACK, bool KEEP>
 __global__ void __launch_bounds__(kDecodeWarps * 32, decode_ctas_per_sm(DK, DV))
 paged_decode_mma_kernel(const DecodeParams p) {
   pdl_trigger();
@@ -154,6 +154,7 @@ paged_decode_mma_kernel(const DecodeParams p) {
   static_assert(STAGES * STAGE_BYTES >= 16 * DV * 4, "merge buffer must fit in the ring");
   const int dk = WIDE ? p.head_dim : DK, dv = WIDE ? p.value_dim : DV;
   static_assert(WIDE || DK == DV, "keys and values of different sizes take the wide forms");
+  static_assert(!KEEP || (WIDE && !WIN), "kept first positions come with the wide, per-row forms");
 
   extern __shared__ __align__(128) uint8_t smem_raw[];
   __shared__ float sm_m[kDecodeWarps][16];
@@ -205,10 +206,9 @@ paged_decode_mma_kernel(const DecodeParams p) {
     hi = max(end, beg);
     return 2;
   };
-  const bool kept = !WIN && p.keep_first > 0;  // two stretches: the range below counts tokens without the gap between them
   // union of the rows' ranges (what is streamed) and their intersection (where no row masks anything)
   int beg, end, ulo = 0, uhi = 0x7fffffff;
-  if (kept) {
+  if constexpr (KEEP) {  // two stretches: the range counts tokens without the gap between them
     beg = p.partitioned ? part * p.ws.partition_size : 0;
     end = ri.span();
     if (beg >= end) return;
@@ -278,7 +278,7 @@ paged_decode_mma_kernel(const DecodeParams p) {
   auto issue_tile = [&](int j, int stage) {
     if (j < n_tiles) {
       const int at = (first_tile + j) * kTileTokens + (lane & 15);
-      const int tok = kept ? ri.token_at(at) : at;
+      const int tok = KEEP ? ri.token_at(at) : at;
       int page = tok >> p.block_shift;
       page = min(page, p.max_blocks_per_seq - 1);
       int64_t blk = table[page];
@@ -286,7 +286,7 @@ paged_decode_mma_kernel(const DecodeParams p) {
       uint32_t koff = (uint32_t)blk * p.block_stride16 + (uint32_t)(tok & block_mask) * p.token_stride16;
       uint32_t voff = (uint32_t)blk * p.v_block_stride16 + (uint32_t)(tok & block_mask) * p.v_token_stride16;
       // zero-fill rows outside the range
-      if (at < beg || at >= end || (kept && tok < ri.beg && tok >= p.keep_first)) koff = voff = 0xFFFFFFFFu;
+      if (at < beg || at >= end || (KEEP && tok < ri.beg && tok >= p.keep_first)) koff = voff = 0xFFFFFFFFu;
       const uint32_t sbase = warp_smem + stage * STAGE_BYTES;
       if constexpr (!WIDE) {  // one layout for both: one row lookup serves K and V
         constexpr int CHUNKS = DK / 8;       // 16-byte chunks per row
@@ -361,7 +361,7 @@ paged_decode_mma_kernel(const DecodeParams p) {
     }
     // ---- scale, softcap, log2 domain, range mask -------------------------------
     const int tok0 = (first_tile + j) * kTileTokens + 2 * tq;
-    const int moved = kept && first_tile + j >= ri.kept ? ri.gap : 0;
+    const int moved = KEEP && first_tile + j >= ri.kept ? ri.gap : 0;
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt) {
 #pragma unroll
@@ -370,7 +370,7 @@ paged_decode_mma_kernel(const DecodeParams p) {
         if (p.softcap > 0.f) v = tanhf(v / p.softcap) * p.softcap * kLog2e;  // :1120-1122,1138
         const int tok = tok0 + nt * 8 + (e & 1);
         bool in = e < 2 ? (tok >= lo0 && tok < hi0) : (tok >= lo1 && tok < hi1);
-        if (kept) in = in && (tok + moved >= ri.beg || tok + moved < p.keep_first);
+        if (KEEP) in = in && (tok + moved >= ri.beg || tok + moved < p.keep_first);
         sacc[nt][e] = in ? v : -INFINITY;
       }
     }
@@ -554,18 +554,18 @@ paged_decode_mma_kernel(const DecodeParams p) {
   }
 }
 
-template <typename T, int DK, int DV, int STAGES, bool WIN, bool WIDE, bool PACK = false>
+template <typename T, int DK, int DV, int STAGES, bool WIN, bool WIDE, bool PACK = false, bool KEEP = false>
 int launch_decode_form(const DecodeParams& p, dim3 grid, cudaStream_t st) {
   constexpr int smem = kDecodeWarps * STAGES * decode_tile_bytes(DK, DV);
   static bool configured_dev[16] = {false};  // cudaFuncSetAttribute is per device
   int dev = 0;
   B200_CUDA_OK(cudaGetDevice(&dev));
   if (!configured_dev[dev & 15]) {
-    B200_CUDA_OK(cudaFuncSetAttribute(paged_decode_mma_kernel<T, DK, DV, STAGES, WIN, WIDE, PACK>,
+    B200_CUDA_OK(cudaFuncSetAttribute(paged_decode_mma_kernel<T, DK, DV, STAGES, WIN, WIDE, PACK, KEEP>,
                                       cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     configured_dev[dev & 15] = true;
   }
-  launch_pdl(paged_decode_mma_kernel<T, DK, DV, STAGES, WIN, WIDE, PACK>, grid, dim3(kDecodeWarps * 32), smem, st, p);
+  launch_pdl(paged_decode_mma_kernel<T, DK, DV, STAGES, WIN, WIDE, PACK, KEEP>, grid, dim3(kDecodeWarps * 32), smem, st, p);
   return check_launch("paged_decode_mma_kernel");
 }
 
@@ -574,5 +574,7 @@ constexpr int decode_key_width(int d) { return d <= 64 ? 64 : d <= 96 ? 96 : d <
 constexpr int decode_value_width(int d) { return d <= 64 ? 64 : d <= 128 ? 128 : d <= 192 ? 192 : 256; }
 int launch_decode_wide(const DecodeParams& p, dim3 grid, cudaStream_t st);         // any group
 int launch_decode_wide_packed(const DecodeParams& p, dim3 grid, cudaStream_t st);  // at most 8 heads a group
+int launch_decode_kept(const DecodeParams& p, dim3 grid, cudaStream_t st);         // the same with kept first positions
+int launch_decode_kept_packed(const DecodeParams& p, dim3 grid, cudaStream_t st);
 
 }  // namespace b200

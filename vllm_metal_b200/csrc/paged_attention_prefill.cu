@@ -108,7 +108,8 @@ __device__ __forceinline__ float tanh_approx(float x) {
 // inline the unrolled softmax body measured several times slower (instruction-fetch bound).
 // WIDE keeps two bf16 terms of every softmax weight: the high terms take the first half of S's columns as usual, the low
 // terms the second half, and the value product runs over both.
-template <int DK, int DV, bool SOFTCAP, bool WIDE, int KV>
+// KEEP: first positions kept beside a window; a flag of its own because the walk over two stretches costs the others 3 to 10%.
+template <int DK, int DV, bool SOFTCAP, bool WIDE, int KV, bool KEEP>
 __global__ void __launch_bounds__(THREADS, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                   const __grid_constant__ CUtensorMap v_map, const Params p) {
@@ -145,9 +146,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
   const int kv_lo = p.sliding_window >= 0 ? max(0, qabs0 + 1 - p.sliding_window) : 0;
   const int j0 = kv_lo / BK, j1 = (kv_hi - 1) / BK;   // KV blocks j0..j1
   // kept first positions: the blocks that hold them and precede the window's come first
-  const int kept = min((p.keep_first + BK - 1) / BK, j0);
+  const int kept = KEEP ? min((p.keep_first + BK - 1) / BK, j0) : 0;
   const int nblk = j1 - j0 + 1 + kept;
-  auto block_at = [&](int it) { return it < kept ? it : j0 + it - kept; };
+  auto block_at = [&](int it) { return KEEP && it < kept ? it : j0 + it - kept; };
 
   extern __shared__ __align__(1024) uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -316,7 +317,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       // this row sees KV positions [row_lo, row_hi); rows past the tile's valid rows see nothing
       const int row_hi = r < nrows ? min(seq_len, qabs + 1) : 0;
       const int row_lo = p.sliding_window >= 0 ? max(0, qabs + 1 - p.sliding_window) : 0;
-      const int row_keep = min(p.keep_first, row_hi);
+      const int row_keep = KEEP ? min(p.keep_first, row_hi) : 0;
       const float sc = p.scale * kLog2e;
       const float cap_in = SOFTCAP ? p.scale / p.softcap : 0.f, cap_out = SOFTCAP ? p.softcap * kLog2e : 0.f;  // tanh(s*scale/c)*c
       const float inv_sc = SOFTCAP ? 1.f / sc : 0.f;
@@ -351,7 +352,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
           for (int c = 0; c < BK; ++c) {
             float x = SOFTCAP ? tanh_approx(s[c] * cap_in) * cap_out * inv_sc : s[c];  // back in raw-score units
             const int kv = kv0 + c;
-            x = (kv >= row_lo && kv < row_hi) || kv < row_keep ? x : -INFINITY;
+            x = (kv >= row_lo && kv < row_hi) || (KEEP && kv < row_keep) ? x : -INFINITY;
             s[c] = x;
             m_raw = fmaxf(m_raw, x);
           }
@@ -491,10 +492,10 @@ static int make_map_rows(CUtensorMap* map, CUtensorMapDataType dt, const void* p
   return B200_OK;
 }
 
-template <int DK, int DV, bool SOFTCAP, bool WIDE, int KV = 128>
+template <int DK, int DV, bool SOFTCAP, bool WIDE, int KV = 128, bool KEEP = false>
 static int launch(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) {
   using SM = Smem<DK, DV, KV>;
-  auto kern = prefill_tc_kernel<DK, DV, SOFTCAP, WIDE, KV>;
+  auto kern = prefill_tc_kernel<DK, DV, SOFTCAP, WIDE, KV, KEEP>;
   static int configured_dev[16] = {0};
   int dev = 0;
   B200_CUDA_OK(cudaGetDevice(&dev));
@@ -563,6 +564,7 @@ bool prefill_tc_supported(const b200_paged_attn_args& a) {
   const int dk = a.head_dim, dv = value_dim(a);
   if (dk % 8 || dv % 8 || dk > 128 || dv > 512) return false;
   // softcap and fp16 stay with the sizes they were written for
+  if (keep_first(a) > 0 && (a.softcap > 0.f || a.dtype == B200_F16)) return false;
   if ((a.softcap > 0.f || a.dtype == B200_F16) && (dk != dv || (dk != 64 && dk != 128))) return false;
   if (a.block_size < 8 || a.block_size > 128 || (128 % a.block_size) != 0) return false;
   // the TMA maps view each cache as one [num_blocks * block_size tokens, H_kv, D] tensor (rows may be wider)
@@ -576,19 +578,29 @@ bool prefill_tc_supported(const b200_paged_attn_args& a) {
   return tc::encode_fn() != nullptr;
 }
 
-int launch_prefill_tc(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) {
+namespace pf {
+// Two terms of every weight, by the sizes that hold keys and values.
+template <bool KEEP>
+static int launch_wide(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) {
   const int dv = value_dim(a);
   const bool k64 = a.head_dim <= 64, v64 = dv <= 64;
+  if (dv > 128 && dv <= 192 && a.block_size <= 64)
+    return k64 ? launch<64, 192, false, true, 64, KEEP>(a, min_qlen, st) : launch<128, 192, false, true, 64, KEEP>(a, min_qlen, st);
+  if (k64)
+    return v64 ? launch<64, 64, false, true, 128, KEEP>(a, min_qlen, st) : launch<64, 128, false, true, 128, KEEP>(a, min_qlen, st);
+  return v64 ? launch<128, 64, false, true, 128, KEEP>(a, min_qlen, st) : launch<128, 128, false, true, 128, KEEP>(a, min_qlen, st);
+}
+}  // namespace pf
+
+int launch_prefill_tc(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) {
+  const int dv = value_dim(a);
+  const bool k64 = a.head_dim <= 64;
   if (a.softcap > 0.f)
     return k64 ? pf::launch<64, 64, true, false>(a, min_qlen, st) : pf::launch<128, 128, true, false>(a, min_qlen, st);
-  // keys and values of different or odd sizes always keep wide weights
+  // keys and values of different or odd sizes and kept first positions always take wide weights
   const bool same = a.head_dim == dv && (dv == 64 || dv == 128);
-  if (a.dtype == B200_BF16 && (a.wide_weights || !same)) {
-    if (dv > 128 && dv <= 192 && a.block_size <= 64)
-      return k64 ? pf::launch<64, 192, false, true, 64>(a, min_qlen, st) : pf::launch<128, 192, false, true, 64>(a, min_qlen, st);
-    if (k64) return v64 ? pf::launch<64, 64, false, true>(a, min_qlen, st) : pf::launch<64, 128, false, true>(a, min_qlen, st);
-    return v64 ? pf::launch<128, 64, false, true>(a, min_qlen, st) : pf::launch<128, 128, false, true>(a, min_qlen, st);
-  }
+  if (keep_first(a) > 0) return pf::launch_wide<true>(a, min_qlen, st);
+  if (a.dtype == B200_BF16 && (a.wide_weights || !same)) return pf::launch_wide<false>(a, min_qlen, st);
   return k64 ? pf::launch<64, 64, false, false>(a, min_qlen, st) : pf::launch<128, 128, false, false>(a, min_qlen, st);
 }
 

@@ -24,14 +24,13 @@ LIB_NAME = "lib_b200_paged_ops.so"
 
 # Parts of the library that stand on their own: a model family that needs no more than such a part can be built and
 # served without compiling the rest (a first call in a fresh checkout).
+_COMMON = ("c_abi", "decoder_ops", "hybrid_ops", "paged_attention_decode", "paged_attention_decode_kept",
+           "paged_attention_decode_kept_packed", "paged_attention_decode_packed", "paged_attention_decode_wide",
+           "paged_attention_generic", "paged_attention_prefill")
 COMPONENTS: dict[str, tuple[str, ...]] = {
-    "hybrid": ("c_abi", "decoder_ops", "hybrid_ops", "latent_attention", "latent_ops", "paged_attention_decode",
-               "paged_attention_decode_packed", "paged_attention_decode_wide", "paged_attention_generic", "paged_attention_prefill", "recurrence"),
-    "streams": ("c_abi", "decoder_ops", "hybrid_ops", "paged_attention_decode", "paged_attention_decode_packed",
-                "paged_attention_decode_wide", "paged_attention_generic", "paged_attention_prefill", "recurrence", "rope_cache", "stream_ops"),
-    "sandwich": ("c_abi", "decoder_ops", "experts", "hybrid_ops", "paged_attention_decode", "paged_attention_decode_packed",
-                 "paged_attention_decode_wide", "paged_attention_generic", "paged_attention_prefill", "residual_step",
-                 "rope_cache"),
+    "hybrid": (*_COMMON, "latent_attention", "latent_ops", "recurrence"),
+    "streams": (*_COMMON, "recurrence", "rope_cache", "stream_ops"),
+    "sandwich": (*_COMMON, "experts", "residual_step", "rope_cache"),
 }
 _wanted: list[str] = []  # the component this process asked for last
 
