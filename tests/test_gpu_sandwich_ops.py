@@ -181,8 +181,8 @@ class Paged:
         return np.stack(out)
 
 
-MASKS = [(40, 7), (16, 0), (17, 1), (1, 3), (5, 64), (128, 16), (129, 131), (64, 5), (33, 400), (300, 12), (-1, 9)]
-SIZES = [(6, 2, 24, 40), (8, 1, 64, 64), (4, 2, 128, 128), (2, 2, 5, 9), (18, 1, 32, 16), (12, 1, 80, 176)]
+MASKS = [(41, 7), (16, 0), (17, 1), (1, 3), (5, 64), (128, 16), (129, 131), (64, 5), (33, 400), (300, 12), (-1, 9)]
+SIZES = [(6, 2, 24, 40), (10, 1, 64, 64), (4, 2, 128, 128), (2, 2, 5, 9), (18, 1, 32, 16), (12, 1, 80, 176)]
 
 
 @BOTH
@@ -200,7 +200,7 @@ def test_window_with_kept_tokens_in_prompts_portions_and_decoding(ops, heads, gr
 @pytest.mark.parametrize("block_size", [8, 32, 64])
 def test_other_pages(ops, block_size, dtype):
     p = Paged(4, 2, 64, 64, [300, 65], dtype, block_size)
-    for mask in ((40, 7), (70, 33)):
+    for mask in ((41, 7), (70, 33)):
         for counts in ([300, 65], [1, 1], [70, 3]):
             p.run(ops, counts, [300, 65], 0.2, mask)
 
@@ -219,7 +219,7 @@ def test_split_keys(ops, mask, dtype):
 
 
 @BOTH
-@pytest.mark.parametrize("heads,groups,dim,vdim", [(6, 2, 24, 40), (8, 1, 64, 64), (2, 2, 5, 9)])
+@pytest.mark.parametrize("heads,groups,dim,vdim", [(6, 2, 24, 40), (10, 1, 64, 64), (2, 2, 5, 9)])
 def test_one_outstanding_key_just_inside_and_outside_every_edge(ops, heads, groups, dim, vdim, dtype):
     """The key every query asks for lies first or last of what is visible, or one past it, and at pages' edges."""
     for (size, keep), n, at in [((30, 6), 150, at) for at in (0, 5, 6, 15, 16, 119, 120, 121, 127, 128, 148, 149)] + \
