@@ -30,10 +30,11 @@ int b200_stream_norm(const float* x, const int64_t* row_ids, const float* weight
 
 /* The element-wise end of a layer's two parallel halves, one launch:
  *   out[r, 0:inner)              = post(gate) * weight * group_norm(y * pre(z))
- *     pre(z) = silu(z) if pre_gate, post(g) = sigmoid(g) if post_gate; group_norm divides each of inner / group_size
+ *     pre(z) = silu(z) if pre_gate, post(g) = sigmoid(g), or silu(g) with post_silu = 1, if post_gate; group_norm divides each of inner / group_size
  *     parts by its own root mean square (group_size = 0: no norm); weight fp32 or NULL.
  *   out[r, act_offset + i]       = act(act_in[r, i]) (* act_mul[r, i] if given), i in [0, act_dim);
- *     act_kind 0: gelu (erf form), 1: silu.  act_in may be the output columns themselves.
+ *     act_kind 0: gelu (erf form), 1: silu, 2: tanh, 3: xIELU, act_a z^2 + z / 2 for z > 0, else act_b (exp(z) - 1 - z) + z / 2.
+ *     act_in may be the output columns themselves.
  *   out[r, i] = 0 for the remaining columns below out_cols (alignment padding of the next product's operand).
  * Any of the two halves may be absent (act_dim = 0; y = NULL: the columns below inner are somebody else's). */
 typedef struct b200_mixer_finish_args {
@@ -51,6 +52,8 @@ typedef struct b200_mixer_finish_args {
   const void* act_mul;
   int64_t mul_stride;
   int32_t act_kind;
+  int32_t post_silu;
+  float act_a, act_b;
 } b200_mixer_finish_args;
 int b200_mixer_finish(const b200_mixer_finish_args* a, void* stream);
 
@@ -71,6 +74,9 @@ int b200_causal_conv(const void* in, const float* weight, const float* bias, voi
  *       out = S^T q' / (max(|n . q'|, exp(-m')) + 1e-6), q' = q_scale q.
  *   kind 2 (lightning attention): S <- decay[h] S + k v^T;  out = S^T q';  no gates (gate_a, bias_a NULL);
  *       rate[h] = -log(decay[h]), finite, is what the chunked forms use.
+ *   kind 3 (RWKV-style): out = (S + diag(u) k v^T)^T q;  then S <- diag(w) S + k v^T  with
+ *       w = exp(-exp(gate_a + bias_a)) per head and key channel; gate_a fp32 [rows, heads * key_dim] whatever dtype, bias_a
+ *       and u = skip [heads * key_dim]; no groups, q_scale is not applied.
  * silu = 1: q, k and v are taken through silu as they are read (token-by-token form only; for the chunked forms the
  * caller does it beforehand).
  * state [slots, heads, key_dim, value_dim]; mLSTM also norm_state [slots, heads, vtiles, key_dim] and max_state
@@ -162,10 +168,14 @@ typedef struct b200_stream_step_args {
 #define B200_MAX_STREAMS 16
 int b200_stream_step(const b200_stream_step_args* a, void* stream);
 
-/* What lies between two sublayers that stand between norms of their own, one launch, fp32 stream x [rows, dim]:
- *   r = y, or with parts > 0 sum_j part_weight[row, j] y[row * parts + j] (+ sigmoid(extra_gate[row]) extra[row]);
- *   x += r / rms(r) * out_norm        (y NULL: x is read only)
- *   h = x / rms(x) * in_norm          (h NULL: nothing follows)
+/* What lies between two sublayers, one launch, fp32 stream x [rows, dim]:
+ *   r = y, or with parts > 0 sum_j part_weight[row, j] y[row * parts + j] (+ sigmoid(extra_gate[row]) extra[row]) (+ bias);
+ *   x += r / rms(r) * out_norm, without out_norm x += r        (y NULL: no result)
+ *   x += table_scale * table[ids[row]], if table (fresh = 1: x starts as that and is not read);  x += add, if add
+ *   h = x / rms(x) * in_norm, each of `groups` parts of a row by its own rms (0: one part; h and h32 NULL: nothing follows);
+ *       h32: as it is in fp32, h: of dtype
+ *   mixes > 0 (batches of one row a request): instead h[s, row, :] = h + (h' - h) * mix_weight[s, :] with h' = mix_state[slots[row],
+ *       dim], zeros for a request's first token, which takes h (all fp32; h [mixes, rows, dim] with mix_stride)
  *   h += conv(h) with taps weights [taps, dim] if conv_weight: the earlier inputs come from state[slots[row], taps - 1, dim]
  *   (oldest first; zeros for a request's first tokens, seq_lens[row] counts this one), which takes h in; for batches of
  *   one row a request.
@@ -189,15 +199,34 @@ typedef struct b200_residual_step_args {
   int32_t rows, dim, parts, taps;
   float eps;
   int32_t dtype;
+  const float* bias;
+  const void* table;
+  const int32_t* ids;
+  const float* add;
+  float* h32;
+  const float* mix_weight;
+  float* mix_state;
+  int64_t mix_stride;
+  float table_scale;
+  int32_t vocab, fresh, groups, mixes;
 } b200_residual_step_args;
 int b200_residual_step(const b200_residual_step_args* a, void* stream);
+
+/* Rows mixed with the row before, for batches with portions: out[s, t, :] = h[t] + (h' - h[t]) * weight[s, :] for s < mixes,
+ * h' = the row before of the same segment, for its first row state[slot, dim] (zeros for a sequence's first token); the slot takes
+ * the segment's last row.  h, weight [mixes, dim] and state fp32; out [mixes, rows, dim] (mix_stride, out_stride) of dtype. */
+#define B200_MAX_MIXES 8
+int b200_token_mix(const float* h, const float* weight, float* state, const int32_t* cu_seqlens, const int32_t* seq_lens,
+                   const int32_t* slots, void* out, int num_seqs, int max_q_len, int dim, int mixes, int64_t h_stride,
+                   int64_t out_stride, int64_t mix_stride, int dtype, void* stream);
 
 #define B200_MAX_EXPERTS 1024
 /* Routed experts.  b200_expert_route, per row: s = softmax(logits[row, 0:experts]); the `top` experts with the largest
  * s + correction (fp32, NULL: 0; ties to the lower number), best first, go to chosen [rows, top] and their s * scale to
- * weights [rows, top]. */
+ * weights [rows, top].  over_chosen = 1: the correction is part of the logits, the largest of them are chosen, and the weights are
+ * the softmax over the chosen ones alone, times scale. */
 int b200_expert_route(const float* logits, int64_t logits_stride, const float* correction, int32_t* chosen, float* weights,
-                      int rows, int experts, int top, float scale, void* stream);
+                      int rows, int experts, int top, float scale, int over_chosen, void* stream);
 
 /* The (row, place) pairs p = row * top + place sorted by expert: pairs [rows * top], first [experts + 1] the start of each
  * expert's stretch, tiles [experts + 1] the running count of the stretches' tiles of tile_rows pairs. */
@@ -256,7 +285,9 @@ int b200_latent_prep(const b200_latent_prep_args* a, void* stream);
 /* Before attention with rotated, then normed heads, per row: the interleaved pairs (2i, 2i + 1) of the first rot_dims
  * dimensions of every query and key head are turned by positions[t] * f_i and scaled by rot_factor, with f_i = freq[2i] +
  * freq[2i + 1] as a high and a low part; the head is divided by its root mean square; a query head also takes
- * q_weight[h] (fp32, NULL: 1).  Queries are updated in place, keys and values go to cache row slot_mapping[t] (negative or out of
+ * q_weight[h] (fp32, NULL: 1).  With q_norm / k_norm (fp32 [dim]) queries / keys are multiplied by them, with norm_values a
+ * value head is divided by its root mean square, and with temp_coef a query is multiplied by
+ * 1 + temp_coef ln(floor((positions[t] + 1) / temp_every) + 1).  Queries are updated in place, keys and values go to cache row slot_mapping[t] (negative or out of
  * range: padding, nothing is cached). */
 typedef struct b200_rope_norm_cache_args {
   void* q;
@@ -273,6 +304,10 @@ typedef struct b200_rope_norm_cache_args {
   int32_t num_tokens, heads, kv_heads, dim, vdim, rot_dims, block_size;
   float rot_factor, eps;
   int32_t dtype;
+  const float* q_norm;
+  const float* k_norm;
+  float temp_coef, temp_every;
+  int32_t norm_values;
 } b200_rope_norm_cache_args;
 int b200_rope_norm_cache(const b200_rope_norm_cache_args* a, void* stream);
 

@@ -25,7 +25,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 6
+#define B200_ABI_VERSION 7
 
 /* Element types of activations / caches (reference: dtype_to_metal,
  * paged_ops.cpp:185-196 -- float, half, bfloat16 are the supported set). */
@@ -176,6 +176,8 @@ typedef struct b200_paged_attn_args {
   int32_t min_q_len;     /* rows of the shortest sequence of the batch if the caller knows it, else 0: where all of them are
                           * the tile kernel's, the per-row kernels are not launched */
   int32_t keep_first;    /* with a window: positions below this stay visible to every later row */
+  const float* slopes;   /* [num_q_heads] or NULL: slopes[h] * (i - j) is taken off the score of position i for position j (not
+                          * together with softcap) */
 } b200_paged_attn_args;
 
 size_t b200_paged_attention_workspace_bytes(const b200_paged_attn_args* args);

@@ -169,7 +169,7 @@ def test_library_exports_every_declared_symbol():
     assert declared == set(EXPORTED_SYMBOLS)
     for name in sorted(declared):
         assert hasattr(lib, name), f"{name} declared in include/*.h but not exported"
-    assert lib.b200_abi_version() == 6  # args.out_dtype .. args.keep_first
+    assert lib.b200_abi_version() == 7  # args.out_dtype .. args.slopes
     assert lib.b200_partition_size() == 512
 
 

@@ -10,7 +10,7 @@ from collections.abc import Sequence
 import torch
 
 from ...lm.hybrid_config import (HybridArgs, LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs,
-                                SideBySideArgs, cached_heads)
+                                SideBySideArgs, TimeMixArgs, cached_heads)
 from .state_cache import RecurrentState
 
 
@@ -45,6 +45,8 @@ class HybridCache:
             elif isinstance(m, (LightningArgs, SideBySideArgs)):
                 r = m.right if isinstance(m, SideBySideArgs) else m
                 self.states[i] = RecurrentState.allocate(num_slots, r.heads, r.dim, r.vdim, self.device)
+            elif isinstance(m, TimeMixArgs):
+                self.states[i] = RecurrentState.allocate(num_slots, m.heads, m.dim, m.dim, self.device, last=args.width)
             a = cached_heads(m)
             if a is not None:
                 self.kv[i] = tuple(torch.zeros((num_blocks, block_size, a.kv_heads, d), dtype=dtype, device=self.device)

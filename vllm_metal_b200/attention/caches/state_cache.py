@@ -1,7 +1,7 @@
 """Per-request state of recurrent layers: fixed-size slots in HBM plus the allocator that hands them out.
 
 A slot holds everything a request carries from step to step in every recurrent layer (32-bit matrix states, the
-normaliser and running maximum of mLSTM, the last inputs of a short convolution).  Nothing is cleared when a slot
+normaliser and running maximum of mLSTM, the last inputs of a short convolution, the last input of time mixing).  Nothing is cleared when a slot
 changes hands: the kernels take a segment that starts at position 0 as having a zero state.  Slot 0 is the padding
 slot (graph warm-up and padded rows write there), like block 0 of the paged pools.
 """
@@ -52,19 +52,22 @@ class RecurrentState:
     normaliser: torch.Tensor | None = None  # fp32 [slots, heads, value tiles, key_dim]
     maximum: torch.Tensor | None = None     # fp32 [slots, heads, value tiles]
     conv: torch.Tensor | None = None        # [slots, taps - 1, channels], the activation type
+    last: torch.Tensor | None = None        # fp32 [slots, width]
 
     @classmethod
     def allocate(cls, num_slots: int, heads: int, key_dim: int, value_dim: int, device, *, normalised: bool = False,
-                 conv_taps: int = 0, conv_channels: int = 0, dtype: torch.dtype = torch.bfloat16) -> RecurrentState:
+                 conv_taps: int = 0, conv_channels: int = 0, dtype: torch.dtype = torch.bfloat16,
+                 last: int = 0) -> RecurrentState:
         n = num_slots + 1
         f32 = dict(dtype=torch.float32, device=device)
         tiles = -(-value_dim // RECURRENCE_TILE_V)
         return cls(torch.zeros((n, heads, key_dim, value_dim), **f32),
                    torch.zeros((n, heads, tiles, key_dim), **f32) if normalised else None,
                    torch.zeros((n, heads, tiles), **f32) if normalised else None,
-                   torch.zeros((n, conv_taps - 1, conv_channels), dtype=dtype, device=device) if conv_taps else None)
+                   torch.zeros((n, conv_taps - 1, conv_channels), dtype=dtype, device=device) if conv_taps else None,
+                   torch.zeros((n, last), **f32) if last else None)
 
     @property
     def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in (self.matrix, self.normaliser, self.maximum, self.conv)
+        return sum(t.numel() * t.element_size() for t in (self.matrix, self.normaliser, self.maximum, self.conv, self.last)
                    if t is not None)

@@ -16,7 +16,7 @@ constexpr int kRouteWarps = 4;
 
 __global__ void __launch_bounds__(kRouteWarps * 32)
 expert_route_kernel(const float* logits, int64_t stride, const float* correction, int32_t* chosen, float* weights, int rows,
-                    int experts, int top, float scale) {
+                    int experts, int top, float scale, int over_chosen) {
   extern __shared__ float sm[];  // per warp: scores [experts], choice scores [experts]
   pdl_trigger();
   pdl_wait();
@@ -28,6 +28,7 @@ expert_route_kernel(const float* logits, int64_t stride, const float* correction
   float m = -INFINITY;
   for (int e = lane; e < experts; e += 32) {
     s[e] = logits[r * stride + e];
+    if (over_chosen) c[e] = s[e] = s[e] + (correction ? correction[e] : 0.f);
     m = fmaxf(m, s[e]);
   }
   m = warp_max(m);
@@ -36,7 +37,7 @@ expert_route_kernel(const float* logits, int64_t stride, const float* correction
     s[e] = expf(s[e] - m);
     sum += s[e];
   }
-  const float inv = 1.f / warp_sum(sum);
+  const float inv = over_chosen ? 1.f : 1.f / warp_sum(sum);
   float best = -INFINITY;  // this lane's best remaining one; it alone looks at its experts again
   int at = 0x7fffffff;
   auto look = [&] {
@@ -47,9 +48,10 @@ expert_route_kernel(const float* logits, int64_t stride, const float* correction
   };
   for (int e = lane; e < experts; e += 32) {
     s[e] *= inv;
-    c[e] = s[e] + (correction ? correction[e] : 0.f);
+    if (!over_chosen) c[e] = s[e] + (correction ? correction[e] : 0.f);
   }
   look();
+  float taken = 0.f;  // on the lane of each choice
   for (int j = 0; j < top; ++j) {
     const uint32_t bits = __float_as_uint(best), key = bits ^ ((int32_t)bits < 0 ? 0xffffffffu : 0x80000000u);  // same order
     const uint32_t top_key = __reduce_max_sync(0xffffffffu, key);
@@ -58,9 +60,15 @@ expert_route_kernel(const float* logits, int64_t stride, const float* correction
     if (lane == i % 32) {
       chosen[r * top + j] = i;
       weights[r * top + j] = s[i] * scale;
+      taken += s[i];
       c[i] = -INFINITY;
       look();
     }
+  }
+  if (over_chosen) {
+    const float f = 1.f / warp_sum(taken);
+    __syncwarp();
+    for (int j = lane; j < top; j += 32) weights[r * top + j] *= f;
   }
 }
 
@@ -213,14 +221,14 @@ using namespace b200;
 extern "C" {
 
 int b200_expert_route(const float* logits, int64_t logits_stride, const float* correction, int32_t* chosen, float* weights,
-                      int rows, int experts, int top, float scale, void* stream) {
+                      int rows, int experts, int top, float scale, int over_chosen, void* stream) {
   B200_CHECK_ARG(logits && chosen && weights, "expert_route: null pointer argument");
   B200_CHECK_ARG(experts >= 1 && experts <= B200_MAX_EXPERTS && top >= 1 && top <= experts,
                  "expert_route: %d of %d experts (at most %d)", top, experts, B200_MAX_EXPERTS);
   if (rows <= 0) return B200_OK;
   B200_CUDA_OK(launch_pdl(expert_route_kernel, dim3((rows + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32),
                           (size_t)kRouteWarps * 2 * experts * sizeof(float), (cudaStream_t)stream, logits, logits_stride,
-                          correction, chosen, weights, rows, experts, top, scale));
+                          correction, chosen, weights, rows, experts, top, scale, over_chosen));
   return check_launch("expert_route");
 }
 

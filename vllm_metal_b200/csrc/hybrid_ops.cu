@@ -10,7 +10,10 @@ namespace {
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ float gelu_erf_f(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
-constexpr int kActGelu = 0, kActSilu = 1;
+constexpr int kActGelu = 0, kActSilu = 1, kActTanh = 2, kActXielu = 3;
+__device__ __forceinline__ float xielu_f(float z, float a, float b) {
+  return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
+}
 
 template <int THREADS>
 __device__ __forceinline__ float block_sum(float v, float* red) {
@@ -132,7 +135,10 @@ mixer_finish_kernel(const b200_mixer_finish_args a, int norm_blocks) {
     auto put = [&](int c, float v) {
       v *= inv;
       if (a.weight) v *= a.weight[c];
-      if (post) v *= sigmoid_f(to_float(post[c]));
+      if (post) {
+        const float z = to_float(post[c]), g = sigmoid_f(z);
+        v *= a.post_silu ? z * g : g;
+      }
       o[c] = from_float<T>(v);
     };
 #pragma unroll
@@ -150,7 +156,10 @@ mixer_finish_kernel(const b200_mixer_finish_args a, int norm_blocks) {
       const int i = base + j * 256 + threadIdx.x;
       if (i >= a.act_dim) continue;
       const float z = to_float(in[i]);
-      const float v = a.act_kind == kActSilu ? z * sigmoid_f(z) : gelu_erf_f(z);
+      const float v = a.act_kind == kActSilu   ? z * sigmoid_f(z)
+                      : a.act_kind == kActGelu ? gelu_erf_f(z)
+                      : a.act_kind == kActTanh ? tanhf(z)
+                                               : xielu_f(z, a.act_a, a.act_b);
       o[a.act_offset + i] = from_float<T>(mul ? v * to_float(mul[i]) : v);
     }
   }
@@ -240,7 +249,10 @@ mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks) {
       for (int e = 0; e < 8; ++e) {
         float x = v[j][e] * inv;
         if (a.weight) x *= w[e];
-        if (post) x *= fast_sigmoid(to_float(vg[j].e[e]));
+        if (post) {
+          const float z = to_float(vg[j].e[e]), g = fast_sigmoid(z);
+          x *= a.post_silu ? z * g : g;
+        }
         res.e[e] = from_float<T>(x);
       }
       *reinterpret_cast<Vec8<T>*>(o + c) = res;
@@ -263,7 +275,10 @@ mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         const float z = to_float(x[j].e[e]);
-        float v = a.act_kind == kActSilu ? z * fast_sigmoid(z) : gelu_erf_f(z);
+        float v = a.act_kind == kActSilu   ? z * fast_sigmoid(z)
+                  : a.act_kind == kActGelu ? gelu_erf_f(z)
+                  : a.act_kind == kActTanh ? tanhf(z)
+                                           : xielu_f(z, a.act_a, a.act_b);
         if (mul) v *= to_float(m[j].e[e]);
         x[j].e[e] = from_float<T>(v);
       }
@@ -495,7 +510,7 @@ int b200_stream_norm(const float* x, const int64_t* row_ids, const float* weight
 int b200_mixer_finish(const b200_mixer_finish_args* a, void* stream) {
   B200_CHECK_ARG(a && a->out, "mixer_finish: no output");
   B200_CHECK_ARG(a->act_dim == 0 || a->act_in, "mixer_finish: no activation input");
-  B200_CHECK_ARG(a->act_kind == kActGelu || a->act_kind == kActSilu, "mixer_finish: unknown activation %d", a->act_kind);
+  B200_CHECK_ARG(a->act_kind >= kActGelu && a->act_kind <= kActXielu, "mixer_finish: unknown activation %d", a->act_kind);
   B200_CHECK_ARG(a->group_size >= 0 && (a->group_size == 0 || a->inner % a->group_size == 0),
                  "mixer_finish: inner %d is not a multiple of the group size %d", a->inner, a->group_size);
   B200_CHECK_ARG(a->out_cols >= a->inner && (a->act_dim == 0 || (a->act_offset >= a->inner &&

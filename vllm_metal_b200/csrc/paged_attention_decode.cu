@@ -11,7 +11,8 @@ static int log2_exact_i(int v) {
 
 // The forms that were there for keys and values of one size; everything else (and 16-bit-wide weights) is bf16 only.
 static bool plain_form(const b200_paged_attn_args& a) {
-  return (a.head_dim == 64 || a.head_dim == 128) && value_dim(a) == a.head_dim && !a.wide_weights && keep_first(a) == 0;
+  return (a.head_dim == 64 || a.head_dim == 128) && value_dim(a) == a.head_dim && !a.wide_weights && keep_first(a) == 0 &&
+         !a.slopes;
 }
 
 bool decode_mma_supported(const b200_paged_attn_args& a) {
@@ -25,6 +26,7 @@ bool decode_mma_supported(const b200_paged_attn_args& a) {
   }
   // kept first positions: bf16, one row a CTA (window batches know one visible stretch a row)
   if (keep_first(a) > 0 && (a.dtype != B200_BF16 || a.window_seqlen_q > 1)) return false;
+  if (a.slopes && (a.dtype != B200_BF16 || a.window_seqlen_q > 1)) return false;  // the same for a distance bias
   const int G = a.num_q_heads / a.num_kv_heads;
   if (G < 1 || G > 16) return false;
   if (log2_exact_i(a.block_size) < 0) return false;
@@ -71,6 +73,7 @@ int launch_decode_mma(const b200_paged_attn_args& a, const SplitWorkspace* ws, c
   p.seq_lens = a.seq_lens;
   p.cu_seqlens_q = a.cu_seqlens_q;
   p.sinks = a.sinks;
+  p.slopes = a.slopes;
   p.num_seqs = a.num_seqs;
   p.num_q_heads = a.num_q_heads;
   p.num_kv_heads = a.num_kv_heads;

@@ -117,6 +117,7 @@ struct DecodeParams {
   const int32_t* seq_lens;
   const int32_t* cu_seqlens_q;
   const float* sinks;
+  const float* slopes;  // distance bias: wide, per-row forms only
   int num_seqs, num_q_heads, num_kv_heads, group;
   int block_shift, max_blocks_per_seq, sliding_window, keep_first;
   int64_t q_stride, out_stride;
@@ -325,6 +326,11 @@ paged_decode_mma_kernel(const DecodeParams p) {
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
 
+  float slope0 = 0.f, slope1 = 0.f;  // log2 units a token
+  if (WIDE && !WIN && p.slopes != nullptr) {
+    if (rv0) slope0 = p.slopes[kvh * G + hl0] * kLog2e;
+    if (rv1) slope1 = p.slopes[kvh * G + hl1] * kLog2e;
+  }
   const float sc_mul = p.softcap > 0.f ? p.scale : p.scale * kLog2e;
 
   // tiles are dealt to warps by absolute index (tile & 3 == warp), so a row's tile -> warp map does not depend on
@@ -369,6 +375,7 @@ paged_decode_mma_kernel(const DecodeParams p) {
         float v = sacc[nt][e] * sc_mul;
         if (p.softcap > 0.f) v = tanhf(v / p.softcap) * p.softcap * kLog2e;  // :1120-1122,1138
         const int tok = tok0 + nt * 8 + (e & 1);
+        if (WIDE && !WIN) v = fmaf(e < 2 ? slope0 : slope1, (float)(tok + moved - (eff0 - 1)), v);
         bool in = e < 2 ? (tok >= lo0 && tok < hi0) : (tok >= lo1 && tok < hi1);
         if (KEEP) in = in && (tok + moved >= ri.beg || tok + moved < p.keep_first);
         sacc[nt][e] = in ? v : -INFINITY;

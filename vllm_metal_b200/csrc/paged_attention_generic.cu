@@ -22,7 +22,7 @@ paged_attention_generic_kernel(T* __restrict__ out, const T* __restrict__ query,
                                const int32_t* __restrict__ block_tables,
                                const int32_t* __restrict__ seq_lens,
                                const int32_t* __restrict__ cu_seqlens_q,
-                               const float* __restrict__ sinks, int num_seqs, int num_q_heads,
+                               const float* __restrict__ sinks, const float* __restrict__ slopes, int num_seqs, int num_q_heads,
                                int num_kv_heads, int head_dim, int v_dim, int block_shift,
                                int max_blocks_per_seq, int sliding_window, int keep_first, int64_t q_stride,
                                int64_t out_stride, int64_t kv_block_stride,
@@ -59,6 +59,7 @@ paged_attention_generic_kernel(T* __restrict__ out, const T* __restrict__ query,
     q[i] = d < head_dim ? to_float(qp[d]) * scale : 0.f;
   }
 
+  const float slope = slopes != nullptr ? slopes[h] : 0.f;
   float m = -INFINITY, l = 0.f;
   float o[kMaxEpl];
 #pragma unroll
@@ -81,6 +82,7 @@ paged_attention_generic_kernel(T* __restrict__ out, const T* __restrict__ query,
     }
     dot = warp_sum(dot);
     if (softcap > 0.f) dot = tanhf(dot / softcap) * softcap;  // :1120-1122
+    if (slopes != nullptr) dot = fmaf(-slope, (float)(eff - 1 - tok), dot);
     const float sc = dot * kLog2e;                            // :1138
     const float m_new = fmaxf(m, sc);
     const float corr = exp2f(m - m_new);  // m = -inf first time -> 0
@@ -214,7 +216,7 @@ int launch_generic(const b200_paged_attn_args& a, const SplitWorkspace* ws, cuda
   return B200_DISPATCH_DTYPE(a.dtype, T, [&]() -> int {
     launch_pdl(paged_attention_generic_kernel<T>, dim3(grid), dim3(kGenericWarps * 32), smem, st, 
         (T*)a.out, (const T*)a.query, (const T*)a.key_cache, (const T*)a.value_cache,
-        a.block_tables, a.seq_lens, a.cu_seqlens_q, a.sinks, a.num_seqs, a.num_q_heads,
+        a.block_tables, a.seq_lens, a.cu_seqlens_q, a.sinks, a.slopes, a.num_seqs, a.num_q_heads,
         a.num_kv_heads, a.head_dim, value_dim(a), shift, a.max_blocks_per_seq, a.sliding_window, keep_first(a), a.q_stride,
         a.out_stride, a.kv_block_stride, a.kv_token_stride, a.kv_head_stride, value_strides(a), a.num_blocks,
         a.scale, a.softcap, w, ws != nullptr);
@@ -258,6 +260,7 @@ static int validate(const b200_paged_attn_args* a) {
                  "paged_attention: unsupported dtype code %d", a->dtype);
   B200_CHECK_ARG(a->num_blocks > 0, "paged_attention: num_blocks must be > 0");
   B200_CHECK_ARG(a->keep_first >= 0, "paged_attention: keep_first must not be negative, got %d", a->keep_first);
+  B200_CHECK_ARG(!a->slopes || a->softcap <= 0.f, "paged_attention: a distance bias beside a softcap is not supported");
   B200_CHECK_ARG(a->window_seqlen_q >= 0, "paged_attention: window_seqlen_q must be >= 1 (1 = per-token decode), got %d",
                  a->window_seqlen_q);
   B200_CHECK_ARG(a->out_dtype == 0 || a->out_dtype == a->dtype || (a->out_dtype == B200_F16 && a->dtype == B200_BF16),

@@ -45,6 +45,7 @@ struct Params {
   const int32_t* seq_lens;
   const int32_t* cu;
   const float* sinks;
+  const float* slopes;
   int num_seqs, num_q_tokens, num_kv_heads, group;
   int block_size, pages_per_tile, max_blocks_per_seq, sliding_window, keep_first, min_qlen;
   int64_t out_stride;
@@ -109,7 +110,8 @@ __device__ __forceinline__ float tanh_approx(float x) {
 // WIDE keeps two bf16 terms of every softmax weight: the high terms take the first half of S's columns as usual, the low
 // terms the second half, and the value product runs over both.
 // KEEP: first positions kept beside a window; a flag of its own because the walk over two stretches costs the others 3 to 10%.
-template <int DK, int DV, bool SOFTCAP, bool WIDE, int KV, bool KEEP>
+// BIAS: slopes[h] * distance comes off the scores, which go through the softmax in log2 units then.
+template <int DK, int DV, bool SOFTCAP, bool WIDE, int KV, bool KEEP, bool BIAS>
 __global__ void __launch_bounds__(THREADS, 1)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
                   const __grid_constant__ CUtensorMap v_map, const Params p) {
@@ -321,6 +323,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
       const float sc = p.scale * kLog2e;
       const float cap_in = SOFTCAP ? p.scale / p.softcap : 0.f, cap_out = SOFTCAP ? p.softcap * kLog2e : 0.f;  // tanh(s*scale/c)*c
       const float inv_sc = SOFTCAP ? 1.f / sc : 0.f;
+      const float slope = BIAS ? p.slopes[h] * kLog2e : 0.f, unit = BIAS ? 1.f : sc;
+      (void)slope;
       (void)cap_in; (void)cap_out; (void)inv_sc;
       const uint32_t t_sp = tmem_base + lane_addr + TM_SP + ti * BK, t_o = tmem_base + lane_addr + TM_O + ti * DV;
       float m_used = -INFINITY, m_true = -INFINITY, l = 0.f;
@@ -340,6 +344,16 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
             for (int q = 0; q < 32; ++q) s[g * 32 + q] = __uint_as_float(v[g][q]);
         }
         const int kv0 = block_at(it) * BK;
+        if (BIAS) {
+          const float2 sc2 = make_float2(sc, sc), slope2 = make_float2(slope, slope);
+          const float at = (float)(kv0 - qabs);  // of the block's first position, seen from this row
+#pragma unroll
+          for (int c = 0; c < BK; c += 2) {
+            const float2 d2 = __fadd2_rn(make_float2(at, at), make_float2((float)c, (float)(c + 1)));
+            const float2 x2 = __ffma2_rn(make_float2(s[c], s[c + 1]), sc2, __fmul2_rn(d2, slope2));
+            s[c] = x2.x, s[c + 1] = x2.y;
+          }
+        }
         // The softmax threads are instruction-issue bound (a polynomial ex2 on the FMA pipe made the kernel 20% SLOWER),
         // so the row is touched as little as possible: the max is taken over the RAW scores (scale > 0 commutes with
         // max), the scale and the max subtraction are one packed fma per column pair, the row sum one packed add.
@@ -360,12 +374,12 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_consta
 #pragma unroll
           for (int c = 0; c < BK; ++c) m_raw = fmaxf(m_raw, s[c]);
         }
-        const float m_blk = m_raw * sc;  // log2 domain (-inf stays -inf: sc > 0)
+        const float m_blk = m_raw * unit;  // log2 domain (-inf stays -inf: unit > 0)
         m_true = fmaxf(m_true, m_blk);
         const float m_new = (m_blk > m_used + kRescaleThreshold) ? m_blk : m_used;
         const float alpha = (m_used == -INFINITY) ? 0.f : ex2(m_used - m_new);
         const float m_eff = (m_new == -INFINITY) ? 0.f : m_new;
-        const float2 sc2 = make_float2(sc, sc), nm2 = make_float2(-m_eff, -m_eff);
+        const float2 sc2 = make_float2(unit, unit), nm2 = make_float2(-m_eff, -m_eff);
         float2 sum2 = make_float2(0.f, 0.f);
         uint32_t pk[WIDE ? 1 : BK / 2];
         if (WIDE) {
@@ -492,10 +506,10 @@ static int make_map_rows(CUtensorMap* map, CUtensorMapDataType dt, const void* p
   return B200_OK;
 }
 
-template <int DK, int DV, bool SOFTCAP, bool WIDE, int KV = 128, bool KEEP = false>
+template <int DK, int DV, bool SOFTCAP, bool WIDE, int KV = 128, bool KEEP = false, bool BIAS = false>
 static int launch(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) {
   using SM = Smem<DK, DV, KV>;
-  auto kern = prefill_tc_kernel<DK, DV, SOFTCAP, WIDE, KV, KEEP>;
+  auto kern = prefill_tc_kernel<DK, DV, SOFTCAP, WIDE, KV, KEEP, BIAS>;
   static int configured_dev[16] = {0};
   int dev = 0;
   B200_CUDA_OK(cudaGetDevice(&dev));
@@ -520,6 +534,7 @@ static int launch(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) 
   p.seq_lens = a.seq_lens;
   p.cu = a.cu_seqlens_q;
   p.sinks = a.sinks;
+  p.slopes = a.slopes;
   p.num_seqs = a.num_seqs;
   p.num_q_tokens = a.num_q_tokens;
   p.num_kv_heads = a.num_kv_heads;
@@ -565,6 +580,7 @@ bool prefill_tc_supported(const b200_paged_attn_args& a) {
   if (dk % 8 || dv % 8 || dk > 128 || dv > 512) return false;
   // softcap and fp16 stay with the sizes they were written for
   if (keep_first(a) > 0 && (a.softcap > 0.f || a.dtype == B200_F16)) return false;
+  if (a.slopes && (a.dtype == B200_F16 || keep_first(a) > 0)) return false;
   if ((a.softcap > 0.f || a.dtype == B200_F16) && (dk != dv || (dk != 64 && dk != 128))) return false;
   if (a.block_size < 8 || a.block_size > 128 || (128 % a.block_size) != 0) return false;
   // the TMA maps view each cache as one [num_blocks * block_size tokens, H_kv, D] tensor (rows may be wider)
@@ -580,15 +596,15 @@ bool prefill_tc_supported(const b200_paged_attn_args& a) {
 
 namespace pf {
 // Two terms of every weight, by the sizes that hold keys and values.
-template <bool KEEP>
+template <bool KEEP, bool BIAS = false>
 static int launch_wide(const b200_paged_attn_args& a, int min_qlen, cudaStream_t st) {
   const int dv = value_dim(a);
   const bool k64 = a.head_dim <= 64, v64 = dv <= 64;
   if (dv > 128 && dv <= 192 && a.block_size <= 64)
-    return k64 ? launch<64, 192, false, true, 64, KEEP>(a, min_qlen, st) : launch<128, 192, false, true, 64, KEEP>(a, min_qlen, st);
+    return k64 ? launch<64, 192, false, true, 64, KEEP, BIAS>(a, min_qlen, st) : launch<128, 192, false, true, 64, KEEP, BIAS>(a, min_qlen, st);
   if (k64)
-    return v64 ? launch<64, 64, false, true, 128, KEEP>(a, min_qlen, st) : launch<64, 128, false, true, 128, KEEP>(a, min_qlen, st);
-  return v64 ? launch<128, 64, false, true, 128, KEEP>(a, min_qlen, st) : launch<128, 128, false, true, 128, KEEP>(a, min_qlen, st);
+    return v64 ? launch<64, 64, false, true, 128, KEEP, BIAS>(a, min_qlen, st) : launch<64, 128, false, true, 128, KEEP, BIAS>(a, min_qlen, st);
+  return v64 ? launch<128, 64, false, true, 128, KEEP, BIAS>(a, min_qlen, st) : launch<128, 128, false, true, 128, KEEP, BIAS>(a, min_qlen, st);
 }
 }  // namespace pf
 
@@ -600,6 +616,7 @@ int launch_prefill_tc(const b200_paged_attn_args& a, int min_qlen, cudaStream_t 
   // keys and values of different or odd sizes and kept first positions always take wide weights
   const bool same = a.head_dim == dv && (dv == 64 || dv == 128);
   if (keep_first(a) > 0) return pf::launch_wide<true>(a, min_qlen, st);
+  if (a.slopes) return pf::launch_wide<false, true>(a, min_qlen, st);
   if (a.dtype == B200_BF16 && (a.wide_weights || !same)) return pf::launch_wide<false>(a, min_qlen, st);
   return k64 ? pf::launch<64, 64, false, false>(a, min_qlen, st) : pf::launch<128, 128, false, false>(a, min_qlen, st);
 }

@@ -1,12 +1,15 @@
 // Gated linear recurrences over per-request state slots (include/b200_hybrid_ops.h): Mamba-2, mLSTM and lightning attention share
 //   S <- decay S + weight k v^T,   out = S^T q
-// and differ in how decay / weight come from the gates (lightning attention has none) and in mLSTM's normaliser.
+// and differ in how decay / weight come from the gates (lightning attention has none) and in mLSTM's normaliser.  RWKV-style
+// time mixing has a decay per key channel and reads the state before the row's own part, which enters with a weight of its own.
 //
 //  * sequential form: one CTA per (64-wide value tile, head, segment); the fp32 state is streamed once per token
 //    (decode: HBM-bound at 2 * key_dim * value_dim * 4 bytes per head), any type and any size.
 //  * chunked forms (bf16 operands), all chunks in parallel: recurrence_tc.cuh (tcgen05, 128 rows) where the key size is
-//    whole 64-wide slices, else recurrence_chunk.cuh (warp-level tensor cores, 64 rows).
+//    whole 64-wide slices, else recurrence_chunk.cuh (warp-level tensor cores, 64 rows); decays per key channel:
+//    recurrence_wkv.cuh.
 #include "recurrence_tc.cuh"
+#include "recurrence_wkv.cuh"
 
 namespace b200 {
 namespace rec {
@@ -34,6 +37,8 @@ sequential_kernel(const b200_recurrence_args a) {
   float* sk = sq + K;                       // [K]
   float* sred = sk + K;                     // [RP][64]
   float* sdot = sred + RP * kTileV;         // [8]
+  float* sdec = sdot + 8;                   // [K] decays, kind 3
+  float* sown = sdec + K;                   // [K] u k, kind 3
   const int64_t slot = a.slots[s];
   float* S = a.state + ((slot * a.num_heads + h) * (int64_t)K) * V + c0 + col;
   float* N = nullptr;
@@ -55,6 +60,12 @@ sequential_kernel(const b200_recurrence_args a) {
       const float qn = to_float(q[n]), kn = to_float(k[n]);
       sq[n] = (KIND == kLightning && a.silu ? silu_f(qn) : qn) * a.q_scale;
       sk[n] = KIND == kLightning && a.silu ? silu_f(kn) : kn;
+      if (KIND == kWkv) {
+        const int hn = h * K + n;
+        sdec[n] = expf(-expf(reinterpret_cast<const float*>(a.gate_a)[r * a.gate_stride + hn] + a.bias_a[hn]));
+        sown[n] = a.skip[hn] * kn;
+        sq[n] = qn;
+      }
     }
     float vv[VEC];
 #pragma unroll
@@ -63,10 +74,13 @@ sequential_kernel(const b200_recurrence_args a) {
       if (KIND == kLightning && a.silu) vv[e] = silu_f(vv[e]);
     }
     const float ga =
-        KIND == kLightning ? 0.f : to_float(reinterpret_cast<const T*>(a.gate_a)[r * a.gate_stride + h]);
+        KIND == kLightning || KIND == kWkv ? 0.f : to_float(reinterpret_cast<const T*>(a.gate_a)[r * a.gate_stride + h]);
     float decay, weight;
     if (KIND == kLightning) {
       decay = a.decay[h];
+      weight = 1.f;
+    } else if (KIND == kWkv) {
+      decay = 1.f;  // per key channel, below
       weight = 1.f;
     } else if (KIND == kSsd) {
       const float dt = softplus_f(ga + a.bias_a[h]);
@@ -102,8 +116,17 @@ sequential_kernel(const b200_recurrence_args a) {
           const int n = n0 + j * RP;
           if (n < K) {
             const float wk = weight * sk[n], qn = sq[n];
+            if (KIND == kWkv) {
+              const float d = sdec[n], own = sown[n];
+#pragma unroll
+              for (int e = 0; e < VEC; ++e) {
+                acc[e] += (st[j][e] + own * vv[e]) * qn;
+                st[j][e] = d * st[j][e] + wk * vv[e];
+              }
+            }
 #pragma unroll
             for (int e = 0; e < VEC; ++e) {
+              if (KIND == kWkv) break;
               st[j][e] = decay * st[j][e] + wk * vv[e];
               acc[e] += st[j][e] * qn;
             }
@@ -151,7 +174,7 @@ int launch_sequential(const b200_recurrence_args& a, cudaStream_t st) {
   const int tiles = (a.value_dim + kTileV - 1) / kTileV;
   const bool vec = a.value_dim % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
   const int rp = vec ? kThreads / (kTileV / 4) : kThreads / kTileV;
-  const size_t smem = (2 * (size_t)a.key_dim + (size_t)rp * kTileV + 8) * sizeof(float);
+  const size_t smem = ((KIND == kWkv ? 4 : 2) * (size_t)a.key_dim + (size_t)rp * kTileV + 8) * sizeof(float);
   B200_CHECK_ARG(smem <= 48 * 1024, "recurrence: key_dim %d is too large", a.key_dim);
   const dim3 grid(tiles, a.num_heads, a.num_seqs);
   B200_CUDA_OK(launch_pdl(vec ? sequential_kernel<T, KIND, 4> : sequential_kernel<T, KIND, 1>, grid, dim3(kThreads),
@@ -169,6 +192,7 @@ template <typename T>
 int run_sequential(const b200_recurrence_args& a, cudaStream_t st) {
   return a.kind == rec::kSsd     ? rec::launch_sequential<T, rec::kSsd>(a, st)
          : a.kind == rec::kMlstm ? rec::launch_sequential<T, rec::kMlstm>(a, st)
+         : a.kind == rec::kWkv   ? rec::launch_sequential<T, rec::kWkv>(a, st)
                                  : rec::launch_sequential<T, rec::kLightning>(a, st);
 }
 }  // namespace
@@ -181,6 +205,7 @@ size_t b200_recurrence_workspace_bytes(const b200_recurrence_args* a) {
 
 int b200_recurrence_chunk(const b200_recurrence_args* a) {
   if (!a) return 0;
+  if (a->kind == rec::kWkv) return rec::can_chunk(*a) ? B200_RECURRENCE_CHUNK : 0;
   return rec::tcr::supported(*a) ? B200_RECURRENCE_CHUNK_TC : rec::can_chunk(*a) ? B200_RECURRENCE_CHUNK : 0;
 }
 
@@ -197,7 +222,7 @@ int b200_recurrence_num_launches(const b200_recurrence_args* a) {
 int b200_recurrence(const b200_recurrence_args* a, void* stream) {
   B200_CHECK_ARG(a && a->q && a->k && a->v && a->state && a->out, "recurrence: null argument");
   B200_CHECK_ARG(a->cu_seqlens && a->seq_lens && a->slots, "recurrence: no segments");
-  B200_CHECK_ARG(a->kind == rec::kSsd || a->kind == rec::kMlstm || a->kind == rec::kLightning,
+  B200_CHECK_ARG(a->kind == rec::kSsd || a->kind == rec::kMlstm || a->kind == rec::kLightning || a->kind == rec::kWkv,
                  "recurrence: unknown kind %d", a->kind);
   B200_CHECK_ARG(a->kind == rec::kLightning || (a->gate_a && a->bias_a), "recurrence: this kind needs its gates");
   B200_CHECK_ARG(!a->silu || (a->kind == rec::kLightning && a->num_chunks <= 0),
@@ -207,6 +232,8 @@ int b200_recurrence(const b200_recurrence_args* a, void* stream) {
   B200_CHECK_ARG(a->key_dim > 0 && a->value_dim > 0, "recurrence: empty state");
   if (a->kind == rec::kSsd)
     B200_CHECK_ARG(a->rate && a->skip, "recurrence: kind 0 needs rate and skip");
+  else if (a->kind == rec::kWkv)
+    B200_CHECK_ARG(a->skip && a->num_groups == a->num_heads, "recurrence: kind 3 needs its bonus and a key per head");
   else if (a->kind == rec::kLightning)
     B200_CHECK_ARG(a->rate && a->decay, "recurrence: kind 2 needs rate and decay");
   else
@@ -221,13 +248,14 @@ int b200_recurrence(const b200_recurrence_args* a, void* stream) {
   }
   if (a->num_chunks > 0) {
     if (a->chunk == B200_RECURRENCE_CHUNK_TC) {
-      B200_CHECK_ARG(rec::tcr::supported(*a), "recurrence: this type or these sizes have no tcgen05 form");
+      B200_CHECK_ARG(a->kind != rec::kWkv && rec::tcr::supported(*a), "recurrence: this type or these sizes have no tcgen05 form");
       return a->kind == rec::kSsd     ? rec::tcr::launch<rec::kSsd>(*a, st)
              : a->kind == rec::kMlstm ? rec::tcr::launch<rec::kMlstm>(*a, st)
                                       : rec::tcr::launch<rec::kLightning>(*a, st);
     }
     B200_CHECK_ARG(a->chunk == B200_RECURRENCE_CHUNK && rec::can_chunk(*a),
                    "recurrence: this type or these sizes have no chunked form of %d rows", a->chunk);
+    if (a->kind == rec::kWkv) return rec::wkv::launch(*a, st);
     return a->kind == rec::kSsd     ? rec::launch_chunked<rec::kSsd>(*a, st)
            : a->kind == rec::kMlstm ? rec::launch_chunked<rec::kMlstm>(*a, st)
                                     : rec::launch_chunked<rec::kLightning>(*a, st);

@@ -21,19 +21,19 @@ constexpr int kPad = 72;    // shared row pitch (bf16): ldmatrix without bank co
 constexpr int kTerms = 3;
 constexpr int kTileElems = 64 * kPad;
 
-// workspace: U / S_in [chunks][heads][K][V], then per (chunk, head): key-sum [K], then {total, amax, m_in, first_m}
+// workspace: U / S_in [chunks][heads][K][V], then per (chunk, head): key-sum (kind 3: decay over the chunk) [K], then {total, amax, m_in, first_m}
 struct Workspace {
   float *state, *keysum, *scal, *gates;  // gates (128-row form): per (chunk, head) {cum, src, top, weight}[128]
   __host__ __device__ Workspace(const b200_recurrence_args& a) {
     const size_t ch = (size_t)a.num_chunks * a.num_heads;
     state = reinterpret_cast<float*>(a.workspace);
     keysum = state + ch * a.key_dim * a.value_dim;
-    scal = keysum + (a.kind == kMlstm ? ch * a.key_dim : 0);
+    scal = keysum + (a.kind == kMlstm || a.kind == kWkv ? ch * a.key_dim : 0);
     gates = scal + 4 * ch;
   }
   static size_t bytes(const b200_recurrence_args& a) {
     const size_t ch = (size_t)a.num_chunks * a.num_heads;
-    return (ch * a.key_dim * a.value_dim + (a.kind == kMlstm ? ch * a.key_dim : 0) + 4 * ch +
+    return (ch * a.key_dim * a.value_dim + (a.kind == kMlstm || a.kind == kWkv ? ch * a.key_dim : 0) + 4 * ch +
             (a.chunk == B200_RECURRENCE_CHUNK_TC ? ch * 4 * B200_RECURRENCE_CHUNK_TC : 0)) * sizeof(float);
   }
 };
@@ -255,19 +255,29 @@ chunk_scan_kernel(const b200_recurrence_args a, int state_blocks) {
     float m = KIND == kMlstm ? scal[2] : 0.f;
     constexpr int AHEAD = 4;
     float4 buf[AHEAD];
+    float kept[KIND == kWkv ? AHEAD : 1];  // decay of this key row over a chunk
+    const float* kp = ws.keysum + ((size_t)cfirst * a.num_heads + h) * K + (KIND == kWkv ? i / V : 0);
+    const size_t kstep = (size_t)a.num_heads * K;
 #pragma unroll
     for (int j = 0; j < AHEAD; ++j)
-      if (j < nc) buf[j] = *reinterpret_cast<const float4*>(u + j * ustep);
+      if (j < nc) {
+        buf[j] = *reinterpret_cast<const float4*>(u + j * ustep);
+        if (KIND == kWkv) kept[KIND == kWkv ? j : 0] = kp[j * kstep];
+      }
     for (int c0 = 0; c0 < nc; c0 += AHEAD) {
 #pragma unroll
       for (int j = 0; j < AHEAD; ++j) {
         const int c = c0 + j;
         if (c >= nc) break;
         const float4 U = buf[j];
-        if (c + AHEAD < nc) buf[j] = *reinterpret_cast<const float4*>(u + (size_t)(c + AHEAD) * ustep);
+        float keep = KIND == kWkv ? kept[KIND == kWkv ? j : 0] : 0.f, add = 1.f;
+        if (c + AHEAD < nc) {
+          buf[j] = *reinterpret_cast<const float4*>(u + (size_t)(c + AHEAD) * ustep);
+          if (KIND == kWkv) kept[KIND == kWkv ? j : 0] = kp[(c + AHEAD) * kstep];
+        }
         *reinterpret_cast<float4*>(u + (size_t)c * ustep) = S;
-        float keep, add = 1.f;
-        if (KIND != kMlstm) {
+        if (KIND == kWkv) {
+        } else if (KIND != kMlstm) {
           keep = expf(scal[c * sstep]);
         } else {
           const float amax = scal[c * sstep + 1], b = fmaxf(m, amax);

@@ -10,6 +10,7 @@ namespace rec {
 constexpr int kSsd = 0;
 constexpr int kMlstm = 1;
 constexpr int kLightning = 2;  // decay per head, no gates
+constexpr int kWkv = 3;        // decay per head, key channel and row; a bonus for the current row
 constexpr int kTileV = 64;  // value columns per CTA; mLSTM's normaliser state has one copy per tile
 
 __device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }

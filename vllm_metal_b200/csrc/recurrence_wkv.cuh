@@ -1,0 +1,404 @@
+// Chunked form of the recurrence whose decay is a vector per row (kind 3), 64-row chunks in three launches as in
+// recurrence_chunk.cuh; the scan is shared.
+//
+// Between a row s and a later row t a key channel decays by w_(s+1) .. w_(t-1).  A quotient of cumulative products would
+// overflow where decays are strong, so a chunk is cut into blocks of 16 rows and only products of decays are ever formed:
+//   up to a block's end      K_s = k_s * prod of the block's later decays
+//   from a block's start     R_t = r_t * prod of the block's earlier decays
+//   over a whole block       D_j
+// A row of block i meets a row of an earlier block j through R_t D_(i-1) .. D_(j+1) K_s: tensor-core products, the D's
+// multiplied into R on the way back through the blocks; after the first block R meets the state on entry.  Within a block the
+// scores are formed in fp32 by the ordinary cores, a lane holding one k_s that decays as the rows go by.  The chunk's own
+// contribution is built up block by block: U <- diag(D_j) U + K_j^T v_j.
+//
+// r, k, v are bf16; every 32-bit factor enters the products as a three-term split, products of two split factors as
+// their six largest terms (24 significant bits).
+#pragma once
+
+#include "recurrence_chunk.cuh"
+
+namespace b200 {
+namespace rec {
+namespace wkv {
+
+constexpr int kBlock = 16, kBlocks = kChunk / kBlock;  // one block a warp
+constexpr int kPitch = 68;                              // of fp32 tiles
+constexpr int kFloatTile = kChunk * kPitch;
+
+struct Decays {  // of one key channel over a block
+  float w[kBlock];
+  __device__ __forceinline__ void load(const b200_recurrence_args& a, int row0, int rows, int first, int channel) {
+    const float bias = a.bias_a[channel];
+    const float* z = reinterpret_cast<const float*>(a.gate_a) + (int64_t)(row0 + first) * a.gate_stride + channel;
+#pragma unroll
+    for (int i = 0; i < kBlock; ++i) w[i] = first + i < rows ? z[i * a.gate_stride] : 0.f;
+#pragma unroll
+    for (int i = 0; i < kBlock; ++i) w[i] = first + i < rows ? expf(-expf(w[i] + bias)) : 1.f;  // rows past the end: no decay
+  }
+};
+
+// K_s of one channel and block, split, into the term tiles; returns D.
+__device__ __forceinline__ float keys_to_block_end(const Decays& d, const bf16* sk, bf16* split, int first, int n) {
+  float run = 1.f;
+#pragma unroll
+  for (int i = kBlock - 1; i >= 0; --i) {
+    const int at = (first + i) * kPad + n;
+    float x = to_float(sk[at]) * run;
+#pragma unroll
+    for (int j = 0; j < kTerms; ++j) {
+      const bf16 b = __float2bfloat16_rn(x);
+      split[j * kTileElems + at] = b;
+      x -= to_float(b);
+    }
+    run *= d.w[i];
+  }
+  return run;
+}
+
+// ---- 1: a chunk's own contribution and its decay -----------------------------------------------------
+constexpr int kStateSmem = (2 + kTerms) * kTileElems * 2 + kBlocks * 64 * 4;
+
+__global__ void __launch_bounds__(128)
+state_kernel(const b200_recurrence_args a) {
+  extern __shared__ __align__(16) uint8_t raw[];
+  bf16* sk = reinterpret_cast<bf16*>(raw);
+  bf16* sv = sk + kTileElems;
+  bf16* ks3 = sv + kTileElems;
+  float* D = reinterpret_cast<float*>(ks3 + kTerms * kTileElems);  // [blocks][64]
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
+  const int K = a.key_dim, V = a.value_dim, c0 = tile * kTileV;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  int row0;
+  const int rows = chunk_rows(a, c, &row0);
+  const Workspace ws(a);
+  const bf16* kp = reinterpret_cast<const bf16*>(a.k) + (int64_t)row0 * a.k_stride + (int64_t)h * K;
+  const bf16* vp = reinterpret_cast<const bf16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)h * V + c0;
+  load_tile(sv, vp, a.v_stride, rows, min(kTileV, V - c0));
+  float* U = ws.state + ((size_t)c * a.num_heads + h) * K * V;
+  float* keep = ws.keysum + ((size_t)c * a.num_heads + h) * K;
+  for (int k0 = 0; k0 < K; k0 += kSlab) {
+    load_tile(sk, kp + k0, a.k_stride, rows, min(kSlab, K - k0));
+    mma::cp_commit();
+    const int n = tid & 63, b0 = (tid >> 6) * 2;
+    Decays d[2];
+    if (k0 + n < K) {
+#pragma unroll
+      for (int b = 0; b < 2; ++b) d[b].load(a, row0, rows, (b0 + b) * kBlock, h * K + k0 + n);
+    } else {
+#pragma unroll
+      for (int b = 0; b < 2; ++b)
+#pragma unroll
+        for (int i = 0; i < kBlock; ++i) d[b].w[i] = 1.f;
+    }
+    mma::cp_wait<0>();
+    __syncthreads();
+#pragma unroll
+    for (int b = 0; b < 2; ++b) D[(b0 + b) * 64 + n] = keys_to_block_end(d[b], sk, ks3, (b0 + b) * kBlock, n);
+    __syncthreads();
+    if (tile == 0 && tid < 64 && k0 + tid < K) {
+      float p = 1.f;
+#pragma unroll
+      for (int j = 0; j < kBlocks; ++j) p *= D[j * 64 + tid];
+      keep[k0 + tid] = p;
+    }
+    float acc[8][4];
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+#pragma unroll
+    for (int j = 0; j < kBlocks; ++j) {
+      if (j > 0) {
+        const float d0 = D[j * 64 + warp * 16 + (lane >> 2)], d1 = D[j * 64 + warp * 16 + (lane >> 2) + 8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+          acc[i][0] *= d0, acc[i][1] *= d0;
+          acc[i][2] *= d1, acc[i][3] *= d1;
+        }
+      }
+      // A[m = key dim][k = row]: stored row by row, so the fragments come transposed
+      uint32_t fa[kTerms][4];
+      const int mat = lane >> 3, krow = j * kBlock + ((mat >> 1) ? 8 : 0) + (lane & 7), kcol = warp * 16 + ((mat & 1) ? 8 : 0);
+#pragma unroll
+      for (int t = 0; t < kTerms; ++t) mma::ldsm4t(fa[t], &ks3[t * kTileElems + krow * kPad + kcol]);
+#pragma unroll
+      for (int n2 = 0; n2 < 4; ++n2) {
+        uint32_t fb[4];
+        mma::ldsm4t(fb, &sv[(j * kBlock + (lane & 15)) * kPad + n2 * 16 + (lane >> 4) * 8]);
+#pragma unroll
+        for (int t = 0; t < kTerms; ++t) {
+          mma::mma16816(acc[2 * n2], fa[t], fb[0], fb[1]);
+          mma::mma16816(acc[2 * n2 + 1], fa[t], fb[2], fb[3]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int col = c0 + i * 8 + (lane & 3) * 2;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int kd = k0 + warp * 16 + (lane >> 2) + half * 8;
+        if (kd < K && col < V)
+          *reinterpret_cast<float2*>(U + (size_t)kd * V + col) = make_float2(acc[i][2 * half], acc[i][2 * half + 1]);
+      }
+    }
+    __syncthreads();  // the tiles are free for the next slab
+  }
+}
+
+// ---- 3: outputs ------------------------------------------------------------------------------------------
+// sr sk sv | K's terms | { R, decays } fp32, over which the state on entry goes later (its three terms) | D, bonus, scores
+constexpr int kBig = 2 * kFloatTile * 4;
+static_assert(kBig >= kTerms * kTileElems * 2, "the state's terms go over R and the decays");
+constexpr int kOutputSmem = (3 + kTerms) * kTileElems * 2 + kBig + (kBlocks * 64 + 64) * 4 + 4 * kBlock * (kBlock + 1) * 4;
+
+__global__ void __launch_bounds__(128)
+output_kernel(const b200_recurrence_args a) {
+  extern __shared__ __align__(16) uint8_t raw[];
+  bf16* sr = reinterpret_cast<bf16*>(raw);
+  bf16* sk = sr + kTileElems;
+  bf16* sv = sk + kTileElems;
+  bf16* ks3 = sv + kTileElems;
+  float* sR = reinterpret_cast<float*>(ks3 + kTerms * kTileElems);
+  float* sw = sR + kFloatTile;
+  bf16* ss = reinterpret_cast<bf16*>(sR);
+  float* D = sw + kFloatTile;
+  float* su = D + kBlocks * 64;
+  float* own = su + 64;  // [warp][16 rows t][17]: scores inside the warp's block
+  pdl_trigger();
+  pdl_wait();
+  const int c = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
+  const int K = a.key_dim, V = a.value_dim, c0 = tile * kTileV;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+  int row0;
+  const int rows = chunk_rows(a, c, &row0);
+  const Workspace ws(a);
+  const bf16* rp = reinterpret_cast<const bf16*>(a.q) + (int64_t)row0 * a.q_stride + (int64_t)h * K;
+  const bf16* kp = reinterpret_cast<const bf16*>(a.k) + (int64_t)row0 * a.k_stride + (int64_t)h * K;
+  const bf16* vp = reinterpret_cast<const bf16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)h * V + c0;
+  const float* S = ws.state + ((size_t)c * a.num_heads + h) * K * V;
+  load_tile(sv, vp, a.v_stride, rows, min(kTileV, V - c0));
+  float* mine = own + warp * kBlock * (kBlock + 1);
+  float sc[2 * kBlocks][4], o[8][4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) sc[i][e] = o[i][e] = 0.f;
+  for (int k0 = 0; k0 < K; k0 += kSlab) {
+    load_tile(sr, rp + k0, a.q_stride, rows, min(kSlab, K - k0));
+    load_tile(sk, kp + k0, a.k_stride, rows, min(kSlab, K - k0));
+    mma::cp_commit();
+    {
+      const int n = tid & 63, b0 = (tid >> 6) * 2;
+      if (tid < 64) su[tid] = k0 + tid < K ? a.skip[h * K + k0 + tid] : 0.f;
+      Decays d[2];
+#pragma unroll
+      for (int b = 0; b < 2; ++b) {
+        if (k0 + n < K) {
+          d[b].load(a, row0, rows, (b0 + b) * kBlock, h * K + k0 + n);
+        } else {
+#pragma unroll
+          for (int i = 0; i < kBlock; ++i) d[b].w[i] = 1.f;
+        }
+      }
+      mma::cp_wait<0>();
+      __syncthreads();
+#pragma unroll
+      for (int b = 0; b < 2; ++b) {
+        const int first = (b0 + b) * kBlock;
+        float run = 1.f;
+#pragma unroll
+        for (int i = 0; i < kBlock; ++i) {
+          sR[(first + i) * kPitch + n] = to_float(sr[(first + i) * kPad + n]) * run;
+          sw[(first + i) * kPitch + n] = d[b].w[i];
+          run *= d[b].w[i];
+        }
+        D[(b0 + b) * 64 + n] = keys_to_block_end(d[b], sk, ks3, first, n);
+      }
+    }
+    __syncthreads();
+    // R of the warp's own rows, as fragments: [k step][row half + column half][pair]
+    float R[4][4][2];
+#pragma unroll
+    for (int ks = 0; ks < 4; ++ks)
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        const float2 x = *reinterpret_cast<const float2*>(&sR[(warp * kBlock + g + (q & 1) * 8) * kPitch + ks * 16 + (q >> 1) * 8 + 2 * tq]);
+        R[ks][q][0] = x.x, R[ks][q][1] = x.y;
+      }
+    {  // scores inside the block: lane = row s, half of the slab's channels
+      const int s = lane & 15, n0 = (lane >> 4) * 32, base = warp * kBlock;
+      float q[32];
+#pragma unroll
+      for (int i = 0; i < 32; i += 8) {
+        const uint4 x4 = *reinterpret_cast<const uint4*>(&sk[(base + s) * kPad + n0 + i]);
+        const bf16* x = reinterpret_cast<const bf16*>(&x4);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) q[i + e] = to_float(x[e]);
+      }
+      float bonus = 0.f;  // the current row against itself
+#pragma unroll
+      for (int i = 0; i < 32; i += 8) {
+        const uint4 x4 = *reinterpret_cast<const uint4*>(&sr[(base + s) * kPad + n0 + i]);
+        const bf16* x = reinterpret_cast<const bf16*>(&x4);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) bonus = fmaf(to_float(x[e]) * su[n0 + i + e], q[i + e], bonus);
+      }
+      bonus += __shfl_xor_sync(0xffffffffu, bonus, 16);
+      if (lane < 16) mine[s * (kBlock + 1) + s] = (k0 > 0 ? mine[s * (kBlock + 1) + s] : 0.f) + bonus;
+#pragma unroll 1
+      for (int t = 1; t < kBlock; ++t) {
+        float dot[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < 32; i += 8) {
+          const uint4 x4 = *reinterpret_cast<const uint4*>(&sr[(base + t) * kPad + n0 + i]);
+          const bf16* x = reinterpret_cast<const bf16*>(&x4);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) dot[e & 3] = fmaf(to_float(x[e]), q[i + e], dot[e & 3]);
+        }
+        float sum = (dot[0] + dot[1]) + (dot[2] + dot[3]);
+        sum += __shfl_xor_sync(0xffffffffu, sum, 16);
+        if (s < t) {
+          if (lane < 16) mine[t * (kBlock + 1) + s] = (k0 > 0 ? mine[t * (kBlock + 1) + s] : 0.f) + sum;
+#pragma unroll
+          for (int i = 0; i < 32; i += 4) {
+            const float4 w = *reinterpret_cast<const float4*>(&sw[(base + t) * kPitch + n0 + i]);
+            q[i] *= w.x, q[i + 1] *= w.y, q[i + 2] *= w.z, q[i + 3] *= w.w;
+          }
+        }
+        __syncwarp();
+      }
+    }
+    // against earlier blocks, nearest first; R picks up a block's decay after it
+    auto split = [&](int ks, uint32_t (&fa)[kTerms][4]) {
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        uint32_t t[kTerms];
+        mma::split_pair<kTerms>(R[ks][q][0], R[ks][q][1], t);
+#pragma unroll
+        for (int j = 0; j < kTerms; ++j) fa[j][q] = t[j];
+      }
+    };
+#pragma unroll
+    for (int j = kBlocks - 2; j >= 0; --j) {
+      if (j >= warp) continue;
+#pragma unroll
+      for (int ks = 0; ks < 4; ++ks) {
+        uint32_t fa[kTerms][4];
+        split(ks, fa);
+#pragma unroll
+        for (int y = 0; y < kTerms; ++y) {
+          uint32_t fb[4];
+          mma::ldsm4(fb, &ks3[y * kTileElems + (j * kBlock + (lane >> 4) * 8 + (lane & 7)) * kPad + ks * 16 + ((lane >> 3) & 1) * 8]);
+#pragma unroll
+          for (int x = 0; x + y < kTerms; ++x) {
+            mma::mma16816(sc[2 * j], fa[x], fb[0], fb[1]);
+            mma::mma16816(sc[2 * j + 1], fa[x], fb[2], fb[3]);
+          }
+        }
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const float2 d = *reinterpret_cast<const float2*>(&D[j * 64 + ks * 16 + (q >> 1) * 8 + 2 * tq]);
+          R[ks][q][0] *= d.x, R[ks][q][1] *= d.y;
+        }
+      }
+    }
+    __syncthreads();  // R and the decays have been read everywhere: the state on entry goes over them
+    for (int i = tid; i < 64 * 16; i += 128) {
+      const int r = i >> 4, cc = (i & 15) * 4;
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (k0 + r < K && c0 + cc < V) x = *reinterpret_cast<const float4*>(S + (size_t)(k0 + r) * V + c0 + cc);
+      uint32_t t0[kTerms], t1[kTerms];
+      mma::split_pair<kTerms>(x.x, x.y, t0);
+      mma::split_pair<kTerms>(x.z, x.w, t1);
+#pragma unroll
+      for (int j = 0; j < kTerms; ++j) *reinterpret_cast<uint2*>(&ss[j * kTileElems + r * kPad + cc]) = make_uint2(t0[j], t1[j]);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int ks = 0; ks < 4; ++ks) {
+      uint32_t fa[kTerms][4];
+      split(ks, fa);
+#pragma unroll
+      for (int n2 = 0; n2 < 4; ++n2)
+#pragma unroll
+        for (int y = 0; y < kTerms; ++y) {
+          uint32_t fb[4];
+          mma::ldsm4t(fb, &ss[y * kTileElems + (ks * 16 + (lane & 15)) * kPad + n2 * 16 + (lane >> 4) * 8]);
+#pragma unroll
+          for (int x = 0; x + y < kTerms; ++x) {
+            mma::mma16816(o[2 * n2], fa[x], fb[0], fb[1]);
+            mma::mma16816(o[2 * n2 + 1], fa[x], fb[2], fb[3]);
+          }
+        }
+    }
+    __syncthreads();
+  }
+  // the block's own scores, on and below the diagonal
+  float dg[2][4];
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int t = g + (e >> 1) * 8, s = i * 8 + 2 * tq + (e & 1);
+      dg[i][e] = s <= t ? mine[t * (kBlock + 1) + s] : 0.f;
+    }
+#pragma unroll
+  for (int j = 0; j < kBlocks; ++j) {
+    if (j > warp) break;
+    uint32_t p[4][kTerms];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const bool diagonal = j == warp;
+      mma::split_pair<kTerms>(diagonal ? dg[i][0] : sc[2 * j + i][0], diagonal ? dg[i][1] : sc[2 * j + i][1], p[2 * i]);
+      mma::split_pair<kTerms>(diagonal ? dg[i][2] : sc[2 * j + i][2], diagonal ? dg[i][3] : sc[2 * j + i][3], p[2 * i + 1]);
+    }
+#pragma unroll
+    for (int n2 = 0; n2 < 4; ++n2) {
+      uint32_t fb[4];
+      mma::ldsm4t(fb, &sv[(j * kBlock + (lane & 15)) * kPad + n2 * 16 + (lane >> 4) * 8]);
+#pragma unroll
+      for (int x = 0; x < kTerms; ++x) {
+        const uint32_t fa[4] = {p[0][x], p[1][x], p[2][x], p[3][x]};
+        mma::mma16816(o[2 * n2], fa, fb[0], fb[1]);
+        mma::mma16816(o[2 * n2 + 1], fa, fb[2], fb[3]);
+      }
+    }
+  }
+  bf16* out = reinterpret_cast<bf16*>(a.out);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int cc = i * 8 + tq * 2;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int t = warp * kBlock + g + e * 8;
+      if (t >= rows || c0 + cc >= V) continue;
+      *reinterpret_cast<__nv_bfloat162*>(out + (int64_t)(row0 + t) * a.out_stride + (int64_t)h * V + c0 + cc) =
+          __floats2bfloat162_rn(o[i][2 * e], o[i][2 * e + 1]);
+    }
+  }
+}
+
+inline int launch(const b200_recurrence_args& a, cudaStream_t st) {
+  B200_CHECK_ARG(a.workspace && a.workspace_bytes >= Workspace::bytes(a), "recurrence: workspace too small");
+  B200_CHECK_ARG(a.chunk_seq && a.chunk_row && a.seq_chunk0, "recurrence: no chunk list");
+  B200_CHECK_ARG(a.num_chunks <= 65535, "recurrence: more than 65535 chunks");
+  static bool attr = false;
+  if (!attr) {
+    B200_CUDA_OK(cudaFuncSetAttribute(state_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kStateSmem));
+    B200_CUDA_OK(cudaFuncSetAttribute(output_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kOutputSmem));
+    attr = true;
+  }
+  const dim3 grid((a.value_dim + kTileV - 1) / kTileV, a.num_heads, a.num_chunks);
+  B200_CUDA_OK(launch_pdl(state_kernel, grid, dim3(128), kStateSmem, st, a));
+  const int blocks = (a.key_dim * a.value_dim / 4 + kScanThreads - 1) / kScanThreads;
+  B200_CUDA_OK(launch_pdl(chunk_scan_kernel<kWkv>, dim3(blocks, a.num_heads, a.num_seqs), dim3(kScanThreads), 0, st, a, blocks));
+  B200_CUDA_OK(launch_pdl(output_kernel, grid, dim3(128), kOutputSmem, st, a));
+  return check_launch("recurrence (decays per key channel)");
+}
+
+}  // namespace wkv
+}  // namespace rec
+}  // namespace b200

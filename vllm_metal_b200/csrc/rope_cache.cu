@@ -112,7 +112,7 @@ norm_rope_cache_kernel(T* __restrict__ q, T* __restrict__ k, const T* __restrict
   }
 }
 
-// ---- the other order: RoPE -> per-head norm without a weight -> cache --------------------------------
+// ---- the other order: RoPE (if any) -> per-head norm -> cache ------------------------------------------
 // Angles from a frequency table (scaled rotations), once per token and CTA.  One CTA per token, a warp per head, a lane
 // holds the pairs lane, lane + 32, ... of the head in registers from load to store.
 template <typename T>
@@ -138,6 +138,24 @@ __device__ __forceinline__ void load_pairs(const T* src, int dim, float2 (&v)[NP
   }
 }
 
+// times `f` and, where given, a weight per dimension
+template <typename T, int NP, bool VEC>
+__device__ __forceinline__ void store_pairs(T* dst, int dim, const float2 (&v)[NP], float f, const float* weight) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int j = 0; j < NP; ++j) {
+    const int e = 2 * (lane + 32 * j);
+    if (e >= dim) continue;
+    const float x = v[j].x * f * (weight ? weight[e] : 1.f), y = v[j].y * f * (weight && e + 1 < dim ? weight[e + 1] : 1.f);
+    if (VEC) {
+      *reinterpret_cast<Pair<T>*>(dst + e) = Pair<T>{from_float<T>(x), from_float<T>(y)};
+    } else {
+      dst[e] = from_float<T>(x);
+      if (e + 1 < dim) dst[e + 1] = from_float<T>(y);
+    }
+  }
+}
+
 template <typename T, int NP, bool VEC>
 __global__ void __launch_bounds__(RC_WARPS * 32)
 rope_norm_cache_kernel(const b200_rope_norm_cache_args a) {
@@ -155,6 +173,8 @@ rope_norm_cache_kernel(const b200_rope_norm_cache_args a) {
     turn[i] = make_float2(a.rot_factor * (cs + fmaf(-s1, sn, c1 * cs)), a.rot_factor * (sn + fmaf(s1, cs, c1 * sn)));
   }
   __syncthreads();
+  float temp = 1.f;
+  if (a.temp_coef != 0.f) temp = 1.f + a.temp_coef * logf((float)floor(((double)a.positions[t] + 1.0) / (double)a.temp_every) + 1.f);
   const int64_t slot = a.slot_mapping[t];
   const bool cached = slot >= 0 && slot < a.num_blocks * a.block_size;
   const int64_t blk = cached ? slot / a.block_size : 0, off = cached ? slot - blk * a.block_size : 0;
@@ -166,6 +186,15 @@ rope_norm_cache_kernel(const b200_rope_norm_cache_args a) {
       const T* src = reinterpret_cast<const T*>(a.v) + (int64_t)t * a.v_stride + (int64_t)hv * a.vdim;
       T* dst = vrow + (int64_t)hv * a.vdim;
       if (!cached) continue;
+      if (a.norm_values) {
+        float2 v[NP];
+        load_pairs<T, NP, VEC>(src, a.vdim, v);
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < NP; ++j) ss += v[j].x * v[j].x + v[j].y * v[j].y;
+        store_pairs<T, NP, VEC>(dst, a.vdim, v, 1.f / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps), nullptr);
+        continue;
+      }
       if (a.vdim % (16 / sizeof(T)) == 0 && (((uintptr_t)src | (uintptr_t)dst) & 15) == 0) {
         for (int i = lane; i < a.vdim / (int)(16 / sizeof(T)); i += 32)
           reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
@@ -193,16 +222,8 @@ rope_norm_cache_kernel(const b200_rope_norm_cache_args a) {
     }
     float f = 1.f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps);
     if (is_q && a.q_weight) f *= a.q_weight[h];
-#pragma unroll
-    for (int j = 0; j < NP; ++j) {
-      const int e = 2 * (lane + 32 * j);
-      if (VEC) {
-        if (e < a.dim) *reinterpret_cast<Pair<T>*>(dst + e) = Pair<T>{from_float<T>(v[j].x * f), from_float<T>(v[j].y * f)};
-      } else {
-        if (e < a.dim) dst[e] = from_float<T>(v[j].x * f);
-        if (e + 1 < a.dim) dst[e + 1] = from_float<T>(v[j].y * f);
-      }
-    }
+    if (is_q) f *= temp;
+    store_pairs<T, NP, VEC>(dst, a.dim, v, f, is_q ? a.q_norm : a.k_norm);
   }
 }
 
@@ -210,9 +231,10 @@ template <typename T, bool VEC>
 int launch_rope_norm_cache(const b200_rope_norm_cache_args& a, cudaStream_t st) {
   const int total = a.heads + 2 * a.kv_heads, need = (total + RC_WARPS - 1) / RC_WARPS;
   const dim3 grid(a.num_tokens, a.num_tokens >= 1024 ? 1 : need);
-  auto* kern = a.dim <= 64    ? rope_norm_cache_kernel<T, 1, VEC>
-               : a.dim <= 128 ? rope_norm_cache_kernel<T, 2, VEC>
-               : a.dim <= 256 ? rope_norm_cache_kernel<T, 4, VEC>
+  const int held = a.norm_values && a.vdim > a.dim ? a.vdim : a.dim;
+  auto* kern = held <= 64    ? rope_norm_cache_kernel<T, 1, VEC>
+               : held <= 128 ? rope_norm_cache_kernel<T, 2, VEC>
+               : held <= 256 ? rope_norm_cache_kernel<T, 4, VEC>
                               : rope_norm_cache_kernel<T, 8, VEC>;
   B200_CUDA_OK(launch_pdl(kern, grid, dim3(RC_WARPS * 32), 0, st, a));
   return check_launch("rope_norm_cache");
@@ -231,13 +253,18 @@ extern "C" int b200_rope_norm_cache(const b200_rope_norm_cache_args* a, void* st
   B200_CHECK_ARG(a->block_size > 0 && a->num_blocks > 0 && a->k_token_stride >= (int64_t)a->kv_heads * a->dim &&
                      a->v_token_stride >= (int64_t)a->kv_heads * a->vdim,
                  "rope_norm_cache: bad cache geometry");
+  B200_CHECK_ARG(!a->norm_values || a->vdim <= RC_MAX_D, "rope_norm_cache: normed values of at most %d columns, got %d", RC_MAX_D,
+                 a->vdim);
+  B200_CHECK_ARG(a->temp_coef == 0.f || a->temp_every > 0.f, "rope_norm_cache: temp_every must be positive");
   if (a->num_tokens <= 0) return B200_OK;
   return B200_DISPATCH_DTYPE(a->dtype, T, [&]() -> int {
     auto ok = [](const void* p, int64_t s0, int64_t s1) {
       return (uintptr_t)p % (2 * sizeof(T)) == 0 && s0 % 2 == 0 && s1 % 2 == 0;
     };
     const bool vec = a->dim % 2 == 0 && ok(a->q, a->q_stride, 0) && ok(a->k, a->k_stride, 0) &&
-                     ok(a->key_cache, a->k_block_stride, a->k_token_stride);
+                     ok(a->key_cache, a->k_block_stride, a->k_token_stride) &&
+                     (!a->norm_values || (a->vdim % 2 == 0 && ok(a->v, a->v_stride, 0) &&
+                                          ok(a->value_cache, a->v_block_stride, a->v_token_stride)));
     return vec ? launch_rope_norm_cache<T, true>(*a, (cudaStream_t)stream)
                : launch_rope_norm_cache<T, false>(*a, (cudaStream_t)stream);
   });

@@ -20,10 +20,17 @@ def _up(n: int) -> int:
     return -(-n // _ALIGN) * _ALIGN
 
 
+def _wide_mm(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    if x.dtype == torch.float32:
+        return torch.mm(x, weight.t())
+    return torch.mm(x, weight.t(), out_dtype=torch.float32)
+
+
 class StackedLinear:
     """``y = x W^T`` for several weights ``[out_i, in]`` that share ``x``; ``split(y)`` gives the parts as views."""
 
-    def __init__(self, parts: dict[str, torch.Tensor], dtype: torch.dtype, device) -> None:
+    def __init__(self, parts: dict[str, torch.Tensor], dtype: torch.dtype, device, bias: torch.Tensor | None = None) -> None:
+        """``bias``: of a single part."""
         self.slices: dict[str, tuple[int, int]] = {}
         at = 0
         for name, w in parts.items():
@@ -36,15 +43,19 @@ class StackedLinear:
                 raise ValueError(f"'{name}' takes {w.shape[1]} inputs, the others {width}")
             lo, hi = self.slices[name]
             self.weight[lo:hi].copy_(w)
+        self.bias = None
+        if bias is not None:
+            self.bias = torch.zeros(at, dtype=dtype, device=device)
+            self.bias[:bias.shape[0]].copy_(bias)
 
     def __call__(self, x: torch.Tensor) -> torch.Tensor:
+        if self.bias is not None:
+            return torch.addmm(self.bias, x, self.weight.t())
         return torch.mm(x, self.weight.t())
 
     def wide(self, x: torch.Tensor) -> torch.Tensor:
         """The product kept in fp32."""
-        if x.dtype == torch.float32:
-            return torch.mm(x, self.weight.t())
-        return torch.mm(x, self.weight.t(), out_dtype=torch.float32)
+        return _wide_mm(x, self.weight)
 
     def split(self, y: torch.Tensor) -> dict[str, torch.Tensor]:
         return {name: y[:, lo:hi] for name, (lo, hi) in self.slices.items()}
@@ -52,6 +63,18 @@ class StackedLinear:
     def span(self, y: torch.Tensor, first: str, last: str) -> torch.Tensor:
         """The columns from part ``first`` to part ``last``, alignment padding (zeros) between them included."""
         return y[:, self.slices[first][0]:self.slices[last][1]]
+
+
+class BatchedLinear:
+    """``y[i] = x[i] W_i^T`` for weights ``[out, in]`` of one size, an input each: one batched product."""
+
+    def __init__(self, weights: list[torch.Tensor], dtype: torch.dtype, device) -> None:
+        self.weight = torch.empty((len(weights), *weights[0].shape), dtype=dtype, device=device)
+        for own, w in zip(self.weight, weights, strict=True):
+            own.copy_(w)
+
+    def __call__(self, x: torch.Tensor) -> torch.Tensor:
+        return torch.bmm(x, self.weight.transpose(1, 2))
 
 
 class SideBySideLinear:
@@ -75,6 +98,10 @@ class SideBySideLinear:
     def __call__(self, y: torch.Tensor) -> torch.Tensor:
         return torch.mm(y, self.weight.t())
 
+    def wide(self, y: torch.Tensor) -> torch.Tensor:
+        """The product kept in fp32."""
+        return _wide_mm(y, self.weight)
+
     def add_into(self, x: torch.Tensor, y: torch.Tensor) -> None:
         if y.dtype == torch.float32:
             torch.addmm(x, y, self.weight.t(), out=x)
@@ -89,6 +116,4 @@ class DenseHead:
         self.weight = weight.to(device=device, dtype=dtype).contiguous()
 
     def __call__(self, x: torch.Tensor) -> torch.Tensor:
-        if x.dtype == torch.float32:
-            return torch.mm(x, self.weight.t())
-        return torch.mm(x, self.weight.t(), out_dtype=torch.float32)
+        return _wide_mm(x, self.weight)

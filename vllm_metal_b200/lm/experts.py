@@ -1,4 +1,4 @@
-"""Feed-forward of routed experts with a gated shared one beside them, over the C-ABI kernels: router product -> choice ->
+"""Feed-forward of routed experts, where the design has it with a gated shared one beside them, over the C-ABI kernels: router product -> choice ->
 sort of the (row, place) pairs -> ONE launch for the way in of all experts and the shared one -> ONE for their way out.
 The weighted sum is left to whoever reads the result (the step to the next sublayer).  Nothing is read back to the host, so
 the block runs under CUDA graphs."""
@@ -21,7 +21,7 @@ class RoutedExperts:
     def __init__(self, r: RoutedArgs, width: int, get, dtype, device) -> None:
         """``get(name, shape)``: the block's tensors by their own names (``e0.gate`` ..., ``router``, ``shared.sg`` ...)."""
         self.r, self.width, self.dtype = r, width, dtype
-        self.correction = get("correction", (r.experts,)).to(device=device, dtype=torch.float32).contiguous()
+        self.correction = get("router.b" if r.over_chosen else "correction", (r.experts,)).to(device=device, dtype=torch.float32).contiguous()
         heads = {"router": get("router", (r.experts, width))}
         self.way_in = torch.empty((r.experts, 2 * r.ff, width), dtype=dtype, device=device)
         self.way_out = torch.zeros((r.experts, width, _pad8(r.ff)), dtype=dtype, device=device)
@@ -54,7 +54,7 @@ class RoutedExperts:
         logits, as ``residual_step`` takes them."""
         r, ops, t = self.r, get_ops(), h.shape[0]
         heads = self.router.split(self.router.wide(h))
-        chosen, weights = ops.expert_route(heads["router"], self.correction, r.experts, r.top, r.scale)
+        chosen, weights = ops.expert_route(heads["router"], self.correction, r.experts, r.top, r.scale, r.over_chosen)
         plan = ops.expert_plan(chosen, r.experts, self.tile_rows(t))
         act, shared_act = ops.expert_product(h, self.way_in, plan, r.top, t, gated=True, shared_weight=self.shared_in)
         y, extra = ops.expert_product(act, self.way_out, plan, r.top, t, gated=False, k=r.ff, shared_x=shared_act,

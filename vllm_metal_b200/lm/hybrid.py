@@ -52,7 +52,7 @@ class HybridModel:
     layer_class = ParallelLayer
 
     def __init__(self, args: HybridArgs, get, dtype: torch.dtype = torch.bfloat16, device="cuda") -> None:
-        """``get(name, shape)`` returns a checkpoint tensor of that shape (or raises)."""
+        """``get(name, shape)`` returns a checkpoint tensor of that shape (or raises); a size of None is the tensor's own."""
         if dtype not in (torch.bfloat16, torch.float32):
             raise ValueError(f"hybrid decoders run in bfloat16 or float32, not {dtype}")
         pin_matmul_precision()
@@ -71,8 +71,9 @@ class HybridModel:
         files = SafetensorsFolder(folder)
 
         def get(name: str, shape: tuple[int, ...]) -> torch.Tensor:
-            if files.shape(name) != tuple(shape):
-                raise ValueError(f"{folder}: tensor '{name}' is {files.shape(name)}, the configuration says {tuple(shape)}")
+            found = files.shape(name)
+            if len(found) != len(shape) or any(n is not None and n != m for n, m in zip(shape, found)):
+                raise ValueError(f"{folder}: tensor '{name}' is {found}, the configuration says {tuple(shape)}")
             return files.tensor(name)
 
         return cls(args, get, dtype, device)

@@ -232,9 +232,58 @@ class RotaryAttentionArgs:
         return b
 
 
-MixerArgs = LatentAttentionArgs | Mamba2Args | MLSTMArgs | LightningArgs | SideBySideArgs | RotaryAttentionArgs
-MIXER_ARGS = {c.kind: c for c in (LatentAttentionArgs, Mamba2Args, MLSTMArgs, LightningArgs, SideBySideArgs,
-                                  RotaryAttentionArgs)}
+@dataclass(frozen=True)
+class TimeMixArgs:
+    """RWKV-style time mixing: a matrix state per head whose decay, per key channel, is a function of the input."""
+
+    heads: int
+    dim: int
+
+    kind = "wkv"
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.dim
+
+    @classmethod
+    def parse(cls, m: dict, where: str) -> TimeMixArgs:
+        a = cls(heads=_take(m, "heads", where), dim=_take(m, "dim", where))
+        _positive(a, where, "heads", "dim")
+        return a
+
+
+@dataclass(frozen=True)
+class BiasedAttentionArgs:
+    """Softmax attention whose scores fall with the distance; normed queries, keys and values, a factor on the queries that
+    grows with the position, a window, and a sigmoid gate on the output."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int        # 0: every earlier token is visible
+    temp_coef: float   # 0: no factor on the queries
+    temp_every: float
+
+    kind = "attention"
+
+    @classmethod
+    def parse(cls, m: dict, where: str) -> BiasedAttentionArgs:
+        a, mask, temp = SoftmaxAttentionArgs.parse(m, where), m.get("mask") or {}, m.get("q_temp")
+        coef, every = (_take(temp, k, f"{where}.q_temp", float) for k in ("coef", "every")) if temp else (0.0, 1.0)
+        b = cls(a.heads, a.kv_heads, a.dim, a.vdim, a.scale, int(mask.get("size") or 0), coef, every)
+        if b.window < 0 or not b.temp_every > 0:
+            raise ConfigError(f"{where}: mask.size {b.window}, q_temp.every {b.temp_every}")
+        return b
+
+    def slopes(self) -> list[float]:
+        """What every token of distance takes off a head's scores."""
+        return [2.0 ** (-8.0 * (h + 1) / self.heads) for h in range(self.heads)]
+
+
+MixerArgs = (LatentAttentionArgs | Mamba2Args | MLSTMArgs | LightningArgs | SideBySideArgs | RotaryAttentionArgs | TimeMixArgs |
+             BiasedAttentionArgs)
 
 
 @dataclass(frozen=True)
@@ -246,15 +295,17 @@ class RoutedArgs:
     ff: int
     scale: float
     shared_ff: int  # 0: none
+    over_chosen: bool = False  # weights: softmax of the (biased) logits of the chosen alone; else of all, times scale
 
     @classmethod
-    def parse(cls, mlp: dict, where: str) -> RoutedArgs:
+    def parse(cls, mlp: dict, where: str, over_chosen: bool = False) -> RoutedArgs:
         where = f"{where}.mlp"
         router = _take(mlp, "router", where, dict)
-        shared = mlp.get("shared")
+        shared = None if over_chosen else mlp.get("shared")
         a = cls(_take(router, "experts", f"{where}.router"), _take(router, "top", f"{where}.router"),
                 _take(_take(mlp, "expert", where, dict), "ff", f"{where}.expert"),
-                _take(router, "scale", f"{where}.router", float), _take(shared, "ff", f"{where}.shared") if shared else 0)
+                1.0 if over_chosen else _take(router, "scale", f"{where}.router", float),
+                _take(shared, "ff", f"{where}.shared") if shared else 0, over_chosen)
         _positive(a, where, "experts", "top", "ff")
         if a.top > a.experts or a.experts > MAX_EXPERTS:
             raise ConfigError(f"{where}: {a.top} of {a.experts} experts (at most {MAX_EXPERTS})")
@@ -271,22 +322,24 @@ def paged_row(mixer: MixerArgs) -> int:
     return a.kv_heads * (a.dim + a.vdim) if a is not None else 0
 
 
-def cached_heads(mixer: MixerArgs) -> SoftmaxAttentionArgs | RotaryAttentionArgs | None:
+def cached_heads(mixer: MixerArgs) -> SoftmaxAttentionArgs | RotaryAttentionArgs | BiasedAttentionArgs | None:
     """The attention whose keys and values (of ``kv_heads``) a layer with this mixer caches, if any."""
     if isinstance(mixer, SideBySideArgs):
         return mixer.left
-    return mixer if isinstance(mixer, RotaryAttentionArgs) else None
+    return mixer if isinstance(mixer, (RotaryAttentionArgs, BiasedAttentionArgs)) else None
 
 
 @dataclass(frozen=True)
 class Design:
     """What the architecture fixes."""
 
-    mixers: tuple[str, ...]
+    mixers: tuple[type, ...]
     # "parallel": mixer and feed-forward from one norm (lm/hybrid.py); "hyper": sublayers around several streams
-    # (lm/streams.py); "sandwich": sublayers between two norms, a short convolution on the mixer's input (lm/sandwich.py)
+    # (lm/streams.py); "sandwich": sublayers between two norms, a short convolution on the mixer's input (lm/sandwich.py);
+    # "prenorm": a grouped norm ahead of every sublayer, looped layers take the embedding in again (lm/prenorm.py)
     layout: str = "parallel"
-    feed_forward: str = "dense"
+    feed_forward: tuple[str, ...] = ("dense",)
+    route_over_chosen: bool = False
 
     @property
     def hyper_connected(self) -> bool:
@@ -294,9 +347,10 @@ class Design:
 
 
 DESIGNS = {
-    "Mapuvik": Design(("latent_attention", "mamba2", "mlstm")),
-    "Tatazen": Design(("lightning", "parallel"), "hyper"),
-    "Kerolorn": Design(("attention",), "sandwich", "moe"),
+    "Mapuvik": Design((LatentAttentionArgs, Mamba2Args, MLSTMArgs)),
+    "Tatazen": Design((LightningArgs, SideBySideArgs), "hyper"),
+    "Kerolorn": Design((RotaryAttentionArgs,), "sandwich", ("moe",)),
+    "Retuvik": Design((TimeMixArgs, BiasedAttentionArgs), "prenorm", ("dense", "moe"), route_over_chosen=True),
 }
 
 
@@ -318,6 +372,10 @@ class HybridArgs:
     streams: int = 1               # copies of the residual stream (hyper-connected designs)
     input_taps: int = 0            # of the convolution on a mixer's input (2: token shift); 0: none
     logit_scale: float = 1.0
+    norm_groups: int = 1           # parts of a row that are normed on their own
+    embedding_scale: float = 1.0
+    passes: tuple[tuple[int, int], ...] = ()  # (layer run, number of the pass) where a pass of the loop begins
+    loop_times: int = 0
 
     @property
     def design(self) -> Design:
@@ -350,16 +408,18 @@ class HybridArgs:
         for i, entry in enumerate(_take(config, "layers", name, list)):
             where = f"layers[{i}]"
             kind = _take(entry, "type", where, str)
-            if kind not in design.mixers:
-                raise ConfigError(f"{where}: unknown mixer '{kind}' (known: {', '.join(sorted(design.mixers))})")
-            mixer = MIXER_ARGS[kind].parse(_take(entry, "mixer", where, dict), where)
+            known = {c.kind: c for c in design.mixers}
+            if kind not in known:
+                raise ConfigError(f"{where}: unknown mixer '{kind}' (known: {', '.join(sorted(known))})")
+            mixer = known[kind].parse(_take(entry, "mixer", where, dict), where)
             ff, routed = 0, None
             if entry.get("mlp") is not None:
                 mlp = entry["mlp"]
-                if mlp.get("kind", "dense") != design.feed_forward:
-                    raise ConfigError(f"{where}: feed-forward kind '{mlp.get('kind')}' is not supported ({design.feed_forward} only)")
-                if design.feed_forward == "moe":
-                    routed = RoutedArgs.parse(mlp, where)
+                if mlp.get("kind", "dense") not in design.feed_forward:
+                    raise ConfigError(f"{where}: feed-forward kind '{mlp.get('kind')}' is not supported "
+                                      f"({', '.join(design.feed_forward)} only)")
+                if mlp.get("kind") == "moe":
+                    routed = RoutedArgs.parse(mlp, where, design.route_over_chosen)
                 else:
                     ff = _take(mlp, "ff", where)
                     if ff < 1:
@@ -391,6 +451,15 @@ class HybridArgs:
                          logit_scale=_take(config, "logit_scale", name, float))
             if not 1 <= extra["input_taps"] <= MAX_INPUT_TAPS:
                 raise ConfigError(f"{name}: canon.taps {extra['input_taps']} outside 1..{MAX_INPUT_TAPS}")
+        elif design.layout == "prenorm":
+            extra = dict(norm_groups=_take(_take(config, "norm", name, dict), "groups", f"{name}: norm"),
+                         embedding_scale=_take(_take(config, "embedding", name, dict), "scale", f"{name}: embedding", float))
+            if extra["norm_groups"] < 1 or _take(config, "width", name) % extra["norm_groups"]:
+                raise ConfigError(f"{name}: width {config['width']} in {extra['norm_groups']} norm groups")
+            if config.get("loop") is not None:
+                start, stop, times = (config["loop"][k] for k in ("start", "stop", "times"))
+                extra |= dict(loop_times=times,
+                              passes=tuple((start + t * (stop - start), t) for t in range(times)) if stop > start else ())
         a = cls(name=name, vocab=_take(config, "vocab", name), width=_take(config, "width", name),
                 eps=_take(_take(config, "norm", name, dict), "eps", name, float), layers=tuple(layers), **extra)
         _positive(a, name, "vocab", "width", "streams")

@@ -5,8 +5,10 @@ from __future__ import annotations
 
 import torch
 
-from .hybrid_config import (HybridArgs, LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs, RotaryAttentionArgs,
-                            SideBySideArgs)
+from .hybrid_config import (BiasedAttentionArgs, HybridArgs, LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs,
+                            RotaryAttentionArgs, SideBySideArgs, TimeMixArgs)
+
+DECAY_RANK = 64  # bottleneck of the decays where nothing says otherwise (a checkpoint has its own)
 
 
 def tensor_shapes(args: HybridArgs) -> dict[str, tuple[int, ...]]:
@@ -41,6 +43,15 @@ def tensor_shapes(args: HybridArgs) -> dict[str, tuple[int, ...]]:
         elif isinstance(m, RotaryAttentionArgs):
             shapes |= {p + "q": (m.heads * m.dim, w), p + "k": (m.kv_heads * m.dim, w), p + "v": (m.kv_heads * m.vdim, w),
                        p + "temp": (m.heads,), p + "o": (w, m.heads * m.vdim)}
+        elif isinstance(m, TimeMixArgs):
+            rank = min(DECAY_RANK, w)
+            shapes |= {p + "mu." + s: (w,) for s in "rkvgw"} | {p + s: (m.inner, w) for s in "rkvg"}
+            shapes |= {p + "w1": (rank, w), p + "w2": (m.inner, rank), p + "w0": (m.inner,), p + "u": (m.heads, m.dim),
+                       p + "norm": (m.inner,), p + "o": (w, m.inner)}
+        elif isinstance(m, BiasedAttentionArgs):
+            shapes |= {p + "q": (m.heads * m.dim, w), p + "k": (m.kv_heads * m.dim, w), p + "v": (m.kv_heads * m.vdim, w),
+                       p + "q.norm": (m.dim,), p + "k.norm": (m.dim,), p + "g": (m.heads * m.vdim, w),
+                       p + "o": (w, m.heads * m.vdim)}
         if layer.ff:
             shapes |= {f"l{i}.mlp.up": (layer.ff, w), f"l{i}.mlp.down": (w, layer.ff)}
         if layer.routed is not None:
@@ -48,13 +59,17 @@ def tensor_shapes(args: HybridArgs) -> dict[str, tuple[int, ...]]:
             units = [(f"e{e}.", r.ff) for e in range(r.experts)] + ([("shared.", r.shared_ff)] if r.shared_ff else [])
             for name, ff in units:
                 shapes |= {p + name + "gate": (ff, w), p + name + "up": (ff, w), p + name + "down": (w, ff)}
-            shapes |= {p + "router": (r.experts, w), p + "correction": (r.experts,)}
+            shapes |= {p + "router": (r.experts, w), p + ("router.b" if r.over_chosen else "correction"): (r.experts,)}
             if r.shared_ff:
                 shapes |= {p + "shared.sg": (1, w)}
         if args.design.layout == "sandwich":
             shapes |= {f"l{i}.norm1b": (w,), f"l{i}.canon1": (w, args.input_taps)}
             if layer.routed is not None:
                 shapes |= {f"l{i}.norm2": (w,), f"l{i}.norm2b": (w,)}
+        if args.design.layout == "prenorm" and (layer.ff or layer.routed is not None):
+            shapes |= {f"l{i}.norm2": (w,)}
+            if layer.ff:
+                shapes |= {f"l{i}.mlp.up.b": (layer.ff,), f"l{i}.mlp.down.b": (w,), f"l{i}.mlp.act": (2,)}
         if args.design.hyper_connected:
             s = args.streams
             shapes |= {f"l{i}.shift": (w,)}
@@ -63,6 +78,8 @@ def tensor_shapes(args: HybridArgs) -> dict[str, tuple[int, ...]]:
             for q in (1, 2) if layer.ff else (1,):
                 shapes |= {f"l{i}.hc{q}.in": (s,), f"l{i}.hc{q}.out": (s,), f"l{i}.hc{q}.mix": (s, s),
                            f"l{i}.rg{q}": (w, w), f"l{i}.rg{q}.b": (w,)}
+    if args.passes:
+        shapes |= {"loop.step": (args.loop_times, w)}
     return shapes | {"final.norm": (w,), "head": (args.vocab, w)}
 
 
@@ -77,8 +94,9 @@ def random_tensors(args: HybridArgs, device="cpu", seed: int = 0):
     number = {name: i for i, name in enumerate(shapes)}
 
     def get(name: str, shape: tuple[int, ...]) -> torch.Tensor:
-        if shapes[name] != tuple(shape):
+        if len(shape) != len(shapes[name]) or any(n is not None and n != m for n, m in zip(shape, shapes[name])):
             raise ValueError(f"tensor '{name}': asked for {shape}, the configuration says {shapes[name]}")
+        shape = shapes[name]
         gen = torch.Generator(device=device).manual_seed(seed * 1000003 + number[name])
         t = torch.empty(shape, dtype=torch.float32, device=device).normal_(0.0, 1.0, generator=gen)
         leaf = name.split(".", 1)[-1]
@@ -96,6 +114,10 @@ def random_tensors(args: HybridArgs, device="cpu", seed: int = 0):
             t = torch.eye(shape[0], device=device) + 0.1 * t
         elif leaf == "shift":
             t = torch.sigmoid(t)
+        elif leaf.startswith("mix.mu."):       # between the row and the one before it
+            t = torch.sigmoid(t)
+        elif leaf == "mix.w0":                 # decays from a few rows to some hundred
+            t = 1.5 * t - 3.0
         elif leaf in ("norm1", "norm"):        # stored around zero
             t = 0.1 * t
         elif leaf == "mix.A_log":
@@ -106,7 +128,7 @@ def random_tensors(args: HybridArgs, device="cpu", seed: int = 0):
             t = t + 2.0
         elif leaf == "mix.conv":
             t = t * shape[1] ** -0.5
-        elif leaf in ("mix.D", "mix.i.b", "mix.conv.b", "embed"):
+        elif leaf in ("mix.D", "mix.i.b", "mix.conv.b", "mix.u", "embed", "step", "mlp.router.b", "mlp.up.b", "mlp.down.b"):
             t = 0.5 * t
         elif len(shape) == 2:
             t = t * shape[1] ** -0.5

@@ -3,7 +3,9 @@ handed, per call, the stacked projections of its input and what its LAYER keeps 
 slots); it leaves its heads' outputs, gated and normed, in the left columns of the layer's output operand.
 
 Interface: ``spans`` names runs of parts the mixer also wants as one view, ``weights`` are to be stacked into the layer's input product, ``out_weight`` belongs to its output product
-(the layer takes both away with ``take_weights``); ``run(parts, up, meta, cache, layer, y, act_offset)``."""
+(the layer takes both away with ``take_weights``); ``run(parts, up, meta, cache, layer, y, act_offset)``.  A mixer with
+``mix_weight [mixes, width]`` reads several mixes of a row with the row before, ``project(mixes [mixes, T, width])`` makes its
+parts of them."""
 
 from __future__ import annotations
 
@@ -13,13 +15,15 @@ import torch
 
 from ..attention.impls.segments import EXPAND_PAGE
 from ..metal import get_ops
-from .hybrid_config import (LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs, RotaryAttentionArgs,
-                            SoftmaxAttentionArgs)
+from .dense import BatchedLinear, SideBySideLinear, StackedLinear
+from .hybrid_config import (BiasedAttentionArgs, LatentAttentionArgs, LightningArgs, Mamba2Args, MLSTMArgs, RotaryAttentionArgs,
+                            SoftmaxAttentionArgs, TimeMixArgs)
 
 Get = Callable[[str, tuple[int, ...]], torch.Tensor]
 
 
 class Mixer:
+    mix_weight: torch.Tensor | None = None
     spans: dict[str, tuple[str, str]] = {}
     weights: dict[str, torch.Tensor]
     out_weight: torch.Tensor
@@ -161,6 +165,66 @@ class RotaryAttentionMixer(Mixer):
             ops.mixer_finish(y, inner, up, act_offset)
 
 
+class TimeMixMixer(Mixer):
+    """RWKV-style time mixing: five mixes of a row with the row before -> products, the decay's through a bottleneck ->
+    recurrence -> per-head norm -> silu gate."""
+
+    MIXES = "rkvgw"
+
+    def __init__(self, m: TimeMixArgs, width: int, eps: float, get: Get, dtype, device) -> None:
+        self.m, self.eps = m, eps
+        f32 = lambda name, *shape: get(name, shape).to(device=device, dtype=torch.float32).contiguous()  # noqa: E731
+        self.mix_weight = torch.stack([f32(f"mu.{s}", width) for s in self.MIXES]).contiguous()
+        self.weights = {}
+        self.out_weight = get("o", (width, m.inner))
+        self.products = BatchedLinear([get(s, (m.inner, width)) for s in self.MIXES[:4]], dtype, device)
+        down = get("w1", (None, width))
+        self.decay_down = StackedLinear({"w": down}, dtype, device)
+        self.decay_up = SideBySideLinear({"w": get("w2", (m.inner, down.shape[0]))}, dtype, device)
+        self.decay_bias, self.bonus = f32("w0", m.inner), f32("u", m.heads, m.dim)
+        self.norm = f32("norm", m.inner)
+
+    def project(self, mixes: torch.Tensor) -> dict[str, torch.Tensor]:
+        r, k, v, g = self.products(mixes[:4])
+        z = self.decay_up.operand(mixes.shape[1])
+        get_ops().mixer_finish(z, 0, self.decay_down(mixes[4]), act="tanh")
+        return {"r": r, "k": k, "v": v, "g": g, "w": self.decay_up.wide(z)}
+
+    def run(self, parts, up, meta, cache, layer: int, y: torch.Tensor, act_offset: int) -> None:
+        m, ops = self.m, get_ops()
+        o = ops.recurrence("wkv", parts["r"], parts["k"], parts["v"], parts["w"], None, meta, cache.states[layer].matrix,
+                           heads=m.heads, groups=m.heads, key_dim=m.dim, value_dim=m.dim, bias_a=self.decay_bias, skip=self.bonus)
+        ops.mixer_finish(y, m.inner, up, act_offset, y=o, post_gate=parts["g"], weight=self.norm, group_size=m.dim, eps=self.eps,
+                         post="silu")
+
+
+class BiasedAttentionMixer(Mixer):
+    """Causal attention over paged keys and values, all three normed per head: scores fall with the distance, queries grow with
+    the position; a sliding window and a sigmoid gate on the output."""
+
+    def __init__(self, m: BiasedAttentionArgs, width: int, eps: float, get: Get, dtype, device) -> None:
+        self.m, self.eps = m, eps
+        self.weights = {"q": get("q", (m.heads * m.dim, width)), "k": get("k", (m.kv_heads * m.dim, width)),
+                        "v": get("v", (m.kv_heads * m.vdim, width)), "g": get("g", (m.heads * m.vdim, width))}
+        self.out_weight = get("o", (width, m.heads * m.vdim))
+        self.q_norm, self.k_norm = (get(n, (m.dim,)).to(device=device, dtype=torch.float32).contiguous() for n in ("q.norm", "k.norm"))
+        self.slopes = torch.tensor(m.slopes(), dtype=torch.float64).to(device=device, dtype=torch.float32)
+
+    def run(self, parts, up, meta, cache, layer: int, y: torch.Tensor, act_offset: int) -> None:
+        m, ops = self.m, get_ops()
+        keys, values = cache.kv[layer]
+        q, k, v = (parts[n].unflatten(1, (h, d)) for n, h, d in (("q", m.heads, m.dim), ("k", m.kv_heads, m.dim),
+                                                                  ("v", m.kv_heads, m.vdim)))
+        ops.rope_norm_cache(q, k, v, keys, values, meta.slot_mapping, meta.positions, None, 1.0, self.eps, q_norm=self.q_norm,
+                            k_norm=self.k_norm, norm_values=True, temperature=(m.temp_coef, m.temp_every))
+        inner = m.heads * m.vdim
+        ops.paged_attention_primitive(q, keys, values, m.kv_heads, m.scale, 0.0, meta.block_tables, meta.seq_lens,
+                                      meta.cu_seqlens_q, meta.block_size, meta.max_seq_len, m.window if m.window > 0 else -1,
+                                      y[:, :inner].unflatten(1, (m.heads, m.vdim)), wide_weights=True, plain_softmax=True,
+                                      min_q_len=meta.min_q_len, slopes=self.slopes)
+        ops.mixer_finish(y, inner, up, act_offset, y=y[:, :inner], post_gate=parts["g"])
+
+
 class LatentAttentionMixer(Mixer):
     """Latent attention: short segments attend in the latent space (queries are taken there by the keys' up-projection),
     long ones get their visible keys and values expanded first, whichever is the smaller work."""
@@ -251,4 +315,5 @@ class LatentAttentionMixer(Mixer):
 
 MIXERS = {c: k for c, k in ((LatentAttentionArgs, LatentAttentionMixer), (Mamba2Args, Mamba2Mixer),
                             (MLSTMArgs, MLSTMMixer), (LightningArgs, LightningMixer),
-                            (SoftmaxAttentionArgs, SoftmaxAttentionMixer), (RotaryAttentionArgs, RotaryAttentionMixer))}
+                            (SoftmaxAttentionArgs, SoftmaxAttentionMixer), (RotaryAttentionArgs, RotaryAttentionMixer),
+                            (TimeMixArgs, TimeMixMixer), (BiasedAttentionArgs, BiasedAttentionMixer))}

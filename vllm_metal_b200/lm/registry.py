@@ -57,10 +57,12 @@ class HybridFamily(ModelFamily):
     @staticmethod
     def model_class(args: HybridArgs) -> type:
         from .hybrid import HybridModel
+        from .prenorm import PreNormModel
         from .sandwich import SandwichModel
         from .streams import StreamModel
 
-        return {"parallel": HybridModel, "hyper": StreamModel, "sandwich": SandwichModel}[args.design.layout]
+        return {"parallel": HybridModel, "hyper": StreamModel, "sandwich": SandwichModel,
+                "prenorm": PreNormModel}[args.design.layout]
 
     def make_cache(self, args, num_blocks, block_size, num_slots, dtype, device):
         from ..attention.caches.hybrid_cache import HybridCache
@@ -94,6 +96,7 @@ FAMILIES: dict[str, ModelFamily] = {
     "Mapuvik": HybridFamily("hybrid"),
     "Tatazen": HybridFamily("streams"),
     "Kerolorn": HybridFamily("sandwich"),
+    "Retuvik": HybridFamily("prenorm"),
     **dict.fromkeys(("LlamaForCausalLM", "MistralForCausalLM", "Qwen3ForCausalLM", "GptOssForCausalLM"), _DECODER),
 }
 

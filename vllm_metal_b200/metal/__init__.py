@@ -28,7 +28,7 @@ from typing import Any
 import torch
 
 from . import constants
-from .hybrid_ops import HYBRID_SYMBOLS, SANDWICH_SYMBOLS, STREAM_SYMBOLS, HybridOps, bind_hybrid
+from .hybrid_ops import HYBRID_SYMBOLS, PRENORM_SYMBOLS, SANDWICH_SYMBOLS, STREAM_SYMBOLS, HybridOps, bind_hybrid
 from .constants import DTYPE_BF16, DTYPE_F16, DTYPE_F32, PA_WINDOW_MAX_HEAD_SIZE as PA_WINDOW_MAX_HEAD, PARTITION_SIZE
 
 logger = logging.getLogger(__name__)
@@ -86,6 +86,7 @@ class PagedAttnArgs(ctypes.Structure):
         ("plain_softmax", ctypes.c_int32),
         ("min_q_len", ctypes.c_int32),
         ("keep_first", ctypes.c_int32),
+        ("slopes", ctypes.c_void_p),
     ]
 
 
@@ -139,6 +140,7 @@ EXPORTED_SYMBOLS = (
     *HYBRID_SYMBOLS,
     *STREAM_SYMBOLS,
     *SANDWICH_SYMBOLS,
+    *PRENORM_SYMBOLS,
 )
 
 
@@ -393,6 +395,7 @@ class _Ops(HybridOps):
         plain_softmax: bool = False,
         min_q_len: int = 0,
         keep_first: int = 0,
+        slopes: torch.Tensor | None = None,
         _force_partitions: int = 0,
         _kernel: int = 0,
     ) -> None:
@@ -402,7 +405,8 @@ class _Ops(HybridOps):
         compression is out of scope for this build and raises.  ``wide_weights``: the tensor-core kernels
         keep 16 instead of 8 significant bits of the softmax weights in the value product.  ``plain_softmax``:
         nothing is added to the softmax denominator.  ``min_q_len``: rows of the shortest sequence, if known (long ones
-        alone need no per-row launch).  ``keep_first``: positions below it stay visible beside a window.  The values' head size may differ from the keys'; ``out`` is then ``[T, H_q, D_v]``.
+        alone need no per-row launch).  ``keep_first``: positions below it stay visible beside a window.  ``slopes``: fp32
+        ``[H_q]``, taken off a score per position of distance.  The values' head size may differ from the keys'; ``out`` is then ``[T, H_q, D_v]``.
         """
         if use_turboquant or key_scale_cache is not None or value_scale_cache is not None:
             if sinks is not None:
@@ -429,6 +433,10 @@ class _Ops(HybridOps):
                     "sinks must be float32; the kernel reads them as device float and "
                     "folds them into a float32 softmax accumulator")
             sinks = sinks.contiguous()
+        if slopes is not None:
+            _require_cuda("slopes", slopes)
+            if slopes.shape != (query.shape[1],) or slopes.dtype != torch.float32 or not slopes.is_contiguous():
+                raise ValueError(f"slopes must be float32, one per query head, got {tuple(slopes.shape)} {slopes.dtype}")
         if window_seqlen_q < 1:
             raise ValueError(
                 f"window_seqlen_q must be >= 1 (1 = per-token decode), got {window_seqlen_q}; "
@@ -517,7 +525,7 @@ class _Ops(HybridOps):
         a.out_dtype = _dtype_code("out", out)
         a.window_seqlen_q = int(window_seqlen_q)
         a.wide_weights, a.plain_softmax = int(bool(wide_weights)), int(bool(plain_softmax))
-        a.min_q_len, a.keep_first = int(min_q_len), int(keep_first)
+        a.min_q_len, a.keep_first, a.slopes = int(min_q_len), int(keep_first), _ptr(slopes)
         if dv != d:
             a.value_dim = dv
             a.v_block_stride, a.v_token_stride, a.v_head_stride = value_cache.stride()[:3]

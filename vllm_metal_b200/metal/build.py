@@ -31,6 +31,7 @@ COMPONENTS: dict[str, tuple[str, ...]] = {
     "hybrid": (*_COMMON, "latent_attention", "latent_ops", "recurrence"),
     "streams": (*_COMMON, "recurrence", "rope_cache", "stream_ops"),
     "sandwich": (*_COMMON, "experts", "residual_step", "rope_cache"),
+    "prenorm": (*_COMMON, "experts", "recurrence", "residual_step", "rope_cache"),
 }
 _wanted: list[str] = []  # the component this process asked for last
 

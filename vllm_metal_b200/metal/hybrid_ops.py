@@ -43,6 +43,8 @@ SANDWICH_SYMBOLS = (
     "b200_expert_product_failed",
 )
 
+PRENORM_SYMBOLS = ("b200_token_mix",)
+
 EXPERT_TILES = (32, 64, 128)  # pairs per tile of the expert products
 
 RECURRENCE_CHUNKS = (64, 128)  # rows per chunk of the two chunked forms
@@ -61,7 +63,7 @@ MixerFinishArgs = _struct(
     P="y pre_gate post_gate weight act_in out",
     L="y_stride pre_stride post_stride act_stride out_stride",
     I="rows inner group_size act_dim act_offset out_cols y_head_dim y_head_stride",
-    F="eps", I2="dtype", P2="act_mul", L2="mul_stride", I3="act_kind")
+    F="eps", I2="dtype", P2="act_mul", L2="mul_stride", I3="act_kind post_silu", F2="act_a act_b")
 RecurrenceArgs = _struct(
     "RecurrenceArgs", "b200_recurrence_args",
     P="q k v gate_a gate_b bias_a bias_b rate skip state norm_state max_state cu_seqlens seq_lens slots chunk_seq "
@@ -86,12 +88,14 @@ LatentPrepArgs = _struct(
 ResidualStepArgs = _struct(
     "ResidualStepArgs", "b200_residual_step_args",
     P="x y part_weight extra extra_gate out_norm in_norm h conv_weight state slots seq_lens row_ids",
-    L="y_stride extra_stride gate_stride h_stride", I="rows dim parts taps", F="eps", I2="dtype")
+    L="y_stride extra_stride gate_stride h_stride", I="rows dim parts taps", F="eps", I2="dtype",
+    P2="bias table ids add h32 mix_weight mix_state", L2="mix_stride", F2="table_scale", I3="vocab fresh groups mixes")
 RopeNormCacheArgs = _struct(
     "RopeNormCacheArgs", "b200_rope_norm_cache_args",
     P="q k v q_weight freq positions slot_mapping key_cache value_cache",
     L="q_stride k_stride v_stride k_block_stride k_token_stride v_block_stride v_token_stride num_blocks",
-    I="num_tokens heads kv_heads dim vdim rot_dims block_size", F="rot_factor eps", I2="dtype")
+    I="num_tokens heads kv_heads dim vdim rot_dims block_size", F="rot_factor eps", I2="dtype",
+    P2="q_norm k_norm", F2="temp_coef temp_every", I3="norm_values")
 ExpertProductArgs = _struct(
     "ExpertProductArgs", "b200_expert_product_args",
     P="x w out shared_x shared_w shared_out pairs first tiles",
@@ -126,7 +130,8 @@ def bind_hybrid(lib: ctypes.CDLL) -> None:
         getattr(lib, f"b200_{name}_workspace_bytes").argtypes = [ctypes.POINTER(struct)]
         getattr(lib, f"b200_{name}_workspace_bytes").restype = ctypes.c_size_t
         getattr(lib, f"b200_{name}_num_launches").argtypes = [ctypes.POINTER(struct)]
-    lib.b200_expert_route.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, f32, vp]
+    lib.b200_expert_route.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, f32, i32, vp]
+    lib.b200_token_mix.argtypes = [vp] * 7 + [i32] * 4 + [i64] * 3 + [i32, vp]
     lib.b200_expert_plan.argtypes = [vp] * 4 + [i32] * 4 + [vp]
     lib.b200_recurrence_chunk.argtypes = [ctypes.POINTER(RecurrenceArgs)]
 
@@ -183,10 +188,11 @@ class HybridOps:
 
     def mixer_finish(self, out, inner: int, act_in=None, act_offset: int = 0, y=None, pre_gate=None, post_gate=None,
                      weight=None, group_size: int = 0, eps: float = 0.0, y_head_dim: int = 0,
-                     y_head_stride: int = 0, act: str = "gelu", act_mul=None) -> None:
-        """Gate -> group norm -> gate into ``out[:, :inner]`` and ``act(act_in)`` ("gelu" / "silu", times ``act_mul``)
-        into ``out[:, act_offset:]``, one launch; ``y`` may be given per head with padding (``y_head_dim`` used of every
-        ``y_head_stride`` columns)."""
+                     y_head_stride: int = 0, act: str = "gelu", act_mul=None, act_weights=(0.0, 0.0),
+                     post: str = "sigmoid") -> None:
+        """Gate -> group norm -> gate (``post``: "sigmoid" / "silu") into ``out[:, :inner]`` and ``act(act_in)`` ("gelu" /
+        "silu" / "tanh" / "xielu" with its two ``act_weights``, times ``act_mul``) into ``out[:, act_offset:]``, one launch;
+        ``y`` may be given per head with padding (``y_head_dim`` used of every ``y_head_stride`` columns)."""
         _rows("out", out)
         a = MixerFinishArgs()
         for name, t in (("y", y), ("pre_gate", pre_gate), ("post_gate", post_gate), ("act_in", act_in),
@@ -205,7 +211,8 @@ class HybridOps:
         a.inner, a.group_size, a.eps, a.dtype = inner, group_size, float(eps), _DTYPE[out.dtype]
         a.act_dim, a.act_offset = (0 if act_in is None else act_in.shape[1]), act_offset
         a.y_head_dim, a.y_head_stride = y_head_dim, y_head_stride
-        a.act_kind, a.mul_stride = ("gelu", "silu").index(act), 0 if act_mul is None else act_mul.stride(0)
+        a.post_silu, (a.act_a, a.act_b) = ("sigmoid", "silu").index(post), act_weights
+        a.act_kind, a.mul_stride = ("gelu", "silu", "tanh", "xielu").index(act), 0 if act_mul is None else act_mul.stride(0)
         if act_mul is not None and act_mul.shape != act_in.shape:
             raise ValueError(f"act_mul is {tuple(act_mul.shape)}, act_in {tuple(act_in.shape)}")
         self._check(self._lib.b200_mixer_finish(ctypes.byref(a), _stream()))
@@ -278,18 +285,22 @@ class HybridOps:
         self.launches += 1
         return h, shifted
 
-    def residual_step(self, x, result=None, in_norm=None, *, eps: float, dtype, rows=None, conv=None, seg=None):
-        """What lies between two sublayers that stand between norms (one launch).  ``result``: what the last one left --
-        ``y [T, dim]`` (or, with ``part_weight [T, parts]``, ``[T * parts, dim]``), optionally ``extra`` with
-        ``extra_gate [T]``, and its ``norm`` -- is added to the fp32 stream ``x [T, dim]``; ``in_norm`` of the next one
-        gives its input, returned.  ``conv`` = (weights [taps, dim], state) with ``seg``: the input plus its convolution, for
-        a batch of single rows.  ``rows`` (int64): only these rows are worked on, the input is packed, ``x`` stays."""
+    def residual_step(self, x, result=None, in_norm=None, *, eps: float, dtype, rows=None, conv=None, seg=None, groups: int = 1,
+                      embed=None, add=None, mix=None, wide: bool = False):
+        """What lies between two sublayers (one launch).  ``result``: what the last one left -- ``y [T, dim]`` (or, with
+        ``part_weight [T, parts]``, ``[T * parts, dim]``), optionally ``extra`` with ``extra_gate [T]``, a ``bias [dim]``, and
+        its ``norm`` (None: as it is) -- is added to the fp32 stream ``x [T, dim]``; then ``embed`` = (ids, table, scale, fresh)
+        -- scaled embedding rows, with which a fresh stream begins -- and the vector ``add``.  ``in_norm`` of the next one, in
+        ``groups`` parts of a row, gives its input, returned (``wide``: in fp32).  For a batch of single rows ``conv`` =
+        (weights [taps, dim], state) with ``seg``: the input plus its convolution; or ``mix`` = (weights [mixes, dim], fp32
+        state [slots, dim]): the input mixed with the row before, ``[mixes, T, dim]``.  ``rows`` (int64): only these rows are
+        worked on, the input is packed, ``x`` stays."""
         _rows("x", x, torch.float32)
         t, dim = x.shape
         if not x.is_contiguous():
             raise ValueError("x must be contiguous")
         a = ResidualStepArgs()
-        a.x, a.dim, a.eps, a.dtype = x.data_ptr(), dim, float(eps), _DTYPE[dtype]
+        a.x, a.dim, a.eps, a.dtype, a.groups = x.data_ptr(), dim, float(eps), _DTYPE[dtype], groups
         a.rows = t if rows is None else rows.shape[0]
         if rows is not None:
             if rows.dtype != torch.int64 or not rows.is_cuda:
@@ -300,7 +311,8 @@ class HybridOps:
             a.parts = 0 if pw is None else pw.shape[1]
             if y.shape != (t * max(1, a.parts), dim):
                 raise ValueError(f"y is {tuple(y.shape)}, the stream has {t} rows of {dim}")
-            a.y, a.y_stride, a.out_norm = y.data_ptr(), y.stride(0), _f32("norm", result["norm"], dim)
+            a.y, a.y_stride, a.out_norm = y.data_ptr(), y.stride(0), _f32("norm", result.get("norm"), dim)
+            a.bias = _f32("bias", result.get("bias"), dim)
             if pw is not None:
                 a.part_weight = _f32("part_weight", pw, t * a.parts)
             if extra is not None:
@@ -309,29 +321,65 @@ class HybridOps:
                     raise ValueError("extra must be [T, dim] and its gate float32 [T]")
                 a.extra, a.extra_stride = extra.data_ptr(), extra.stride(0)
                 a.extra_gate, a.gate_stride = gate.data_ptr(), gate.stride(0)
+        if embed is not None:
+            ids, table, scale, fresh = embed
+            if ids.dtype != torch.int32 or ids.shape != (t,) or _rows("table", table, dtype).shape[1] != dim or \
+                    not table.is_contiguous():
+                raise ValueError(f"embed: int32 ids, one per row, and a contiguous table of {dim} columns")
+            a.ids, a.table, a.table_scale = ids.data_ptr(), table.data_ptr(), float(scale)
+            a.vocab, a.fresh = table.shape[0], int(fresh)
+        a.add = _f32("add", add, dim)
         h = None
         if in_norm is not None:
-            h = torch.empty((a.rows, dim), dtype=dtype, device=x.device)
-            a.h, a.h_stride, a.in_norm = h.data_ptr(), h.stride(0), _f32("in_norm", in_norm, dim)
+            a.in_norm = _f32("in_norm", in_norm, dim)
+            shape = (a.rows, dim) if mix is None else (mix[0].shape[0], a.rows, dim)
+            h = torch.empty(shape, dtype=torch.float32 if wide else dtype, device=x.device)
+            a.h_stride = h.stride(-2)
+            if wide:
+                a.h32 = h.data_ptr()
+            else:
+                a.h = h.data_ptr()
+        if (conv is not None or mix is not None) and seg.cu_seqlens_q.shape[0] - 1 != t:
+            raise ValueError("the fused convolution or mix takes one row per request")
         if conv is not None:
             weight, state = conv
             taps = weight.shape[0]
             if state.dtype != dtype or tuple(state.shape[1:]) != (taps - 1, dim) or not state.is_contiguous():
                 raise ValueError(f"state must be contiguous [slots, {taps - 1}, {dim}] of the activation type")
-            if seg.cu_seqlens_q.shape[0] - 1 != t:
-                raise ValueError("the fused convolution takes one row per request")
             a.conv_weight, a.taps = _f32("conv weight", weight, taps * dim), taps
             a.state = state.data_ptr() if state.numel() else None
+        if mix is not None:
+            weight, state = mix
+            a.mixes, a.mix_weight = weight.shape[0], _f32("mix weight", weight, weight.shape[0] * dim)
+            a.mix_state, a.mix_stride = _f32("mix state", state, state.shape[0] * dim), h.stride(0)
+        if conv is not None or mix is not None:
             a.slots, a.seq_lens = seg.state_slots.data_ptr(), seg.seq_lens.data_ptr()
         self._check(self._lib.b200_residual_step(ctypes.byref(a), _stream()))
         self.launches += 1
         return h
 
+    def token_mix(self, h, weight, state, seg, dtype) -> torch.Tensor:
+        """``h`` (fp32 ``[T, dim]``) mixed with the row before of its segment, once per row of ``weight [mixes, dim]``; the fp32
+        ``state [slots, dim]`` carries a segment's last row: ``[mixes, T, dim]`` of ``dtype``."""
+        _rows("h", h, torch.float32)
+        t, dim = h.shape
+        mixes = weight.shape[0]
+        out = torch.empty((mixes, t, dim), dtype=dtype, device=h.device)
+        self._check(self._lib.b200_token_mix(
+            h.data_ptr(), _f32("mix weight", weight, mixes * dim), _f32("mix state", state, state.shape[0] * dim),
+            seg.cu_seqlens_q.data_ptr(), seg.seq_lens.data_ptr(), seg.state_slots.data_ptr(), out.data_ptr(),
+            seg.cu_seqlens_q.shape[0] - 1, seg.max_q_len, dim, mixes, h.stride(0), out.stride(1), out.stride(0), _DTYPE[dtype],
+            _stream()))
+        self.launches += 1
+        return out
+
     def rope_norm_cache(self, q, k, v, key_cache, value_cache, slot_mapping, positions, freq, factor: float, eps: float,
-                        q_weight=None) -> None:
-        """Heads rotated (interleaved pairs, ``freq [pairs, 2]`` high and low parts, times ``factor``), then divided by
-        their root mean square, queries times ``q_weight [H]``: ``q [T, H, D]`` in place, ``k [T, G, D]`` and
-        ``v [T, G, V]`` into the paged caches."""
+                        q_weight=None, *, q_norm=None, k_norm=None, norm_values: bool = False,
+                        temperature=(0.0, 1.0)) -> None:
+        """Heads rotated (interleaved pairs, ``freq [pairs, 2]`` high and low parts, times ``factor``; None: not at all), then
+        divided by their root mean square, queries times ``q_weight [H]``, with weights ``q_norm`` / ``k_norm`` ``[D]``:
+        ``q [T, H, D]`` in place, ``k [T, G, D]`` and ``v [T, G, V]`` into the paged caches.  ``norm_values``: value heads are
+        divided by theirs as well.  ``temperature`` = (coef, every): queries times 1 + coef ln(floor((p + 1) / every) + 1)."""
         t, heads, dim = q.shape
         groups, vdim = v.shape[1:]
         for name, x in (("q", q), ("k", k), ("v", v)):
@@ -347,8 +395,10 @@ class HybridOps:
         a = RopeNormCacheArgs()
         a.q, a.k, a.v, a.key_cache, a.value_cache = (x.data_ptr() for x in (q, k, v, key_cache, value_cache))
         a.q_weight = _f32("q_weight", q_weight, heads)
-        a.rot_dims = freq.numel()
-        a.freq = _f32("freq", freq, freq.numel()) if freq.numel() else None
+        a.rot_dims = 0 if freq is None else freq.numel()
+        a.freq = _f32("freq", freq, freq.numel()) if a.rot_dims else None
+        a.q_norm, a.k_norm = _f32("q_norm", q_norm, dim), _f32("k_norm", k_norm, dim)
+        a.norm_values, (a.temp_coef, a.temp_every) = int(norm_values), temperature
         a.positions, a.slot_mapping = positions.data_ptr(), slot_mapping.data_ptr()
         a.q_stride, a.k_stride, a.v_stride = q.stride(0), k.stride(0), v.stride(0)
         a.k_block_stride, a.k_token_stride = key_cache.stride()[:2]
@@ -359,8 +409,9 @@ class HybridOps:
         self._check(self._lib.b200_rope_norm_cache(ctypes.byref(a), _stream()))
         self.launches += 1
 
-    def expert_route(self, logits, correction, experts: int, top: int, scale: float):
-        """``(chosen int32 [T, top], weights fp32 [T, top])`` of fp32 router logits (their first ``experts`` columns)."""
+    def expert_route(self, logits, correction, experts: int, top: int, scale: float, over_chosen: bool = False):
+        """``(chosen int32 [T, top], weights fp32 [T, top])`` of fp32 router logits (their first ``experts`` columns).
+        ``over_chosen``: the correction is part of the logits and the weights are the softmax over the chosen ones alone."""
         _rows("logits", logits, torch.float32)
         t = logits.shape[0]
         if logits.shape[1] < experts:
@@ -369,7 +420,7 @@ class HybridOps:
         weights = torch.empty((t, top), dtype=torch.float32, device=logits.device)
         self._check(self._lib.b200_expert_route(
             logits.data_ptr(), logits.stride(0), _f32("correction", correction, experts), chosen.data_ptr(),
-            weights.data_ptr(), t, experts, top, float(scale), _stream()))
+            weights.data_ptr(), t, experts, top, float(scale), int(over_chosen), _stream()))
         self.launches += 1
         return chosen, weights
 
@@ -446,16 +497,19 @@ class HybridOps:
                    value_dim: int, bias_a=None, bias_b=None, rate=None, skip=None, norm_state=None, max_state=None,
                    q_scale: float = 1.0, gate_cap: float = 0.0, decay=None, silu=None,
                    force_sequential: bool = False, chunk: int = 0) -> torch.Tensor:
-        """Linear recurrence (``kind`` "ssd" / "mlstm" gated, "lightning" with ``decay`` per head and ``rate`` =
-        -log(decay); there ``silu``, a view that covers q, k and v, says they still have to go through silu: as they are
+        """Linear recurrence (``kind`` "ssd" / "mlstm" gated, "wkv" with decays per head and key channel from the fp32 ``gate_a
+        [T, heads * key_dim]`` and ``bias_a``, ``skip`` the current row's bonus, "lightning" with ``decay`` per head and ``rate``
+        = -log(decay); there ``silu``, a view that covers q, k and v, says they still have to go through silu: as they are
         read where no chunk is involved, else in place beforehand) over the segments of ``seg``: outputs ``[T, heads *
         value_dim]``, the slots' fp32 states updated in place.  Segments longer than ``seg.chunk_limit`` rows run in
         chunks on tensor cores where type and sizes allow (``chunk``: a form by its rows per chunk, 0 = auto)."""
         a = RecurrenceArgs()
         for name, t in (("q", q), ("k", k), ("v", v), ("gate_a", gate_a), ("gate_b", gate_b)):
             if t is not None:
-                _rows(name, t, v.dtype)
+                _rows(name, t, torch.float32 if kind == "wkv" and name == "gate_a" else v.dtype)
                 setattr(a, name, t.data_ptr())
+        if kind == "wkv" and gate_a.shape != (v.shape[0], heads * key_dim):
+            raise ValueError(f"recurrence: gates must be [T, {heads * key_dim}], got {tuple(gate_a.shape)}")
         if gate_b is not None and gate_b.stride(0) != gate_a.stride(0):
             raise ValueError("both gates must share one row stride")
         if q.shape[1] != groups * key_dim or v.shape[1] != heads * value_dim:
@@ -464,8 +518,9 @@ class HybridOps:
         if tuple(state.shape) != (slots, heads, key_dim, value_dim):
             raise ValueError(f"state must be [slots, {heads}, {key_dim}, {value_dim}], got {tuple(state.shape)}")
         tiles = -(-value_dim // RECURRENCE_TILE_V)
-        a.bias_a, a.bias_b = _f32("bias_a", bias_a, heads), _f32("bias_b", bias_b, heads)
-        a.rate, a.skip = _f32("rate", rate, heads), _f32("skip", skip, heads)
+        wide = heads * (key_dim if kind == "wkv" else 1)
+        a.bias_a, a.bias_b = _f32("bias_a", bias_a, wide), _f32("bias_b", bias_b, heads)
+        a.rate, a.skip = _f32("rate", rate, heads), _f32("skip", skip, wide)
         a.state = _f32("state", state, state.numel())
         a.norm_state = _f32("norm_state", norm_state, slots * heads * tiles * key_dim)
         a.max_state = _f32("max_state", max_state, slots * heads * tiles)
@@ -475,7 +530,7 @@ class HybridOps:
         a.out, a.out_stride = out.data_ptr(), out.stride(0)
         a.q_stride, a.k_stride, a.v_stride = q.stride(0), k.stride(0), v.stride(0)
         a.gate_stride = 0 if gate_a is None else gate_a.stride(0)
-        a.kind, a.dtype = {"ssd": 0, "mlstm": 1, "lightning": 2}[kind], _DTYPE[v.dtype]
+        a.kind, a.dtype = {"ssd": 0, "mlstm": 1, "lightning": 2, "wkv": 3}[kind], _DTYPE[v.dtype]
         a.decay = _f32("decay", decay, heads)
         a.num_tokens, a.num_seqs = v.shape[0], seg.cu_seqlens_q.shape[0] - 1
         a.num_heads, a.num_groups, a.key_dim, a.value_dim = heads, groups, key_dim, value_dim
