@@ -70,7 +70,8 @@ def make_engine(config: dict, tensors: dict[str, torch.Tensor], dtype=torch.bflo
 
     family = family_of(config)
     args = family.parse(config)
-    model = family.model_class(args)(args, lambda name, shape: tensors[name].reshape(shape), dtype, "cuda")
+    model = family.model_class(args)(args, lambda name, shape: tensors[name] if None in shape else tensors[name].reshape(shape),
+                                     dtype, "cuda")
     cache = family.make_cache(args, max_tokens // block_size + 1, block_size, max_num_seqs, dtype, "cuda")
     return Engine(model, cache, vocab=args.vocab, max_num_seqs=max_num_seqs, max_model_len=max_tokens, **kw)
 

@@ -175,9 +175,10 @@ def test_library_exports_every_declared_symbol():
 
 def test_args_struct_matches_header_layout():
     # 10 pointers/size_t + 12 int32 + 6 int64 + 2 float + 4 int32 (out_dtype .. value_dim) + 3 int64 (value strides) + 3 int32
-    # (plain_softmax, min_q_len, keep_first), padded to 8
-    assert ctypes.sizeof(PagedAttnArgs) == 10 * 8 + 12 * 4 + 6 * 8 + 2 * 4 + 4 * 4 + 3 * 8 + 4 * 4
-    assert PagedAttnArgs.keep_first.offset == ctypes.sizeof(PagedAttnArgs) - 8
+    # (plain_softmax, min_q_len, keep_first), padded to 8, + 1 pointer (slopes)
+    assert ctypes.sizeof(PagedAttnArgs) == 10 * 8 + 12 * 4 + 6 * 8 + 2 * 4 + 4 * 4 + 3 * 8 + 4 * 4 + 8
+    assert PagedAttnArgs.slopes.offset == ctypes.sizeof(PagedAttnArgs) - 8
+    assert PagedAttnArgs.keep_first.offset == ctypes.sizeof(PagedAttnArgs) - 16
     assert PagedAttnArgs.out_dtype.offset == 10 * 8 + 12 * 4 + 6 * 8 + 2 * 4
     assert PagedAttnArgs.window_seqlen_q.offset == PagedAttnArgs.out_dtype.offset + 4
     assert PagedAttnArgs.q_stride.offset == 10 * 8 + 12 * 4
