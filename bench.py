@@ -665,7 +665,7 @@ def run_b200(args) -> None:
 
 
 def run_design(args, module: str, sizes: str) -> None:
-    """--hybrid / --streams / --sandwich: one JSON line with prefill / decode throughput and every kernel's roofline, per size."""
+    """--hybrid / --streams / --sandwich / --prenorm: one JSON line with prefill / decode throughput and every kernel's roofline, per size."""
     if args.impl == "reference" or args.gpus != 1:
         _emit(json.dumps({"impl": args.impl, "unavailable": "these decoders: one GPU, no reference arm"}))
         return
@@ -715,6 +715,9 @@ def main() -> None:
     ap.add_argument("--sandwich", action="store_true",
                     help="sandwich-norm decoders with routed experts and the closest transformer with routed experts")
     ap.add_argument("--sandwich-sizes", default="s,m,w", help="sizes of profiles/bench_sandwich.py")
+    ap.add_argument("--prenorm", action="store_true",
+                    help="pre-norm decoders with time mixing and the closest hyper-connected decoder, one stream")
+    ap.add_argument("--prenorm-sizes", default="s,m,w", help="sizes of profiles/bench_prenorm.py")
     args = ap.parse_args()
     if args.hybrid:
         run_design(args, "bench_hybrid", args.hybrid_sizes)
@@ -724,6 +727,9 @@ def main() -> None:
         return
     if args.sandwich:
         run_design(args, "bench_sandwich", args.sandwich_sizes)
+        return
+    if args.prenorm:
+        run_design(args, "bench_prenorm", args.prenorm_sizes)
         return
     select_config(args.config)
     if args.gpus < CONFIGS[args.config][6] and args.impl == "b200":

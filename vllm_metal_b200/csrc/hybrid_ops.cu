@@ -181,6 +181,13 @@ struct alignas(16) Vec8 {
 };
 __device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 
+// In 16-bit results: near zero the first terms of the series, where exp(z) - 1 - z would cancel.
+__device__ __forceinline__ float fast_xielu(float z, float a, float b) {
+  const float near0 = z * z * fmaf(z, fmaf(z, fmaf(z, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f);
+  const float low = z > -0.0625f ? near0 : __expf(z) - 1.f - z;
+  return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, low, 0.5f * z);
+}
+
 template <typename T, int LANES, int VPL, int ACT>
 __global__ void __launch_bounds__(256)
 mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks) {
@@ -224,13 +231,14 @@ mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks) {
       }
     }
     if (a.group_size > 0) {
-      ss = warp_sum(ss);
+#pragma unroll
+      for (int off = (LANES < 32 ? LANES : 32) / 2; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
       if (LANES > 32) {
         if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
         __syncthreads();
         ss = 0.f;
 #pragma unroll
-        for (int i = 0; i < LANES / 32; ++i) ss += red[threadIdx.x / LANES * (LANES / 32) + i];
+        for (int i = 0; i < (LANES > 32 ? LANES / 32 : 1); ++i) ss += red[threadIdx.x / LANES * (LANES / 32) + i];
       }
       inv = 1.f / sqrtf(ss / (float)gs + a.eps);
     }
@@ -278,7 +286,7 @@ mixer_finish_vec_kernel(const b200_mixer_finish_args a, int norm_blocks) {
         float v = a.act_kind == kActSilu   ? z * fast_sigmoid(z)
                   : a.act_kind == kActGelu ? gelu_erf_f(z)
                   : a.act_kind == kActTanh ? tanhf(z)
-                                           : xielu_f(z, a.act_a, a.act_b);
+                                           : fast_xielu(z, a.act_a, a.act_b);
         if (mul) v *= to_float(m[j].e[e]);
         x[j].e[e] = from_float<T>(v);
       }
@@ -302,13 +310,15 @@ bool finish_vec_ok(const b200_mixer_finish_args& a) {
 template <typename T>
 int launch_finish_vec(const b200_mixer_finish_args& a, cudaStream_t st) {
   const int gs = a.group_size > 0 ? a.group_size : 2048, groups = a.y ? (a.inner + gs - 1) / gs : 0;
-  const int lanes = gs <= 256 ? 32 : gs <= 512 ? 64 : gs <= 1024 ? 128 : 256;
+  const int lanes = gs <= 64 ? 8 : gs <= 128 ? 16 : gs <= 256 ? 32 : gs <= 512 ? 64 : gs <= 1024 ? 128 : 256;
   const int vpl = gs <= 2048 ? 1 : gs <= 4096 ? 2 : 4, act = a.rows >= 256 ? 2 : 1;
   const int nb = (groups * lanes + 255) / 256, ab = (a.act_dim + act * 2048 - 1) / (act * 2048);
   auto pick = [&](auto act_tag) {
     constexpr int A = decltype(act_tag)::value;
     return vpl == 4      ? mixer_finish_vec_kernel<T, 256, 4, A>
            : vpl == 2    ? mixer_finish_vec_kernel<T, 256, 2, A>
+           : lanes == 8 ? mixer_finish_vec_kernel<T, 8, 1, A>
+           : lanes == 16 ? mixer_finish_vec_kernel<T, 16, 1, A>
            : lanes == 32 ? mixer_finish_vec_kernel<T, 32, 1, A>
            : lanes == 64 ? mixer_finish_vec_kernel<T, 64, 1, A>
            : lanes == 128 ? mixer_finish_vec_kernel<T, 128, 1, A>

@@ -253,7 +253,7 @@ chunk_scan_kernel(const b200_recurrence_args a, int state_blocks) {
     const size_t ustep = (size_t)a.num_heads * K * V;
     float4 S = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *st;
     float m = KIND == kMlstm ? scal[2] : 0.f;
-    constexpr int AHEAD = 4;
+    constexpr int AHEAD = KIND == kWkv ? 8 : 4;
     float4 buf[AHEAD];
     float kept[KIND == kWkv ? AHEAD : 1];  // decay of this key row over a chunk
     const float* kp = ws.keysum + ((size_t)cfirst * a.num_heads + h) * K + (KIND == kWkv ? i / V : 0);

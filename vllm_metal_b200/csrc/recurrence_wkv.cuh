@@ -21,13 +21,29 @@ namespace b200 {
 namespace rec {
 namespace wkv {
 
-constexpr int kBlock = 16, kBlocks = kChunk / kBlock;  // one block a warp
+constexpr int kThreads = 256;
+constexpr int kBlock = 16, kBlocks = kChunk / kBlock;  // two warps a block
 constexpr int kPitch = 68;                              // of fp32 tiles
 constexpr int kFloatTile = kChunk * kPitch;
 
+// As rec::load_tile, by all threads here.
+__device__ __forceinline__ void load_rows(bf16* dst, const bf16* src, int64_t stride, int rows, int cols) {
+#pragma unroll
+  for (int i = threadIdx.x; i < 64 * 8; i += kThreads) {
+    const int r = i >> 3, c = (i & 7) * 8;
+    const bool live = r < rows && c < cols;
+    mma::cp_async16(dst + r * kPad + c, live ? src + (int64_t)r * stride + c : src, live);
+  }
+}
+
 struct Decays {  // of one key channel over a block
   float w[kBlock];
-  __device__ __forceinline__ void load(const b200_recurrence_args& a, int row0, int rows, int first, int channel) {
+  __device__ __forceinline__ void load(const b200_recurrence_args& a, int row0, int rows, int first, int channel, bool live) {
+    if (!live) {
+#pragma unroll
+      for (int i = 0; i < kBlock; ++i) w[i] = 1.f;
+      return;
+    }
     const float bias = a.bias_a[channel];
     const float* z = reinterpret_cast<const float*>(a.gate_a) + (int64_t)(row0 + first) * a.gate_stride + channel;
 #pragma unroll
@@ -58,7 +74,7 @@ __device__ __forceinline__ float keys_to_block_end(const Decays& d, const bf16* 
 // ---- 1: a chunk's own contribution and its decay -----------------------------------------------------
 constexpr int kStateSmem = (2 + kTerms) * kTileElems * 2 + kBlocks * 64 * 4;
 
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kThreads, 3)
 state_kernel(const b200_recurrence_args a) {
   extern __shared__ __align__(16) uint8_t raw[];
   bf16* sk = reinterpret_cast<bf16*>(raw);
@@ -69,33 +85,24 @@ state_kernel(const b200_recurrence_args a) {
   pdl_wait();
   const int c = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
   const int K = a.key_dim, V = a.value_dim, c0 = tile * kTileV;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, m0 = (warp >> 1) * 16, v0 = (warp & 1) * 32;
   int row0;
   const int rows = chunk_rows(a, c, &row0);
   const Workspace ws(a);
   const bf16* kp = reinterpret_cast<const bf16*>(a.k) + (int64_t)row0 * a.k_stride + (int64_t)h * K;
   const bf16* vp = reinterpret_cast<const bf16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)h * V + c0;
-  load_tile(sv, vp, a.v_stride, rows, min(kTileV, V - c0));
+  load_rows(sv, vp, a.v_stride, rows, min(kTileV, V - c0));
   float* U = ws.state + ((size_t)c * a.num_heads + h) * K * V;
   float* keep = ws.keysum + ((size_t)c * a.num_heads + h) * K;
+  const int n = tid & 63, b = tid >> 6;
   for (int k0 = 0; k0 < K; k0 += kSlab) {
-    load_tile(sk, kp + k0, a.k_stride, rows, min(kSlab, K - k0));
+    load_rows(sk, kp + k0, a.k_stride, rows, min(kSlab, K - k0));
     mma::cp_commit();
-    const int n = tid & 63, b0 = (tid >> 6) * 2;
-    Decays d[2];
-    if (k0 + n < K) {
-#pragma unroll
-      for (int b = 0; b < 2; ++b) d[b].load(a, row0, rows, (b0 + b) * kBlock, h * K + k0 + n);
-    } else {
-#pragma unroll
-      for (int b = 0; b < 2; ++b)
-#pragma unroll
-        for (int i = 0; i < kBlock; ++i) d[b].w[i] = 1.f;
-    }
+    Decays d;
+    d.load(a, row0, rows, b * kBlock, h * K + k0 + n, k0 + n < K);
     mma::cp_wait<0>();
     __syncthreads();
-#pragma unroll
-    for (int b = 0; b < 2; ++b) D[(b0 + b) * 64 + n] = keys_to_block_end(d[b], sk, ks3, (b0 + b) * kBlock, n);
+    D[b * 64 + n] = keys_to_block_end(d, sk, ks3, b * kBlock, n);
     __syncthreads();
     if (tile == 0 && tid < 64 && k0 + tid < K) {
       float p = 1.f;
@@ -103,30 +110,30 @@ state_kernel(const b200_recurrence_args a) {
       for (int j = 0; j < kBlocks; ++j) p *= D[j * 64 + tid];
       keep[k0 + tid] = p;
     }
-    float acc[8][4];
+    float acc[4][4];
 #pragma unroll
-    for (int i = 0; i < 8; ++i)
+    for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
 #pragma unroll
     for (int j = 0; j < kBlocks; ++j) {
       if (j > 0) {
-        const float d0 = D[j * 64 + warp * 16 + (lane >> 2)], d1 = D[j * 64 + warp * 16 + (lane >> 2) + 8];
+        const float d0 = D[j * 64 + m0 + (lane >> 2)], d1 = D[j * 64 + m0 + (lane >> 2) + 8];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
+        for (int i = 0; i < 4; ++i) {
           acc[i][0] *= d0, acc[i][1] *= d0;
           acc[i][2] *= d1, acc[i][3] *= d1;
         }
       }
       // A[m = key dim][k = row]: stored row by row, so the fragments come transposed
       uint32_t fa[kTerms][4];
-      const int mat = lane >> 3, krow = j * kBlock + ((mat >> 1) ? 8 : 0) + (lane & 7), kcol = warp * 16 + ((mat & 1) ? 8 : 0);
+      const int mat = lane >> 3, krow = j * kBlock + ((mat >> 1) ? 8 : 0) + (lane & 7), kcol = m0 + ((mat & 1) ? 8 : 0);
 #pragma unroll
       for (int t = 0; t < kTerms; ++t) mma::ldsm4t(fa[t], &ks3[t * kTileElems + krow * kPad + kcol]);
 #pragma unroll
-      for (int n2 = 0; n2 < 4; ++n2) {
+      for (int n2 = 0; n2 < 2; ++n2) {
         uint32_t fb[4];
-        mma::ldsm4t(fb, &sv[(j * kBlock + (lane & 15)) * kPad + n2 * 16 + (lane >> 4) * 8]);
+        mma::ldsm4t(fb, &sv[(j * kBlock + (lane & 15)) * kPad + v0 + n2 * 16 + (lane >> 4) * 8]);
 #pragma unroll
         for (int t = 0; t < kTerms; ++t) {
           mma::mma16816(acc[2 * n2], fa[t], fb[0], fb[1]);
@@ -135,11 +142,11 @@ state_kernel(const b200_recurrence_args a) {
       }
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int col = c0 + i * 8 + (lane & 3) * 2;
+    for (int i = 0; i < 4; ++i) {
+      const int col = c0 + v0 + i * 8 + (lane & 3) * 2;
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
-        const int kd = k0 + warp * 16 + (lane >> 2) + half * 8;
+        const int kd = k0 + m0 + (lane >> 2) + half * 8;
         if (kd < K && col < V)
           *reinterpret_cast<float2*>(U + (size_t)kd * V + col) = make_float2(acc[i][2 * half], acc[i][2 * half + 1]);
       }
@@ -149,12 +156,17 @@ state_kernel(const b200_recurrence_args a) {
 }
 
 // ---- 3: outputs ------------------------------------------------------------------------------------------
+// Two warps share a block: each takes half of a slab's key channels through all the products -- they are linear in the scores --
+// and the two halves of the outputs meet at the end.
 // sr sk sv | K's terms | { R, decays } fp32, over which the state on entry goes later (its three terms) | D, bonus, scores
 constexpr int kBig = 2 * kFloatTile * 4;
+constexpr int kScorePitch = kBlock + 1, kSwapPitch = 36;
 static_assert(kBig >= kTerms * kTileElems * 2, "the state's terms go over R and the decays");
-constexpr int kOutputSmem = (3 + kTerms) * kTileElems * 2 + kBig + (kBlocks * 64 + 64) * 4 + 4 * kBlock * (kBlock + 1) * 4;
+static_assert(kBig >= 2 * kBlocks * kBlock * kSwapPitch * 4, "so do the halves of the outputs");
+constexpr int kOutputSmem =
+    (3 + kTerms) * kTileElems * 2 + kBig + (kBlocks * 64 + 64) * 4 + 2 * kBlocks * kBlock * kScorePitch * 4;
 
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kThreads, 2)
 output_kernel(const b200_recurrence_args a) {
   extern __shared__ __align__(16) uint8_t raw[];
   bf16* sr = reinterpret_cast<bf16*>(raw);
@@ -166,12 +178,13 @@ output_kernel(const b200_recurrence_args a) {
   bf16* ss = reinterpret_cast<bf16*>(sR);
   float* D = sw + kFloatTile;
   float* su = D + kBlocks * 64;
-  float* own = su + 64;  // [warp][16 rows t][17]: scores inside the warp's block
+  float* own = su + 64;  // [warp][16 rows t][17]: scores inside the block, from the warp's channels
   pdl_trigger();
   pdl_wait();
   const int c = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
   const int K = a.key_dim, V = a.value_dim, c0 = tile * kTileV;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+  const int block = warp >> 1, half = warp & 1, base = block * kBlock;
   int row0;
   const int rows = chunk_rows(a, c, &row0);
   const Workspace ws(a);
@@ -179,60 +192,59 @@ output_kernel(const b200_recurrence_args a) {
   const bf16* kp = reinterpret_cast<const bf16*>(a.k) + (int64_t)row0 * a.k_stride + (int64_t)h * K;
   const bf16* vp = reinterpret_cast<const bf16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)h * V + c0;
   const float* S = ws.state + ((size_t)c * a.num_heads + h) * K * V;
-  load_tile(sv, vp, a.v_stride, rows, min(kTileV, V - c0));
-  float* mine = own + warp * kBlock * (kBlock + 1);
-  float sc[2 * kBlocks][4], o[8][4];
+  load_rows(sv, vp, a.v_stride, rows, min(kTileV, V - c0));
+  float* mine = own + warp * kBlock * kScorePitch;
+  float sc[2 * (kBlocks - 1)][4], o[8][4];
 #pragma unroll
   for (int i = 0; i < 8; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) sc[i][e] = o[i][e] = 0.f;
+    for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
+#pragma unroll
+  for (int i = 0; i < 2 * (kBlocks - 1); ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) sc[i][e] = 0.f;
   for (int k0 = 0; k0 < K; k0 += kSlab) {
-    load_tile(sr, rp + k0, a.q_stride, rows, min(kSlab, K - k0));
-    load_tile(sk, kp + k0, a.k_stride, rows, min(kSlab, K - k0));
+    load_rows(sr, rp + k0, a.q_stride, rows, min(kSlab, K - k0));
+    load_rows(sk, kp + k0, a.k_stride, rows, min(kSlab, K - k0));
     mma::cp_commit();
+    float4 sx[4];  // the slab's state on entry, for later
     {
-      const int n = tid & 63, b0 = (tid >> 6) * 2;
+      const int n = tid & 63, b = tid >> 6, first = b * kBlock;
       if (tid < 64) su[tid] = k0 + tid < K ? a.skip[h * K + k0 + tid] : 0.f;
-      Decays d[2];
+      Decays d;
+      d.load(a, row0, rows, first, h * K + k0 + n, k0 + n < K);
 #pragma unroll
-      for (int b = 0; b < 2; ++b) {
-        if (k0 + n < K) {
-          d[b].load(a, row0, rows, (b0 + b) * kBlock, h * K + k0 + n);
-        } else {
-#pragma unroll
-          for (int i = 0; i < kBlock; ++i) d[b].w[i] = 1.f;
-        }
+      for (int i = 0; i < 4; ++i) {
+        const int r = (tid >> 4) + i * 16, cc = (tid & 15) * 4;
+        sx[i] = k0 + r < K && c0 + cc < V ? *reinterpret_cast<const float4*>(S + (size_t)(k0 + r) * V + c0 + cc)
+                                          : make_float4(0.f, 0.f, 0.f, 0.f);
       }
       mma::cp_wait<0>();
       __syncthreads();
+      float run = 1.f;
 #pragma unroll
-      for (int b = 0; b < 2; ++b) {
-        const int first = (b0 + b) * kBlock;
-        float run = 1.f;
-#pragma unroll
-        for (int i = 0; i < kBlock; ++i) {
-          sR[(first + i) * kPitch + n] = to_float(sr[(first + i) * kPad + n]) * run;
-          sw[(first + i) * kPitch + n] = d[b].w[i];
-          run *= d[b].w[i];
-        }
-        D[(b0 + b) * 64 + n] = keys_to_block_end(d[b], sk, ks3, first, n);
+      for (int i = 0; i < kBlock; ++i) {
+        sR[(first + i) * kPitch + n] = to_float(sr[(first + i) * kPad + n]) * run;
+        sw[(first + i) * kPitch + n] = d.w[i];
+        run *= d.w[i];
       }
+      D[b * 64 + n] = keys_to_block_end(d, sk, ks3, first, n);
     }
     __syncthreads();
-    // R of the warp's own rows, as fragments: [k step][row half + column half][pair]
-    float R[4][4][2];
+    // R of the block's rows and the warp's channels, as fragments: [k step][row half + column half][pair]
+    float R[2][4][2];
 #pragma unroll
-    for (int ks = 0; ks < 4; ++ks)
+    for (int ks = 0; ks < 2; ++ks)
 #pragma unroll
       for (int q = 0; q < 4; ++q) {
-        const float2 x = *reinterpret_cast<const float2*>(&sR[(warp * kBlock + g + (q & 1) * 8) * kPitch + ks * 16 + (q >> 1) * 8 + 2 * tq]);
+        const float2 x = *reinterpret_cast<const float2*>(&sR[(base + g + (q & 1) * 8) * kPitch + half * 32 + ks * 16 + (q >> 1) * 8 + 2 * tq]);
         R[ks][q][0] = x.x, R[ks][q][1] = x.y;
       }
-    {  // scores inside the block: lane = row s, half of the slab's channels
-      const int s = lane & 15, n0 = (lane >> 4) * 32, base = warp * kBlock;
-      float q[32];
+    {  // scores inside the block: lane = row s, 16 of the warp's channels
+      const int s = lane & 15, n0 = half * 32 + (lane >> 4) * 16;
+      float q[16];
 #pragma unroll
-      for (int i = 0; i < 32; i += 8) {
+      for (int i = 0; i < 16; i += 8) {
         const uint4 x4 = *reinterpret_cast<const uint4*>(&sk[(base + s) * kPad + n0 + i]);
         const bf16* x = reinterpret_cast<const bf16*>(&x4);
 #pragma unroll
@@ -240,19 +252,19 @@ output_kernel(const b200_recurrence_args a) {
       }
       float bonus = 0.f;  // the current row against itself
 #pragma unroll
-      for (int i = 0; i < 32; i += 8) {
+      for (int i = 0; i < 16; i += 8) {
         const uint4 x4 = *reinterpret_cast<const uint4*>(&sr[(base + s) * kPad + n0 + i]);
         const bf16* x = reinterpret_cast<const bf16*>(&x4);
 #pragma unroll
         for (int e = 0; e < 8; ++e) bonus = fmaf(to_float(x[e]) * su[n0 + i + e], q[i + e], bonus);
       }
       bonus += __shfl_xor_sync(0xffffffffu, bonus, 16);
-      if (lane < 16) mine[s * (kBlock + 1) + s] = (k0 > 0 ? mine[s * (kBlock + 1) + s] : 0.f) + bonus;
-#pragma unroll 1
+      if (lane < 16) mine[s * kScorePitch + s] = (k0 > 0 ? mine[s * kScorePitch + s] : 0.f) + bonus;
+#pragma unroll 3
       for (int t = 1; t < kBlock; ++t) {
         float dot[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int i = 0; i < 32; i += 8) {
+        for (int i = 0; i < 16; i += 8) {
           const uint4 x4 = *reinterpret_cast<const uint4*>(&sr[(base + t) * kPad + n0 + i]);
           const bf16* x = reinterpret_cast<const bf16*>(&x4);
 #pragma unroll
@@ -260,15 +272,12 @@ output_kernel(const b200_recurrence_args a) {
         }
         float sum = (dot[0] + dot[1]) + (dot[2] + dot[3]);
         sum += __shfl_xor_sync(0xffffffffu, sum, 16);
-        if (s < t) {
-          if (lane < 16) mine[t * (kBlock + 1) + s] = (k0 > 0 ? mine[t * (kBlock + 1) + s] : 0.f) + sum;
+        if (lane < 16 && s < t) mine[t * kScorePitch + s] = (k0 > 0 ? mine[t * kScorePitch + s] : 0.f) + sum;
 #pragma unroll
-          for (int i = 0; i < 32; i += 4) {
-            const float4 w = *reinterpret_cast<const float4*>(&sw[(base + t) * kPitch + n0 + i]);
-            q[i] *= w.x, q[i + 1] *= w.y, q[i + 2] *= w.z, q[i + 3] *= w.w;
-          }
+        for (int i = 0; i < 16; i += 4) {  // a row's own key does not decay before the row after the next reads it
+          const float4 w = *reinterpret_cast<const float4*>(&sw[(base + t) * kPitch + n0 + i]);
+          q[i] *= s < t ? w.x : 1.f, q[i + 1] *= s < t ? w.y : 1.f, q[i + 2] *= s < t ? w.z : 1.f, q[i + 3] *= s < t ? w.w : 1.f;
         }
-        __syncwarp();
       }
     }
     // against earlier blocks, nearest first; R picks up a block's decay after it
@@ -283,15 +292,16 @@ output_kernel(const b200_recurrence_args a) {
     };
 #pragma unroll
     for (int j = kBlocks - 2; j >= 0; --j) {
-      if (j >= warp) continue;
+      if (j >= block) continue;
 #pragma unroll
-      for (int ks = 0; ks < 4; ++ks) {
+      for (int ks = 0; ks < 2; ++ks) {
+        const int col = half * 32 + ks * 16;
         uint32_t fa[kTerms][4];
         split(ks, fa);
 #pragma unroll
         for (int y = 0; y < kTerms; ++y) {
           uint32_t fb[4];
-          mma::ldsm4(fb, &ks3[y * kTileElems + (j * kBlock + (lane >> 4) * 8 + (lane & 7)) * kPad + ks * 16 + ((lane >> 3) & 1) * 8]);
+          mma::ldsm4(fb, &ks3[y * kTileElems + (j * kBlock + (lane >> 4) * 8 + (lane & 7)) * kPad + col + ((lane >> 3) & 1) * 8]);
 #pragma unroll
           for (int x = 0; x + y < kTerms; ++x) {
             mma::mma16816(sc[2 * j], fa[x], fb[0], fb[1]);
@@ -300,25 +310,24 @@ output_kernel(const b200_recurrence_args a) {
         }
 #pragma unroll
         for (int q = 0; q < 4; ++q) {
-          const float2 d = *reinterpret_cast<const float2*>(&D[j * 64 + ks * 16 + (q >> 1) * 8 + 2 * tq]);
+          const float2 d = *reinterpret_cast<const float2*>(&D[j * 64 + col + (q >> 1) * 8 + 2 * tq]);
           R[ks][q][0] *= d.x, R[ks][q][1] *= d.y;
         }
       }
     }
     __syncthreads();  // R and the decays have been read everywhere: the state on entry goes over them
-    for (int i = tid; i < 64 * 16; i += 128) {
-      const int r = i >> 4, cc = (i & 15) * 4;
-      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (k0 + r < K && c0 + cc < V) x = *reinterpret_cast<const float4*>(S + (size_t)(k0 + r) * V + c0 + cc);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = (tid >> 4) + i * 16, cc = (tid & 15) * 4;
       uint32_t t0[kTerms], t1[kTerms];
-      mma::split_pair<kTerms>(x.x, x.y, t0);
-      mma::split_pair<kTerms>(x.z, x.w, t1);
+      mma::split_pair<kTerms>(sx[i].x, sx[i].y, t0);
+      mma::split_pair<kTerms>(sx[i].z, sx[i].w, t1);
 #pragma unroll
       for (int j = 0; j < kTerms; ++j) *reinterpret_cast<uint2*>(&ss[j * kTileElems + r * kPad + cc]) = make_uint2(t0[j], t1[j]);
     }
     __syncthreads();
 #pragma unroll
-    for (int ks = 0; ks < 4; ++ks) {
+    for (int ks = 0; ks < 2; ++ks) {
       uint32_t fa[kTerms][4];
       split(ks, fa);
 #pragma unroll
@@ -326,7 +335,7 @@ output_kernel(const b200_recurrence_args a) {
 #pragma unroll
         for (int y = 0; y < kTerms; ++y) {
           uint32_t fb[4];
-          mma::ldsm4t(fb, &ss[y * kTileElems + (ks * 16 + (lane & 15)) * kPad + n2 * 16 + (lane >> 4) * 8]);
+          mma::ldsm4t(fb, &ss[y * kTileElems + (half * 32 + ks * 16 + (lane & 15)) * kPad + n2 * 16 + (lane >> 4) * 8]);
 #pragma unroll
           for (int x = 0; x + y < kTerms; ++x) {
             mma::mma16816(o[2 * n2], fa[x], fb[0], fb[1]);
@@ -336,25 +345,13 @@ output_kernel(const b200_recurrence_args a) {
     }
     __syncthreads();
   }
-  // the block's own scores, on and below the diagonal
-  float dg[2][4];
-#pragma unroll
-  for (int i = 0; i < 2; ++i)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int t = g + (e >> 1) * 8, s = i * 8 + 2 * tq + (e & 1);
-      dg[i][e] = s <= t ? mine[t * (kBlock + 1) + s] : 0.f;
-    }
-#pragma unroll
-  for (int j = 0; j < kBlocks; ++j) {
-    if (j > warp) break;
+  // the scores' share of the outputs; those of the block itself on and below the diagonal
+  auto values = [&](int j, const float (&lo)[4], const float (&hi)[4]) {  // scores of columns 0..7 and 8..15 of block j
     uint32_t p[4][kTerms];
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const bool diagonal = j == warp;
-      mma::split_pair<kTerms>(diagonal ? dg[i][0] : sc[2 * j + i][0], diagonal ? dg[i][1] : sc[2 * j + i][1], p[2 * i]);
-      mma::split_pair<kTerms>(diagonal ? dg[i][2] : sc[2 * j + i][2], diagonal ? dg[i][3] : sc[2 * j + i][3], p[2 * i + 1]);
-    }
+    mma::split_pair<kTerms>(lo[0], lo[1], p[0]);
+    mma::split_pair<kTerms>(lo[2], lo[3], p[1]);
+    mma::split_pair<kTerms>(hi[0], hi[1], p[2]);
+    mma::split_pair<kTerms>(hi[2], hi[3], p[3]);
 #pragma unroll
     for (int n2 = 0; n2 < 4; ++n2) {
       uint32_t fb[4];
@@ -366,17 +363,44 @@ output_kernel(const b200_recurrence_args a) {
         mma::mma16816(o[2 * n2 + 1], fa, fb[2], fb[3]);
       }
     }
+  };
+#pragma unroll
+  for (int j = 0; j < kBlocks - 1; ++j)
+    if (j < block) values(j, sc[2 * j], sc[2 * j + 1]);
+  float dg[2][4];
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int t = g + (e >> 1) * 8, s = i * 8 + 2 * tq + (e & 1);
+      dg[i][e] = s <= t ? mine[t * kScorePitch + s] : 0.f;
+    }
+  values(block, dg[0], dg[1]);
+  // a warp leaves its partner the 32 columns that it does not store
+  float* swap = sR + warp * kBlock * kSwapPitch;
+  const float* other = sR + (warp ^ 1) * kBlock * kSwapPitch;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int cc = i * 8 + 2 * tq;
+    float2 lo, hi;
+    lo.x = half ? o[i][0] : o[i + 4][0], lo.y = half ? o[i][1] : o[i + 4][1];
+    hi.x = half ? o[i][2] : o[i + 4][2], hi.y = half ? o[i][3] : o[i + 4][3];
+    *reinterpret_cast<float2*>(&swap[g * kSwapPitch + cc]) = lo;
+    *reinterpret_cast<float2*>(&swap[(g + 8) * kSwapPitch + cc]) = hi;
   }
+  __syncthreads();
   bf16* out = reinterpret_cast<bf16*>(a.out);
 #pragma unroll
-  for (int i = 0; i < 8; ++i) {
-    const int cc = i * 8 + tq * 2;
+  for (int i = 0; i < 4; ++i) {
+    const int cc = i * 8 + 2 * tq, col = half * 32 + cc;
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      const int t = warp * kBlock + g + e * 8;
-      if (t >= rows || c0 + cc >= V) continue;
-      *reinterpret_cast<__nv_bfloat162*>(out + (int64_t)(row0 + t) * a.out_stride + (int64_t)h * V + c0 + cc) =
-          __floats2bfloat162_rn(o[i][2 * e], o[i][2 * e + 1]);
+      const int t = base + g + e * 8;
+      if (t >= rows || c0 + col >= V) continue;
+      const float2 x = *reinterpret_cast<const float2*>(&other[(g + e * 8) * kSwapPitch + cc]);
+      const float y0 = half ? o[i + 4][2 * e] : o[i][2 * e], y1 = half ? o[i + 4][2 * e + 1] : o[i][2 * e + 1];
+      *reinterpret_cast<__nv_bfloat162*>(out + (int64_t)(row0 + t) * a.out_stride + (int64_t)h * V + c0 + col) =
+          __floats2bfloat162_rn(y0 + x.x, y1 + x.y);
     }
   }
 }
@@ -392,10 +416,10 @@ inline int launch(const b200_recurrence_args& a, cudaStream_t st) {
     attr = true;
   }
   const dim3 grid((a.value_dim + kTileV - 1) / kTileV, a.num_heads, a.num_chunks);
-  B200_CUDA_OK(launch_pdl(state_kernel, grid, dim3(128), kStateSmem, st, a));
+  B200_CUDA_OK(launch_pdl(state_kernel, grid, dim3(kThreads), kStateSmem, st, a));
   const int blocks = (a.key_dim * a.value_dim / 4 + kScanThreads - 1) / kScanThreads;
   B200_CUDA_OK(launch_pdl(chunk_scan_kernel<kWkv>, dim3(blocks, a.num_heads, a.num_seqs), dim3(kScanThreads), 0, st, a, blocks));
-  B200_CUDA_OK(launch_pdl(output_kernel, grid, dim3(128), kOutputSmem, st, a));
+  B200_CUDA_OK(launch_pdl(output_kernel, grid, dim3(kThreads), kOutputSmem, st, a));
   return check_launch("recurrence (decays per key channel)");
 }
 
