@@ -72,43 +72,52 @@ __device__ __forceinline__ float keys_to_block_end(const Decays& d, const bf16* 
 }
 
 // ---- 1: a chunk's own contribution and its decay -----------------------------------------------------
-constexpr int kStateSmem = (2 + kTerms) * kTileElems * 2 + kBlocks * 64 * 4;
+// A CTA has one slab of key channels; the value tiles pass by it.
+constexpr int kStateSmem = (3 + kTerms) * kTileElems * 2 + kBlocks * 64 * 4;
 
 __global__ void __launch_bounds__(kThreads, 3)
 state_kernel(const b200_recurrence_args a) {
   extern __shared__ __align__(16) uint8_t raw[];
   bf16* sk = reinterpret_cast<bf16*>(raw);
-  bf16* sv = sk + kTileElems;
-  bf16* ks3 = sv + kTileElems;
+  bf16* sv2 = sk + kTileElems;  // two tiles, one being filled
+  bf16* ks3 = sv2 + 2 * kTileElems;
   float* D = reinterpret_cast<float*>(ks3 + kTerms * kTileElems);  // [blocks][64]
   pdl_trigger();
   pdl_wait();
-  const int c = blockIdx.z, h = blockIdx.y, tile = blockIdx.x;
-  const int K = a.key_dim, V = a.value_dim, c0 = tile * kTileV;
+  const int c = blockIdx.z, h = blockIdx.y, k0 = blockIdx.x * kSlab;
+  const int K = a.key_dim, V = a.value_dim, tiles = (V + kTileV - 1) / kTileV;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, m0 = (warp >> 1) * 16, v0 = (warp & 1) * 32;
   int row0;
   const int rows = chunk_rows(a, c, &row0);
   const Workspace ws(a);
   const bf16* kp = reinterpret_cast<const bf16*>(a.k) + (int64_t)row0 * a.k_stride + (int64_t)h * K;
-  const bf16* vp = reinterpret_cast<const bf16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)h * V + c0;
-  load_rows(sv, vp, a.v_stride, rows, min(kTileV, V - c0));
+  const bf16* vp = reinterpret_cast<const bf16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)h * V;
   float* U = ws.state + ((size_t)c * a.num_heads + h) * K * V;
-  float* keep = ws.keysum + ((size_t)c * a.num_heads + h) * K;
-  const int n = tid & 63, b = tid >> 6;
-  for (int k0 = 0; k0 < K; k0 += kSlab) {
-    load_rows(sk, kp + k0, a.k_stride, rows, min(kSlab, K - k0));
-    mma::cp_commit();
+  load_rows(sk, kp + k0, a.k_stride, rows, min(kSlab, K - k0));
+  load_rows(sv2, vp, a.v_stride, rows, min(kTileV, V));
+  mma::cp_commit();
+  {
+    const int n = tid & 63, b = tid >> 6;
     Decays d;
     d.load(a, row0, rows, b * kBlock, h * K + k0 + n, k0 + n < K);
     mma::cp_wait<0>();
     __syncthreads();
     D[b * 64 + n] = keys_to_block_end(d, sk, ks3, b * kBlock, n);
-    __syncthreads();
+  }
+  for (int tile = 0; tile < tiles; ++tile) {
+    const int c0 = tile * kTileV;
+    if (tile > 0) mma::cp_wait<0>();
+    __syncthreads();  // this tile is there, and the one before it has been read
+    const bf16* sv = sv2 + (tile & 1) * kTileElems;
+    if (tile + 1 < tiles) {
+      load_rows(sv2 + (~tile & 1) * kTileElems, vp + c0 + kTileV, a.v_stride, rows, min(kTileV, V - c0 - kTileV));
+      mma::cp_commit();
+    }
     if (tile == 0 && tid < 64 && k0 + tid < K) {
       float p = 1.f;
 #pragma unroll
       for (int j = 0; j < kBlocks; ++j) p *= D[j * 64 + tid];
-      keep[k0 + tid] = p;
+      ws.keysum[((size_t)c * a.num_heads + h) * K + k0 + tid] = p;
     }
     float acc[4][4];
 #pragma unroll
@@ -151,7 +160,6 @@ state_kernel(const b200_recurrence_args a) {
           *reinterpret_cast<float2*>(U + (size_t)kd * V + col) = make_float2(acc[i][2 * half], acc[i][2 * half + 1]);
       }
     }
-    __syncthreads();  // the tiles are free for the next slab
   }
 }
 
@@ -416,7 +424,8 @@ inline int launch(const b200_recurrence_args& a, cudaStream_t st) {
     attr = true;
   }
   const dim3 grid((a.value_dim + kTileV - 1) / kTileV, a.num_heads, a.num_chunks);
-  B200_CUDA_OK(launch_pdl(state_kernel, grid, dim3(kThreads), kStateSmem, st, a));
+  const dim3 slabs((a.key_dim + kSlab - 1) / kSlab, a.num_heads, a.num_chunks);
+  B200_CUDA_OK(launch_pdl(state_kernel, slabs, dim3(kThreads), kStateSmem, st, a));
   const int blocks = (a.key_dim * a.value_dim / 4 + kScanThreads - 1) / kScanThreads;
   B200_CUDA_OK(launch_pdl(chunk_scan_kernel<kWkv>, dim3(blocks, a.num_heads, a.num_seqs), dim3(kScanThreads), 0, st, a, blocks));
   B200_CUDA_OK(launch_pdl(output_kernel, grid, dim3(kThreads), kOutputSmem, st, a));
